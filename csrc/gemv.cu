@@ -23,15 +23,6 @@
 
 #include "common.cuh"
 
-__device__ TrlError g_trl_error = {0, 0, 0, 0};
-int g_trl_use_pdl = 1;
-#ifdef TRL_TRACE
-__device__ TrlTraceRec g_trl_trace[TRL_TRACE_CAP];
-__device__ unsigned int g_trl_trace_n = 0;
-__device__ unsigned int g_trl_trace_cur = 0;
-__device__ unsigned long long g_trl_last_exit = 0;
-#endif
-
 enum { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_STORE_F32 = 3, EPI_PUSH = 4 };
 
 namespace {
@@ -775,20 +766,6 @@ TRL_API int trl_gemv_bf16(const void* x, int ldx, const void* w, const void* nor
   return 0;
 }
 
-TRL_API void trl_set_pdl(int on) { g_trl_use_pdl = on; }
-
-TRL_API int trl_error_read(int* out4, int clear) {
-  TrlError h;
-  cudaError_t e = cudaMemcpyFromSymbol(&h, g_trl_error, sizeof(h));
-  if (e != cudaSuccess) return (int)e;
-  out4[0] = h.code, out4[1] = h.a, out4[2] = h.b, out4[3] = h.c;
-  if (clear && h.code != 0) {
-    TrlError z = {0, 0, 0, 0};
-    cudaMemcpyToSymbol(g_trl_error, &z, sizeof(z));
-  }
-  return 0;
-}
-
 // Row-parallel GEMV whose epilogue pushes fp32 partial rows into every rank's one-shot
 // all-reduce slot (see comm.cu); trl_allreduce_finish completes the sum on each rank.
 TRL_API int trl_gemv_nvfp4_push(const void* x, int ldx, const void* wq, const void* wscale, const void* tscale,
@@ -808,25 +785,4 @@ TRL_API int trl_gemv_nvfp4_push(const void* x, int ldx, const void* wq, const vo
     if (e != cudaSuccess) return (int)e;
   }
   return 0;
-}
-
-// Timeline records of the launches since the last reset (builds with -DTRL_TRACE; otherwise
-// returns 0 records).  out: n x 16 uint64 {kind, entry, dependency wait done, exit, mark 0, mark 1,
-// latest exit of any CTA of the launches before, unused, marks 2..9} in ns.
-TRL_API int trl_trace_read(void* out, int cap, int reset) {
-#ifdef TRL_TRACE
-  unsigned int n = 0;
-  if (cudaMemcpyFromSymbol(&n, g_trl_trace_n, sizeof(n)) != cudaSuccess) return -1;
-  if ((int)n > cap) n = cap;
-  if (n > TRL_TRACE_CAP) n = TRL_TRACE_CAP;
-  if (n && cudaMemcpyFromSymbol(out, g_trl_trace, (size_t)n * sizeof(TrlTraceRec)) != cudaSuccess) return -1;
-  if (reset) {
-    const unsigned int z = 0;
-    cudaMemcpyToSymbol(g_trl_trace_n, &z, sizeof(z));
-  }
-  return (int)n;
-#else
-  (void)out, (void)cap, (void)reset;
-  return 0;
-#endif
 }
