@@ -6,7 +6,8 @@ into ``tilerl_b200/_C.so`` (plain C ABI, loaded with ctypes; no torch headers, s
 a full rebuild takes well under a minute).  The host-side C++ runtime
 (``csrc/runtime.cpp``: paged allocator, block-table builder) is linked into the
 same library.  The library is built in-tree so a source snapshot of the
-repository carries it to the GPU machine.
+repository carries it to the GPU machine.  ``ensure`` builds a smaller library for one
+architecture where the full one is missing.
 """
 from __future__ import annotations
 
@@ -15,6 +16,7 @@ import os
 import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
+from typing import Optional
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CSRC = os.path.join(ROOT, "csrc")
@@ -27,6 +29,10 @@ NVCC_FLAGS = [
     # global loads bypass L1: see "global loads and programmatic dependent launch" in csrc/common.cuh
     "-Xptxas", "-dlcm=cg",
 ]
+
+
+# Sources of a library that serves one architecture only (a first call in a fresh checkout compiles no more)
+GROUPS = {"Zinutar": ("core.cu", "stream.cu", "linear_rows.cu", "attn_sigmoid.cu", "misc.cu", "runtime.cpp")}
 
 
 def _nvcc() -> str:
@@ -52,7 +58,29 @@ def _stamp(path: str) -> str:
     return h.hexdigest()
 
 
-def build(force: bool = False, verbose: bool = False, extra_flags=(), trace: bool = False, bounds: bool = False) -> str:
+def _digest(sources, flags) -> str:
+    return hashlib.sha1("".join(_stamp(os.path.join(CSRC, f)) for f in sources).encode() + " ".join(flags).encode()).hexdigest()
+
+
+def _current(path: str, sources, flags=()) -> bool:
+    """``path`` was linked from these sources as they are now."""
+    try:
+        with open(path + ".stamp") as f:
+            return os.path.exists(path) and f.read() == _digest(sources, flags)
+    except OSError:
+        return False
+
+
+def ensure(architecture: str) -> str:
+    """The library that serves ``architecture``: the full one if it is built and current, else one of just the
+    sources that architecture needs (built if missing or stale)."""
+    if _current(OUT, _sources()):
+        return OUT
+    return build(group=architecture if architecture in GROUPS else None)
+
+
+def build(force: bool = False, verbose: bool = False, extra_flags=(), trace: bool = False, bounds: bool = False,
+          group: Optional[str] = None) -> str:
     """``trace=True`` builds ``tilerl_b200/_C_trace.so`` with ``-DTRL_TRACE`` (per-launch timestamps of a
     tick, read by ``tilerl_b200.utils.tick_trace``) next to the normal library.  ``bounds=True`` builds
     ``tilerl_b200/_C_bounds.so`` with ``-DTRL_DEBUG_BOUNDS``: the indices the kernels take from tables
@@ -61,6 +89,9 @@ def build(force: bool = False, verbose: bool = False, extra_flags=(), trace: boo
     assert not (trace and bounds)
     variant = "_trace" if trace else ("_bounds" if bounds else "")
     obj_dir = OBJ + variant
+    sources = sorted(GROUPS[group]) if group else _sources()
+    if group:
+        variant += "_" + group.lower()
     out_path = OUT.replace("_C.so", f"_C{variant}.so")
     if trace:
         extra_flags = tuple(extra_flags) + ("-DTRL_TRACE",)
@@ -70,7 +101,7 @@ def build(force: bool = False, verbose: bool = False, extra_flags=(), trace: boo
     nvcc = _nvcc()
     jobs = []
     objs = []
-    for src in _sources():
+    for src in sources:
         sp = os.path.join(CSRC, src)
         op = os.path.join(obj_dir, src + ".o")
         st = op + ".stamp"
@@ -94,12 +125,14 @@ def build(force: bool = False, verbose: bool = False, extra_flags=(), trace: boo
     if jobs:
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(run, jobs))
-    if jobs or not os.path.exists(out_path):
+    if jobs or not _current(out_path, sources, extra_flags):
         cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-rdc=true",
                "-Xcompiler", "-fPIC", *objs, "-o", out_path]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed: {' '.join(cmd)}\n{r.stdout}\n{r.stderr}")
+        with open(out_path + ".stamp", "w") as f:
+            f.write(_digest(sources, extra_flags))
     return out_path
 
 

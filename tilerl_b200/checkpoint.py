@@ -37,10 +37,12 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import ATTN, ModelConfig
+from .config import ATTN, ModelConfig, ZinutarConfig
 from .formats import (FP8BlockTensor, NVFP4Tensor, dequantize_fp8_block, dequantize_nvfp4,
                       quantize_nvfp4)
 from .models.hybrid import HybridModel, linear_names, quantize_weight
+from .models.zinutar import ZinutarModel
+from .zinutar_layout import tensor_shapes
 
 
 class CheckpointError(ValueError):
@@ -255,8 +257,27 @@ def assemble_master(cfg: ModelConfig, reader: _Reader) -> Dict[str, torch.Tensor
     return out
 
 
+def load_zinutar(cfg: ZinutarConfig, path: str, device="cpu", dtype: Optional[torch.dtype] = None) -> ZinutarModel:
+    """Dense checkpoint of a Zinutar model (tensor names and shapes: ``zinutar_layout.tensor_shapes``)."""
+    reader = _Reader(path)
+    lacks = [n for n in tensor_shapes(cfg) if not reader.has(n)]
+    if lacks:
+        raise CheckpointError(f"checkpoint lacks {len(lacks)} tensors, first {lacks[0]}")
+    if dtype is None:
+        dtype = torch.bfloat16 if torch.device(device).type == "cuda" else torch.float32
+    try:
+        return ZinutarModel.from_tensors(cfg, reader.get, device, dtype)
+    except ValueError as e:
+        raise CheckpointError(str(e)) from None
+
+
 def load_checkpoint(cfg: ModelConfig, path: str, *, device="cpu", tp_rank: int = 0, tp: int = 1,
-                    keep_master: bool = False) -> HybridModel:
+                    keep_master: bool = False, dtype: Optional[torch.dtype] = None) -> HybridModel:
+    """``dtype``: compute dtype of designs that run in more than one (default: bf16 on a GPU, fp32 on CPU)."""
+    if isinstance(cfg, ZinutarConfig):
+        if tp > 1 or keep_master:
+            raise CheckpointError("Zinutar models are served on one GPU per process, without training masters")
+        return load_zinutar(cfg, path, device, dtype)
     cj = os.path.join(path, "config.json")
     if os.path.exists(cj):
         with open(cj) as f:
@@ -307,7 +328,10 @@ def save_checkpoint(model: HybridModel, path: str) -> None:
     from safetensors.torch import save_file
     os.makedirs(path, exist_ok=True)
     tensors: Dict[str, torch.Tensor] = {}
-    for k, v in model.params.items():
+    dense = isinstance(model, ZinutarModel)
+    if dense:
+        tensors = {k: v.detach().to(torch.bfloat16).cpu().contiguous() for k, v in model.tensors()}
+    for k, v in ({} if dense else model.params).items():
         if k.startswith("master."):
             continue
         if isinstance(v, NVFP4Tensor):
@@ -323,6 +347,9 @@ def save_checkpoint(model: HybridModel, path: str) -> None:
     os.replace(tmp, os.path.join(path, "model.safetensors"))
     cfg = model.cfg
     with open(os.path.join(path, "config.json"), "w") as f:
+        if dense:
+            json.dump(cfg.to_json(), f, indent=1)
+            return
         json.dump({"model_type": "tilerl_b200_hybrid", "name": cfg.name, "num_hidden_layers": cfg.n_layers,
                    "hidden_size": cfg.hidden, "num_attention_heads": cfg.n_q_heads,
                    "num_key_value_heads": cfg.n_kv_heads, "head_dim": cfg.head_dim,

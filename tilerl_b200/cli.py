@@ -13,7 +13,7 @@ from typing import List, Optional
 
 
 def _add_model_flags(p: argparse.ArgumentParser) -> None:
-    p.add_argument("--model", default="tiny", help="model config name (see tilerl_b200.config)")
+    p.add_argument("--model", default="tiny", help="model config name (see tilerl_b200.config), or a checkpoint directory with a config.json")
     p.add_argument("--checkpoint", default=None, help="HF-style checkpoint directory")
     p.add_argument("--tokenizer", default=None, help="tokenizer.json (default: byte tokenizer)")
     p.add_argument("--device", default=None, help="cuda | cpu (default: cuda when available)")
@@ -209,6 +209,11 @@ def _device(args) -> str:
     return "cuda" if torch.cuda.is_available() else "cpu"
 
 
+def _checkpoint(args) -> Optional[str]:
+    """``--checkpoint``, or the directory given as ``--model``."""
+    return args.checkpoint or (args.model if os.path.isdir(args.model) else None)
+
+
 def ssd_slots(path: str, capacity_bytes: int, slot_bytes: int) -> int:
     """Pages the spill file may hold: ``capacity_bytes`` of them, or, with no capacity given, half of the
     free space of the file's filesystem; at least one, at most 2^24."""
@@ -254,7 +259,7 @@ def cmd_serve(args) -> int:
         except ImportError:
             pass                      # no NVML binding in this environment: nothing to check with
     ops = make_ops(dev)
-    model = build_model(cfg, dev, seed=args.seed, checkpoint=args.checkpoint, ops=ops if dev != "cpu" else None)
+    model = build_model(cfg, dev, seed=args.seed, checkpoint=_checkpoint(args), ops=ops if dev != "cpu" else None)
     drafter = None
     if args.draft_checkpoint:
         from .spec import load_drafter
@@ -324,7 +329,7 @@ def cmd_train(args) -> int:
     import torch
     from . import evals, rl
     from .checkpoint import load_adapter, save_adapter, save_checkpoint
-    from .config import get_config
+    from .config import ZinutarConfig, get_config
     from .factory import build_engine, build_model, make_ops
     from .ledger import Run, runs_dir
     from .optim import make_optimizer
@@ -355,6 +360,8 @@ def cmd_train(args) -> int:
     if flags.get("allow_short_rollouts"):        # (a smoke recipe runs into its cap on purpose)
         args.allow_short_rollouts = True
     cfg = get_config(flags.get("model", args.model))
+    if isinstance(cfg, ZinutarConfig):
+        raise SystemExit("Zinutar models are served (serve, generate, bench), not trained")
     if not args.dry_run and flags.get("reward") in ("gsm8k", "boxed") and not args.data and (flags.get("rl") or flags.get("opd")):
         raise SystemExit(f"reward {flags['reward']!r} scores completions against gold answers: give --data rows.jsonl "
                          "with {prompt, answer} rows")
@@ -635,7 +642,7 @@ def cmd_bench(args) -> int:
     from .factory import build_engine, build_model, make_ops
     dev = _device(args)
     ops = make_ops(dev)
-    model = build_model(cfg, dev, seed=args.seed, checkpoint=args.checkpoint, ops=ops if dev != "cpu" else None)
+    model = build_model(cfg, dev, seed=args.seed, checkpoint=_checkpoint(args), ops=ops if dev != "cpu" else None)
     out = []
     for b in [int(x) for x in args.batches.split(",")]:
         eng = build_engine(model, ops, device=dev, slots=b + 1, max_ctx=args.prompt_len + args.gen + 32, prefix=False)

@@ -1,4 +1,5 @@
-"""Model configuration for the hybrid (gated-GQA attention + Gated-DeltaNet) decoder.
+"""Model configurations: the hybrid (gated-GQA attention + Gated-DeltaNet) decoder, and Zinutar
+(:class:`ZinutarConfig`, a looped decoder of parallel blocks; no counterpart in the reference).
 
 One frozen dataclass describes every shape the kernels, the KV pools, the
 tensor-parallel shard tables and the cost model derive from.  Layer kinds are
@@ -10,8 +11,10 @@ Parity: reference ``src/tilerl/config.py:11`` (``ModelConfig``), ``:114``
 """
 from __future__ import annotations
 
+import json
+import os
 from dataclasses import dataclass, replace
-from typing import Tuple
+from typing import Dict, Optional, Tuple
 
 ATTN = "attn"
 GDN = "gdn"
@@ -206,15 +209,220 @@ def small_gpu_tp() -> ModelConfig:
     )
 
 
+# ---- Zinutar: looped parallel-block decoder with sigmoid-weighted attention ------------------------
+@dataclass(frozen=True)
+class AttnSpec:
+    """One attention mixer without softmax: ``heads`` query heads over ``kv_heads`` key / value heads
+    (contiguous groups), query / key width ``dim``, value width ``vdim``, score factor ``scale``."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+
+    def __post_init__(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) <= 0 or self.heads % self.kv_heads:
+            raise ValueError(f"attention needs positive sizes and heads a multiple of kv_heads: {self}")
+
+    @property
+    def group(self) -> int:
+        return self.heads // self.kv_heads
+
+
+@dataclass(frozen=True)
+class MlpSpec:
+    """Feed-forward of width ``ff`` without a gate; ``kind`` names its form."""
+    ff: int
+    kind: str = "dense"
+
+    def __post_init__(self) -> None:
+        if self.kind != "dense":
+            raise ValueError(f"unknown feed-forward kind {self.kind!r}")
+        if self.ff <= 0:
+            raise ValueError("feed-forward width must be positive")
+
+
+@dataclass(frozen=True)
+class BlockSpec:
+    """One layer: an attention mixer and an optional feed-forward, both reading the same normed input."""
+    mixer: AttnSpec
+    mlp: Optional[MlpSpec] = None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers ``start .. stop-1`` run ``times`` times in a row with shared weights."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer: ``layer`` names its weights, ``kv`` its own cache, ``inject`` whether the
+    embedding output is added to the stream right before it."""
+    layer: int
+    kv: int
+    inject: bool = False
+
+
+def _fields(d: Dict, known, where: str) -> None:
+    extra = sorted(set(d) - set(known))
+    if extra:
+        raise ValueError(f"{where}: unknown keys {extra}")
+
+
+@dataclass(frozen=True)
+class ZinutarConfig:
+    """Sizes and constants of a Zinutar model.  Every layer has its own mixer and feed-forward sizes;
+    :attr:`runs` spells the executions out in order, one KV cache each."""
+    name: str
+    hidden: int
+    vocab: int
+    layers: Tuple[BlockSpec, ...]
+    loop: Optional[LoopSpec] = None
+    rms_eps: float = 1e-5
+    max_ctx: int = 1 << 20
+
+    architecture = "Zinutar"
+    tie_embeddings = False
+    quant = "bf16"
+    lm_head_quant = "bf16"
+    # no recurrent layers: the state pool of the engine degenerates to slot bookkeeping
+    n_gdn_layers = 0
+    gdn_k_heads = gdn_v_heads = gdn_head_dim = gdn_conv_dim = 0
+
+    def __post_init__(self) -> None:
+        object.__setattr__(self, "layers", tuple(self.layers))
+        if self.hidden <= 0 or self.vocab <= 0 or not self.layers:
+            raise ValueError("a model needs a positive width and vocabulary and at least one layer")
+        lo = self.loop
+        if lo is not None and not (0 <= lo.start < lo.stop <= len(self.layers) and lo.times >= 1):
+            raise ValueError(f"loop {lo} does not fit {len(self.layers)} layers")
+
+    @property
+    def runs(self) -> Tuple[LayerRun, ...]:
+        lo, n = self.loop or LoopSpec(0, 1, 1), len(self.layers)
+        order = [(i, False) for i in range(lo.start)]
+        for t in range(lo.times):
+            order += [(i, t > 0 and i == lo.start) for i in range(lo.start, lo.stop)]
+        order += [(i, False) for i in range(lo.stop, n)]
+        return tuple(LayerRun(i, kv, inj) for kv, (i, inj) in enumerate(order))
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def n_attn_layers(self) -> int:
+        """KV caches a sequence holds: one per execution of an attention layer."""
+        return len(self.runs)
+
+    @property
+    def n_q_heads(self) -> int:
+        return max(b.mixer.heads for b in self.layers)
+
+    @property
+    def n_kv_heads(self) -> int:
+        return max(b.mixer.kv_heads for b in self.layers)
+
+    def n_params(self) -> int:
+        h = self.hidden
+        n = 2 * self.vocab * h + 2 * h
+        for b in self.layers:
+            a = b.mixer
+            n += h + h * (a.heads + a.kv_heads) * a.dim + h * (a.kv_heads + a.heads) * a.vdim + a.heads
+            if b.mlp is not None:
+                n += 2 * h * b.mlp.ff + 4
+        return n
+
+    # ---- config.json -----------------------------------------------------------------------
+    @classmethod
+    def from_json(cls, j: Dict, name: str = "zinutar", max_ctx: Optional[int] = None) -> "ZinutarConfig":
+        blocks = []
+        for i, l in enumerate(j["layers"]):
+            if l["type"] != "attention":
+                raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+            m, f = l["mixer"], l.get("mlp")
+            _fields(m, ("heads", "kv_heads", "dim", "vdim", "scale"), f"layer {i} mixer")
+            if f is not None:
+                _fields(f, ("ff", "kind"), f"layer {i} mlp")
+            blocks.append(BlockSpec(AttnSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]),
+                                             float(m["scale"])),
+                                    None if f is None else MlpSpec(int(f["ff"]), f["kind"])))
+        lo = j.get("loop")
+        return cls(name=name, hidden=int(j["width"]), vocab=int(j["vocab"]), layers=tuple(blocks),
+                   loop=None if lo is None else LoopSpec(int(lo["start"]), int(lo["stop"]), int(lo["times"])),
+                   rms_eps=float(j["norm"]["eps"]), **({} if max_ctx is None else {"max_ctx": max_ctx}))
+
+    def to_json(self) -> Dict:
+        out: Dict = {"architecture": self.architecture, "width": self.hidden, "vocab": self.vocab,
+                     "norm": {"eps": self.rms_eps}, "layers": []}
+        for b in self.layers:
+            a = b.mixer
+            out["layers"].append({"type": "attention",
+                                  "mixer": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim,
+                                            "scale": a.scale},
+                                  "mlp": None if b.mlp is None else {"kind": b.mlp.kind, "ff": b.mlp.ff}})
+        if self.loop is not None:
+            out["loop"] = {"start": self.loop.start, "stop": self.loop.stop, "times": self.loop.times}
+        return out
+
+
+def zinutar_uniform(name: str, *, hidden: int, vocab: int, n_layers: int, heads: int, kv_heads: int, dim: int, ff: int,
+                    vdim: Optional[int] = None, loop: Optional[LoopSpec] = None, **kw) -> ZinutarConfig:
+    """A Zinutar model whose layers all have one size, scores scaled by ``1 / sqrt(dim)``."""
+    blk = BlockSpec(AttnSpec(heads, kv_heads, dim, vdim or dim, dim ** -0.5), MlpSpec(ff))
+    return ZinutarConfig(name=name, hidden=hidden, vocab=vocab, layers=(blk,) * n_layers, loop=loop, **kw)
+
+
+def zinutar_tiny() -> ZinutarConfig:
+    """Smoke model: three layers of different sizes (one without a feed-forward), the first two looped
+    twice, byte vocabulary of 320."""
+    return ZinutarConfig(
+        name="zinutar-tiny", hidden=72, vocab=320, rms_eps=1e-5, max_ctx=4096, loop=LoopSpec(0, 2, 2),
+        layers=(BlockSpec(AttnSpec(6, 2, 24, 16, 0.3), MlpSpec(100)), BlockSpec(AttnSpec(4, 4, 16, 40, 0.2), None),
+                BlockSpec(AttnSpec(5, 1, 32, 32, 0.25), MlpSpec(136))))
+
+
+def zinutar_small() -> ZinutarConfig:
+    """Four layers of a 1B-class width; profiler captures and GPU engine tests."""
+    return zinutar_uniform("zinutar-small", hidden=2048, vocab=32768, n_layers=4, heads=16, kv_heads=4, dim=128, ff=8192,
+                           loop=LoopSpec(1, 3, 2))
+
+
+def zinutar_8b() -> ZinutarConfig:
+    """Layers of an 8B-class dense decoder (width 4096, 16 query / 4 kv heads x 256, ff 14336), 32 of them."""
+    return zinutar_uniform("zinutar-8b", hidden=4096, vocab=128256, n_layers=32, heads=16, kv_heads=4, dim=256, ff=14336)
+
+
+ARCHITECTURES = {ZinutarConfig.architecture: ZinutarConfig}
+
 _REGISTRY = {
+    "zinutar-tiny": zinutar_tiny, "zinutar-small": zinutar_small, "zinutar-8b": zinutar_8b,
     "qwen38-27b": qwen38_27b, "qwen36-27b": qwen36_27b, "tiny": tiny,
     "tiny-hybrid": tiny_hybrid, "small-gpu": small_gpu, "small-gpu-tp": small_gpu_tp,
     "tiny-agent": lambda: tiny(65536),
 }
 
 
-def get_config(name: str) -> ModelConfig:
-    try:
+def config_from_dir(path: str):
+    """The configuration a checkpoint directory describes in its ``config.json``: by ``architecture`` for designs
+    whose file spells every size out, else by the registry name that ``save_checkpoint`` wrote."""
+    with open(os.path.join(path, "config.json")) as f:
+        j = json.load(f)
+    arch = j.get("architecture")
+    if arch in ARCHITECTURES:
+        return ARCHITECTURES[arch].from_json(j, name=os.path.basename(os.path.normpath(path)))
+    if j.get("name") in _REGISTRY:
+        return _REGISTRY[j["name"]]()
+    raise ValueError(f"{path}/config.json names neither a known architecture ({sorted(ARCHITECTURES)}) nor a known model")
+
+
+def get_config(name: str):
+    """Configuration by registry name, or by a checkpoint directory that holds a ``config.json``."""
+    if name in _REGISTRY:
         return _REGISTRY[name]()
-    except KeyError:
-        raise ValueError(f"unknown model {name!r}; known: {sorted(_REGISTRY)}") from None
+    if os.path.exists(os.path.join(name, "config.json")):
+        return config_from_dir(name)
+    raise ValueError(f"unknown model {name!r}; known: {sorted(_REGISTRY)}, or a directory with a config.json")

@@ -131,6 +131,16 @@ class _Req:
 
 
 @dataclass
+class _Tick:
+    """What one forward of a tick leaves behind."""
+    logits: Optional[torch.Tensor] = None
+    argmax: Optional[List[int]] = None        # greedy tokens, when the captured tick computed them
+    taps: Optional[dict] = None
+    accept: Optional[List[int]] = None        # per sequence: drafts accepted, counted (and the state plane selected) on the device
+    sparse: bool = False                      # this tick's attention reads selected pages
+
+
+@dataclass
 class Result:
     rid: int
     tokens: List[int]
@@ -173,6 +183,7 @@ class Engine:
         self._waiting: Deque[_Req] = deque()
         self._running: List[_Req] = []
         self._reqs: Dict[int, _Req] = {}
+        self._fed: Dict[str, _Req] = {}       # open requests of feed()
         self._thread: Optional[threading.Thread] = None
         self._stop = threading.Event()
         self._wake = threading.Event()
@@ -387,6 +398,58 @@ class Engine:
                 self.last_tick_ms = dict(prep=(t1 - t0) * 1e3, run=(time.perf_counter() - t1) * 1e3)
             return True
 
+    # ---- given tokens: replay of a recorded trace -------------------------------------------------
+    def feed(self, entries: Sequence[Tuple[str, Sequence[int], Sequence[int]]],
+             end: Sequence[str] = ()) -> Optional[torch.Tensor]:
+        """One tick over tokens the caller gives instead of sampling them.  ``entries``: (key, next tokens of that
+        request, places among them whose logits are wanted).  A request is admitted with its first tokens and
+        keeps its pages and slot until its key is listed in ``end``; the tick is batched, paged and executed
+        (captured decode tick or eager forward) like any other.  Returns the wanted logits ``[n, vocab]`` (fp32)
+        in order, or None when none are wanted.  A bad entry raises before anything is run or allocated."""
+        with self._lock:
+            keys = [k for k, _, _ in entries]
+            if len(set(keys)) != len(keys):
+                raise ValueError("a request appears twice in one step")
+            for k in end:
+                if k not in self._fed and k not in keys:
+                    raise ValueError(f"request {k!r} is not open")
+            for key, tokens, want in entries:
+                n0 = len(self._fed[key].prompt) if key in self._fed else 0
+                if not len(tokens) or any(not 0 <= int(t) < self.model.cfg.vocab for t in tokens):
+                    raise ValueError(f"request {key!r}: no tokens, or a token outside the vocabulary")
+                if any(not 0 <= int(w) < len(tokens) for w in want):
+                    raise ValueError(f"request {key!r}: a wanted place outside its tokens")
+                if n0 + len(tokens) > self.model.cfg.max_ctx:
+                    raise ValueError(f"request {key!r} exceeds the model context")
+            plan, rows, off = [], [], 0
+            for key, tokens, want in entries:
+                r = self._fed.get(key)
+                if r is None:
+                    r = _Req(self._next, [], SamplingParams(), state=PREFILL, slot=self.states.alloc_slot())
+                    self._next += 1
+                    self._fed[key] = r
+                start, toks = r.n_computed, [int(t) for t in tokens]
+                if not self._grow(r, start + len(toks)):
+                    raise PoolExhausted("KV pool has no free block for the fed tokens")
+                r.state = DECODE if start and len(toks) == 1 else PREFILL
+                plan.append((r, toks, start))
+                rows += [off + int(w) for w in want]
+                off += len(toks)
+            logits = None
+            if plan:
+                logits = self._forward(plan, rows=rows).logits
+                if logits is not None and hasattr(self.ops, "full_logits"):
+                    logits = self.ops.full_logits(logits)
+                logits = logits if rows else None
+                self._check_device_error()
+                for r, toks, start in plan:
+                    r.prompt += toks
+                    r.n_computed = start + len(toks)
+                self.counters["ticks"] += 1
+            for k in end:
+                self._give_back(self._fed.pop(k))
+            return logits
+
     def _check_device_error(self) -> None:
         """A kernel's bounded wait that ran out (a TP peer that never pushed its partial rows, a
         copy that never landed) leaves a record in the device error word and returns: the tick then
@@ -503,57 +566,58 @@ class Engine:
             budget -= len(toks)
         return plan
 
-    def _run(self, plan) -> None:
-        verify = self.spec_width > 0 and any(r.state == DECODE and len(t) > 1 for r, t, _ in plan)
+    def _forward(self, plan, verify: bool = False, rows: Optional[List[int]] = None) -> "_Tick":
+        """Run the model on one tick's tokens, ``plan = [(request, tokens, start position)]``: a replay of the
+        captured decode or verify tick when one fits, else an eager forward.  ``rows``: token rows whose logits
+        are wanted (default: each sequence's last; every row of a verify tick)."""
         decode_only = all(r.state == DECODE for r, _, _ in plan)
         seqs = [dict(tokens=t, start=s, blocks=r.blocks, slot=r.slot,
                      keep=verify and r.state == DECODE) for r, t, s in plan]
-        logits = None
-        if self.graph is not None and decode_only and not verify and self.sparse is None:
-            logits = self.graph.run(seqs)
-            if logits is not None:
-                self.counters["graph_ticks"] += 1
-        taps = hidden = None
-        amax = None
-        vout = None
-        dev_accept = None       # per sequence: drafts accepted, counted (and the state plane selected) on the device
-        sparse_tick = False     # True when this tick's attention reads selected pages
-        if logits is None and self.vgraph is not None and decode_only and verify and self.sparse is None:
-            greedy = all(self._is_plain_greedy(r) for r, _, _ in plan)
-            vout = self.vgraph.run(seqs, need_logits=not greedy)
-        if vout is not None:
-            self.counters["graph_ticks"] += 1
-            logits, taps = vout.logits, vout.taps
-            amax = vout.argmax if greedy else None
-            dev_accept = vout.accept if greedy else None
-        elif logits is not None:
-            logits, amax = logits.logits, logits.argmax
-            if not all(self._is_plain_greedy(r) for r, _, _ in plan):
-                amax = None
-        else:
-            keep = max(len(t) for _, t, _ in plan) if verify else 0
-            batch = Batch.build(seqs, self.device, keep_steps=keep)
-            self.io_h2d += batch.h2d_bytes
-            if self.sparse is not None:
-                batch.sparse = self.sparse.for_batch(batch, [r.rid for r, _, _ in plan])
-                sparse_tick = batch.sparse is not None
-            aux = tuple(self.drafter.aux_layers) if self.drafter is not None else ()
-            res = self.model.forward(batch, self.ops, self.kv, self.states,
-                                     last_only=not verify, aux_layers=aux)
-            if aux:
-                logits, hidden, taps = res
-            else:
-                logits = res
-            if all(self._is_plain_greedy(r) for r, _, _ in plan):
-                amax = [int(v) for v in self.ops.argmax(logits).tolist()]  # one device sync per tick
-                self.io_d2h += 4 * len(amax)
+        out = _Tick()
+        if decode_only and self.sparse is None:
+            if self.graph is not None and not verify:
+                g = self.graph.run(seqs)
+                if g is not None:
+                    self.counters["graph_ticks"] += 1
+                    out.logits, out.argmax = (g.logits, g.argmax) if rows is None else (g.logits[rows], None)
+                    return out
+            if self.vgraph is not None and verify:
+                greedy = all(self._is_plain_greedy(r) for r, _, _ in plan)
+                v = self.vgraph.run(seqs, need_logits=not greedy)
+                if v is not None:
+                    self.counters["graph_ticks"] += 1
+                    out.logits, out.taps = v.logits, v.taps
+                    out.argmax = v.argmax if greedy else None
+                    out.accept = v.accept if greedy else None
+                    return out
+        keep = max(len(t) for _, t, _ in plan) if verify else 0
+        batch = Batch.build(seqs, self.device, keep_steps=keep)
+        self.io_h2d += batch.h2d_bytes
+        if self.sparse is not None:
+            batch.sparse = self.sparse.for_batch(batch, [r.rid for r, _, _ in plan])
+            out.sparse = batch.sparse is not None
+        aux = tuple(self.drafter.aux_layers) if self.drafter is not None else ()
+        res = self.model.forward(batch, self.ops, self.kv, self.states, last_only=not verify, aux_layers=aux,
+                                 rows=rows)
+        out.logits, _, out.taps = res if aux else (res, None, None)
+        return out
+
+    def _run(self, plan) -> None:
+        verify = self.spec_width > 0 and any(r.state == DECODE and len(t) > 1 for r, t, _ in plan)
+        tick = self._forward(plan, verify)
+        logits, taps, amax, dev_accept = tick.logits, tick.taps, tick.argmax, tick.accept
+        if not all(self._is_plain_greedy(r) for r, _, _ in plan):
+            amax = None
+        elif amax is None:
+            amax = [int(v) for v in self.ops.argmax(logits).tolist()]  # one device sync per tick
+            self.io_d2h += 4 * len(amax)
         if amax is None and hasattr(self.ops, "full_logits"):
             logits = self.ops.full_logits(logits)   # sampling needs every vocab shard
         self._presampled = self._presample(plan, logits, verify) if amax is None else {}
         kinds = {r.state for r, _, _ in plan}
         key = "mixed_ticks" if len(kinds) > 1 else ("decode_ticks" if DECODE in kinds else "prefill_ticks")
         self.counters[key] += 1
-        self.counters["sparse_ticks" if sparse_tick else "dense_ticks"] += 1
+        self.counters["sparse_ticks" if tick.sparse else "dense_ticks"] += 1
         if verify:
             self.counters["verify_ticks"] += 1
         tok_off = 0
@@ -726,16 +790,7 @@ class Engine:
         the client sees no difference but the delay."""
         self._events += 1
         self._running.remove(r)
-        for b in r.blocks:
-            self.kv.release(b)
-        r.blocks = []
-        if r.slot > 0:
-            self.states.release(r.slot)
-            r.slot = -1
-        if self.drafter is not None and hasattr(self.drafter, "release"):
-            self.drafter.release(r.rid)
-        if self.sparse is not None:
-            self.sparse.release(r.rid)
+        self._give_back(r)
         r.resumed = len(r.out) if r.out else 0
         r.n_computed, r.prefix_tokens, r.drafts, r.state = 0, 0, [], WAITING
         self._waiting.appendleft(r)
@@ -746,6 +801,10 @@ class Engine:
         r.finish_reason = reason
         r.state = DONE
         r.t_done = time.monotonic()
+        self._give_back(r)
+
+    def _give_back(self, r: _Req) -> None:
+        """Return a request's pages, state slot and side tables to their pools."""
         for b in r.blocks:
             self.kv.release(b)
         r.blocks = []

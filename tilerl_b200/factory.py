@@ -4,7 +4,8 @@
 a checkpoint directory or from a seeded random initialisation.  Random weights
 are generated tensor by tensor directly on the target device and quantised
 there, so the 27B never exists in full precision anywhere (its fp32 master
-would be 108 GB).  ``fit_blocks`` derives the KV page count from free device
+would be 108 GB).  A Zinutar configuration goes to :class:`~tilerl_b200.models.zinutar.ZinutarModel` and the
+packed KV pool, every other one to the hybrid model.  ``fit_blocks`` derives the KV page count from free device
 memory; ``build_engine`` creates pools, prefix store, CUDA-graph runner and the
 engine.
 
@@ -13,16 +14,18 @@ Parity: reference ``src/tilerl/build.py`` -- ``build_model:76``, ``_shard:46``,
 """
 from __future__ import annotations
 
+import os
 import zlib
 from typing import Dict, Optional
 
 import torch
 
-from .config import ModelConfig, get_config
+from .config import ModelConfig, ZinutarConfig, get_config
 from .engine import Engine, StepLimits
 from .formats import NVFP4Tensor
-from .kv import GdnStatePool, NoPrefixStore, PagedKvPool, PrefixStore
+from .kv import GdnStatePool, NoPrefixStore, PrefixStore, kv_pages, make_kv_pool
 from .models.hybrid import HybridModel, linear_names, param_shapes, quantize_weight
+from .models.zinutar import ZinutarModel
 from .ops.backend import RefOps
 from .ops.ref import KV_BLOCK
 
@@ -102,11 +105,23 @@ def materialize(model: HybridModel, ops) -> None:
 
 def build_model(model: str | ModelConfig, device="cpu", *, seed: int = 0, checkpoint: Optional[str] = None,
                 tp_rank: int = 0, tp: int = 1, ops=None, keep_master: bool = False,
-                master_only: bool = False) -> HybridModel:
+                master_only: bool = False, dtype: Optional[torch.dtype] = None):
+    """``model``: a configuration, its registry name, or a checkpoint directory (which is then also where the
+    weights come from).  ``dtype``: compute dtype of designs that run in more than one."""
     cfg = get_config(model) if isinstance(model, str) else model
+    if isinstance(model, str) and checkpoint is None and os.path.isdir(model):
+        checkpoint = model
+    if isinstance(cfg, ZinutarConfig):
+        if tp > 1 or keep_master or master_only:
+            raise ValueError("Zinutar models are served on one GPU per process; tensor parallelism and training are not built")
+        if checkpoint is None:
+            on_gpu = torch.device(device).type == "cuda"
+            return ZinutarModel.build_random(cfg, seed, device, act_dtype=dtype or (torch.bfloat16 if on_gpu else torch.float32))
+    elif dtype is not None and dtype != (torch.bfloat16 if torch.device(device).type == "cuda" else torch.float32):
+        raise ValueError(f"{cfg.name} does not run in {dtype} on {device}")
     if checkpoint:
         from .checkpoint import load_checkpoint
-        return load_checkpoint(cfg, checkpoint, device=device, tp_rank=tp_rank, tp=tp, keep_master=keep_master)
+        return load_checkpoint(cfg, checkpoint, device=device, tp_rank=tp_rank, tp=tp, keep_master=keep_master, dtype=dtype)
     m = build_random_streaming(cfg, device, seed, tp_rank, tp, ops, keep_master, master_only)
     if ops is not None and not master_only:
         materialize(m, ops)
@@ -116,6 +131,9 @@ def build_model(model: str | ModelConfig, device="cpu", *, seed: int = 0, checkp
 def fit_blocks(cfg: ModelConfig, free_bytes: int, slots: int, *, planes: int = 1, tp: int = 1,
                pool_fraction: float = 2.0 / 3.0, max_blocks: int = 1 << 20, kv_fp8: bool = False) -> int:
     """KV pages that fit in ``pool_fraction`` of what is left after the GDN state slots."""
+    if isinstance(cfg, ZinutarConfig):
+        per_block = sum(p.n_kv * p.nbytes for p in kv_pages(cfg, 2))
+        return int(max(2, min(max_blocks, free_bytes * pool_fraction // per_block)))
     from .parallel.mesh import tp_dims
     d = tp_dims(cfg, tp)
     gd = cfg.gdn_head_dim
@@ -128,6 +146,7 @@ def fit_blocks(cfg: ModelConfig, free_bytes: int, slots: int, *, planes: int = 1
 
 
 def make_ops(device, tp_comm=None):
+    """The op backend of a device."""
     device = torch.device(device)
     if device.type == "cuda":
         from .ops.cuda import CudaOps
@@ -160,8 +179,10 @@ def build_engine(model: HybridModel, ops=None, *, device=None, blocks: Optional[
     on_gpu = device.type == "cuda"
     if kv_fp8 and sparse is not None and on_gpu:
         raise ValueError("sparse page selection reads a bf16 KV pool on the device: use --kv-format bf16 with --sparse-k")
-    kv = PagedKvPool(cfg, blocks, device, dtype=torch.bfloat16 if on_gpu else torch.float32, n_kv_heads=d.n_kv,
-                     fp8=kv_fp8)
+    kv = make_kv_pool(cfg, blocks, device, getattr(model, "act_dtype", torch.bfloat16 if on_gpu else torch.float32),
+                      n_kv_heads=d.n_kv, fp8=kv_fp8)
+    if sparse is not None and isinstance(cfg, ZinutarConfig):
+        raise ValueError("sparse page selection is not built for the packed KV pool")
     st = GdnStatePool(cfg, slots + 1, device, planes=planes,
                       ring_dtype=torch.bfloat16 if on_gpu else torch.float32,
                       n_v_heads=d.gdn_nv or None, n_k_heads=d.gdn_nk or None)

@@ -15,7 +15,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Dict, List, Optional
 
-from .config import ATTN, ModelConfig
+from .config import ATTN, ModelConfig, ZinutarConfig
 from .formats import FORMATS, nbytes
 from .parallel.mesh import tp_dims
 
@@ -51,8 +51,33 @@ def _linear(name: str, count: int, m: int, n: int, k: int, fmt: str, comm: float
     return Row(name, count, w + act, 2.0 * m * n * k, comm)
 
 
+def _zinutar_rows(cfg: ZinutarConfig, m: int, pairs: float, kv_read: float, head_rows_m: int) -> List[Row]:
+    """One forward of ``m`` tokens: ``pairs`` (query token, key) pairs, ``kv_read`` key tokens whose pages are read."""
+    from .kv import kv_pages
+    from .zinutar_layout import BlockLayout, head_rows, stream_width
+    w = stream_width(cfg)
+    rows = [Row("embedding + norm", 1, m * w * (2 + 4), 0)]
+    for i in range(cfg.n_layers):
+        runs = [r for r in cfg.runs if r.layer == i]
+        if not runs:
+            continue
+        l, pg = BlockLayout.of(cfg.layers[i]), kv_pages(cfg, 2)[runs[0].kv]
+        per_token = pg.n_kv * pg.nbytes / 16
+        n = len(runs)
+        rows += [Row(f"L{i} in (norm fused)", n, l.n_in * w * 2 + m * (w * 4 + l.n_in * 2), 2.0 * m * l.n_in * w),
+                 Row(f"L{i} attn.kv write + polynorm", n, m * (per_token * 2 + 4.0 * l.ff), 0),
+                 Row(f"L{i} attn.sigmoid", n, kv_read * per_token + m * l.heads * (l.dk + l.dv) * 2.0,
+                     2.0 * pairs * l.heads * (l.dk + l.dv)),
+                 Row(f"L{i} out (+stream)", n, l.n_out * w * 2 + m * (l.n_out * 2 + w * 8), 2.0 * m * l.n_out * w)]
+    rows.append(Row("lm_head", 1, head_rows(cfg) * w * 2 + head_rows_m * (w * 4 + head_rows(cfg) * 4), 2.0 * head_rows_m * head_rows(cfg) * w))
+    return rows
+
+
 def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
     """One decode (or verify) tick on one TP rank."""
+    if isinstance(cfg, ZinutarConfig):
+        b, c = s.batch, s.ctx
+        return _zinutar_rows(cfg, b * s.width, b * s.width * c, b * c, b * s.width)
     d = tp_dims(cfg, s.tp)
     m = s.batch * s.width
     h = cfg.hidden
@@ -87,6 +112,8 @@ def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
 def prefill_rows(cfg: ModelConfig, tokens: int, tp: int = 1, terms: int = 2) -> List[Row]:
     """One prefill of ``tokens`` tokens (one sequence) on one TP rank; ``terms`` NVFP4
     activation terms per token multiply the tensor-core work."""
+    if isinstance(cfg, ZinutarConfig):
+        return _zinutar_rows(cfg, tokens, tokens * (tokens + 1) / 2, tokens, 1)
     d = tp_dims(cfg, tp)
     h, m = cfg.hidden, tokens
     fmt = _lin_format(cfg)

@@ -3,6 +3,8 @@
 * :class:`PagedKvPool` -- ``k/v [attn_layers, blocks, hkv, 16, D]`` (bf16, or e4m3
   with one fp32 scale per (block, head, token)); free list + refcounts; block 0
   is a reserved pad page that CUDA-graph padding rows write into.
+* :class:`PackedKvPool` -- the same allocator over pages that hold K, its norm factors and V of one head
+  back to back, with per-layer head counts and widths (:class:`KvPage`; no counterpart in the reference).
 * :class:`GdnStatePool` -- ``states [slots, gdn_layers, planes, nv, dk, dv]`` fp32
   and a raw-qkv ring ``[slots, gdn_layers, R, C]`` indexed by ``position % R``.
   ``planes > 1`` keeps the state after each token of a speculative-verify tick;
@@ -27,7 +29,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from .config import ModelConfig
+from .config import ModelConfig, ZinutarConfig
 from .ops.ref import KV_BLOCK
 
 RING = 16  # conv ring rows; >= spec width + conv taps
@@ -69,6 +71,9 @@ class PagedKvPool:
         if fp8:
             self.k_scale = torch.ones(shape[:-1], dtype=torch.float32, device=device)
             self.v_scale = torch.ones(shape[:-1], dtype=torch.float32, device=device)
+        self._init_allocator()
+
+    def _init_allocator(self) -> None:
         self._pager = _native_pager(self.num_blocks)     # C++ free list + refcounts when the library is built
         if self._pager is None:
             self._ref = [0] * self.num_blocks
@@ -147,6 +152,11 @@ class PagedKvPool:
         return self.k[attn_idx], self.v[attn_idx]
 
     # ---- host tier hooks -------------------------------------------------------
+    @property
+    def page_shape(self) -> List[int]:
+        """Shape of each of the two tensors of :meth:`read_block`."""
+        return list(self.k[:, 0].shape)
+
     def read_block(self, b: int) -> Tuple[torch.Tensor, torch.Tensor]:
         if self.fp8:     # tiers move the dequantised page; the scales are re-derived on the way back
             return (self.k[:, b].float() * self.k_scale[:, b].unsqueeze(-1),
@@ -163,6 +173,121 @@ class PagedKvPool:
             return
         self.k[:, b].copy_(k)
         self.v[:, b].copy_(v)
+
+
+@dataclass(frozen=True)
+class KvPage:
+    """Byte layout of one page of one KV head in a :class:`PackedKvPool`: 16 K rows, the 16 fp32 reciprocal
+    root mean squares of those rows, 16 V rows, back to back, so that one bulk copy brings a page whole.
+
+    Rows are made of 16-byte chunks and row ``r`` is rotated by ``r``: chunk ``c`` sits at chunk
+    ``(c + r) % chunks`` of its row.  Eight rows read at one chunk index then fall into different shared-memory
+    banks.  Widths are padded to 16 elements; the padding holds zeros."""
+    n_kv: int
+    dim: int
+    vdim: int
+    itemsize: int
+
+    @staticmethod
+    def pad(n: int) -> int:
+        return (n + 15) // 16 * 16
+
+    @property
+    def k_chunks(self) -> int:
+        return self.pad(self.dim) * self.itemsize // 16
+
+    @property
+    def v_chunks(self) -> int:
+        return self.pad(self.vdim) * self.itemsize // 16
+
+    @property
+    def rms_offset(self) -> int:
+        return KV_BLOCK * self.k_chunks * 16
+
+    @property
+    def v_offset(self) -> int:
+        return self.rms_offset + KV_BLOCK * 4
+
+    @property
+    def nbytes(self) -> int:
+        return self.v_offset + KV_BLOCK * self.v_chunks * 16
+
+    def _index(self, width: int, chunks: int, base: int) -> torch.Tensor:
+        """Element index inside the page of ``[16 rows, width]`` values that start at byte ``base``."""
+        per = 16 // self.itemsize
+        r = torch.arange(KV_BLOCK)[:, None]
+        d = torch.arange(width)[None, :]
+        return base // self.itemsize + (r * chunks + (d // per + r) % chunks) * per + d % per
+
+    def k_index(self) -> torch.Tensor:
+        return self._index(self.pad(self.dim), self.k_chunks, 0)
+
+    def v_index(self) -> torch.Tensor:
+        return self._index(self.pad(self.vdim), self.v_chunks, self.v_offset)
+
+    def rms_index(self) -> torch.Tensor:
+        """Index of the 16 reciprocal root mean squares in the page seen as fp32."""
+        return self.rms_offset // 4 + torch.arange(KV_BLOCK)
+
+
+def kv_pages(cfg, itemsize: int) -> Tuple[KvPage, ...]:
+    """Page layout of every KV cache of a design whose layers differ in size (one per layer execution)."""
+    return tuple(KvPage(a.kv_heads, a.dim, a.vdim, itemsize)
+                 for a in (cfg.layers[run.layer].mixer for run in cfg.runs))
+
+
+class PackedKvPool(PagedKvPool):
+    """Paged pool whose caches may differ in head count and widths: cache ``i`` is a contiguous
+    ``[blocks, kv heads, page bytes]`` slice of one byte buffer (layout: :class:`KvPage`).  K is stored as
+    projected, with the norm's reciprocal root mean square beside it.  Allocator, reference counts and tier
+    hooks are the parent's."""
+    fp8 = False
+
+    def __init__(self, cfg, num_blocks: int, device="cpu", dtype=torch.bfloat16):
+        self.cfg, self.num_blocks, self.dtype = cfg, int(num_blocks), dtype
+        self.pages = kv_pages(cfg, torch.empty(0, dtype=dtype).element_size())
+        self.hkv = max(p.n_kv for p in self.pages)
+        sizes = [self.num_blocks * p.n_kv * p.nbytes for p in self.pages]
+        self.k = torch.zeros(sum(sizes), dtype=torch.uint8, device=device)
+        self.v = self.k[:0]                  # K and V share the pages
+        offs = [0]
+        for n in sizes:
+            offs.append(offs[-1] + n)
+        self._layers = [self.k[offs[i]:offs[i + 1]].view(self.num_blocks, p.n_kv, p.nbytes)
+                        for i, p in enumerate(self.pages)]
+        self._init_allocator()
+
+    def block_bytes(self) -> int:
+        return sum(p.n_kv * p.nbytes for p in self.pages)
+
+    def layer(self, attn_idx: int) -> torch.Tensor:
+        return self._layers[attn_idx]
+
+    @property
+    def page_shape(self) -> List[int]:
+        return [self.block_bytes() // 2]
+
+    def read_block(self, b: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        """The block's bytes over all caches, in two equal halves (the tiers move pairs of tensors)."""
+        flat = torch.cat([l[b].reshape(-1) for l in self._layers])
+        return flat.view(2, -1)[0].clone(), flat.view(2, -1)[1].clone()
+
+    def write_block(self, b: int, k: torch.Tensor, v: torch.Tensor) -> None:
+        flat, o = torch.cat([k.reshape(-1), v.reshape(-1)]), 0
+        for l in self._layers:
+            n = l[b].numel()
+            l[b].copy_(flat[o:o + n].view_as(l[b]))
+            o += n
+
+
+def make_kv_pool(cfg, num_blocks: int, device="cpu", dtype=torch.bfloat16, *, fp8: bool = False,
+                 n_kv_heads: Optional[int] = None) -> PagedKvPool:
+    """The pool a configuration's layers keep K / V in."""
+    if isinstance(cfg, ZinutarConfig):
+        if fp8:
+            raise ValueError("the packed KV pool holds bf16 or fp32 pages, not fp8")
+        return PackedKvPool(cfg, num_blocks, device, dtype)
+    return PagedKvPool(cfg, num_blocks, device, dtype=dtype, n_kv_heads=n_kv_heads, fp8=fp8)
 
 
 class GdnStatePool:

@@ -226,7 +226,7 @@ class KvBootStore:
                 torch.save([t.cpu() for t in e.snapshot], os.path.join(self.root, snap_fn))
             entries.append({"tokens": list(e.tokens), "pages": pages, "snapshot": snap_fn})
         man = {"fingerprint": weights_fingerprint(engine.model), "entries": entries,
-               "page_shape": list(pool.k[:, 0].shape), "dtype": str(pool.k.dtype)}
+               "page_shape": list(pool.page_shape), "dtype": str(pool.k.dtype)}
         with open(os.path.join(self.root, "manifest.json.tmp"), "w") as f:
             json.dump(man, f)
         os.replace(os.path.join(self.root, "manifest.json.tmp"), os.path.join(self.root, "manifest.json"))

@@ -17,7 +17,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
-from .config import ModelConfig
+from .config import ModelConfig, ZinutarConfig
 from .formats import nbytes, weight_specs
 from .parallel.mesh import is_sharded, tp_dims
 
@@ -50,6 +50,9 @@ def weight_bytes(cfg: ModelConfig, tp: int = 1, tiled_copy: bool = True) -> int:
 
 
 def kv_block_bytes(cfg: ModelConfig, tp: int = 1, fp8: bool = False) -> int:
+    if isinstance(cfg, ZinutarConfig):
+        from .kv import kv_pages
+        return sum(p.n_kv * p.nbytes for p in kv_pages(cfg, 2))
     d = tp_dims(cfg, tp)
     per = d.n_kv * 16 * cfg.head_dim * (1 if fp8 else 2) * 2
     if fp8:
@@ -58,6 +61,8 @@ def kv_block_bytes(cfg: ModelConfig, tp: int = 1, fp8: bool = False) -> int:
 
 
 def state_slot_bytes(cfg: ModelConfig, tp: int = 1, planes: int = 1) -> int:
+    if not cfg.n_gdn_layers:
+        return 0
     d = tp_dims(cfg, tp)
     gd = cfg.gdn_head_dim
     return cfg.n_gdn_layers * (planes * d.gdn_nv * gd * gd * 4 + 16 * d.gdn_conv_dim * 2)
@@ -88,6 +93,19 @@ def indexer_bytes(cfg: ModelConfig, *, heads: int = 4, dim: int = 128, tp: int =
     return max(1, cfg.n_attn_layers) * (d.n_q + d.n_kv) * cfg.head_dim * heads * dim * itemsize
 
 
+def workspace_bytes(cfg: ModelConfig, tokens: int, tp: int = 1) -> int:
+    """Activation buffers of a tick of ``tokens`` tokens and the logits of 64 rows."""
+    if isinstance(cfg, ZinutarConfig):
+        from .zinutar_layout import BlockLayout, head_rows, stream_width
+        ls = [BlockLayout.of(b) for b in cfg.layers]
+        # fp32 stream and embedding output, bf16 normed row, fused projection rows, block middle
+        per = stream_width(cfg) * (4 + 4 + 2) + 2 * max(l.n_in for l in ls) + 2 * max(l.n_out for l in ls)
+        return tokens * per + head_rows(cfg) * 4 * 64
+    d = tp_dims(cfg, tp)
+    widest = max(d.qkv_rows, d.gdn_in_rows, 2 * d.ffn)
+    return tokens * (widest * 2 + cfg.hidden * 8 + d.ffn * 2) + d.vocab_local * 4 * 64
+
+
 def plan(cfg: ModelConfig, *, device_bytes: int = B200_BYTES, tp: int = 1, slots: int = 64, planes: int = 1,
          max_batched_tokens: int = 8192, reserve_bytes: int = 2 * GIB, pool_fraction: float = 2 / 3,
          state_fraction: float = 1 / 4, kv_fp8: bool = False, blocks: Optional[int] = None,
@@ -107,9 +125,7 @@ def plan(cfg: ModelConfig, *, device_bytes: int = B200_BYTES, tp: int = 1, slots
     if host_pages:
         p.notes.append(f"host KV tier: {host_pages * kv_block_bytes(cfg, tp, kv_fp8) / GIB:.2f} GiB of pinned host memory "
                        f"for {host_pages:,} pages")
-    d = tp_dims(cfg, tp)
-    widest = max(d.qkv_rows, d.gdn_in_rows, 2 * d.ffn)
-    p.rows["workspace"] = max_batched_tokens * (widest * 2 + cfg.hidden * 8 + d.ffn * 2) + d.vocab_local * 4 * 64
+    p.rows["workspace"] = workspace_bytes(cfg, max_batched_tokens, tp)
     p.rows["reserve"] = reserve_bytes
     left = device_bytes - p.total
     if left <= 0:
@@ -151,6 +167,8 @@ def train_plan(cfg: ModelConfig, *, mode: str = "lora", rank: int = 16, zero: in
     matrices, Adafactor for the vectors)."""
     if optimizer not in ("adamw", "adafactor", "iso"):
         raise ValueError(f"unknown optimizer {optimizer!r}")
+    if isinstance(cfg, ZinutarConfig):
+        raise ValueError("Zinutar models are served, not trained")
     n = cfg.n_params()
     rows: Dict[str, int] = {}
     if mode == "lora":

@@ -188,8 +188,9 @@ class HybridModel:
 
     # ---- serving forward ------------------------------------------------------------------
     def forward(self, batch, ops, kv_pool, state_pool, *, last_only: bool = True,
-                aux_layers: Sequence[int] = (), return_hidden: bool = False):
-        """Returns logits ``[B or T, vocab]`` (fp32).  ``aux_layers``: also return the
+                aux_layers: Sequence[int] = (), return_hidden: bool = False, rows=None):
+        """Returns logits ``[B or T, vocab]`` (fp32), or those of the token rows listed in ``rows`` (None when the
+        list is empty).  ``aux_layers``: also return the
         residual stream after those layers (taps for the block drafter)."""
         cfg, P, d = self.cfg, self.params, self.dims
         eps = cfg.rms_eps
@@ -218,9 +219,12 @@ class HybridModel:
                 settle()
                 taps[i] = x.clone()  # the residual stream is updated in place
         settle()
-        xs = x[batch.last_idx.long()] if last_only else x
+        if rows is not None:
+            xs = x[rows] if len(rows) else None
+        else:
+            xs = x[batch.last_idx.long()] if last_only else x
         head = P["embed"] if cfg.tie_embeddings else P["lm_head"]
-        logits = ops.lm_head(xs, P["final_norm"], head, eps)[..., :cfg.vocab]
+        logits = None if xs is None else ops.lm_head(xs, P["final_norm"], head, eps)[..., :cfg.vocab]
         if aux_layers or return_hidden:
             return logits, x, taps
         return logits

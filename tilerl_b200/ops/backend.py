@@ -96,6 +96,46 @@ class RefOps:
         out = ref.paged_attention(q, gate, kc, vc, table, batch.seq_ids, pos, scale)
         return out.to(self.act_dtype)
 
+    # -- fp32 stream with parallel blocks (models/zinutar.py) --------------------------------------
+    def embed_norm(self, table, norm_w, ids, eps, n, keep):
+        e = ref.embedding(table, ids)
+        x = e * ref.rms_factor(e, n, eps)[:, None] * norm_w
+        return x, (x.clone() if keep else None)
+
+    def stream_add(self, x, y):
+        x += y
+
+    def stream_linear(self, x, norm_w, w, eps, n):
+        h = (x * ref.rms_factor(x, n, eps)[:, None] * norm_w).to(self.act_dtype)
+        return ref.linear(h, w).to(self.act_dtype)
+
+    def block_mid(self, proj, act, l, batch, pool, kv_idx, eps):
+        """K / V of the tick's tokens into the pool; returns the input of the block's output projection with
+        the feed-forward columns filled in."""
+        t = proj.shape[0]
+        k = proj[:, l.k0:l.v0].view(t, l.kv_heads, l.dk)
+        v = proj[:, l.v0:l.up0].view(t, l.kv_heads, l.dv)
+        ref.packed_kv_write(pool.layer(kv_idx), pool.pages[kv_idx], k.to(pool.dtype), v.to(pool.dtype), batch.slot_mapping, eps)
+        mid = torch.zeros(t, l.n_out, dtype=self.act_dtype, device=proj.device)
+        if l.ff:
+            mid[:, l.attn_cols:l.attn_cols + l.ff] = ref.polynorm(proj[:, l.up0:l.up0 + l.ff], act, eps).to(self.act_dtype)
+        return mid
+
+    def sigmoid_attention(self, proj, mid, bias, l, batch, pool, kv_idx, eps):
+        q = proj[:, :l.k0].view(-1, l.heads, l.dk).float()
+        q = q * ref.rms_factor(q, l.dim, eps)[..., None]
+        for i in range(proj.shape[0]):
+            k, v = ref.packed_kv_gather(pool.layer(kv_idx), pool.pages[kv_idx], pool.dtype,
+                                        batch.block_table[int(batch.seq_ids[i])], int(batch.positions[i]) + 1)
+            mid[i, :l.attn_cols] = ref.sigmoid_attention(q[i], k, v, bias, l.scale).reshape(-1).to(self.act_dtype)
+
+    def stream_accumulate(self, a, w, x):
+        x += ref.linear(a, w)
+
+    def stream_head(self, x, norm_w, w, eps, n):
+        h = (x * ref.rms_factor(x, n, eps)[:, None] * norm_w).to(self.act_dtype)
+        return ref.linear(h, w)
+
     def gdn(self, inp, lp, batch, spool, gdn_idx, cfg, nk, nv):
         d = cfg.gdn_head_dim
         out = torch.zeros(inp.shape[0], nv * d, dtype=torch.float32, device=inp.device)

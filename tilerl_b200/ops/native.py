@@ -74,12 +74,29 @@ _SIGS = {
     "trl_quant_nvfp4": [P, I, L, L, P, P, P, P, I, P],
     "trl_dequant_nvfp4": [P, P, P, P, L, L, P],
     "trl_add": [P, P, P, L, P],
+    # fp32 stream, parallel blocks, sigmoid attention (csrc/stream.cu, linear_rows.cu, attn_sigmoid.cu)
+    "trl_embed_norm": [P, P, P, P, P, I, I, I, I, F, I, P],
+    "trl_stream_norm": [P, P, P, I, I, I, F, I, P],
+    "trl_stream_add": [P, P, L, P],
+    "trl_block_mid": [P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P],
+    "trl_linear_rows": [P, I, P, P, F, I, P, I, I, I, I, I, P],
+    "trl_sigmoid_attn_rows": [I, I],
+    "trl_sigmoid_attn": [P, I, P, I, P, I, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P],
+    "trl_sigmoid_attn_f32": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P],
     "trl_decode_advance": [P, P, P, P, P, P, I, I, P, I, P, P],
 }
 
 
 _RESTYPE = {"trl_set_pdl": None, "trl_gdn_set_wy": None, "trl_gemv2_set_trigger": None, "trl_gdn_set_mma": None, "trl_pager_create": c_void_p, "trl_pager_destroy": None,
             "trl_batch_ints": c_longlong, "trl_batch_fill": c_longlong}
+
+
+def use(path: str) -> None:
+    """Load the library from ``path`` instead (before anything else of it is used)."""
+    global _PATH
+    if _LIB is not None and path != _PATH:
+        raise RuntimeError("the kernel library is already loaded")
+    _PATH = path
 
 
 def loadable() -> bool:

@@ -202,6 +202,58 @@ def dense_attention(q, k, v, gate, scale: float, q_pos=None, k_pos=None):
     return o.reshape(b, t, hq * d)
 
 
+# ---- sigmoid-weighted attention over packed pages ------------------------------------------------
+def rms_factor(x, n: int, eps: float):
+    """Reciprocal root mean square over the last dim, of which the first ``n`` values count (the rest are
+    padding zeros)."""
+    return torch.rsqrt(_f(x).pow(2).sum(-1) / n + eps)
+
+
+def packed_kv_write(cache, page, k, v, slot_mapping, eps: float):
+    """Write rows ``k [T, hkv, dk]`` / ``v [T, hkv, dv]`` (padded widths) into a packed cache
+    ``[blocks, hkv, page bytes]``: K unnormalised with its reciprocal root mean square beside it."""
+    el = cache.view(k.dtype)
+    f32 = cache.view(torch.float32)
+    ki, vi, ri = page.k_index().to(k.device), page.v_index().to(k.device), page.rms_index().to(k.device)
+    fac = rms_factor(k, page.dim, eps)
+    for t in range(k.shape[0]):
+        s = int(slot_mapping[t])
+        if s < 0:
+            continue
+        b, o = divmod(s, KV_BLOCK)
+        el[b][:, ki[o]] = k[t]
+        el[b][:, vi[o]] = v[t]
+        f32[b, :, ri[o]] = fac[t]
+
+
+def packed_kv_gather(cache, page, dtype, block_row, length: int):
+    """``(normalised K [length, hkv, dk], V [length, hkv, dv])`` of one sequence, fp32."""
+    nb = (length + KV_BLOCK - 1) // KV_BLOCK
+    pages = cache[block_row[:nb].long()]                              # [nb, hkv, bytes]
+    el, dev = pages.view(dtype), cache.device
+    k = _f(el[..., page.k_index().to(dev)])                           # [nb, hkv, 16, dk]
+    v = _f(el[..., page.v_index().to(dev)])
+    r = pages.view(torch.float32)[..., page.rms_index().to(dev)]      # [nb, hkv, 16]
+    flat = lambda a: a.transpose(1, 2).reshape(nb * KV_BLOCK, a.shape[1], *a.shape[3:])[:length]
+    return flat(k) * flat(r)[..., None], flat(v)
+
+
+def sigmoid_attention(q, k, v, bias, scale: float):
+    """One query token over the keys it sees: ``q [hq, dk]`` and ``k [n, hkv, dk]`` already normalised,
+    ``v [n, hkv, dv]``; weights ``sigmoid(q.k * scale + bias[head])``, summed without normalisation."""
+    hq, hkv = q.shape[0], k.shape[1]
+    s = torch.einsum("hgd,nhd->hgn", q.view(hkv, hq // hkv, -1), k) * scale + _f(bias).view(hkv, -1)[..., None]
+    return torch.einsum("hgn,nhd->hgd", torch.sigmoid(s), v).reshape(hq, -1)
+
+
+def polynorm(z, act, eps: float):
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` with ``N`` the RMS norm over the last dim, ``act = (a, b, c, e)``."""
+    z = _f(z)
+    n = lambda p: p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)
+    a, b, c, e = (float(x) for x in act)
+    return a * n(z) + b * n(z * z) + c * n(z * z * z) + e
+
+
 # ---- Quest-style page index (sparse KV) ---------------------------------------------------
 def page_bounds(kcache_block):
     """Per (kv head) element-wise min and max over a page's tokens: ``[hkv, 2, D]``."""
