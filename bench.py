@@ -190,7 +190,15 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN)
     ap.add_argument("--gen", type=int, default=GEN_LEN)
     ap.add_argument("--no-control", action="store_true", help="skip the unfused same-box control at N > 1")
-    args = ap.parse_args()
+    ap.add_argument("--design", default=None, choices=["zinutar"],
+                    help="measure another design beside the closest hybrid form at equal size instead (tilerl_b200/suites/zinutar.py; "
+                         "its own flags follow)")
+    args, rest = ap.parse_known_args()
+    if args.design == "zinutar":
+        from tilerl_b200.suites.zinutar import main as design_main
+        return design_main(rest)
+    if rest:
+        ap.error(f"unrecognized arguments: {' '.join(rest)}")
     if args.impl == "reference":
         return reference_arm(args)
     if args.impl not in ("ours", "unfused"):

@@ -22,9 +22,10 @@
 
 namespace {
 
-constexpr int KVB = 16, TILE = 64, TPAGES = TILE / KVB;
+constexpr int KVB = 16, TILE = 64, TPAGES = TILE / KVB, RMS_BYTES = 128;
 constexpr long long SA_WAIT_CYCLES = 4000000000LL;
 constexpr int SA_SMEM = 216 * 1024;
+constexpr float LOG2E = 1.4426950408889634f;
 
 struct SigArgs {
   const bf16* q;                       // fused projection rows, query heads first
@@ -79,22 +80,29 @@ __device__ __forceinline__ uint32_t sa_try_wait(uint32_t bar, uint32_t parity) {
                : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
   return ok;
 }
-// chunk c of a row rotated by `rot` (= row % n): both below n
-__device__ __forceinline__ int rotate(int c, int rot, int n) {
-  const int x = c + rot;
-  return x >= n ? x - n : x;
+// where chunk c of row r sits in a packed page row of n chunks
+__device__ __forceinline__ int page_chunk(int c, int r, int n) { return n % 8 == 0 ? c ^ (r & 7) : (c + r) % n; }
+// sigmoid of a score given as t = -log2(e) x: 1 / (1 + 2^t)
+__device__ __forceinline__ float sigmoid_weight(float t) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(t));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return r;
 }
-__device__ __forceinline__ float sigmoid_weight(float s) { return __fdividef(1.f, 1.f + __expf(-s)); }
 
-template <int D, int WM, int WN>
+// FULL: K and V rows are D wide, so every chunk place is a constant away from one of four addresses a thread keeps.
+template <int D, int WM, int WN, bool FULL>
 __global__ void __launch_bounds__((WM * WN + 1) * 32)
 sig_attn_kernel(const SigArgs a) {
   constexpr int ROWS = 16 * WM, NP = TPAGES / WN, NWC = WM * WN, THREADS = (NWC + 1) * 32;
-  extern __shared__ __align__(128) unsigned char sa_smem[];
+  extern __shared__ unsigned char sa_smem_raw[];
   __shared__ float s_q[ROWS];                              // query factor x scale
   __shared__ __align__(8) uint64_t s_bar[8];               // full[4], empty[4]
   __shared__ volatile int s_ok;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int kch = FULL ? D / 8 : a.kch, vch = FULL ? D / 8 : a.vch, page_bytes = FULL ? KVB * D * 4 + RMS_BYTES : a.page_bytes;
+  const uint32_t raw_a = (uint32_t)__cvta_generic_to_shared(sa_smem_raw);
+  unsigned char* sa_smem = sa_smem_raw + (((raw_a + 127u) & ~127u) - raw_a);
   const uint32_t bar_a = (uint32_t)__cvta_generic_to_shared(s_bar);
   if (threadIdx.x == 0) {
     for (int st = 0; st < a.n_stages; ++st) {
@@ -117,19 +125,19 @@ sig_attn_kernel(const SigArgs a) {
   if (split >= used) return;
   const int lo = split * pps * KVB, hi = min(kv_len, (split + 1) * pps * KVB);
   const int n_tiles = (hi - lo + TILE - 1) / TILE;
-  const int qld = a.kch * 16 + 16;                          // Q row stride in bytes: an odd number of 16-byte units
+  const int qld = kch * 16 + 16;                          // Q row stride in bytes: an odd number of 16-byte units
   const uint32_t q_a = (uint32_t)__cvta_generic_to_shared(sa_smem);
-  const int q_bytes = (ROWS * qld + 127) / 128 * 128, stage_bytes = TPAGES * a.page_bytes;
+  const int q_bytes = (ROWS * qld + 127) / 128 * 128, stage_bytes = TPAGES * page_bytes;
   unsigned char* ring = sa_smem + q_bytes;
   const uint32_t ring_a = q_a + q_bytes;
-  const int v_off = KVB * a.kch * 16 + KVB * 4;
+  const int v_off = KVB * kch * 16 + RMS_BYTES;
 
   // query rows as projected, and their norm factors
   for (int r = warp; r < ROWS; r += NWC + 1) {
     const int row = row0 + r;
     float ss = 0.f;
-    const bf16* src = a.q + (size_t)(q0 + row / G) * a.ldq + (size_t)(kvh * G + row % G) * (a.kch * 8);
-    for (int c = lane; c < a.kch; c += 32) {
+    const bf16* src = a.q + (size_t)(q0 + row / G) * a.ldq + (size_t)(kvh * G + row % G) * (kch * 8);
+    for (int c = lane; c < kch; c += 32) {
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (row < n_rows) v = *reinterpret_cast<const uint4*>(src + c * 8);
       *reinterpret_cast<uint4*>(sa_smem + r * qld + c * 16) = v;
@@ -149,8 +157,8 @@ sig_attn_kernel(const SigArgs a) {
     const int last = n_tiles - 1, tail = hi & (KVB - 1);
     if (tail && last < a.n_stages) {
       const int pg = ((hi - 1 - lo) / KVB) % TPAGES;
-      unsigned char* v = ring + last * stage_bytes + pg * a.page_bytes + v_off;
-      for (int x = tail * a.vch + threadIdx.x; x < KVB * a.vch; x += THREADS)
+      unsigned char* v = ring + last * stage_bytes + pg * page_bytes + v_off;
+      for (int x = tail * vch + threadIdx.x; x < KVB * vch; x += THREADS)
         *reinterpret_cast<uint4*>(v + x * 16) = make_uint4(0u, 0u, 0u, 0u);
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -191,8 +199,8 @@ sig_attn_kernel(const SigArgs a) {
       if (lane < n_pg) {
         const int p = j0 / KVB + lane, keys = min(KVB, hi - p * KVB);
         const int blk = trl_checked(table[p], a.n_blocks, 6);
-        src = a.pages + ((size_t)blk * a.n_kv + kvh) * a.page_bytes;
-        bytes = (uint32_t)(v_off + keys * a.vch * 16);
+        src = a.pages + ((size_t)blk * a.n_kv + kvh) * page_bytes;
+        bytes = (uint32_t)(v_off + keys * vch * 16);
       }
       const uint32_t total = __reduce_add_sync(0xffffffffu, bytes);
       const uint32_t full = bar_a + 8u * st;
@@ -200,7 +208,7 @@ sig_attn_kernel(const SigArgs a) {
       __syncwarp();
       if (lane < n_pg)
         asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                     ::"r"(ring_a + st * stage_bytes + lane * a.page_bytes), "l"(src), "r"(bytes), "r"(full) : "memory");
+                     ::"r"(ring_a + st * stage_bytes + lane * page_bytes), "l"(src), "r"(bytes), "r"(full) : "memory");
       if (++st == a.n_stages) st = 0, ph ^= 1u;
     }
   } else {
@@ -213,22 +221,42 @@ sig_attn_kernel(const SigArgs a) {
       const int r = r_lo + 8 * i, row = row0 + r;
       const bool in = row < n_rows;
       pos[i] = in ? a.positions[q0 + row / G] : -1;
-      qf[i] = s_q[r];
-      bs[i] = in ? a.bias[kvh * G + row % G] : 0.f;
+      qf[i] = s_q[r] * -LOG2E;
+      bs[i] = in ? a.bias[kvh * G + row % G] * -LOG2E : 0.f;
     }
     const int my_rows = min(16, n_rows - row0 - wm * 16);   // keys this warp's rows see
     const int my_hi = my_rows > 0 ? min(hi, a.positions[q0 + (row0 + wm * 16 + my_rows - 1) / G] + 1) : 0;
+    const int my_lo = my_rows > 0 ? a.positions[q0 + (row0 + wm * 16) / G] : 0;       // the first of them sees keys <= my_lo
     const uint32_t qa = q_a + (wm * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * qld + (lane >> 4) * 16;
-    const int kr = (lane & 7) + (lane >> 4) * 8, krot = kr % a.kch, kcl = (lane >> 3) & 1;
-    const int vr = (lane & 7) + ((lane >> 3) & 1) * 8, vrot = vr % a.vch, vcl = lane >> 4;
+    const int kr = (lane & 7) + (lane >> 4) * 8, kcl = (lane >> 3) & 1;
+    const int vr = (lane & 7) + ((lane >> 3) & 1) * 8, vcl = lane >> 4;
+    uint32_t ka[4], va[4];                                  // FULL: offsets of chunks kcl + {0, 2, 4, 6} of this lane's rows
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      ka[i] = (uint32_t)(kr * kch * 16 + ((kcl ^ (kr & 7) ^ (2 * i)) << 4));
+      va[i] = (uint32_t)(v_off + vr * vch * 16 + ((vcl ^ (vr & 7) ^ (2 * i)) << 4));
+    }
+    const int krot = kr % kch, vrot = vr % vch;
+    auto place = [](int c, int r, int rot, int n) {         // page_chunk without a division (rot = r % n)
+      const int x = c + rot;
+      return n % 8 == 0 ? c ^ (r & 7) : (x >= n ? x - n : x);
+    };
+    auto k_off = [&](int c) {                               // c even
+      if constexpr (FULL) return ka[(c >> 1) & 3] + (uint32_t)((c >> 3) * 128);
+      else return (uint32_t)((kr * kch + place(c + kcl, kr, krot, kch)) * 16);
+    };
+    auto v_at = [&](int c) {
+      if constexpr (FULL) return va[(c >> 1) & 3] + (uint32_t)((c >> 3) * 128);
+      else return (uint32_t)(v_off + (vr * vch + place(c + vcl, vr, vrot, vch)) * 16);
+    };
     int st = 0;
     uint32_t ph = 0;
     for (int kt = 0; kt < n_tiles; ++kt) {
       if (!bounded_wait(bar_a + 8u * st, ph, 500 + st)) break;
       const int jw = lo + kt * TILE + wn * NP * KVB;        // first key of this warp's pages
       if (jw < my_hi) {
-        const uint32_t base = ring_a + st * stage_bytes + wn * NP * a.page_bytes;
-        const unsigned char* base_p = ring + st * stage_bytes + wn * NP * a.page_bytes;
+        const uint32_t base = ring_a + st * stage_bytes + wn * NP * page_bytes;
+        const unsigned char* base_p = ring + st * stage_bytes + wn * NP * page_bytes;
         // ---- scores of NP x 16 keys (pages past the range hold stale bytes: masked below)
         float sc[NP][2][4];
 #pragma unroll
@@ -237,14 +265,14 @@ sig_attn_kernel(const SigArgs a) {
           for (int n8 = 0; n8 < 2; ++n8) sc[p][n8][0] = sc[p][n8][1] = sc[p][n8][2] = sc[p][n8][3] = 0.f;
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
-          if (kk * 2 < a.kch) {
+          if (FULL || kk * 2 < kch) {
             uint32_t qv[4];
             ldsm4(qv, qa + kk * 32);
-            const uint32_t ko = (uint32_t)((kr * a.kch + rotate(kk * 2 + kcl, krot, a.kch)) * 16);
+            const uint32_t ko = k_off(kk * 2);
 #pragma unroll
             for (int p = 0; p < NP; ++p) {
               uint32_t b[4];
-              ldsm4(b, base + p * a.page_bytes + ko);
+              ldsm4(b, base + p * page_bytes + ko);
               mma16(sc[p][0], qv, b[0], b[1]);
               mma16(sc[p][1], qv, b[2], b[3]);
             }
@@ -254,7 +282,8 @@ sig_attn_kernel(const SigArgs a) {
 #pragma unroll
         for (int p = 0; p < NP; ++p) {
           if (jw + p * KVB < my_hi) {
-            const float* kf = reinterpret_cast<const float*>(base_p + p * a.page_bytes + KVB * a.kch * 16);
+            const float* kf = reinterpret_cast<const float*>(base_p + p * page_bytes + KVB * kch * 16);
+            const bool edge = jw + p * KVB + KVB - 1 > my_lo;   // some row does not see all of this page
             uint32_t wh[4], wl[4];
 #pragma unroll
             for (int n8 = 0; n8 < 2; ++n8) {
@@ -262,20 +291,24 @@ sig_attn_kernel(const SigArgs a) {
               const float2 f = *reinterpret_cast<const float2*>(kf + c);
 #pragma unroll
               for (int i = 0; i < 2; ++i) {
-                const float w0 = j <= pos[i] ? sigmoid_weight(sc[p][n8][2 * i] * (qf[i] * f.x) + bs[i]) : 0.f;
-                const float w1 = j + 1 <= pos[i] ? sigmoid_weight(sc[p][n8][2 * i + 1] * (qf[i] * f.y) + bs[i]) : 0.f;
+                float w0 = sigmoid_weight(fmaf(sc[p][n8][2 * i], qf[i] * f.x, bs[i]));
+                float w1 = sigmoid_weight(fmaf(sc[p][n8][2 * i + 1], qf[i] * f.y, bs[i]));
+                if (edge) {                                 // (a select: stale bytes past the range may be anything)
+                  w0 = j <= pos[i] ? w0 : 0.f;
+                  w1 = j + 1 <= pos[i] ? w1 : 0.f;
+                }
                 const uint32_t h = f2_to_bf162_bits(w0, w1);
                 const float2 hf = bf162_bits_to_f2(h);
                 wh[n8 * 2 + i] = h;
                 wl[n8 * 2 + i] = f2_to_bf162_bits(w0 - hf.x, w1 - hf.y);
               }
             }
-            const uint32_t vb = base + p * a.page_bytes + v_off;
+            const uint32_t vb = base + p * page_bytes;
 #pragma unroll
             for (int nd = 0; nd < D / 8; nd += 2) {
-              if (nd < a.vch) {
+              if (FULL || nd < vch) {
                 uint32_t b[4];
-                ldsm4t(b, vb + (uint32_t)((vr * a.vch + rotate(nd + vcl, vrot, a.vch)) * 16));
+                ldsm4t(b, vb + v_at(nd));
                 mma16(o[nd], wh, b[0], b[1]);
                 mma16(o[nd + 1], wh, b[2], b[3]);
                 mma16(o[nd], wl, b[0], b[1]);
@@ -296,7 +329,7 @@ sig_attn_kernel(const SigArgs a) {
     while (clock64() - t_begin < 2000000LL) {
     }
   }
-  const int dv = a.vch * 8;
+  const int dv = vch * 8;
   auto dst_part = [&](int row) {
     const int t = q0 + row / G, h = kvh * G + row % G;
     return a.part + (((size_t)t * a.n_q + h) * a.n_splits + split) * dv;
@@ -310,7 +343,7 @@ sig_attn_kernel(const SigArgs a) {
       if (row >= n_rows) continue;
 #pragma unroll
       for (int nd = 0; nd < D / 8; ++nd) {
-        if (nd < a.vch) {
+        if (FULL || nd < vch) {
           const int d = nd * 8 + (lane & 3) * 2;
           if (used == 1) *reinterpret_cast<uint32_t*>(dst_out(row) + d) = f2_to_bf162_bits(o[nd][2 * i], o[nd][2 * i + 1]);
           else *reinterpret_cast<float2*>(dst_part(row) + d) = make_float2(o[nd][2 * i], o[nd][2 * i + 1]);
@@ -323,7 +356,7 @@ sig_attn_kernel(const SigArgs a) {
     if (warp < NWC) {
 #pragma unroll
       for (int nd = 0; nd < D / 8; ++nd) {
-        if (nd < a.vch) {
+        if (FULL || nd < vch) {
           const int d = nd * 8 + (lane & 3) * 2, r = wm * 16 + (lane >> 2);
           *reinterpret_cast<float2*>(so + ((size_t)wn * ROWS + r) * dv + d) = make_float2(o[nd][0], o[nd][1]);
           *reinterpret_cast<float2*>(so + ((size_t)wn * ROWS + r + 8) * dv + d) = make_float2(o[nd][2], o[nd][3]);
@@ -406,15 +439,15 @@ sig_attn_f32_kernel(const float* q, int ldq, const unsigned char* pages, int pag
     const unsigned char* page = pages + ((size_t)blk * n_kv + kvh) * page_bytes;
     const float* kp = reinterpret_cast<const float*>(page);
     const float* fp = kp + KVB * dk;
-    const float* vp = fp + KVB;
+    const float* vp = fp + RMS_BYTES / 4;
     __syncthreads();
     for (int x = threadIdx.x; x < KVB * dk; x += 256) {
       const int kr = x / dk, d = x % dk;
-      sk[kr * (dk + 1) + d] = kr < keys ? kp[(kr * kch + (d / 4 + kr) % kch) * 4 + d % 4] : 0.f;
+      sk[kr * (dk + 1) + d] = kr < keys ? kp[(kr * kch + page_chunk(d / 4, kr, kch)) * 4 + d % 4] : 0.f;
     }
     for (int x = threadIdx.x; x < KVB * dv; x += 256) {
       const int kr = x / dv, d = x % dv;
-      sv[x] = kr < keys ? vp[(kr * vch + (d / 4 + kr) % vch) * 4 + d % 4] : 0.f;
+      sv[x] = kr < keys ? vp[(kr * vch + page_chunk(d / 4, kr, vch)) * 4 + d % 4] : 0.f;
     }
     if (threadIdx.x < KVB) s_f[threadIdx.x] = threadIdx.x < keys ? fp[threadIdx.x] : 0.f;
     __syncthreads();
@@ -436,8 +469,8 @@ sig_attn_f32_kernel(const float* q, int ldq, const unsigned char* pages, int pag
       if (c + 16 * i < dv) out[(size_t)t * ldo + (size_t)h * dv + c + 16 * i] = acc[i];
 }
 
-template <int D, int WM, int WN>
-cudaError_t sig_launch(SigArgs a, int tiles, int B, const int* seq_ids, int n_tok, cudaStream_t st) {
+template <int D, int WM, int WN, bool FULL>
+cudaError_t sig_launch_as(SigArgs a, int tiles, int B, const int* seq_ids, int n_tok, cudaStream_t st) {
   constexpr int ROWS = 16 * WM;
   const size_t q_bytes = (size_t)(ROWS * (a.kch * 16 + 16) + 127) / 128 * 128, stage = (size_t)TPAGES * a.page_bytes;
   const size_t room = WM == 1 ? 104 * 1024 : (size_t)SA_SMEM;   // decode blocks: two on an SM where three stages allow it
@@ -446,17 +479,23 @@ cudaError_t sig_launch(SigArgs a, int tiles, int B, const int* seq_ids, int n_to
   if (WM == 1 && stages < 3 && q_bytes + 3 * stage <= (size_t)SA_SMEM) stages = 3;
   if (q_bytes + stages * stage > (size_t)SA_SMEM) return cudaErrorInvalidValue;
   a.n_stages = stages;
-  auto kern = sig_attn_kernel<D, WM, WN>;
+  auto kern = sig_attn_kernel<D, WM, WN, FULL>;
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SA_SMEM);
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SA_SMEM + 128);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  cudaError_t e = trl_launch(kern, dim3(tiles * a.n_splits, a.n_kv, B), dim3((WM * WN + 1) * 32), q_bytes + stages * stage, st, a);
+  cudaError_t e = trl_launch(kern, dim3(tiles * a.n_splits, a.n_kv, B), dim3((WM * WN + 1) * 32), q_bytes + stages * stage + 128, st, a);
   if (e == cudaSuccess && a.n_splits > 1)
     e = trl_launch(sig_combine_kernel, dim3(n_tok, a.n_q), dim3(128), 0, st, a, seq_ids, ROWS);
   return e;
+}
+
+template <int D, int WM, int WN>
+cudaError_t sig_launch(const SigArgs& a, int tiles, int B, const int* seq_ids, int n_tok, cudaStream_t st) {
+  if (a.kch == D / 8 && a.vch == D / 8) return sig_launch_as<D, WM, WN, true>(a, tiles, B, seq_ids, n_tok, st);
+  return sig_launch_as<D, WM, WN, false>(a, tiles, B, seq_ids, n_tok, st);
 }
 
 }  // namespace
@@ -479,7 +518,7 @@ TRL_API int trl_sigmoid_attn(const void* q, int ldq, const void* pages, int n_bl
     return (int)cudaErrorInvalidValue;
   SigArgs a;
   a.q = (const bf16*)q, a.ldq = ldq, a.pages = (const unsigned char*)pages, a.kch = dk / 8, a.vch = dv / 8;
-  a.page_bytes = KVB * (a.kch + a.vch) * 16 + KVB * 4, a.n_blocks = n_blocks;
+  a.page_bytes = KVB * (a.kch + a.vch) * 16 + RMS_BYTES, a.n_blocks = n_blocks;
   a.table = (const int*)table, a.max_blocks = max_blocks;
   a.q_start = (const int*)q_start, a.q_len = (const int*)q_len, a.positions = (const int*)positions;
   a.bias = (const float*)bias, a.out = (bf16*)out, a.ldo = ldo, a.part = (float*)part;
@@ -506,7 +545,7 @@ TRL_API int trl_sigmoid_attn_f32(const void* q, int ldq, const void* pages, int 
   if (B <= 0 || max_q_len <= 0 || n_kv <= 0 || n_q % n_kv || dk % 16 || dv % 16 || dk > F_MAXD || dv > F_MAXD || dk <= 0 ||
       dv <= 0 || dim <= 0 || dim > dk || n_blocks <= 0)
     return (int)cudaErrorInvalidValue;
-  const int kch = dk / 4, vch = dv / 4, page_bytes = KVB * (kch + vch) * 16 + KVB * 4;
+  const int kch = dk / 4, vch = dv / 4, page_bytes = KVB * (kch + vch) * 16 + RMS_BYTES;
   const size_t smem = (size_t)((F_ROWS + KVB) * (dk + 1) + KVB * dv) * sizeof(float);
   static bool configured = false;
   if (!configured) {

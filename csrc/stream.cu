@@ -8,7 +8,10 @@
 
 namespace {
 
-constexpr int KVB = 16;
+constexpr int KVB = 16, RMS_BYTES = 128;
+
+// where chunk c of row r sits in a packed page row of n chunks
+__device__ __forceinline__ int page_chunk(int c, int r, int n) { return n % 8 == 0 ? c ^ (r & 7) : (c + r) % n; }
 
 // 16-byte chunk of activations <-> fp32
 template <typename T> struct Chunk;
@@ -161,18 +164,18 @@ block_mid_kernel(const T* proj, const float* __restrict__ act, T* mid, const int
     const uint4* vs = reinterpret_cast<const uint4*>(row + a.v0) + (size_t)h * a.vch;
     uint4* kd = reinterpret_cast<uint4*>(page) + r * a.kch;
     unsigned char* rms = page + KVB * a.kch * 16;
-    uint4* vd = reinterpret_cast<uint4*>(rms + KVB * 4) + r * a.vch;
+    uint4* vd = reinterpret_cast<uint4*>(rms + RMS_BYTES) + r * a.vch;
     float ss = 0.f;
     for (int c = lane; c < a.kch; c += 32) {
       const uint4 v = ks[c];
       Chunk<T>::get(v, f);
 #pragma unroll
       for (int i = 0; i < C; ++i) ss += f[i] * f[i];
-      kd[(c + r) % a.kch] = v;
+      kd[page_chunk(c, r, a.kch)] = v;
     }
     ss = warp_sum(ss);
     if (lane == 0) reinterpret_cast<float*>(rms)[r] = inv_rms(ss, a.dim, a.eps);
-    for (int c = lane; c < a.vch; c += 32) vd[(c + r) % a.vch] = vs[c];
+    for (int c = lane; c < a.vch; c += 32) vd[page_chunk(c, r, a.vch)] = vs[c];
     return;
   }
   // ---- PolyNorm: a N(z) + b N(z^2) + c N(z^3) + e; columns past ff are zero
@@ -268,7 +271,7 @@ TRL_API int trl_block_mid(const void* proj, int ldp, const void* act, void* mid,
   MidArgs a;
   a.ldp = ldp, a.ldm = ldm, a.k0 = k0, a.v0 = v0, a.up0 = up0, a.attn_cols = attn_cols, a.ff = ff;
   a.n_kv = n_kv, a.dim = dim, a.kch = dk / per, a.vch = dv / per, a.n_blocks = n_blocks, a.eps = eps;
-  a.page_bytes = KVB * (a.kch + a.vch) * 16 + KVB * 4;
+  a.page_bytes = KVB * (a.kch + a.vch) * 16 + RMS_BYTES;
   cudaStream_t st = (cudaStream_t)stream;
   // few tokens: wide blocks, so that a token's feed-forward row is one round of loads
   const int threads = (T <= 64 && ff > 4096) ? 1024 : 256;

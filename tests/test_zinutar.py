@@ -46,11 +46,12 @@ def test_packed_pages_place_every_element_once(dim, vdim, itemsize):
     pg = KvPage(3, dim, vdim, itemsize)
     byte = lambda idx, size: (idx.reshape(-1, 1) * size + torch.arange(size)).reshape(-1)
     used = torch.cat([byte(pg.k_index(), itemsize), byte(pg.v_index(), itemsize), byte(pg.rms_index(), 4)])
-    assert sorted(used.tolist()) == list(range(pg.nbytes))          # a bijection onto the page's bytes
-    assert pg.nbytes % 16 == 0 and pg.v_offset % 16 == 0
+    spare = range(pg.rms_offset + 64, pg.v_offset)
+    assert sorted(used.tolist() + list(spare)) == list(range(pg.nbytes))      # every other byte of the page once
+    assert pg.nbytes % 128 == 0 and pg.v_offset % 128 == 0
     # eight rows at one chunk index fall into different 16-byte bank groups when a row is a multiple of 128 bytes
-    if pg.k_chunks % 8 == 0:
-        groups = (pg.k_index()[:8, 0] * itemsize // 16) % 8
+    for c in range(pg.k_chunks if pg.k_chunks % 8 == 0 else 0):
+        groups = (pg.k_index()[:8, c * 16 // itemsize] * itemsize // 16) % 8
         assert len(set(groups.tolist())) == 8
 
 

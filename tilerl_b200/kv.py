@@ -33,6 +33,7 @@ from .config import ModelConfig, ZinutarConfig
 from .ops.ref import KV_BLOCK
 
 RING = 16  # conv ring rows; >= spec width + conv taps
+RMS_BYTES = 128  # of a packed page: 16 fp32 norm factors, padded so that K and V rows start on 128-byte lines
 
 
 class PoolExhausted(RuntimeError):
@@ -178,11 +179,12 @@ class PagedKvPool:
 @dataclass(frozen=True)
 class KvPage:
     """Byte layout of one page of one KV head in a :class:`PackedKvPool`: 16 K rows, the 16 fp32 reciprocal
-    root mean squares of those rows, 16 V rows, back to back, so that one bulk copy brings a page whole.
+    root mean squares of those rows (64 bytes, and 64 unused ones), 16 V rows, back to back, so that one bulk copy
+    brings a page whole.
 
-    Rows are made of 16-byte chunks and row ``r`` is rotated by ``r``: chunk ``c`` sits at chunk
-    ``(c + r) % chunks`` of its row.  Eight rows read at one chunk index then fall into different shared-memory
-    banks.  Widths are padded to 16 elements; the padding holds zeros."""
+    Rows are made of 16-byte chunks whose order depends on the row, so that eight rows read at one chunk index fall
+    into different shared-memory banks: chunk ``c`` of row ``r`` sits at ``c ^ (r % 8)`` when a row is a multiple of
+    eight chunks, at ``(c + r) % chunks`` otherwise.  Widths are padded to 16 elements; the padding holds zeros."""
     n_kv: int
     dim: int
     vdim: int
@@ -206,7 +208,7 @@ class KvPage:
 
     @property
     def v_offset(self) -> int:
-        return self.rms_offset + KV_BLOCK * 4
+        return self.rms_offset + RMS_BYTES
 
     @property
     def nbytes(self) -> int:
@@ -217,7 +219,8 @@ class KvPage:
         per = 16 // self.itemsize
         r = torch.arange(KV_BLOCK)[:, None]
         d = torch.arange(width)[None, :]
-        return base // self.itemsize + (r * chunks + (d // per + r) % chunks) * per + d % per
+        c = (d // per) ^ (r % 8) if chunks % 8 == 0 else (d // per + r) % chunks
+        return base // self.itemsize + (r * chunks + c) * per + d % per
 
     def k_index(self) -> torch.Tensor:
         return self._index(self.pad(self.dim), self.k_chunks, 0)

@@ -4,8 +4,9 @@ Mixed into :class:`tilerl_b200.ops.cuda.CudaOps`.  The activation type is that o
 type) or fp32 (true fp32 everywhere: library products without TF32, fp32 kernels).
 
 A layer is five launches in a decode tick: fused in-projection with the norm in its prologue, block middle (K / V
-write, PolyNorm), attention, the sum of its splits, out-projection added to the stream.  More than
-``ROWS_MAX`` rows take library products (``torch.mm``) between the same kernels.  No counterpart in the reference.
+write, PolyNorm), attention, the sum of its splits, out-projection added to the stream.  More rows than the
+weight-streaming projection serves take library products (``torch.mm``) between the same kernels.  No counterpart in the
+reference.
 """
 from __future__ import annotations
 
@@ -13,8 +14,11 @@ import torch
 
 from . import native as N
 
-ROWS_MAX = 16           # rows the weight-streaming projection serves
-ROWS_NORM_MAX = 4       # rows whose norm it folds in (every block recomputes it)
+# Rows the weight-streaming projection serves: measured against the library product at the sizes of a 1B and an 8B
+# model (in projection of 4096 columns: 1 row 39 us against 44, 8 rows 45 against 44; out projection of 18688 columns:
+# 4 rows 48 against 44, 8 rows 70 against 42, the staged activations leave room for one block per SM)
+ROWS_MAX, ROWS_MAX_LONG, LONG_ELEMENTS = 8, 4, 100_000
+ROWS_NORM_MAX = 2       # rows whose norm it folds in (every block recomputes it)
 EPI_STORE, EPI_STORE_F32, EPI_ADD_F32 = 0, 1, 2
 SHORT_ROWS = 16         # (token, head of the group) rows of a sequence up to which attention splits keys over warps
 
@@ -47,14 +51,19 @@ class StreamOps:
                                          y.stride(0), x.shape[0], w.shape[0], w.shape[1], epi, N.stream()), "linear_rows")
         N.count()
 
+    @staticmethod
+    def _streams(rows: int, w) -> bool:
+        """This many rows go through the weight-streaming projection."""
+        return w.dtype == torch.bfloat16 and rows <= (ROWS_MAX if rows * w.shape[1] <= LONG_ELEMENTS else ROWS_MAX_LONG)
+
     def _project(self, x, norm_w, w, eps, n, y, epi):
         """``y = norm(x) @ W^T`` from stream rows ``x``."""
         t = x.shape[0]
-        if w.dtype == torch.bfloat16 and t <= ROWS_NORM_MAX:
+        if t <= ROWS_NORM_MAX and self._streams(t, w):
             self._linear_rows(x, w, y, epi, norm_w, eps, n)
             return y
         h = self._stream_norm(x, norm_w, eps, n, w.dtype)
-        if w.dtype == torch.bfloat16 and t <= ROWS_MAX:
+        if self._streams(t, w):
             self._linear_rows(h, w, y, epi)
         elif y.dtype == w.dtype:
             torch.mm(h, w.t(), out=y)
@@ -72,7 +81,7 @@ class StreamOps:
 
     def stream_accumulate(self, a, w, x):
         """``x += a @ W^T`` (fp32)."""
-        if w.dtype == torch.bfloat16 and a.shape[0] <= ROWS_MAX:
+        if self._streams(a.shape[0], w):
             self._linear_rows(a, w, x, EPI_ADD_F32)
         elif w.dtype == torch.float32:
             x.addmm_(a, w.t())
@@ -114,7 +123,7 @@ class StreamOps:
             rows = self.lib.trl_sigmoid_attn_rows(l.dk, l.dv) if wide else 16
             tiles = max((lens[i] * g + rows - 1) // rows for i in sel)
             splits = self._sigmoid_splits(sum((lens[i] * g + rows - 1) // rows for i in sel) * l.kv_heads,
-                                          max(kvs[i] for i in sel), wide)
+                                          max(kvs[i] for i in sel), wide, pool.pages[kv_idx].nbytes)
             part = self.ws.get("attn_part", (t * l.heads * splits * l.dv,), torch.float32) if splits > 1 else None
             N.check(self.lib.trl_sigmoid_attn(
                 proj.data_ptr(), proj.stride(0), cache.data_ptr(), cache.shape[0], table.data_ptr(), table.stride(0),
@@ -124,10 +133,10 @@ class StreamOps:
                 l.scale, st), "sigmoid_attn")
             N.count(2 if splits > 1 else 1)
 
-    def _sigmoid_splits(self, blocks: int, longest: int, wide: int) -> int:
+    def _sigmoid_splits(self, blocks: int, longest: int, wide: int, page_bytes: int) -> int:
         """Key splits that fill the GPU; a split holds at least 128 keys (256 for prompt tiles).  In a captured tick
         (``attn_splits`` set) the context may grow later: the kernel itself leaves splits without keys out."""
-        per_sm = 1 if wide else 2
+        per_sm = 1 if wide or 3 * 4 * page_bytes > 96 * 1024 else 2
         if not self.attn_splits:
             per_split = 256 if wide else 128
             longest = (longest + per_split - 1) // per_split

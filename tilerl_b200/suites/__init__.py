@@ -8,6 +8,8 @@ JSON line:
   continuous batching of long prompts, sparse top-k KV decode at long context;
 * ``tick`` (:mod:`.tick`): eager decode ticks (and one prefill) with a per-op event breakdown, the
   command profiler captures of single kernels are taken on;
+* ``zinutar`` (:mod:`.zinutar`): the Zinutar design beside the hybrid's attention-only form at equal size,
+  whole models and single kernels;
 * ``grpo`` (:mod:`.grpo`): one-GPU GRPO step with LoRA adapters, split rollout / train;
 * ``grpo-zero3`` (:mod:`.grpo_zero3`, started under ``torchrun``): GRPO step with ZeRO-3 training
   and a tensor-parallel NVFP4 rollout engine on the same GPUs.
@@ -25,6 +27,7 @@ SUITES = {
     "batch": ("serve", ["--what", "batch"]),
     "sparse": ("serve", ["--what", "sparse"]),
     "tick": ("tick", []),
+    "zinutar": ("zinutar", []),
     "grpo": ("grpo", []),
     "grpo-zero3": ("grpo_zero3", []),
 }

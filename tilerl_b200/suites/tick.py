@@ -28,13 +28,13 @@ def main(argv=None):
     from tilerl_b200.batch import Batch
     from tilerl_b200.config import get_config
     from tilerl_b200.factory import build_model, make_ops
-    from tilerl_b200.kv import GdnStatePool, PagedKvPool
+    from tilerl_b200.kv import GdnStatePool, make_kv_pool
     dev = torch.device("cuda", 0)
     cfg = get_config(args.model)
     ops = make_ops(dev)
     model = build_model(cfg, dev, seed=0, ops=ops)
     nblk = (args.ctx + args.ticks + max(args.prefill, 1) + 32) // 16 + 1
-    kv = PagedKvPool(cfg, args.batch * nblk + 2, dev)
+    kv = make_kv_pool(cfg, args.batch * nblk + 2, dev)
     st = GdnStatePool(cfg, args.batch + 1, dev)
     rows = [dict(blocks=list(range(1 + r * nblk, 1 + (r + 1) * nblk)), slot=r + 1) for r in range(args.batch)]
     times = collections.defaultdict(float)
