@@ -112,7 +112,7 @@ sig_attn_kernel(const SigArgs a) {
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     s_ok = 1;
   }
-  pdl_launch_dependents(25);
+  pdl_enter(25);
   pdl_wait();
   const int n_tiles_x = gridDim.x / a.n_splits;
   const int tile = n_tiles_x - 1 - (int)blockIdx.x / a.n_splits, split = blockIdx.x % a.n_splits;   // longest key ranges first
@@ -324,6 +324,7 @@ sig_attn_kernel(const SigArgs a) {
     }
   }
   __syncthreads();
+  pdl_trigger();                                            // (not earlier: waiting blocks would take the room of working ones)
   if (!s_ok) {                                              // copies may still be in flight towards this block
     const long long t_begin = clock64();
     while (clock64() - t_begin < 2000000LL) {
@@ -484,6 +485,8 @@ cudaError_t sig_launch_as(SigArgs a, int tiles, int B, const int* seq_ids, int n
   if (!configured) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SA_SMEM + 128);
     if (e != cudaSuccess) return e;
+    cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    cudaFuncSetAttribute(sig_combine_kernel, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     configured = true;
   }
   cudaError_t e = trl_launch(kern, dim3(tiles * a.n_splits, a.n_kv, B), dim3((WM * WN + 1) * 32), q_bytes + stages * stage + 128, st, a);

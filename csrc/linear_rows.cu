@@ -2,21 +2,23 @@
 //
 //   y[m, n] (store bf16 | store fp32 | += fp32) = sum_k x'[m, k] * W[n, k]
 //
-// x' is the row itself (bf16) or rms(x) * norm_w of an fp32 stream row, rounded to bf16.  The weights are
-// streamed once, straight into mma.sync A fragments: a warp owns 16 weight rows and a share of K; lane (g, t)
-// loads 16 bytes (8 consecutive k) of rows g and g + 8 per 32-wide step.  The order of k does not matter to a
-// dot product, so the 8 values serve two MMAs under a fixed permutation of k that the activation chunk (read
-// from shared memory as one 16-byte load) shares.  KW warps of a block split K and meet in shared memory in a
-// fixed order, so a run repeats bit for bit.  A block stages the activations once and walks its row tiles, the next
-// tile's first weights in flight while one is summed up.  The first weight loads are issued before the dependency wait:
-// weights are constants of the tick.
+// x' is the row itself (bf16) or rms(x) * norm_w of an fp32 stream row, rounded to bf16.  The weights are streamed
+// once: a warp owns 16 weight rows and a share of K, and every lane copies the 16-byte pieces it will itself feed to
+// mma.sync (8 consecutive k of rows g and g + 8 per 32-wide step) into its own slots of a shared-memory ring, so no
+// barrier sits between the copies and the products, and the bytes in flight do not depend on how much of the SM's
+// memory is left to L1 (register loads lost half their rate behind a kernel that takes all of it as shared memory).
+// The order of k does not matter to a dot product, so the 8 values serve two MMAs under a fixed permutation of k that
+// the activation chunk (one 16-byte load) shares.  KW warps of a block split K and meet in shared memory in a fixed
+// order, so a run repeats bit for bit.  A block stages the activations once and walks its row tiles; the ring runs on
+// across tiles, and its first fill is issued before the dependency wait: weights are constants of the tick.
 // Reference parity: it projects out of a bf16 residual (no counterpart).
 #include "common.cuh"
 
 namespace {
 
-constexpr int LR_THREADS = 256, LR_WARPS = LR_THREADS / 32, LR_U = 8, LR_PAD = 32;
-constexpr int LR_SMEM = 160 * 1024;
+constexpr int LR_THREADS = 256, LR_WARPS = LR_THREADS / 32, LR_U = 4, LR_PAD = 32;
+constexpr int LR_SLOT = LR_U * 2 * 512;                        // bytes of a ring stage of one warp
+constexpr int LR_SMEM = 216 * 1024;
 enum { LR_STORE = 0, LR_STORE_F32 = 1, LR_ADD_F32 = 2 };
 
 __device__ __forceinline__ void lr_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -25,42 +27,52 @@ __device__ __forceinline__ void lr_mma(float (&c)[4], uint32_t a0, uint32_t a1, 
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <bool NORM, int NT, int EPI>
-__global__ void __launch_bounds__(LR_THREADS, 2)
+__device__ __forceinline__ void lr_copy(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ uint4 lr_lds(uint32_t a) {
+  uint4 v;
+  asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(a) : "memory");
+  return v;
+}
+
+template <bool NORM, int NT, int EPI, int DEPTH>
+__global__ void __launch_bounds__(LR_THREADS)
 linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const float* __restrict__ norm_w, float eps, int n_norm,
-                   void* y, int ldy, int M, int N, int K, int kseg, int KW, int n_tiles) {
+                   void* y, int ldy, int M, int N, int K, int KW, int n_tiles) {
   extern __shared__ __align__(16) unsigned char lr_smem[];
   __shared__ float red[32];
   __shared__ float s_r[16];
   __shared__ float s_part[LR_WARPS * 16 * NT * 8];
-  bf16* xs = reinterpret_cast<bf16*>(lr_smem);                 // [M][kseg + LR_PAD]
+  bf16* xs = reinterpret_cast<bf16*>(lr_smem + LR_WARPS * DEPTH * LR_SLOT);     // [M][K + LR_PAD]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
-  const int RW = LR_WARPS / KW, wr = warp / KW, wk = warp % KW;
-  const int nseg = (K + kseg - 1) / kseg, ldxs = kseg + LR_PAD;
-  const bf16 *wa, *wb;
-  auto rows_of = [&](int tile) {
-    const int r0 = (tile * RW + wr) * 16;
-    wa = w + (size_t)min(r0 + g, N - 1) * K + (t << 3), wb = w + (size_t)min(r0 + g + 8, N - 1) * K + (t << 3);
-  };
-  // this warp's 32-wide steps of segment s
-  int jb, je;
-  auto range = [&](int s) {
-    const int steps = min(kseg, K - s * kseg) >> 5, per = (steps + KW - 1) / KW;
-    jb = min(steps, wk * per), je = min(steps, jb + per);
-  };
-  uint4 va[LR_U], vb[LR_U];
-  auto load = [&](int s, int j0) {
+  const int RW = LR_WARPS / KW, wr = warp / KW, wk = warp % KW, ldxs = K + LR_PAD;
+  const uint32_t ring = (uint32_t)__cvta_generic_to_shared(lr_smem) + warp * DEPTH * LR_SLOT + lane * 16;
+  const int steps = K >> 5, per = (steps + KW - 1) / KW, jb = min(steps, wk * per), je = min(steps, jb + per);
+  // fetch cursor: runs DEPTH - 1 blocks of LR_U steps ahead of the products, across row tiles
+  int f_tile = blockIdx.x, f_j = jb, f_slot = 0;
+  auto fetch = [&]() {
+    if (f_tile < n_tiles && jb < je) {
+      const int r0 = (f_tile * RW + wr) * 16;
+      const bf16* wa = w + (size_t)min(r0 + g, N - 1) * K + (t << 3);
+      const bf16* wb = w + (size_t)min(r0 + g + 8, N - 1) * K + (t << 3);
 #pragma unroll
-    for (int u = 0; u < LR_U; ++u) {
-      const int j = min(j0 + u, je - 1);
-      const size_t o = (size_t)s * kseg + ((size_t)j << 5);
-      va[u] = ldg_stream_16(wa + o), vb[u] = ldg_stream_16(wb + o);
+      for (int u = 0; u < LR_U; ++u) {
+        if (f_j + u < je) {
+          const size_t o = (size_t)(f_j + u) << 5;
+          lr_copy(ring + f_slot * LR_SLOT + u * 1024, wa + o);
+          lr_copy(ring + f_slot * LR_SLOT + u * 1024 + 512, wb + o);
+        }
+      }
+      f_j += LR_U;
+      if (f_j >= je) f_j = jb, f_tile += gridDim.x;
     }
+    f_slot = f_slot + 1 == DEPTH ? 0 : f_slot + 1;
+    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  rows_of(blockIdx.x);
-  range(0);
-  if (jb < je) load(0, jb);
-  pdl_launch_dependents(24);
+#pragma unroll
+  for (int i = 0; i < DEPTH - 1; ++i) fetch();
+  pdl_enter(24);
   pdl_wait();
   if (NORM) {
     for (int m = 0; m < M; ++m) {
@@ -73,60 +85,53 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
       ss = block_sum(ss, red);
       if (threadIdx.x == 0) s_r[m] = 1.f / sqrtf(ss / (float)n_norm + eps);
     }
-  }
-  auto stage = [&](int s) {
-    __syncthreads();                                           // s_r written; the previous segment is consumed
-    const int kc = min(kseg, K - s * kseg);
-    for (int m = 0; m < M; ++m) {
-      bf16* dst = xs + (size_t)m * ldxs;
-      if (NORM) {
-        const float* xr = reinterpret_cast<const float*>(xin) + (size_t)m * ldx + s * kseg;
-        const float* nw = norm_w + s * kseg;
-        const float r = s_r[m];
-        for (int c = threadIdx.x; c < kc / 4; c += LR_THREADS) {
-          const float4 v = *reinterpret_cast<const float4*>(xr + 4 * c), q = *reinterpret_cast<const float4*>(nw + 4 * c);
-          *reinterpret_cast<uint2*>(dst + 4 * c) =
-              make_uint2(f2_to_bf162_bits(v.x * r * q.x, v.y * r * q.y), f2_to_bf162_bits(v.z * r * q.z, v.w * r * q.w));
-        }
-      } else {
-        const bf16* xr = reinterpret_cast<const bf16*>(xin) + (size_t)m * ldx + s * kseg;
-        for (int c = threadIdx.x; c < kc / 8; c += LR_THREADS)
-          *reinterpret_cast<uint4*>(dst + 8 * c) = *reinterpret_cast<const uint4*>(xr + 8 * c);
-      }
-    }
     __syncthreads();
-  };
-  if (nseg == 1) stage(0);
+  }
+  for (int m = 0; m < M; ++m) {
+    bf16* dst = xs + (size_t)m * ldxs;
+    if (NORM) {
+      const float* xr = reinterpret_cast<const float*>(xin) + (size_t)m * ldx;
+      const float r = s_r[m];
+      for (int c = threadIdx.x; c < K / 4; c += LR_THREADS) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + 4 * c), q = *reinterpret_cast<const float4*>(norm_w + 4 * c);
+        *reinterpret_cast<uint2*>(dst + 4 * c) =
+            make_uint2(f2_to_bf162_bits(v.x * r * q.x, v.y * r * q.y), f2_to_bf162_bits(v.z * r * q.z, v.w * r * q.w));
+      }
+    } else {
+      const bf16* xr = reinterpret_cast<const bf16*>(xin) + (size_t)m * ldx;
+      for (int c = threadIdx.x; c < K / 8; c += LR_THREADS)
+        *reinterpret_cast<uint4*>(dst + 8 * c) = *reinterpret_cast<const uint4*>(xr + 8 * c);
+    }
+  }
+  __syncthreads();
+  int slot = 0;
   for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
+    if (tile + (int)gridDim.x >= n_tiles) pdl_trigger();       // last tile: dependents may take the room this block leaves
     float acc[NT][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    for (int s = 0; s < nseg; ++s) {
-      if (nseg > 1) {
-        stage(s);
-        range(s);
-        if ((s > 0 || tile != blockIdx.x) && jb < je) load(s, jb);
+    for (int j0 = jb; j0 < je; j0 += LR_U) {
+      fetch();
+      asm volatile("cp.async.wait_group %0;" ::"n"(DEPTH - 1) : "memory");
+      uint4 va[LR_U], vb[LR_U];
+#pragma unroll
+      for (int u = 0; u < LR_U; ++u) {
+        va[u] = lr_lds(ring + slot * LR_SLOT + u * 1024);
+        vb[u] = lr_lds(ring + slot * LR_SLOT + u * 1024 + 512);
       }
-      for (int j0 = jb; j0 < je; j0 += LR_U) {
-        if (j0 > jb) load(s, j0);
+      slot = slot + 1 == DEPTH ? 0 : slot + 1;
 #pragma unroll
-        for (int u = 0; u < LR_U; ++u) {
-          if (j0 + u < je) {
+      for (int u = 0; u < LR_U; ++u) {
+        if (j0 + u < je) {
 #pragma unroll
-            for (int i = 0; i < NT; ++i) {
-              uint4 xv = make_uint4(0u, 0u, 0u, 0u);           // rows past M count as zeros
-              if (i * 8 + g < M) xv = *reinterpret_cast<const uint4*>(xs + (size_t)(i * 8 + g) * ldxs + ((j0 + u) << 5) + (t << 3));
-              lr_mma(acc[i], va[u].x, vb[u].x, va[u].y, vb[u].y, xv.x, xv.y);
-              lr_mma(acc[i], va[u].z, vb[u].z, va[u].w, vb[u].w, xv.z, xv.w);
-            }
+          for (int i = 0; i < NT; ++i) {
+            uint4 xv = make_uint4(0u, 0u, 0u, 0u);             // rows past M count as zeros
+            if (i * 8 + g < M) xv = *reinterpret_cast<const uint4*>(xs + (size_t)(i * 8 + g) * ldxs + ((j0 + u) << 5) + (t << 3));
+            lr_mma(acc[i], va[u].x, vb[u].x, va[u].y, vb[u].y, xv.x, xv.y);
+            lr_mma(acc[i], va[u].z, vb[u].z, va[u].w, vb[u].w, xv.z, xv.w);
           }
         }
       }
-    }
-    const int next = tile + gridDim.x;
-    if (next < n_tiles) {
-      rows_of(next);
-      if (nseg == 1 && jb < je) load(0, jb);                   // in flight while this tile is summed up
     }
     // accumulator e of tile i: weight row g + 8 (e / 2), activation row 8 i + 2 t + e % 2
 #pragma unroll
@@ -146,6 +151,7 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
     }
     __syncthreads();
   }
+  asm volatile("cp.async.wait_all;" ::: "memory");
 }
 
 int lr_sms() {
@@ -160,39 +166,45 @@ int lr_sms() {
 
 }  // namespace
 
+// Most rows the projection takes for K columns (0: none): the staged rows and a two-stage ring fit shared memory.
+TRL_API int trl_linear_rows_max(int K) {
+  return max(0, min(16, (LR_SMEM - LR_WARPS * 2 * LR_SLOT) / ((K + LR_PAD) * 2)));
+}
+
 // x: bf16 [M, ldx], or the fp32 stream when norm_w is given (its row norm counts n_norm columns).  w: bf16 [N, K],
-// K a multiple of 64.  epi: 0 store bf16, 1 store fp32, 2 add to fp32.  M <= 16.
+// K a multiple of 64.  epi: 0 store bf16, 1 store fp32, 2 add to fp32.  M <= trl_linear_rows_max(K).
 TRL_API int trl_linear_rows(const void* x, int ldx, const void* w, const void* norm_w, float eps, int n_norm, void* y, int ldy,
                             int M, int N, int K, int epi, void* stream) {
-  if (M < 1 || M > 16 || N < 1 || K < 64 || K % 64 || ldx % 8 || epi < 0 || epi > 2 || (norm_w && n_norm < 1) ||
-      ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
+  if (M < 1 || N < 1 || K < 64 || K % 64 || M > trl_linear_rows_max(K) || ldx % 8 || epi < 0 || epi > 2 ||
+      (norm_w && n_norm < 1) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return (int)cudaErrorInvalidValue;
   const int groups = (N + 15) / 16;
   // split K over the warps of a block: shares of at least 16 steps, more splits where there are few rows
   int KW = 1;
   while (KW < LR_WARPS && (K / 32 / (2 * KW) >= 16 || (long)groups * KW < 2L * lr_sms() * LR_WARPS)) KW *= 2;
-  const int RW = LR_WARPS / KW, n_tiles = (groups + RW - 1) / RW;
-  const int cap = (LR_SMEM / (2 * M) - LR_PAD) / 32 * 32;
-  const int nseg = (K + cap - 1) / cap, kseg = ((K + nseg - 1) / nseg + 31) / 32 * 32;
-  const size_t smem = (size_t)M * (kseg + LR_PAD) * sizeof(bf16);
-  const int nt = M <= 8 ? 1 : 2;
-  const int grid = min(n_tiles, lr_sms() * (smem <= 96 * 1024 ? 2 : 1));   // one round of blocks walks all row tiles
+  const int RW = LR_WARPS / KW, n_tiles = (groups + RW - 1) / RW, grid = min(n_tiles, lr_sms());
+  const size_t xb = (size_t)M * (K + LR_PAD) * sizeof(bf16);
+  const int nt = M <= 8 ? 1 : 2, depth = xb + LR_WARPS * 4 * LR_SLOT <= LR_SMEM ? 4 : 2;
+  const size_t smem = xb + (size_t)LR_WARPS * depth * LR_SLOT;
   cudaError_t e = cudaErrorInvalidValue;
-#define LR_CASE(NO, NTT, EP)                                                                                            \
-  if ((norm_w != nullptr) == NO && nt == NTT && epi == EP) {                                                            \
-    auto kern = linear_rows_kernel<NO, NTT, EP>;                                                                        \
+#define LR_CASE(NO, NTT, EP, DE)                                                                                        \
+  if ((norm_w != nullptr) == NO && nt == NTT && epi == EP && depth == DE) {                                             \
+    auto kern = linear_rows_kernel<NO, NTT, EP, DE>;                                                                    \
     static bool configured = false;                                                                                     \
     if (!configured) {                                                                                                  \
-      e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, LR_SMEM + 4096);                      \
+      e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, LR_SMEM);                             \
       if (e != cudaSuccess) return (int)e;                                                                              \
+      cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, 100);                                  \
       configured = true;                                                                                                \
     }                                                                                                                   \
     e = trl_launch(kern, dim3(grid), dim3(LR_THREADS), smem, (cudaStream_t)stream, x, ldx, (const bf16*)w,              \
-                   (const float*)norm_w, eps, n_norm, y, ldy, M, N, K, kseg, KW, n_tiles);                                       \
+                   (const float*)norm_w, eps, n_norm, y, ldy, M, N, K, KW, n_tiles);                                    \
   }
-  LR_CASE(true, 1, LR_STORE) LR_CASE(true, 1, LR_STORE_F32) LR_CASE(true, 2, LR_STORE) LR_CASE(true, 2, LR_STORE_F32)
-  LR_CASE(false, 1, LR_STORE) LR_CASE(false, 1, LR_STORE_F32) LR_CASE(false, 1, LR_ADD_F32)
-  LR_CASE(false, 2, LR_STORE) LR_CASE(false, 2, LR_STORE_F32) LR_CASE(false, 2, LR_ADD_F32)
+#define LR_BOTH(NO, NTT, EP) LR_CASE(NO, NTT, EP, 2) LR_CASE(NO, NTT, EP, 4)
+  LR_BOTH(true, 1, LR_STORE) LR_BOTH(true, 1, LR_STORE_F32) LR_BOTH(true, 2, LR_STORE) LR_BOTH(true, 2, LR_STORE_F32)
+  LR_BOTH(false, 1, LR_STORE) LR_BOTH(false, 1, LR_STORE_F32) LR_BOTH(false, 1, LR_ADD_F32)
+  LR_BOTH(false, 2, LR_STORE) LR_BOTH(false, 2, LR_STORE_F32) LR_BOTH(false, 2, LR_ADD_F32)
+#undef LR_BOTH
 #undef LR_CASE
   return (int)e;
 }

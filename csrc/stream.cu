@@ -276,6 +276,11 @@ TRL_API int trl_block_mid(const void* proj, int ldp, const void* act, void* mid,
   // few tokens: wide blocks, so that a token's feed-forward row is one round of loads
   const int threads = (T <= 64 && ff > 4096) ? 1024 : 256;
   const dim3 grid(T, 1 + (n_kv + threads / 32 - 1) / (threads / 32));
+  static bool configured = false;
+  if (!configured) {
+    cudaFuncSetAttribute(block_mid_kernel<bf16>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    configured = true;
+  }
   if (f32)
     return (int)trl_launch(block_mid_kernel<float>, grid, dim3(threads), 0, st, (const float*)proj, (const float*)act,
                            (float*)mid, (const int*)slot_mapping, (unsigned char*)pages, a);

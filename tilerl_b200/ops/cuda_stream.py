@@ -14,10 +14,9 @@ import torch
 
 from . import native as N
 
-# Rows the weight-streaming projection serves: measured against the library product at the sizes of a 1B and an 8B
-# model (in projection of 4096 columns: 1 row 39 us against 44, 8 rows 45 against 44; out projection of 18688 columns:
-# 4 rows 48 against 44, 8 rows 70 against 42, the staged activations leave room for one block per SM)
-ROWS_MAX, ROWS_MAX_LONG, LONG_ELEMENTS = 8, 4, 100_000
+# Rows the weight-streaming projection serves.  Decode ticks of 2048- and 4096-wide models, against library products in
+# its place: 1 row 0.47 / 0.62 ms against 0.70 / 0.70, 4 rows 0.56 / 0.73 against 0.72 / 0.73, 8 rows even.
+ROWS_MAX = 4
 ROWS_NORM_MAX = 2       # rows whose norm it folds in (every block recomputes it)
 EPI_STORE, EPI_STORE_F32, EPI_ADD_F32 = 0, 1, 2
 SHORT_ROWS = 16         # (token, head of the group) rows of a sequence up to which attention splits keys over warps
@@ -51,10 +50,9 @@ class StreamOps:
                                          y.stride(0), x.shape[0], w.shape[0], w.shape[1], epi, N.stream()), "linear_rows")
         N.count()
 
-    @staticmethod
-    def _streams(rows: int, w) -> bool:
+    def _streams(self, rows: int, w) -> bool:
         """This many rows go through the weight-streaming projection."""
-        return w.dtype == torch.bfloat16 and rows <= (ROWS_MAX if rows * w.shape[1] <= LONG_ELEMENTS else ROWS_MAX_LONG)
+        return w.dtype == torch.bfloat16 and rows <= ROWS_MAX and rows <= self.lib.trl_linear_rows_max(w.shape[1])
 
     def _project(self, x, norm_w, w, eps, n, y, epi):
         """``y = norm(x) @ W^T`` from stream rows ``x``."""

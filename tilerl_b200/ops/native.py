@@ -80,6 +80,7 @@ _SIGS = {
     "trl_stream_add": [P, P, L, P],
     "trl_block_mid": [P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P],
     "trl_linear_rows": [P, I, P, P, F, I, P, I, I, I, I, I, P],
+    "trl_linear_rows_max": [I],
     "trl_sigmoid_attn_rows": [I, I],
     "trl_sigmoid_attn": [P, I, P, I, P, I, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P],
     "trl_sigmoid_attn_f32": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P],

@@ -82,7 +82,8 @@ register("any", "cpu", {op: Kernel(fn, _REF) for op, fn in {
     "paged_attention_prefill": "paged_attention", "gdn": "gdn_sequence", "gdn_chunked": "gdn_chunked",
     "gdn_backward": "gdn_recurrent_backward", "sample": "sample", "sample_nucleus": "sample_nucleus_model",
     "cross_entropy": "cross_entropy_grad", "cross_entropy_sharded": "cross_entropy_sharded",
-    "page_bounds": "page_bounds", "select_pages": "select_pages",
+    "page_bounds": "page_bounds", "select_pages": "select_pages", "sigmoid_attention": "sigmoid_attention",
+    "polynorm": "polynorm", "packed_kv_write": "packed_kv_write",
 }.items()})
 register("any", "cpu", {
     "quantize_nvfp4": Kernel("quantize_nvfp4", "tilerl_b200/formats.py"),
@@ -105,7 +106,13 @@ register("bf16", "sm100", {
     "linear_bf16_gemv": Kernel("gemv_bf16_kernel", "csrc/gemv.cu", "trl_gemv_bf16"),
     "linear_bf16_gemv_rows16": Kernel("gemv_bf16_mma_kernel", "csrc/gemv.cu", "trl_gemv_bf16",
                                       note="3..16 rows (batched / verify lm_head): one mma.sync pass over the weights"),
+    "linear_stream_rows": Kernel("linear_rows_kernel", "csrc/linear_rows.cu", "trl_linear_rows",
+                                 note="few rows out of / into an fp32 stream: norm prologue, cp.async weight ring, mma.sync"),
     "linear_bf16_gemm": Kernel("torch.matmul (cuBLAS)", "tilerl_b200/ops/gemm.py", note="plain library GEMM"),
+})
+register("fp32", "sm100", {
+    "sigmoid_attention": Kernel("sig_attn_f32_kernel", "csrc/attn_sigmoid.cu", "trl_sigmoid_attn_f32", note="fp32 packed pool"),
+    "linear_fp32_gemm": Kernel("torch.mm (cuBLAS, no TF32)", "tilerl_b200/ops/cuda_stream.py", note="plain library GEMM"),
 })
 register("fp8", "sm100", {
     "linear_fp8": Kernel("gemm_fp8_kernel", "csrc/gemm_fp8.cu", "trl_gemm_fp8",
@@ -149,6 +156,12 @@ register("any", "sm100", {
     "zero_all_gather": Kernel("zero_allgather_kernel", "csrc/zero.cu", "trl_zero_allgather", "tilerl_b200.parallel.zero3"),
     "zero_reduce_scatter": Kernel("zero_reduce_scatter_kernel", "csrc/zero.cu", "trl_zero_reduce_scatter",
                                   "tilerl_b200.parallel.zero3"),
+    "embed_norm": Kernel("embed_norm_kernel", "csrc/stream.cu", "trl_embed_norm", note="fp32 stream; bf16 or fp32 table"),
+    "stream_norm": Kernel("stream_norm_kernel", "csrc/stream.cu", "trl_stream_norm"),
+    "stream_add": Kernel("stream_add_kernel", "csrc/stream.cu", "trl_stream_add"),
+    "block_mid": Kernel("block_mid_kernel", "csrc/stream.cu", "trl_block_mid", note="packed K / V write + PolyNorm"),
+    "sigmoid_attention": Kernel("sig_attn_kernel + sig_combine_kernel", "csrc/attn_sigmoid.cu", "trl_sigmoid_attn",
+                                note="bf16 packed pool; narrow row tiles for decoding, wide ones for prompts, key splits"),
     "batch_fill": Kernel("trl_batch_fill", "csrc/runtime.cpp", "trl_batch_fill", note="host runtime"),
     "pager": Kernel("trl_pager_*", "csrc/runtime.cpp", "trl_pager_alloc", note="host runtime"),
 })
