@@ -128,7 +128,8 @@ def _run(ops, cfg, l, lens, starts, dtype, seed=0, blocks=None):
 
 
 SHAPES = [(4, 2, 64, 64, 3.0, 96), (6, 2, 24, 40, 2.0, 100), (8, 1, 128, 128, 1.0, 0), (20, 1, 16, 96, 4.0, 40),
-          (2, 2, 256, 256, 0.5, 20000), (4, 4, 256, 48, 0.5, 72), (3, 1, 80, 192, 1.0, 33), (5, 5, 8, 8, 6.0, 16)]
+          (2, 2, 256, 256, 0.5, 20000), (4, 4, 256, 48, 0.5, 72), (3, 1, 80, 192, 1.0, 33), (5, 5, 8, 8, 6.0, 16),
+          (3, 3, 40, 16, 2.0, 0)]
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 8e-3)])
