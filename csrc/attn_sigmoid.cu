@@ -18,11 +18,11 @@
 //   sig_attn_f32_kernel         the same attention in fp32 (CUDA cores) on an fp32 pool.
 //
 // Reference parity: the reference's attention is softmax only (no counterpart).
-#include "common.cuh"
+#include "packed.cuh"
 
 namespace {
 
-constexpr int KVB = 16, TILE = 64, TPAGES = TILE / KVB, RMS_BYTES = 128;
+constexpr int TILE = 64, TPAGES = TILE / KVB, RMS_BYTES = 128;
 constexpr long long SA_WAIT_CYCLES = 4000000000LL;
 constexpr int SA_SMEM = 216 * 1024;
 constexpr float LOG2E = 1.4426950408889634f;
@@ -59,19 +59,6 @@ __device__ __forceinline__ int tile_keys(int row0, int rows, int n_rows, int G, 
   return positions[q0 + (min(row0 + rows, n_rows) - 1) / G] + 1;
 }
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ uint32_t sa_try_wait(uint32_t bar, uint32_t parity) {
   uint32_t ok;
   asm volatile("{ .reg .pred p;\n"
@@ -80,8 +67,6 @@ __device__ __forceinline__ uint32_t sa_try_wait(uint32_t bar, uint32_t parity) {
                : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
   return ok;
 }
-// where chunk c of row r sits in a packed page row of n chunks
-__device__ __forceinline__ int page_chunk(int c, int r, int n) { return n % 8 == 0 ? c ^ (r & 7) : (c + r) % n; }
 // sigmoid of a score given as t = -log2(e) x: 1 / (1 + 2^t)
 __device__ __forceinline__ float sigmoid_weight(float t) {
   float e, r;

@@ -1,0 +1,39 @@
+// Arguments and gates of the decayed-scan kernels (scan.cu, scan_mma.cu).
+#pragma once
+#include "packed.cuh"
+
+enum { SCAN_MAMBA2 = 0, SCAN_MLSTM = 1 };
+
+// Mirrored by tilerl_b200/ops/cuda_mixers.py::ScanArgs, field by field.
+struct ScanArgs {
+  const void* rows;                    // [T, ld]: q, k, v columns at q0, k0, v0
+  const float* gates;                  // [T, ldg] raw gates: dt, or i then f
+  const float *gate_b, *a_log, *skip;  // per head (gate_b: per gate)
+  float* states;                       // the layer's record of slot 0, plane 0
+  const int *cur, *keep_flags, *q_start, *q_len, *slots;
+  float* o;                            // [T, heads * dv]
+  long slot_stride, plane_stride;      // floats
+  int ld, q0, k0, v0, ldg;
+  int heads, per, dk, dv;              // per: heads that share q and k
+  int min_len, max_len;
+  float cap, q_scale;
+};
+
+inline bool scan_args_bad(const ScanArgs& a, int kind) {
+  return a.heads <= 0 || a.per <= 0 || a.heads % a.per || a.dk <= 0 || a.dk % 16 || a.dk > 256 || a.dv <= 0 || a.dv % 16 ||
+         a.ldg < a.heads * (kind + 1) || !a.rows || !a.gates || !a.states || !a.o || !a.gate_b || (kind == SCAN_MAMBA2 && (!a.a_log || !a.skip)) ||
+         (kind == SCAN_MLSTM && !(a.cap > 0.f)) || kind < 0 || kind > 1;
+}
+
+// Mamba-2: (keep, dt) of a token and head.  mLSTM: (log forget gate, log input gate).
+template <int KIND>
+__device__ __forceinline__ void scan_gates(const ScanArgs& a, int t, int h, float& g0, float& g1) {
+  const float* row = a.gates + (size_t)t * a.ldg;
+  if (KIND == SCAN_MAMBA2) {
+    g1 = softplus_x(row[h] + a.gate_b[h]);
+    g0 = expf(-expf(a.a_log[h]) * g1);
+  } else {
+    g1 = a.cap * tanhf((row[h] + a.gate_b[h]) / a.cap);
+    g0 = -softplus_x(-a.cap * tanhf((row[a.heads + h] + a.gate_b[a.heads + h]) / a.cap));
+  }
+}

@@ -4,43 +4,11 @@
 // PolyNorm(up) into the feed-forward columns of the output projection's input.
 // Stream rows are `ld` wide (a multiple of 64) with zeros past the model width `n`.
 // Reference parity: the reference keeps a bf16 residual and has no PolyNorm (no counterpart).
-#include "common.cuh"
+#include "packed.cuh"
 
 namespace {
 
-constexpr int KVB = 16, RMS_BYTES = 128;
-
-// where chunk c of row r sits in a packed page row of n chunks
-__device__ __forceinline__ int page_chunk(int c, int r, int n) { return n % 8 == 0 ? c ^ (r & 7) : (c + r) % n; }
-
-// 16-byte chunk of activations <-> fp32
-template <typename T> struct Chunk;
-template <> struct Chunk<bf16> {
-  static constexpr int N = 8;
-  static __device__ __forceinline__ void get(const uint4& v, float (&f)[8]) {
-    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 a = bf162_bits_to_f2(w[i]);
-      f[2 * i] = a.x, f[2 * i + 1] = a.y;
-    }
-  }
-  static __device__ __forceinline__ uint4 put(const float (&f)[8]) {
-    return make_uint4(f2_to_bf162_bits(f[0], f[1]), f2_to_bf162_bits(f[2], f[3]), f2_to_bf162_bits(f[4], f[5]),
-                      f2_to_bf162_bits(f[6], f[7]));
-  }
-};
-template <> struct Chunk<float> {
-  static constexpr int N = 4;
-  static __device__ __forceinline__ void get(const uint4& v, float (&f)[4]) {
-    f[0] = __uint_as_float(v.x), f[1] = __uint_as_float(v.y), f[2] = __uint_as_float(v.z), f[3] = __uint_as_float(v.w);
-  }
-  static __device__ __forceinline__ uint4 put(const float (&f)[4]) {
-    return make_uint4(__float_as_uint(f[0]), __float_as_uint(f[1]), __float_as_uint(f[2]), __float_as_uint(f[3]));
-  }
-};
-
-__device__ __forceinline__ float inv_rms(float ss, int n, float eps) { return 1.f / sqrtf(ss / (float)n + eps); }
+constexpr int RMS_BYTES = 128;
 
 // x = rms(table[id]) * w, optionally kept a second time (the embedding output re-entering a loop)
 template <typename T>

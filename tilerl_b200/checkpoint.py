@@ -37,12 +37,13 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import ATTN, ModelConfig, ZinutarConfig
+from .config import ATTN, ModelConfig, StreamDesign, ZinutarConfig
 from .formats import (FP8BlockTensor, NVFP4Tensor, dequantize_fp8_block, dequantize_nvfp4,
                       quantize_nvfp4)
 from .models.hybrid import HybridModel, linear_names, quantize_weight
+from .models.fetotar import FetotarModel
 from .models.zinutar import ZinutarModel
-from .zinutar_layout import tensor_shapes
+from . import fetotar_layout, zinutar_layout
 
 
 class CheckpointError(ValueError):
@@ -257,16 +258,17 @@ def assemble_master(cfg: ModelConfig, reader: _Reader) -> Dict[str, torch.Tensor
     return out
 
 
-def load_zinutar(cfg: ZinutarConfig, path: str, device="cpu", dtype: Optional[torch.dtype] = None) -> ZinutarModel:
-    """Dense checkpoint of a Zinutar model (tensor names and shapes: ``zinutar_layout.tensor_shapes``)."""
+def load_stream_design(cfg: StreamDesign, path: str, device="cpu", dtype: Optional[torch.dtype] = None):
+    """Dense checkpoint of a stream design (tensor names and shapes: ``tensor_shapes`` of its layout module)."""
+    model, layout = (ZinutarModel, zinutar_layout) if isinstance(cfg, ZinutarConfig) else (FetotarModel, fetotar_layout)
     reader = _Reader(path)
-    lacks = [n for n in tensor_shapes(cfg) if not reader.has(n)]
+    lacks = [n for n in layout.tensor_shapes(cfg) if not reader.has(n)]
     if lacks:
         raise CheckpointError(f"checkpoint lacks {len(lacks)} tensors, first {lacks[0]}")
     if dtype is None:
         dtype = torch.bfloat16 if torch.device(device).type == "cuda" else torch.float32
     try:
-        return ZinutarModel.from_tensors(cfg, reader.get, device, dtype)
+        return model.from_tensors(cfg, reader.get, device, dtype)
     except ValueError as e:
         raise CheckpointError(str(e)) from None
 
@@ -274,10 +276,10 @@ def load_zinutar(cfg: ZinutarConfig, path: str, device="cpu", dtype: Optional[to
 def load_checkpoint(cfg: ModelConfig, path: str, *, device="cpu", tp_rank: int = 0, tp: int = 1,
                     keep_master: bool = False, dtype: Optional[torch.dtype] = None) -> HybridModel:
     """``dtype``: compute dtype of designs that run in more than one (default: bf16 on a GPU, fp32 on CPU)."""
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, StreamDesign):
         if tp > 1 or keep_master:
-            raise CheckpointError("Zinutar models are served on one GPU per process, without training masters")
-        return load_zinutar(cfg, path, device, dtype)
+            raise CheckpointError(f"{cfg.architecture} models are served on one GPU per process, without training masters")
+        return load_stream_design(cfg, path, device, dtype)
     cj = os.path.join(path, "config.json")
     if os.path.exists(cj):
         with open(cj) as f:
@@ -328,7 +330,7 @@ def save_checkpoint(model: HybridModel, path: str) -> None:
     from safetensors.torch import save_file
     os.makedirs(path, exist_ok=True)
     tensors: Dict[str, torch.Tensor] = {}
-    dense = isinstance(model, ZinutarModel)
+    dense = isinstance(model.cfg, StreamDesign)
     if dense:
         tensors = {k: v.detach().to(torch.bfloat16).cpu().contiguous() for k, v in model.tensors()}
     for k, v in ({} if dense else model.params).items():

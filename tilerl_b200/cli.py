@@ -329,7 +329,7 @@ def cmd_train(args) -> int:
     import torch
     from . import evals, rl
     from .checkpoint import load_adapter, save_adapter, save_checkpoint
-    from .config import ZinutarConfig, get_config
+    from .config import StreamDesign, get_config
     from .factory import build_engine, build_model, make_ops
     from .ledger import Run, runs_dir
     from .optim import make_optimizer
@@ -360,8 +360,8 @@ def cmd_train(args) -> int:
     if flags.get("allow_short_rollouts"):        # (a smoke recipe runs into its cap on purpose)
         args.allow_short_rollouts = True
     cfg = get_config(flags.get("model", args.model))
-    if isinstance(cfg, ZinutarConfig):
-        raise SystemExit("Zinutar models are served (serve, generate, bench), not trained")
+    if isinstance(cfg, StreamDesign):
+        raise SystemExit(f"{cfg.architecture} models are served (serve, generate, bench), not trained")
     if not args.dry_run and flags.get("reward") in ("gsm8k", "boxed") and not args.data and (flags.get("rl") or flags.get("opd")):
         raise SystemExit(f"reward {flags['reward']!r} scores completions against gold answers: give --data rows.jsonl "
                          "with {prompt, answer} rows")

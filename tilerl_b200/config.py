@@ -1,5 +1,7 @@
-"""Model configurations: the hybrid (gated-GQA attention + Gated-DeltaNet) decoder, and Zinutar
-(:class:`ZinutarConfig`, a looped decoder of parallel blocks; no counterpart in the reference).
+"""Model configurations: the hybrid (gated-GQA attention + Gated-DeltaNet) decoder, and the stream designs
+(:class:`StreamDesign`: an fp32 residual stream, served in bf16 or fp32 on one GPU per process; no counterpart in the
+reference): Zinutar (:class:`ZinutarConfig`, a looped decoder of parallel blocks) and Fetotar (:class:`FetotarConfig`,
+sandwich-normed layers of latent attention, Mamba-2 and mLSTM with a per-layer token input).
 
 One frozen dataclass describes every shape the kernels, the KV pools, the
 tensor-parallel shard tables and the cost model derive from.  Layer kinds are
@@ -15,6 +17,8 @@ import json
 import os
 from dataclasses import dataclass, replace
 from typing import Dict, Optional, Tuple
+
+from .mixers import MIXERS, ClampedGluSpec, LatentAttnSpec, LayerSpec, Mamba2Spec, MlstmSpec, RotarySpec, YarnSpec, take
 
 ATTN = "attn"
 GDN = "gdn"
@@ -209,6 +213,19 @@ def small_gpu_tp() -> ModelConfig:
     )
 
 
+# ---- stream designs ----------------------------------------------------------------------------------
+class StreamDesign:
+    """What designs with an fp32 residual stream have in common: their ``config.json`` spells every size out, weights
+    are served in bf16 (or fp32), one process serves one GPU, and they are not trained here."""
+    architecture = ""
+    tie_embeddings = False
+    quant = "bf16"
+    lm_head_quant = "bf16"
+    # no Gated-DeltaNet layers: recurrent state, where a design has any, lives in a RecurrentPool
+    n_gdn_layers = 0
+    gdn_k_heads = gdn_v_heads = gdn_head_dim = gdn_conv_dim = 0
+
+
 # ---- Zinutar: looped parallel-block decoder with sigmoid-weighted attention ------------------------
 @dataclass(frozen=True)
 class AttnSpec:
@@ -273,7 +290,7 @@ def _fields(d: Dict, known, where: str) -> None:
 
 
 @dataclass(frozen=True)
-class ZinutarConfig:
+class ZinutarConfig(StreamDesign):
     """Sizes and constants of a Zinutar model.  Every layer has its own mixer and feed-forward sizes;
     :attr:`runs` spells the executions out in order, one KV cache each."""
     name: str
@@ -285,12 +302,6 @@ class ZinutarConfig:
     max_ctx: int = 1 << 20
 
     architecture = "Zinutar"
-    tie_embeddings = False
-    quant = "bf16"
-    lm_head_quant = "bf16"
-    # no recurrent layers: the state pool of the engine degenerates to slot bookkeeping
-    n_gdn_layers = 0
-    gdn_k_heads = gdn_v_heads = gdn_head_dim = gdn_conv_dim = 0
 
     def __post_init__(self) -> None:
         object.__setattr__(self, "layers", tuple(self.layers))
@@ -396,9 +407,119 @@ def zinutar_8b() -> ZinutarConfig:
     return zinutar_uniform("zinutar-8b", hidden=4096, vocab=128256, n_layers=32, heads=16, kv_heads=4, dim=256, ff=14336)
 
 
-ARCHITECTURES = {ZinutarConfig.architecture: ZinutarConfig}
+# ---- Fetotar: sandwich-normed layers of three mixers, with a per-layer token input ---------------------
+@dataclass(frozen=True)
+class FetotarConfig(StreamDesign):
+    """Sizes and constants of a Fetotar model.  Every layer has its own mixer and feed-forward; attention layers number
+    the KV caches, recurrent layers the states, both in layer order."""
+    name: str
+    hidden: int
+    vocab: int
+    layers: Tuple[LayerSpec, ...]
+    side_dim: int                   # width of a layer's share of the per-token side embedding
+    embed_scale: float = 1.0
+    norm_eps: float = 1e-6
+    max_ctx: int = 1 << 20
+
+    architecture = "Fetotar"
+
+    def __post_init__(self) -> None:
+        object.__setattr__(self, "layers", tuple(self.layers))
+        if self.hidden <= 0 or self.vocab <= 0 or self.side_dim <= 0 or not self.layers:
+            raise ValueError("a model needs positive sizes and at least one layer")
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def attn_mixers(self) -> Tuple[LatentAttnSpec, ...]:
+        return tuple(l.mixer for l in self.layers if not l.mixer.recurrent)
+
+    @property
+    def recurrent_mixers(self) -> Tuple[object, ...]:
+        return tuple(l.mixer for l in self.layers if l.mixer.recurrent)
+
+    @property
+    def n_attn_layers(self) -> int:
+        return len(self.attn_mixers)
+
+    @property
+    def n_q_heads(self) -> int:
+        return max([m.heads for m in self.attn_mixers] + [1])
+
+    n_kv_heads = 1                  # one latent per token, whatever the heads
+
+    def cache_index(self, layer: int) -> int:
+        """Number of the layer's cache (attention) or state (recurrent)."""
+        kind = self.layers[layer].mixer.recurrent
+        return sum(l.mixer.recurrent == kind for l in self.layers[:layer])
+
+    def n_params(self) -> int:
+        from .fetotar_layout import tensor_shapes
+        n = 0
+        for shape in tensor_shapes(self).values():
+            k = 1
+            for x in shape:
+                k *= x
+            n += k
+        return n
+
+    # ---- config.json -----------------------------------------------------------------------
+    @classmethod
+    def from_json(cls, j: Dict, name: str = "fetotar", max_ctx: Optional[int] = None) -> "FetotarConfig":
+        take(j, ("architecture", "width", "vocab", "norm", "embedding", "token_side", "layers"), "configuration")
+        layers = []
+        for i, l in enumerate(j["layers"]):
+            l = take({"mlp": None, **l}, ("type", "mixer", "mlp"), f"layer {i}")
+            if l["type"] not in MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+            layers.append(LayerSpec(MIXERS[l["type"]].from_json(l["mixer"], f"layer {i} mixer"),
+                                    None if l["mlp"] is None else ClampedGluSpec.from_json(l["mlp"], f"layer {i} mlp")))
+        take(j["norm"], ("eps",), "norm"), take(j["embedding"], ("scale",), "embedding"), take(j["token_side"], ("dim",), "token_side")
+        return cls(name=name, hidden=int(j["width"]), vocab=int(j["vocab"]), layers=tuple(layers),
+                   side_dim=int(j["token_side"]["dim"]), embed_scale=float(j["embedding"]["scale"]),
+                   norm_eps=float(j["norm"]["eps"]), **({} if max_ctx is None else {"max_ctx": max_ctx}))
+
+    def to_json(self) -> Dict:
+        return {"architecture": self.architecture, "width": self.hidden, "vocab": self.vocab, "norm": {"eps": self.norm_eps},
+                "embedding": {"scale": self.embed_scale}, "token_side": {"dim": self.side_dim},
+                "layers": [{"type": l.mixer.type, "mixer": l.mixer.to_json(), "mlp": None if l.mlp is None else l.mlp.to_json()}
+                           for l in self.layers]}
+
+
+def fetotar_tiny() -> FetotarConfig:
+    """Smoke model: every mixer once, with and without a feed-forward, byte vocabulary of 320."""
+    rot = RotarySpec(16, 10000.0, YarnSpec(4.0, 64.0, 8.0, 1.0))
+    return FetotarConfig(
+        name="fetotar-tiny", hidden=72, vocab=320, side_dim=20, embed_scale=1.5, norm_eps=1e-5, max_ctx=4096,
+        layers=(LayerSpec(Mamba2Spec(4, 16, 24, 2, 4, 2), ClampedGluSpec(100, 2.0)),
+                LayerSpec(LatentAttnSpec(5, 24, 16, 32, 40, 48, 0.16, 24, rot), None),
+                LayerSpec(MlstmSpec(3, 24, 16, 10.0), ClampedGluSpec(64, 3.0))))
+
+
+def fetotar_uniform(name: str, *, hidden: int, vocab: int, ff: int, heads: int, repeats: int, window: int, dim: int = 128,
+                    rot_dim: int = 64, kv_rank: int = 512, q_rank: int = 1536, side_dim: int = 256, state: int = 128,
+                    **kw) -> FetotarConfig:
+    """A model of ``repeats`` x (mLSTM, latent attention, Mamba-2) layers of one width, each with a feed-forward; recurrent
+    heads are ``dim`` wide on both sides."""
+    attn = LatentAttnSpec(heads, dim, rot_dim, dim, q_rank, kv_rank, (dim + rot_dim) ** -0.5, window,
+                          RotarySpec(rot_dim, 10000.0, YarnSpec(16.0, 4096.0, 32.0, 1.0)))
+    glu = ClampedGluSpec(ff, 7.0)
+    return FetotarConfig(name=name, hidden=hidden, vocab=vocab, side_dim=side_dim, **kw, layers=repeats * (
+        LayerSpec(MlstmSpec(heads, dim, dim, 15.0), glu), LayerSpec(attn, glu),
+        LayerSpec(Mamba2Spec(heads, dim, state, max(1, heads // 8), 4, 1), glu)))
+
+
+def fetotar_small() -> FetotarConfig:
+    """Three layers of a 1B-class width; profiler captures and GPU engine tests."""
+    return fetotar_uniform("fetotar-small", hidden=2048, vocab=32768, ff=6144, heads=16, repeats=1, window=1024, q_rank=768)
+
+
+ARCHITECTURES = {c.architecture: c for c in (ZinutarConfig, FetotarConfig)}
 
 _REGISTRY = {
+    "fetotar-tiny": fetotar_tiny, "fetotar-small": fetotar_small,
     "zinutar-tiny": zinutar_tiny, "zinutar-small": zinutar_small, "zinutar-8b": zinutar_8b,
     "qwen38-27b": qwen38_27b, "qwen36-27b": qwen36_27b, "tiny": tiny,
     "tiny-hybrid": tiny_hybrid, "small-gpu": small_gpu, "small-gpu-tp": small_gpu_tp,

@@ -779,7 +779,7 @@ class Engine:
             return
         boundary = (len(r.prompt) - 1) // KV_BLOCK * KV_BLOCK
         if boundary and r.n_computed == boundary:
-            snap = self.states.snapshot(r.slot) if self.model.cfg.n_gdn_layers else None
+            snap = self.states.snapshot(r.slot) if self.states.recurrent else None
             self.prefix.insert(r.prompt[:boundary], r.blocks, snap)
             r.published = True
 

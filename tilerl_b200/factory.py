@@ -4,8 +4,8 @@
 a checkpoint directory or from a seeded random initialisation.  Random weights
 are generated tensor by tensor directly on the target device and quantised
 there, so the 27B never exists in full precision anywhere (its fp32 master
-would be 108 GB).  A Zinutar configuration goes to :class:`~tilerl_b200.models.zinutar.ZinutarModel` and the
-packed KV pool, every other one to the hybrid model.  ``fit_blocks`` derives the KV page count from free device
+would be 108 GB).  A stream design goes to its model class (``STREAM_MODELS``) and the
+packed KV pool, every other configuration to the hybrid model.  ``fit_blocks`` derives the KV page count from free device
 memory; ``build_engine`` creates pools, prefix store, CUDA-graph runner and the
 engine.
 
@@ -20,14 +20,18 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import ModelConfig, ZinutarConfig, get_config
+from .config import FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig, get_config
 from .engine import Engine, StepLimits
 from .formats import NVFP4Tensor
-from .kv import GdnStatePool, NoPrefixStore, PrefixStore, kv_pages, make_kv_pool
+from .kv import NoPrefixStore, PrefixStore, kv_pages, make_kv_pool, make_state_pool
+from .models.fetotar import FetotarModel
 from .models.hybrid import HybridModel, linear_names, param_shapes, quantize_weight
 from .models.zinutar import ZinutarModel
 from .ops.backend import RefOps
 from .ops.ref import KV_BLOCK
+
+
+STREAM_MODELS = {ZinutarConfig: ZinutarModel, FetotarConfig: FetotarModel}
 
 
 def _seed_for(name: str, seed: int) -> int:
@@ -111,12 +115,12 @@ def build_model(model: str | ModelConfig, device="cpu", *, seed: int = 0, checkp
     cfg = get_config(model) if isinstance(model, str) else model
     if isinstance(model, str) and checkpoint is None and os.path.isdir(model):
         checkpoint = model
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, StreamDesign):
         if tp > 1 or keep_master or master_only:
-            raise ValueError("Zinutar models are served on one GPU per process; tensor parallelism and training are not built")
+            raise ValueError(f"{cfg.architecture} models are served on one GPU per process; tensor parallelism and training are not built")
         if checkpoint is None:
             on_gpu = torch.device(device).type == "cuda"
-            return ZinutarModel.build_random(cfg, seed, device, act_dtype=dtype or (torch.bfloat16 if on_gpu else torch.float32))
+            return STREAM_MODELS[type(cfg)].build_random(cfg, seed, device, act_dtype=dtype or (torch.bfloat16 if on_gpu else torch.float32))
     elif dtype is not None and dtype != (torch.bfloat16 if torch.device(device).type == "cuda" else torch.float32):
         raise ValueError(f"{cfg.name} does not run in {dtype} on {device}")
     if checkpoint:
@@ -131,9 +135,11 @@ def build_model(model: str | ModelConfig, device="cpu", *, seed: int = 0, checkp
 def fit_blocks(cfg: ModelConfig, free_bytes: int, slots: int, *, planes: int = 1, tp: int = 1,
                pool_fraction: float = 2.0 / 3.0, max_blocks: int = 1 << 20, kv_fp8: bool = False) -> int:
     """KV pages that fit in ``pool_fraction`` of what is left after the GDN state slots."""
-    if isinstance(cfg, ZinutarConfig):
-        per_block = sum(p.n_kv * p.nbytes for p in kv_pages(cfg, 2))
-        return int(max(2, min(max_blocks, free_bytes * pool_fraction // per_block)))
+    if isinstance(cfg, StreamDesign):
+        from .memory import state_slot_bytes
+        per_block = max(1, sum(p.n_kv * p.nbytes for p in kv_pages(cfg, 2)))
+        left = max(0, free_bytes - slots * state_slot_bytes(cfg, 1, planes))
+        return int(max(2, min(max_blocks, left * pool_fraction // per_block)))
     from .parallel.mesh import tp_dims
     d = tp_dims(cfg, tp)
     gd = cfg.gdn_head_dim
@@ -181,11 +187,11 @@ def build_engine(model: HybridModel, ops=None, *, device=None, blocks: Optional[
         raise ValueError("sparse page selection reads a bf16 KV pool on the device: use --kv-format bf16 with --sparse-k")
     kv = make_kv_pool(cfg, blocks, device, getattr(model, "act_dtype", torch.bfloat16 if on_gpu else torch.float32),
                       n_kv_heads=d.n_kv, fp8=kv_fp8)
-    if sparse is not None and isinstance(cfg, ZinutarConfig):
+    if sparse is not None and isinstance(cfg, StreamDesign):
         raise ValueError("sparse page selection is not built for the packed KV pool")
-    st = GdnStatePool(cfg, slots + 1, device, planes=planes,
-                      ring_dtype=torch.bfloat16 if on_gpu else torch.float32,
-                      n_v_heads=d.gdn_nv or None, n_k_heads=d.gdn_nk or None)
+    ring_dtype = model.act_dtype if isinstance(cfg, StreamDesign) else (torch.bfloat16 if on_gpu else torch.float32)
+    st = make_state_pool(cfg, slots + 1, device, planes=planes, ring_dtype=ring_dtype,
+                         n_v_heads=d.gdn_nv or None, n_k_heads=d.gdn_nk or None)
     runner = vrunner = None
     if graph and on_gpu:
         from .graph import DecodeGraphRunner, VerifyGraphRunner

@@ -11,6 +11,8 @@
   ``cur[slot]`` names the live plane, so adopting "the state after n accepted
   tokens" is one int32 write instead of a 144 MiB copy, and the conv window
   needs no rollback at all because the ring is addressed by absolute position.
+* :class:`RecurrentPool` -- the same slots and planes for layers whose state differs in form and size (decayed scans);
+  no counterpart in the reference.
 * :class:`PrefixStore` -- rolling-hash cache of whole 16-token blocks; an entry
   owns refcounted block ids *and* a GDN snapshot taken at the same boundary
   (a hybrid model needs both to resume).
@@ -29,7 +31,8 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from .config import ModelConfig, ZinutarConfig
+from .config import FetotarConfig, ModelConfig, StreamDesign
+from .fetotar_layout import LatentLayout, layout_of, state_layouts
 from .ops.ref import KV_BLOCK
 
 RING = 16  # conv ring rows; >= spec width + conv taps
@@ -176,6 +179,15 @@ class PagedKvPool:
         self.v[:, b].copy_(v)
 
 
+def _page_index(width: int, chunks: int, base: int, itemsize: int) -> torch.Tensor:
+    """Element index inside a packed page of ``[16 rows, width]`` values that start at byte ``base``."""
+    per = 16 // itemsize
+    r = torch.arange(KV_BLOCK)[:, None]
+    d = torch.arange(width)[None, :]
+    c = (d // per) ^ (r % 8) if chunks % 8 == 0 else (d // per + r) % chunks
+    return base // itemsize + (r * chunks + c) * per + d % per
+
+
 @dataclass(frozen=True)
 class KvPage:
     """Byte layout of one page of one KV head in a :class:`PackedKvPool`: 16 K rows, the 16 fp32 reciprocal
@@ -214,27 +226,51 @@ class KvPage:
     def nbytes(self) -> int:
         return self.v_offset + KV_BLOCK * self.v_chunks * 16
 
-    def _index(self, width: int, chunks: int, base: int) -> torch.Tensor:
-        """Element index inside the page of ``[16 rows, width]`` values that start at byte ``base``."""
-        per = 16 // self.itemsize
-        r = torch.arange(KV_BLOCK)[:, None]
-        d = torch.arange(width)[None, :]
-        c = (d // per) ^ (r % 8) if chunks % 8 == 0 else (d // per + r) % chunks
-        return base // self.itemsize + (r * chunks + c) * per + d % per
-
     def k_index(self) -> torch.Tensor:
-        return self._index(self.pad(self.dim), self.k_chunks, 0)
+        return _page_index(self.pad(self.dim), self.k_chunks, 0, self.itemsize)
 
     def v_index(self) -> torch.Tensor:
-        return self._index(self.pad(self.vdim), self.v_chunks, self.v_offset)
+        return _page_index(self.pad(self.vdim), self.v_chunks, self.v_offset, self.itemsize)
 
     def rms_index(self) -> torch.Tensor:
         """Index of the 16 reciprocal root mean squares in the page seen as fp32."""
         return self.rms_offset // 4 + torch.arange(KV_BLOCK)
 
 
-def kv_pages(cfg, itemsize: int) -> Tuple[KvPage, ...]:
-    """Page layout of every KV cache of a design whose layers differ in size (one per layer execution)."""
+@dataclass(frozen=True)
+class LatentPage:
+    """Byte layout of one page of cached latents in a :class:`PackedKvPool`: 16 rows of ``kv`` latent and ``rd`` rotated-key
+    values, shared by every head; the order of a row's 16-byte chunks is that of :class:`KvPage`."""
+    kv: int
+    rd: int
+    itemsize: int
+    n_kv: int = 1
+
+    @staticmethod
+    def of(l: LatentLayout, itemsize: int) -> "LatentPage":
+        return LatentPage(l.kv, l.rd, itemsize)
+
+    @property
+    def width(self) -> int:
+        return self.kv + self.rd
+
+    @property
+    def chunks(self) -> int:
+        return self.width * self.itemsize // 16
+
+    @property
+    def nbytes(self) -> int:
+        return KV_BLOCK * self.chunks * 16
+
+    def index(self) -> torch.Tensor:
+        """Element index inside the page of its ``[16, width]`` values."""
+        return _page_index(self.width, self.chunks, 0, self.itemsize)
+
+
+def kv_pages(cfg, itemsize: int) -> Tuple[object, ...]:
+    """Page layout of every KV cache of a design whose layers differ in size (one per execution of an attention layer)."""
+    if isinstance(cfg, FetotarConfig):
+        return tuple(LatentPage.of(layout_of(m), itemsize) for m in cfg.attn_mixers)
     return tuple(KvPage(a.kv_heads, a.dim, a.vdim, itemsize)
                  for a in (cfg.layers[run.layer].mixer for run in cfg.runs))
 
@@ -249,7 +285,7 @@ class PackedKvPool(PagedKvPool):
     def __init__(self, cfg, num_blocks: int, device="cpu", dtype=torch.bfloat16):
         self.cfg, self.num_blocks, self.dtype = cfg, int(num_blocks), dtype
         self.pages = kv_pages(cfg, torch.empty(0, dtype=dtype).element_size())
-        self.hkv = max(p.n_kv for p in self.pages)
+        self.hkv = max([p.n_kv for p in self.pages] + [1])
         sizes = [self.num_blocks * p.n_kv * p.nbytes for p in self.pages]
         self.k = torch.zeros(sum(sizes), dtype=torch.uint8, device=device)
         self.v = self.k[:0]                  # K and V share the pages
@@ -272,7 +308,7 @@ class PackedKvPool(PagedKvPool):
 
     def read_block(self, b: int) -> Tuple[torch.Tensor, torch.Tensor]:
         """The block's bytes over all caches, in two equal halves (the tiers move pairs of tensors)."""
-        flat = torch.cat([l[b].reshape(-1) for l in self._layers])
+        flat = torch.cat([l[b].reshape(-1) for l in self._layers] or [self.k])
         return flat.view(2, -1)[0].clone(), flat.view(2, -1)[1].clone()
 
     def write_block(self, b: int, k: torch.Tensor, v: torch.Tensor) -> None:
@@ -286,7 +322,7 @@ class PackedKvPool(PagedKvPool):
 def make_kv_pool(cfg, num_blocks: int, device="cpu", dtype=torch.bfloat16, *, fp8: bool = False,
                  n_kv_heads: Optional[int] = None) -> PagedKvPool:
     """The pool a configuration's layers keep K / V in."""
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, StreamDesign):
         if fp8:
             raise ValueError("the packed KV pool holds bf16 or fp32 pages, not fp8")
         return PackedKvPool(cfg, num_blocks, device, dtype)
@@ -300,6 +336,7 @@ class GdnStatePool:
         self.cfg = cfg
         self.num_slots = int(num_slots)
         self.planes = int(planes)
+        self.recurrent = cfg.n_gdn_layers > 0     # False: the slots hold nothing
         self.nv = n_v_heads or cfg.gdn_v_heads
         self.nk = n_k_heads or cfg.gdn_k_heads
         ng = max(1, cfg.n_gdn_layers)
@@ -346,6 +383,84 @@ class GdnStatePool:
         self.states[slot, :, 0].copy_(snap[0])
         self.cur[slot] = 0
         self.ring[slot].copy_(snap[1])
+
+
+class RecurrentPool:
+    """State slots of decayed-scan layers that differ in form and size: ``states [slots, planes, floats]`` fp32, every
+    layer's record at a fixed offset (``fetotar_layout``: ``S [heads, dk, dv]``, then an mLSTM's key sum and running
+    maximum), and a ring ``[slots, rows, channels]`` of convolution inputs indexed by ``position % rows``.  ``planes`` and
+    ``cur`` work as in :class:`GdnStatePool`."""
+
+    def __init__(self, cfg: FetotarConfig, num_slots: int, device="cpu", planes: int = 1, ring_dtype=torch.bfloat16):
+        self.cfg, self.num_slots, self.planes = cfg, int(num_slots), int(planes)
+        self.layouts = state_layouts(cfg)
+        self.recurrent = bool(self.layouts)
+        self.offsets, self.channels, n, c = [], [], 0, 0
+        for l in self.layouts:
+            self.offsets.append(n)
+            self.channels.append(c)
+            n += l.state_floats
+            c += l.conv_c
+        rows = max([l.taps - 1 for l in self.layouts] + [0]) + self.planes
+        self.ring_rows = max(RING, 1 << (rows - 1).bit_length())
+        self.states = torch.zeros(self.num_slots, self.planes, max(1, n), dtype=torch.float32, device=device)
+        self.ring = torch.zeros(self.num_slots, self.ring_rows, max(1, c), dtype=ring_dtype, device=device)
+        self.cur = torch.zeros(self.num_slots, dtype=torch.int32, device=device)
+        self._free = list(range(self.num_slots - 1, 0, -1))  # slot 0 = pad slot
+
+    @property
+    def free_slots(self) -> int:
+        return len(self._free)
+
+    def alloc_slot(self) -> int:
+        if not self._free:
+            raise PoolExhausted("state pool has no free slot")
+        s = self._free.pop()
+        self.states[s].zero_()
+        self.ring[s].zero_()
+        self.cur[s] = 0
+        return s
+
+    def release(self, s: int) -> None:
+        assert s != 0 and s not in self._free
+        self._free.append(s)
+
+    def slot_bytes(self) -> int:
+        return self.states[0].numel() * 4 + self.ring[0].numel() * self.ring.element_size()
+
+    def view(self, idx: int, slot: int, plane: int) -> List[torch.Tensor]:
+        """The parts of one layer's state: ``S`` and, for an mLSTM, the copies of ``n`` and ``m``."""
+        l, o = self.layouts[idx], self.offsets[idx]
+        rec = self.states[slot, plane, o:o + l.state_floats]
+        k = l.heads * l.dk * l.dv
+        parts = [rec[:k].view(l.heads, l.dk, l.dv)]
+        if l.kind == "mlstm":
+            c = l.heads * l.copies
+            parts += [rec[k:k + c * l.dk].view(l.heads, l.copies, l.dk), rec[k + c * l.dk:k + c * (l.dk + 1)].view(l.heads, l.copies)]
+        return parts
+
+    def ring_view(self, idx: int, slot: int) -> torch.Tensor:
+        return self.ring[slot, :, self.channels[idx]:self.channels[idx] + self.layouts[idx].conv_c]
+
+    def select_step(self, slot: int, step: int) -> None:
+        """Adopt the state stored after token ``step`` (0-based) of the last verify tick."""
+        self.cur[slot] = step
+
+    def snapshot(self, slot: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        return self.states[slot, int(self.cur[slot])].clone(), self.ring[slot].clone()
+
+    def restore(self, slot: int, snap: Tuple[torch.Tensor, torch.Tensor]) -> None:
+        self.states[slot, 0].copy_(snap[0])
+        self.cur[slot] = 0
+        self.ring[slot].copy_(snap[1])
+
+
+def make_state_pool(cfg, num_slots: int, device="cpu", *, planes: int = 1, ring_dtype=torch.bfloat16,
+                    n_v_heads: Optional[int] = None, n_k_heads: Optional[int] = None):
+    """The pool a configuration's recurrent layers keep their state in (it also hands out the slots of designs without any)."""
+    if isinstance(cfg, FetotarConfig):
+        return RecurrentPool(cfg, num_slots, device, planes=planes, ring_dtype=ring_dtype)
+    return GdnStatePool(cfg, num_slots, device, planes=planes, ring_dtype=ring_dtype, n_v_heads=n_v_heads, n_k_heads=n_k_heads)
 
 
 # ---- prefix store ------------------------------------------------------------------

@@ -17,7 +17,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
-from .config import ModelConfig, ZinutarConfig
+from .config import FetotarConfig, ModelConfig, StreamDesign
 from .formats import nbytes, weight_specs
 from .parallel.mesh import is_sharded, tp_dims
 
@@ -50,7 +50,7 @@ def weight_bytes(cfg: ModelConfig, tp: int = 1, tiled_copy: bool = True) -> int:
 
 
 def kv_block_bytes(cfg: ModelConfig, tp: int = 1, fp8: bool = False) -> int:
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, StreamDesign):
         from .kv import kv_pages
         return sum(p.n_kv * p.nbytes for p in kv_pages(cfg, 2))
     d = tp_dims(cfg, tp)
@@ -61,6 +61,9 @@ def kv_block_bytes(cfg: ModelConfig, tp: int = 1, fp8: bool = False) -> int:
 
 
 def state_slot_bytes(cfg: ModelConfig, tp: int = 1, planes: int = 1) -> int:
+    if isinstance(cfg, FetotarConfig):
+        from .fetotar_layout import state_layouts
+        return sum(planes * l.state_floats * 4 + 16 * l.conv_c * 2 for l in state_layouts(cfg))
     if not cfg.n_gdn_layers:
         return 0
     d = tp_dims(cfg, tp)
@@ -95,7 +98,16 @@ def indexer_bytes(cfg: ModelConfig, *, heads: int = 4, dim: int = 128, tp: int =
 
 def workspace_bytes(cfg: ModelConfig, tokens: int, tp: int = 1) -> int:
     """Activation buffers of a tick of ``tokens`` tokens and the logits of 64 rows."""
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, FetotarConfig):
+        from .fetotar_layout import head_rows, layouts, pad, side_width, stream_width
+        ls, glu = layouts(cfg), max([pad(b.mlp.ff, 64) for b in cfg.layers if b.mlp is not None] + [0])
+        # fp32 stream and branch output, bf16 normed row, fused projection rows, mixer output, feed-forward, side input;
+        # attention: query heads, latent queries and sums, a prompt's expanded keys / values; scans: fp32 rows, convolution
+        per = stream_width(cfg) * (4 + 4 + 2) + 2 * max(l.n_in for l in ls) + 2 * max(l.n_out for l in ls) + 6 * glu + 2 * side_width(cfg)
+        per += max([2 * l.heads * (l.dq + l.row + 2 * l.kv + l.dk + l.dv) for l in ls if l.kind == "latent"] + [0])
+        per += max([4 * l.heads * l.dv + 2 * l.conv_c for l in ls if l.kind != "latent"] + [0])
+        return tokens * per + head_rows(cfg) * 4 * 64
+    if isinstance(cfg, StreamDesign):
         from .zinutar_layout import BlockLayout, head_rows, stream_width
         ls = [BlockLayout.of(b) for b in cfg.layers]
         # fp32 stream and embedding output, bf16 normed row, fused projection rows, block middle
@@ -167,8 +179,8 @@ def train_plan(cfg: ModelConfig, *, mode: str = "lora", rank: int = 16, zero: in
     matrices, Adafactor for the vectors)."""
     if optimizer not in ("adamw", "adafactor", "iso"):
         raise ValueError(f"unknown optimizer {optimizer!r}")
-    if isinstance(cfg, ZinutarConfig):
-        raise ValueError("Zinutar models are served, not trained")
+    if isinstance(cfg, StreamDesign):
+        raise ValueError(f"{cfg.architecture} models are served, not trained")
     n = cfg.n_params()
     rows: Dict[str, int] = {}
     if mode == "lora":

@@ -18,6 +18,7 @@ from typing import Optional
 import torch
 
 from . import ref
+from .ref_mixers import RefMixers
 
 
 class TPContext:
@@ -27,7 +28,7 @@ class TPContext:
         self.rank, self.world, self.group = rank, world, group
 
 
-class RefOps:
+class RefOps(RefMixers):
     name = "ref"
 
     def __init__(self, tp: Optional[TPContext] = None, act_dtype=torch.float32):

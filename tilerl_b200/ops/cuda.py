@@ -26,6 +26,7 @@ import torch
 
 from ..formats import FP8BlockTensor, NVFP4Tensor
 from . import native as N
+from .cuda_mixers import MixerOps
 from .cuda_stream import StreamOps
 
 EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_STORE_F32 = 0, 1, 2, 3
@@ -68,7 +69,7 @@ class Workspace:
         return t[:n].view(*shape)
 
 
-class CudaOps(StreamOps):
+class CudaOps(StreamOps, MixerOps):
     name = "cuda"
 
     def __init__(self, device="cuda", tp=None, comm=None, attn_splits: int = 0, use_tc_gemm: bool = True,

@@ -1,0 +1,169 @@
+"""CUDA ops of sandwich-normed stream designs (``models/fetotar.py``): joins, latent attention, decayed scans.
+
+Mixed into :class:`tilerl_b200.ops.cuda.CudaOps` beside :class:`~tilerl_b200.ops.cuda_stream.StreamOps`, whose projections
+they use.  The activation type is that of the weights: bf16 (the serving type) or fp32 (true fp32 everywhere).  No
+counterpart in the reference.
+"""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from . import native as N
+from .cuda_stream import EPI_STORE_F32
+
+MAMBA2, MLSTM = 0, 1
+
+
+class ScanArgs(ctypes.Structure):
+    """``ScanArgs`` of ``csrc/scan.cuh``."""
+    _fields_ = ([(n, ctypes.c_void_p) for n in ("rows", "gates", "gate_b", "a_log", "skip", "states", "cur", "keep_flags",
+                                                "q_start", "q_len", "slots", "o")]
+                + [(n, ctypes.c_long) for n in ("slot_stride", "plane_stride")]
+                + [(n, ctypes.c_int) for n in ("ld", "q0", "k0", "v0", "ldg", "heads", "per", "dk", "dv", "min_len", "max_len")]
+                + [(n, ctypes.c_float) for n in ("cap", "q_scale")])
+
+
+def _f32(t: torch.Tensor) -> int:
+    return int(t.dtype == torch.float32)
+
+
+def _norm_kind(norm) -> int:
+    return 0 if norm is None else norm.shape[0]
+
+
+class MixerOps:
+    # ---- stream ----------------------------------------------------------------------
+    def _join(self, x, y, post, nxt, h, table, ids, scale, eps, n):
+        t, ld = x.shape
+        N.check(self.lib.trl_join(x.data_ptr(), N.ptr(y), N.ptr(post), _norm_kind(post), N.ptr(nxt), _norm_kind(nxt), h.data_ptr(),
+                                  N.ptr(table), N.ptr(ids), scale, 0 if table is None else table.shape[0], t, ld, n, eps, _f32(h),
+                                  N.stream()), "join")
+        N.count()
+        return h
+
+    def embed_stream(self, table, ids, scale, norm, eps, n):
+        t, ld = ids.shape[0], table.shape[1]
+        x, h = self.ws.get("stream", (t, ld), torch.float32), self.ws.get(f"join_h_{table.dtype}", (t, ld), table.dtype)
+        self._join_dtype = table.dtype
+        return x, self._join(x, None, None, norm, h, table, ids, scale, eps, n)
+
+    def join(self, x, y, post, nxt, eps, n):
+        """``x += norm_post(y)``; returns ``norm_nxt(x)`` (or x rounded) as the next projection's input."""
+        h = self.ws.get(f"join_h_{self._join_dtype}", tuple(x.shape), self._join_dtype)
+        return self._join(x, y, post, nxt, h, None, None, 1.0, eps, n)
+
+    def _mm(self, a, w, y):
+        if y.dtype == w.dtype:
+            torch.mm(a, w.t(), out=y)
+        else:
+            torch.mm(a, w.t(), out_dtype=y.dtype, out=y)
+        return y
+
+    def project_gates(self, h, w, n_in):
+        t, ng = h.shape[0], w.shape[0] - n_in
+        proj = self.ws.get(f"block_proj_{w.dtype}", (t, n_in), w.dtype)
+        gates = self.ws.get("mix_gates", (t, max(ng, 1)), torch.float32)
+        self._mm(h, w[:n_in], proj)
+        if ng:
+            self._mm(h, w[n_in:], gates)
+        return proj, gates
+
+    def project_f32(self, a, w):
+        y = self.ws.get("branch", (a.shape[0], w.shape[0]), torch.float32)
+        if self._streams(a.shape[0], w):
+            self._linear_rows(a, w, y, EPI_STORE_F32)
+            return y
+        return self._mm(a, w, y)
+
+    def project_logits(self, h, w):
+        logits = self.ws.get("logits", (h.shape[0], w.shape[0]), torch.float32)
+        h = h.contiguous()
+        if self._streams(h.shape[0], w):
+            self._linear_rows(h, w, logits, EPI_STORE_F32)
+            return logits
+        return self._mm(h, w, logits)
+
+    def clamped_glu(self, h, w, limit):
+        t, n = h.shape[0], w.shape[0]
+        out = self.ws.get(f"glu_{w.dtype}", (t, n // 2), w.dtype)
+        gu = self._mm(h, w, self.ws.get(f"gate_up_{w.dtype}", (t, n), w.dtype))
+        N.check(self.lib.trl_clamped_glu(gu.data_ptr(), out.data_ptr(), out.numel(), limit, _f32(w), N.stream()), "clamped_glu")
+        N.count()
+        return out
+
+    def side_input(self, h, w, table, ids, layer, dim):
+        t, n = h.shape[0], w.shape[0]
+        out = self.ws.get(f"side_{w.dtype}", (t, n), w.dtype)
+        z = self._mm(h, w, self.ws.get(f"side_z_{w.dtype}", (t, n), w.dtype))
+        N.check(self.lib.trl_side_input(z.data_ptr(), table.data_ptr(), ids.data_ptr(), out.data_ptr(), t, n, dim, table.shape[1],
+                                        layer * ((dim + 7) // 8 * 8), table.shape[0], _f32(w), N.stream()), "side_input")
+        N.count()
+        return out
+
+    # ---- latent attention ----------------------------------------------------------------
+    def latent_prep(self, proj, l, q_norm, kv_norm, uq, freqs, rot, batch, pool, idx, eps):
+        t, cache, st = proj.shape[0], pool.layer(idx), N.stream()
+        cq = self.ws.get(f"latent_cq_{proj.dtype}", (t, l.c0), proj.dtype)
+        N.check(self.lib.trl_latent_prep(
+            proj.data_ptr(), proj.stride(0), q_norm.data_ptr(), kv_norm.data_ptr(), freqs.data_ptr(), batch.positions.data_ptr(),
+            batch.slot_mapping.data_ptr(), cq.data_ptr(), cache.data_ptr(), cache.shape[0], t, l.c0, l.kr0, l.q_rank, l.kv_rank, l.kv,
+            l.rd, freqs.numel(), rot.amplitude, eps, _f32(proj), st), "latent_prep")
+        q = self._mm(cq, uq, self.ws.get(f"latent_q_{proj.dtype}", (t, uq.shape[0]), proj.dtype))
+        N.check(self.lib.trl_latent_rope(q.data_ptr(), freqs.data_ptr(), batch.positions.data_ptr(), t, l.heads, l.dq, l.dk, freqs.numel(),
+                                         rot.amplitude, _f32(q), st), "latent_rope")
+        N.count(2)
+        return q.view(t, l.heads, l.dq)
+
+    def latent_attention(self, q, proj, up, l, batch, pool, idx):
+        t, cache, table, dt, st = proj.shape[0], pool.layer(idx), batch.block_table, proj.dtype, N.stream()
+        uk, uv = up[:l.heads * l.dk].view(l.heads, l.dk, l.kv), up[l.heads * l.dk:].view(l.heads, l.dv, l.kv)
+        ql = self.ws.get(f"latent_ql_{dt}", (l.heads, t, l.kv), dt)
+        oc = self.ws.get(f"latent_oc_{dt}", (l.heads, t, l.kv), dt)
+        ov = self.ws.get(f"latent_ov_{dt}", (l.heads, t, l.dv), dt)
+        torch.bmm(q.transpose(0, 1)[:, :, :l.dk], uk, out=ql)
+        N.check(self.lib.trl_latent_attn(
+            ql.data_ptr(), t * l.kv, l.kv, q.data_ptr(), l.dq, l.dk, cache.data_ptr(), l.kv, l.rd, cache.shape[0], table.data_ptr(),
+            table.stride(0), batch.q_start.data_ptr(), batch.q_len.data_ptr(), batch.positions.data_ptr(), oc.data_ptr(), t * l.kv, l.kv,
+            batch.n_seqs, batch.max_q_len, l.heads, l.window, l.scale, _f32(proj), st), "latent_attn")
+        torch.bmm(oc, uv.transpose(1, 2), out=ov)
+        out = self.ws.get(f"mix_out_{dt}", (t, l.n_out), dt)
+        N.check(self.lib.trl_latent_gate(ov.data_ptr(), proj[:, l.g0:].data_ptr(), proj.stride(0), out.data_ptr(), l.n_out, t, l.heads,
+                                         l.dv, _f32(proj), st), "latent_gate")
+        N.count(2)
+        return out
+
+    # ---- recurrent mixers ------------------------------------------------------------------
+    def recurrent_mix(self, proj, gates, w, l, batch, pool, idx, eps):
+        t, dt, st = proj.shape[0], proj.dtype, N.stream()
+        kind = MAMBA2 if l.kind == "mamba2" else MLSTM
+        ring = pool.ring_view(idx, 0) if kind == MAMBA2 else None
+        o = self.ws.get("scan_o", (t, l.heads * l.dv), torch.float32)
+        a = ScanArgs()
+        if kind == MAMBA2:
+            rows = self.ws.get(f"scan_conv_{dt}", (t, l.conv_c), dt)
+            N.check(self.lib.trl_scan_conv(
+                proj.data_ptr(), proj.stride(0), w["conv"].data_ptr(), w["conv_b"].data_ptr(), ring.data_ptr(), pool.ring.stride(0),
+                pool.ring_rows, pool.ring.stride(1), batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(),
+                batch.state_slots.data_ptr(), rows.data_ptr(), t, l.conv_c, l.taps, _f32(proj), st), "scan_conv")
+            N.count()
+            a.q0, a.k0, a.v0, a.per, a.q_scale, a.cap = l.q0, l.k0, 0, l.heads // l.groups, 1.0, 1.0
+        else:
+            rows = proj
+            a.q0, a.k0, a.v0, a.per, a.q_scale, a.cap = 0, l.k0, l.v0, 1, l.dim ** -0.5, l.cap
+        a.rows, a.ld, a.gates, a.ldg = rows.data_ptr(), rows.stride(0), gates.data_ptr(), gates.stride(0)
+        a.gate_b, a.a_log, a.skip = w["gate_b"].data_ptr(), N.ptr(w["a_log"]), N.ptr(w["skip"])
+        a.states, a.slot_stride, a.plane_stride = pool.states.data_ptr() + 4 * pool.offsets[idx], pool.states.stride(0), pool.states.stride(1)
+        a.cur, a.keep_flags = pool.cur.data_ptr(), N.ptr(batch.keep_flags) if batch.keep_steps else None
+        a.q_start, a.q_len, a.slots = batch.q_start.data_ptr(), batch.q_len.data_ptr(), batch.state_slots.data_ptr()
+        a.o, a.heads, a.dk, a.dv, a.min_len, a.max_len = o.data_ptr(), l.heads, l.dk, l.dv, 1, 1 << 30
+        N.check(self.lib.trl_scan_serial(ctypes.byref(a), batch.n_seqs, kind, _f32(proj), st), "scan_serial")
+        out = self.ws.get(f"mix_out_{dt}", (t, l.n_out), dt)
+        N.check(self.lib.trl_scan_norm(
+            o.data_ptr(), proj[:, l.g0:].data_ptr(), proj.stride(0), w["norm"].data_ptr(), out.data_ptr(), l.n_out, t, l.heads, l.vdim, l.dv,
+            l.norm_groups, eps, proj.data_ptr(), N.ptr(ring), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1), l.conv_c,
+            batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(), batch.q_len.data_ptr(),
+            batch.state_slots.data_ptr(), kind, _f32(proj), st), "scan_norm")
+        N.count(2)
+        return out

@@ -84,6 +84,17 @@ _SIGS = {
     "trl_sigmoid_attn_rows": [I, I],
     "trl_sigmoid_attn": [P, I, P, I, P, I, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P],
     "trl_sigmoid_attn_f32": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P],
+    # sandwich-normed layers: joins, latent attention, decayed scans (csrc/join.cu, latent.cu, scan.cu)
+    "trl_join": [P, P, P, I, P, I, P, P, P, F, I, I, I, I, F, I, P],
+    "trl_clamped_glu": [P, P, L, F, I, P],
+    "trl_side_input": [P, P, P, P, I, I, I, L, I, I, I, P],
+    "trl_latent_prep": [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, P],
+    "trl_latent_rope": [P, P, P, I, I, I, I, I, F, I, P],
+    "trl_latent_gate": [P, P, I, P, I, I, I, I, I, P],
+    "trl_latent_attn": [P, L, L, P, I, I, P, I, I, I, P, I, P, P, P, P, L, L, I, I, I, I, F, I, P],
+    "trl_scan_conv": [P, I, P, P, P, L, I, I, P, P, P, P, P, I, I, I, I, P],
+    "trl_scan_serial": [P, I, I, I, P],
+    "trl_scan_norm": [P, P, I, P, P, I, I, I, I, I, I, F, P, P, L, I, I, I, P, P, P, P, P, I, I, P],
     "trl_decode_advance": [P, P, P, P, P, P, I, I, P, I, P, P],
 }
 

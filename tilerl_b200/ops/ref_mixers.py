@@ -1,0 +1,232 @@
+"""fp32 torch form of the stream designs' mechanisms (latent attention, decayed scans, norms, gates) and, on top of
+them, the op surface :class:`RefMixers` that ``models/fetotar.py`` calls; mixed into
+:class:`~tilerl_b200.ops.backend.RefOps`.  The CUDA twin is :mod:`tilerl_b200.ops.cuda_mixers`.  No counterpart in the
+reference.
+"""
+from __future__ import annotations
+
+import math
+
+import torch
+import torch.nn.functional as F
+
+from . import ref
+from .ref import KV_BLOCK
+
+
+# ---- element-wise and norms --------------------------------------------------------------------------
+def stream_norm(x, norm, eps: float, n: int):
+    """``norm``: ``[2, width]`` weight and bias of a layer norm, ``[1, width]`` weight of an RMS norm, None for the row
+    itself.  The first ``n`` columns count; columns past them come out as zeros (weights and biases are zero there)."""
+    if norm is None:
+        return x
+    if norm.shape[0] == 1:
+        return x * ref.rms_factor(x, n, eps)[:, None] * norm[0]
+    mean = x[:, :n].sum(-1, keepdim=True) / n
+    var = (x[:, :n] - mean).pow(2).sum(-1, keepdim=True) / n
+    return (x - mean) * torch.rsqrt(var + eps) * norm[0] + norm[1]
+
+
+def clamped_glu(gate_up, limit: float):
+    """Rows ``2j`` = gate, ``2j + 1`` = up: ``g sigmoid(1.702 g) (u + 1)`` with ``g`` bounded above, ``u`` on both sides."""
+    g, u = gate_up[..., 0::2].clamp(max=limit), gate_up[..., 1::2].clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z.pow(3))))
+
+
+# ---- latent attention ----------------------------------------------------------------------------------
+def rotate_pairs(x, positions, freqs, amplitude: float):
+    """Turn the leading ``2 len(freqs)`` columns of ``x [T, ..., width]`` in neighbouring pairs."""
+    ang = positions.to(torch.float64)[:, None] * freqs.to(positions.device)[None, :]
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [freqs.numel()]
+    c, s = (ang.cos() * amplitude).float().view(shape), (ang.sin() * amplitude).float().view(shape)
+    k = 2 * freqs.numel()
+    u, v = x[..., 0:k:2], x[..., 1:k:2]
+    out = x.clone()
+    out[..., 0:k:2], out[..., 1:k:2] = u * c - v * s, v * c + u * s
+    return out
+
+
+def latent_write(cache, page, rows, slot_mapping):
+    """Cached rows ``[T, width]`` into ``cache [blocks, 1, page bytes]``."""
+    el, idx = cache.view(rows.dtype), page.index().to(rows.device)
+    for t in range(rows.shape[0]):
+        s = int(slot_mapping[t])
+        if s >= 0:
+            el[s // KV_BLOCK, 0, idx[s % KV_BLOCK]] = rows[t]
+
+
+def latent_gather(cache, page, dtype, block_row, lo: int, hi: int):
+    """Cached rows of positions ``lo .. hi - 1`` of one sequence, fp32."""
+    first = lo // KV_BLOCK
+    pages = cache[block_row[first:(hi + KV_BLOCK - 1) // KV_BLOCK].long()]
+    rows = pages.view(dtype)[:, 0, page.index().to(cache.device)].float().reshape(-1, page.width)
+    return rows[lo - first * KV_BLOCK:hi - first * KV_BLOCK]
+
+
+def latent_attention(q, rows, kv: int, scale: float):
+    """One query token over the rows it sees: ``q [heads, kv + rd]`` (the unrotated part already mapped into the latent),
+    ``rows [n, kv + rd]``; softmax-weighted sum of the latents ``[heads, kv]``."""
+    return torch.softmax(q @ rows.t() * scale, dim=-1) @ rows[:, :kv]
+
+
+# ---- decayed scans ---------------------------------------------------------------------------------------
+def conv_rows(rows, taps, bias):
+    """``rows [k, C]`` (oldest first), ``taps [k, C]`` -> silu of the depthwise convolution's newest output."""
+    return F.silu((rows * taps).sum(0) + bias)
+
+
+def mamba2_step(state, x, b, c, dt, a_log, skip):
+    """``state [H, N, V]``; ``x [H, V]``, ``b, c [H, N]`` (groups expanded), ``dt [H]``."""
+    s = torch.exp(-torch.exp(a_log) * dt)[:, None, None] * state + (dt[:, None] * b)[:, :, None] * x[:, None, :]
+    return s, torch.einsum("hnv,hn->hv", s, c) + skip[:, None] * x
+
+
+def mlstm_gates(raw, bias, cap: float):
+    """Raw gates ``[..., 2H]`` -> (log input gate, log forget gate)."""
+    z = cap * torch.tanh((raw + bias) / cap)
+    h = raw.shape[-1] // 2
+    return z[..., :h], F.logsigmoid(z[..., h:])
+
+
+def mlstm_step(state, n, m, q, k, v, i, f):
+    """``state [H, D, V]``, ``n [H, D]``, ``m [H]``."""
+    new = torch.maximum(f + m, i)
+    keep, add = torch.exp(f + m - new), torch.exp(i - new)
+    s = keep[:, None, None] * state + (add[:, None] * k)[:, :, None] * v[:, None, :]
+    n = keep[:, None] * n + add[:, None] * k
+    den = torch.maximum((n * q).sum(-1).abs(), torch.exp(-new)) + 1e-6
+    return s, n, new, torch.einsum("hdv,hd->hv", s, q) / den[:, None]
+
+
+def grouped_rms(y, heads: int, vdim: int, dv: int, groups: int, eps: float):
+    """RMS norm without a weight over ``groups`` equal parts of the true columns of ``y [T, heads * dv]``."""
+    t = y.shape[0]
+    v = y.view(t, heads, dv)[:, :, :vdim].reshape(t, groups, -1)
+    out = torch.zeros_like(y)
+    out.view(t, heads, dv)[:, :, :vdim] = (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)).view(t, heads, vdim)
+    return out
+
+
+class RefMixers:
+    """Ops of an fp32 stream with sandwich norms, and its mixers (mixed into RefOps: ``act_dtype``)."""
+
+    # ---- stream ----------------------------------------------------------------------
+    def embed_stream(self, table, ids, scale, norm, eps, n):
+        """(stream, first normed row): the scaled embedding."""
+        x = ref.embedding(table, ids) * scale
+        return x, stream_norm(x, norm, eps, n).to(self.act_dtype)
+
+    def join(self, x, y, post, nxt, eps, n):
+        """``x += norm_post(y)``; the next projection's input ``norm_nxt(x)``."""
+        x += stream_norm(y, post, eps, n)
+        return stream_norm(x, nxt, eps, n).to(self.act_dtype)
+
+    def project_gates(self, h, w, n_in):
+        """(fused projection rows, fp32 gate rows)."""
+        return ref.linear(h, w[:n_in]).to(self.act_dtype), ref.linear(h, w[n_in:])
+
+    def project_f32(self, a, w):
+        return ref.linear(a, w)
+
+    def project_logits(self, h, w):
+        return ref.linear(h, w)
+
+    def clamped_glu(self, h, w, limit):
+        return clamped_glu(ref.linear(h, w), limit).to(self.act_dtype)
+
+    def side_input(self, h, w, table, ids, layer, dim):
+        """``gelu(W h) * side[token, layer]``, zero past ``dim``."""
+        z = ref.linear(h, w)
+        stride = (dim + 7) // 8 * 8
+        e = torch.zeros_like(z)
+        e[:, :dim] = table[ids.long()][:, layer * stride:layer * stride + dim].float()
+        return (gelu_tanh(z) * e).to(self.act_dtype)
+
+    # ---- latent attention ----------------------------------------------------------------
+    def latent_prep(self, proj, l, q_norm, kv_norm, uq, freqs, rot, batch, pool, idx, eps):
+        """Normed latents and the rotated shared key into the cache; returns the query heads ``[T, heads, dk + rd]`` with
+        their rotated part turned."""
+        t = proj.shape[0]
+        cq = proj[:, :l.c0].float()
+        cq = (cq * ref.rms_factor(cq, l.q_rank, eps)[:, None] * q_norm).to(self.act_dtype)
+        c = proj[:, l.c0:l.kr0].float()
+        c = c * ref.rms_factor(c, l.kv_rank, eps)[:, None] * kv_norm
+        kr = rotate_pairs(proj[:, l.kr0:l.g0].float(), batch.positions, freqs, rot.amplitude)
+        latent_write(pool.layer(idx), pool.pages[idx], torch.cat([c, kr], 1).to(pool.dtype), batch.slot_mapping)
+        q = ref.linear(cq, uq).view(t, l.heads, l.dq)
+        q[:, :, l.dk:] = rotate_pairs(q[:, :, l.dk:], batch.positions, freqs, rot.amplitude)
+        return q.to(self.act_dtype)
+
+    def latent_attention(self, q, proj, up, l, batch, pool, idx):
+        """Gated attention output, padded to the output projection's columns."""
+        t = proj.shape[0]
+        uk, uv = up.float().split([l.heads * l.dk, l.heads * l.dv])
+        uk, uv = uk.view(l.heads, l.dk, l.kv), uv.view(l.heads, l.dv, l.kv)
+        ql = torch.cat([torch.einsum("thd,hdc->thc", q[:, :, :l.dk].float(), uk), q[:, :, l.dk:].float()], -1)
+        out = torch.zeros(t, l.n_out, dtype=self.act_dtype, device=proj.device)
+        for i in range(t):
+            p = int(batch.positions[i])
+            rows = latent_gather(pool.layer(idx), pool.pages[idx], pool.dtype, batch.block_table[int(batch.seq_ids[i])],
+                                 max(0, p + 1 - l.window), p + 1)
+            o = torch.einsum("hc,hdc->hd", latent_attention(ql[i], rows, l.kv, l.scale), uv).reshape(-1)
+            out[i, :l.heads * l.dv] = (o * torch.sigmoid(proj[i, l.g0:l.n_in].float())).to(self.act_dtype)
+        return out
+
+    # ---- recurrent mixers ------------------------------------------------------------------
+    def recurrent_mix(self, proj, gates, w, l, batch, pool, idx, eps):
+        """Normed and gated output of a decayed scan; state and convolution inputs move on in ``pool``."""
+        t, dev = proj.shape[0], proj.device
+        y = torch.zeros(t, l.heads * l.dv, dtype=torch.float32, device=dev)
+        gate = proj[:, l.g0:l.n_in].float()
+        for r in range(batch.n_seqs):
+            s0, n = int(batch.q_start[r]), int(batch.q_len[r])
+            if n == 0:
+                continue
+            slot = int(batch.state_slots[r])
+            keep = bool(batch.keep_steps) and batch.keep_rows[r]
+            state = pool.view(idx, slot, int(pool.cur[slot]))
+            parts = [a.clone() for a in state]
+            ring = pool.ring_view(idx, slot)
+            for j in range(n):
+                tt = s0 + j
+                if l.kind == "mamba2":
+                    parts, y[tt] = self._mamba2_token(proj[tt], gates[tt], w, l, parts, ring, int(batch.positions[tt]))
+                else:
+                    parts, y[tt] = self._mlstm_token(proj[tt], gates[tt], w, l, parts)
+                if keep:
+                    for a, b in zip(pool.view(idx, slot, j), parts):
+                        a.copy_(b)
+            if not keep:
+                for a, b in zip(state, parts):
+                    a.copy_(b)
+        if l.kind == "mamba2":
+            y = y * F.silu(gate)
+        y = grouped_rms(y, l.heads, l.vdim, l.dv, l.norm_groups, eps) * w["norm"]
+        if l.kind == "mlstm":
+            y = y * torch.sigmoid(gate)
+        out = torch.zeros(t, l.n_out, dtype=self.act_dtype, device=dev)
+        out[:, :l.heads * l.dv] = y.to(self.act_dtype)
+        return out
+
+    def _mamba2_token(self, row, gates, w, l, parts, ring, pos):
+        rows = ring.shape[0]
+        ring[pos % rows] = row[:l.conv_c].to(ring.dtype)
+        taken = [ring[(pos - j) % rows].float() if pos >= j else torch.zeros(l.conv_c) for j in range(l.taps - 1, -1, -1)]
+        c = conv_rows(torch.stack(taken), w["conv"], w["conv_b"]).to(self.act_dtype).float()
+        per = l.heads // l.groups
+        x = c[:l.k0].view(l.heads, l.dv)
+        b, cc = (a.view(l.groups, l.dk).repeat_interleave(per, 0) for a in (c[l.k0:l.q0], c[l.q0:]))
+        s, y = mamba2_step(parts[0], x, b, cc, F.softplus(gates[:l.heads].float() + w["gate_b"]), w["a_log"], w["skip"])
+        return [s], y.reshape(-1)
+
+    def _mlstm_token(self, row, gates, w, l, parts):
+        row = row.float()
+        q = row[:l.k0].view(l.heads, l.dk) * l.dim ** -0.5
+        k, v = row[l.k0:l.v0].view(l.heads, l.dk), row[l.v0:l.g0].view(l.heads, l.dv)
+        i, f = mlstm_gates(gates[:2 * l.heads].float(), w["gate_b"], l.cap)
+        s, n, m, o = mlstm_step(parts[0], parts[1][:, 0], parts[2][:, 0], q, k, v, i, f)
+        return [s, n[:, None].expand_as(parts[1]), m[:, None].expand_as(parts[2])], o.reshape(-1)
