@@ -15,7 +15,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Dict, List, Optional
 
-from .config import ATTN, ModelConfig, ZinutarConfig
+from .config import ATTN, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig
 from .formats import FORMATS, nbytes
 from .parallel.mesh import tp_dims
 
@@ -73,10 +73,40 @@ def _zinutar_rows(cfg: ZinutarConfig, m: int, pairs: float, kv_read: float, head
     return rows
 
 
+def _fetotar_rows(cfg: FetotarConfig, m: int, ctx: int, n_seqs: int, head_rows_m: int) -> List[Row]:
+    """One forward of ``m`` tokens in ``n_seqs`` sequences that end at ``ctx`` tokens each."""
+    from .fetotar_layout import head_rows, layout_of, pad, side_width, stream_width
+    w, q = stream_width(cfg), m // n_seqs
+    lin = lambda name, n, k, out=2: Row(name, 1, n * k * 2 + m * (k * 2 + n * out), 2.0 * m * n * k)
+    rows = [Row("embedding + norm", 1, m * w * (2 + 4 + 2), 0)]
+    for i, b in enumerate(cfg.layers):
+        l = layout_of(b.mixer)
+        rows.append(lin(f"L{i} in", l.n_in + pad(l.n_gates, 8), w))
+        if l.kind == "latent":
+            seen = sum(min(p + 1, l.window) for p in range(ctx - q, ctx))        # (query, key) pairs of one sequence
+            keys = min(ctx, q + l.window - 1)
+            rows += [Row(f"L{i} attn.latents into the cache", 1, m * (l.c0 + l.row) * 4.0, 0), lin(f"L{i} attn.queries", l.heads * l.dq, l.c0),
+                     Row(f"L{i} attn.latent", 1, n_seqs * keys * l.row * 2 + m * l.heads * (l.dq + l.dv) * 2.0,
+                         2.0 * n_seqs * seen * l.heads * (l.dq + l.dv)),
+                     Row(f"L{i} attn.key / value maps", 1, l.heads * (l.dk + l.dv) * l.kv * 2.0, 2.0 * m * l.heads * (l.dk + l.dv) * l.kv)]
+        else:
+            rows.append(Row(f"L{i} {l.kind}.scan", 1, n_seqs * l.state_floats * 8.0 + m * (l.n_in * 2 + l.heads * l.dv * 6.0),
+                            4.0 * m * l.heads * l.dk * l.dv))
+        rows += [lin(f"L{i} o", w, l.n_out, 4), Row(f"L{i} joins", 2 + (b.mlp is not None), m * w * (4 + 8 + 2.0), 0)]
+        if b.mlp is not None:
+            ff = pad(b.mlp.ff, 64)
+            rows += [lin(f"L{i} gate_up", 2 * ff, w), lin(f"L{i} down", w, ff, 4)]
+        rows += [lin(f"L{i} side gate", side_width(cfg), w), lin(f"L{i} side proj", w, side_width(cfg), 4)]
+    rows.append(Row("lm_head", 1, head_rows(cfg) * w * 2 + head_rows_m * (w * 2 + head_rows(cfg) * 4), 2.0 * head_rows_m * head_rows(cfg) * w))
+    return rows
+
+
 def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
     """One decode (or verify) tick on one TP rank."""
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, StreamDesign):
         b, c = s.batch, s.ctx
+        if isinstance(cfg, FetotarConfig):
+            return _fetotar_rows(cfg, b * s.width, c, b, b * s.width)
         return _zinutar_rows(cfg, b * s.width, b * s.width * c, b * c, b * s.width)
     d = tp_dims(cfg, s.tp)
     m = s.batch * s.width
@@ -112,7 +142,9 @@ def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
 def prefill_rows(cfg: ModelConfig, tokens: int, tp: int = 1, terms: int = 2) -> List[Row]:
     """One prefill of ``tokens`` tokens (one sequence) on one TP rank; ``terms`` NVFP4
     activation terms per token multiply the tensor-core work."""
-    if isinstance(cfg, ZinutarConfig):
+    if isinstance(cfg, FetotarConfig):
+        return _fetotar_rows(cfg, tokens, tokens, 1, 1)
+    if isinstance(cfg, StreamDesign):
         return _zinutar_rows(cfg, tokens, tokens * (tokens + 1) / 2, tokens, 1)
     d = tp_dims(cfg, tp)
     h, m = cfg.hidden, tokens
