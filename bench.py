@@ -190,13 +190,13 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN)
     ap.add_argument("--gen", type=int, default=GEN_LEN)
     ap.add_argument("--no-control", action="store_true", help="skip the unfused same-box control at N > 1")
-    ap.add_argument("--design", default=None, choices=["zinutar"],
-                    help="measure another design beside the closest hybrid form at equal size instead (tilerl_b200/suites/zinutar.py; "
+    ap.add_argument("--design", default=None, choices=["zinutar", "fetotar"],
+                    help="measure another design beside the closest hybrid form at equal size instead (tilerl_b200/suites/<design>.py; "
                          "its own flags follow)")
     args, rest = ap.parse_known_args()
-    if args.design == "zinutar":
-        from tilerl_b200.suites.zinutar import main as design_main
-        return design_main(rest)
+    if args.design:
+        import importlib
+        return importlib.import_module(f"tilerl_b200.suites.{args.design}").main(rest)
     if rest:
         ap.error(f"unrecognized arguments: {' '.join(rest)}")
     if args.impl == "reference":

@@ -183,18 +183,15 @@ latent_attn_kernel(const T* ql, long ql_h, long ql_t, const T* q, int dq, int dk
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
     const float now = fmaxf(top, m);
-    if (now == -INFINITY) {                        // nothing of this row's window so far (all 16 threads of the row agree)
-      s_w[r][c] = 0.f;
-    } else {
-      const float w = expf(s - now), back = expf(top - now);
-      s_w[r][c] = w;
-      float ws = w;
+    // (no branch: the two rows of a warp may differ in whether anything of their window has come by)
+    const float ref = now == -INFINITY ? 0.f : now, w = expf(s - ref), back = expf(top - ref);
+    s_w[r][c] = w;
+    float ws = w;
 #pragma unroll
-      for (int o = 8; o > 0; o >>= 1) ws += __shfl_xor_sync(0xffffffffu, ws, o);
-      sum = sum * back + ws, top = now;
+    for (int o = 8; o > 0; o >>= 1) ws += __shfl_xor_sync(0xffffffffu, ws, o);
+    sum = sum * back + ws, top = now;
 #pragma unroll
-      for (int i = 0; i < F_MAXKV / 16; ++i) acc[i] *= back;
-    }
+    for (int i = 0; i < F_MAXKV / 16; ++i) acc[i] *= back;
     __syncwarp();                                  // a row's 16 threads share a warp
 #pragma unroll
     for (int i = 0; i < F_MAXKV / 16; ++i) {

@@ -1,0 +1,709 @@
+// Latent attention in bf16 on tensor cores (mma.sync), in its two forms.  Cache and symbols: latent.cu.
+//
+// Few query tokens (decoding, verify windows, short portions): queries are mapped into the latent and every head reads the
+// same cached rows, so a page is fetched once for all heads.
+//   latent_absorb_kernel  q W_uk per head, and the rotated part beside it: query rows [kv | rd] of every (token, head).
+//   latent_decode_kernel  one block = 16 (token, head) rows of a sequence and a share of the window's keys.  Pages come
+//                         through a ring of stages (one bulk copy each, from a producing warp); each of four warps (eight,
+//                         for latents above 256) owns one page of a stage and keeps its own softmax, merged at the end.
+//   latent_out_kernel     merges the shares, maps the sum back (W_uv) and applies the output gate.
+// Prompts: keys and values of the window are expanded once for all query tokens.
+//   latent_gather_kernel  cached rows of a range of positions, dense; the expansion itself is one library product.
+//   latent_prompt_kernel  windowed softmax attention per head, 128 query tokens x 64 keys, output gate in the epilogue.
+//
+// Scores, softmax and sums are fp32; weights enter the value product as a bf16 pair (value and rest).
+// Reference parity: the reference's attention keeps full keys and values (no counterpart).
+#include "packed.cuh"
+
+namespace {
+
+constexpr int TILE = 64, TPAGES = TILE / KVB;
+constexpr long long LD_WAIT_CYCLES = 4000000000LL;
+constexpr int LD_SMEM = 216 * 1024;
+constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ bool in_class(int n, int lo, int hi) { return n >= lo && n <= hi; }
+
+// grid (head, 128 latent columns, TT tokens), 128 threads: 16 column groups of 8 x 8 groups of query dimensions
+template <int TT>
+__global__ void __launch_bounds__(128)
+latent_absorb_kernel(const bf16* q, int dq, int dk, int rd, const bf16* __restrict__ uk, int kv, const int* seq_ids, const int* q_len,
+                     int max_len, bf16* ql, int T, int heads) {
+  extern __shared__ float s_ab[];                      // [TT][dk], then [8][TT][128]
+  pdl_launch_dependents(44);
+  const int h = blockIdx.x, c0 = blockIdx.y * 128, t0 = blockIdx.z * TT, n = min(TT, T - t0), tid = threadIdx.x;
+  pdl_wait();
+  bool any = false;
+  for (int t = 0; t < n; ++t) any |= q_len[seq_ids[t0 + t]] <= max_len;
+  if (!any) return;
+  const int D = kv + rd;
+  for (int x = tid; x < TT * dk; x += 128) {
+    const int t = x / dk, d = x % dk;
+    s_ab[x] = t < n ? __bfloat162float(q[((size_t)(t0 + t) * heads + h) * dq + d]) : 0.f;
+  }
+  if (blockIdx.y == 0)                                 // the rotated part as it is
+    for (int x = tid; x < n * (rd / 8); x += 128) {
+      const int t = x / (rd / 8), c = x % (rd / 8);
+      *reinterpret_cast<uint4*>(ql + ((size_t)(t0 + t) * heads + h) * D + kv + c * 8) =
+          *reinterpret_cast<const uint4*>(q + ((size_t)(t0 + t) * heads + h) * dq + dk + c * 8);
+    }
+  __syncthreads();
+  const int c = (tid & 15) * 8, g = tid >> 4;
+  float acc[TT][8];
+#pragma unroll
+  for (int t = 0; t < TT; ++t)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[t][e] = 0.f;
+  if (c0 + c < kv) {
+    const bf16* w = uk + (size_t)h * dk * kv + c0 + c;
+#pragma unroll 4
+    for (int d = g; d < dk; d += 8) {
+      float f[8];
+      Chunk<bf16>::get(*reinterpret_cast<const uint4*>(w + (size_t)d * kv), f);
+#pragma unroll
+      for (int t = 0; t < TT; ++t) {
+        const float x = s_ab[t * dk + d];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[t][e] = fmaf(x, f[e], acc[t][e]);
+      }
+    }
+  }
+  float* part = s_ab + TT * dk;
+#pragma unroll
+  for (int t = 0; t < TT; ++t)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) part[(g * TT + t) * 128 + c + e] = acc[t][e];
+  __syncthreads();
+  for (int x = tid; x < n * 128; x += 128) {
+    const int t = x >> 7, cc = x & 127;
+    if (c0 + cc >= kv) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v += part[(k * TT + t) * 128 + cc];
+    ql[((size_t)(t0 + t) * heads + h) * D + c0 + cc] = __float2bfloat16(v);
+  }
+}
+
+struct DecArgs {
+  const bf16* ql;                      // [T, heads, kv + rd]
+  const unsigned char* pages;
+  int kch, vch, n_blocks;              // 16-byte chunks of a cached row, of its latent part
+  const int* table;
+  int max_blocks;
+  const int *q_start, *q_len, *positions;
+  float* part;                         // [T, heads, n_splits, kv]
+  float2* ml;                          // [T, heads, n_splits]: running maximum (log2), sum
+  int heads, n_splits, n_stages, window, min_len, max_len;
+  float scale2;                        // scale x log2(e)
+};
+
+// First page and number of stages of a row tile's keys, and the stages of one split.
+__device__ __forceinline__ void tile_range(int p_first, int p_last, int window, int& page0, int& stages) {
+  page0 = max(0, p_first - window + 1) / KVB;
+  stages = (p_last / KVB - page0) / TPAGES + 1;
+}
+__device__ __forceinline__ int stages_per_split(int stages, int n_splits) {
+  const int want = max(1, min(n_splits, (stages + 1) / 2));        // at least 128 keys each
+  return (stages + want - 1) / want;
+}
+__device__ __forceinline__ uint32_t ld_try_wait(uint32_t bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile("{ .reg .pred p;\n"
+               "  mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+               "  selp.u32 %0, 1, 0, p; }\n"
+               : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
+  return ok;
+}
+
+template <int OD, int HALVES>
+__global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(const DecArgs a) {
+  constexpr int NW = 4 * HALVES, THREADS = (NW + 1) * 32;
+  extern __shared__ unsigned char ld_raw[];
+  __shared__ __align__(8) uint64_t s_bar[8];               // full[4], empty[4]
+  __shared__ float s_m[4][16], s_l[4][16];
+  __shared__ volatile int s_ok;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const uint32_t raw_a = (uint32_t)__cvta_generic_to_shared(ld_raw);
+  unsigned char* smem = ld_raw + (((raw_a + 127u) & ~127u) - raw_a);
+  const uint32_t smem_a = (raw_a + 127u) & ~127u, bar_a = (uint32_t)__cvta_generic_to_shared(s_bar);
+  if (threadIdx.x == 0) {
+    for (int st = 0; st < a.n_stages; ++st) {
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(bar_a + 8u * st));
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar_a + 32u + 8u * st), "r"(NW));
+    }
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    s_ok = 1;
+  }
+  pdl_enter(45);
+  pdl_wait();
+  const int tile = blockIdx.x / a.n_splits, split = blockIdx.x % a.n_splits, seq = blockIdx.y;
+  const int T = a.q_len[seq], n_rows = T * a.heads, row0 = tile * 16;
+  if (!in_class(T, a.min_len, a.max_len) || row0 >= n_rows) return;
+  const int q0 = a.q_start[seq], rows = min(16, n_rows - row0);
+  const int p_first = a.positions[q0 + row0 / a.heads], p_last = a.positions[q0 + (row0 + rows - 1) / a.heads];
+  int page0, stages;
+  tile_range(p_first, p_last, a.window, page0, stages);
+  const int sps = stages_per_split(stages, a.n_splits);
+  const int s0 = split * sps, s1 = min(stages, s0 + sps);
+  if (s0 >= s1) return;
+  const int row_b = a.kch * 16, page_b = KVB * row_b, stage_b = TPAGES * page_b, qld = row_b + 16;
+  const int kv = a.vch * 8, D = a.kch * 8;
+  const int q_bytes = (16 * qld + 127) / 128 * 128;
+  unsigned char* ring = smem + q_bytes;
+  const uint32_t ring_a = smem_a + q_bytes;
+  const int lo = (page0 + s0 * TPAGES) * KVB, hi = min(p_last + 1, (page0 + s1 * TPAGES) * KVB);
+  for (int x = threadIdx.x; x < 16 * a.kch; x += THREADS) {
+    const int r = x / a.kch, c = x % a.kch, row = row0 + r;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (r < rows) v = *reinterpret_cast<const uint4*>(a.ql + ((size_t)(q0 + row / a.heads) * a.heads + row % a.heads) * D + c * 8);
+    *reinterpret_cast<uint4*>(smem + r * qld + c * 16) = v;
+  }
+  {
+    // The last page brings only the rows that exist (the pool may hold anything past them, and 0 x row must be 0): if
+    // nothing was copied into that place before, its tail starts as zeros.
+    const int last = s1 - s0 - 1, tail = hi & (KVB - 1);
+    if (tail && last < a.n_stages) {
+      const int pg = ((hi - 1 - lo) / KVB) % TPAGES;
+      unsigned char* p = ring + last * stage_b + pg * page_b;
+      for (int x = tail * a.kch + threadIdx.x; x < KVB * a.kch; x += THREADS) *reinterpret_cast<uint4*>(p + x * 16) = make_uint4(0u, 0u, 0u, 0u);
+    }
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  }
+  __syncthreads();
+  auto bounded_wait = [&](uint32_t bar, uint32_t parity, int what) {
+    if (ld_try_wait(bar, parity)) return true;
+    const long long t_begin = clock64();
+    for (uint32_t it = 1; !ld_try_wait(bar, parity); ++it) {
+      if ((it & 63) == 0) {
+        if (!s_ok) return false;
+        if (clock64() - t_begin > LD_WAIT_CYCLES) {
+          trl_set_error(TRL_ERR_MBAR_TIMEOUT, (int)blockIdx.x, what, (int)parity);
+          s_ok = 0;
+          return false;
+        }
+      }
+    }
+    return true;
+  };
+  const int kw = warp & 3, half = warp >> 2;               // key page of a stage, column half
+  float o[OD / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < OD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  if (warp == NW) {
+    // ---------------- producer ----------------
+    const int* table = a.table + (size_t)seq * a.max_blocks;
+    int st = 0;
+    uint32_t ph = 0;
+    for (int k = s0; k < s1; ++k) {
+      if (k - s0 >= a.n_stages && !bounded_wait(bar_a + 32u + 8u * st, ph ^ 1u, 530 + st)) break;
+      const int j0 = (page0 + k * TPAGES) * KVB, n_pg = min(TPAGES, (hi - j0 + KVB - 1) / KVB);
+      uint32_t bytes = 0;
+      const unsigned char* src = nullptr;
+      if (lane < n_pg) {
+        const int p = j0 / KVB + lane;
+        src = a.pages + (size_t)trl_checked(table[p], a.n_blocks, 11) * page_b;
+        bytes = (uint32_t)(min(KVB, hi - p * KVB) * row_b);
+      }
+      const uint32_t total = __reduce_add_sync(0xffffffffu, bytes), full = bar_a + 8u * st;
+      if (lane == 0) asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(full), "r"(total) : "memory");
+      __syncwarp();
+      if (lane < n_pg)
+        asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                     ::"r"(ring_a + st * stage_b + lane * page_b), "l"(src), "r"(bytes), "r"(full) : "memory");
+      if (++st == a.n_stages) st = 0, ph ^= 1u;
+    }
+  } else {
+    // ---------------- consumers ----------------
+    int pos[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int r = (lane >> 2) + 8 * i;
+      pos[i] = r < rows ? a.positions[q0 + (row0 + r) / a.heads] : -1;
+    }
+    const uint32_t qa = smem_a + ((lane & 7) + ((lane >> 3) & 1) * 8) * qld + (lane >> 4) * 16;
+    const int kr = (lane & 7) + (lane >> 4) * 8, kcl = (lane >> 3) & 1;
+    const int vr = (lane & 7) + ((lane >> 3) & 1) * 8, vcl = lane >> 4;
+    const int krot = kr % a.kch, vrot = vr % a.kch, nc = a.kch;
+    const bool xored = nc % 8 == 0;
+    auto place = [&](int c, int r, int rot) {              // page_chunk without a division (rot = r % nc)
+      const int x = c + rot;
+      return xored ? c ^ (r & 7) : (x >= nc ? x - nc : x);
+    };
+    const int vc0 = half * (OD / 8), vch = min(OD / 8, a.vch - vc0);      // this warp's output chunks
+    int st = 0;
+    uint32_t ph = 0;
+    for (int k = s0; k < s1; ++k) {
+      if (!bounded_wait(bar_a + 8u * st, ph, 520 + st)) break;
+      const int j0 = (page0 + k * TPAGES + kw) * KVB;
+      if (j0 < hi) {
+        const uint32_t base = ring_a + st * stage_b + kw * page_b;
+        float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll 4
+        for (int kk = 0; kk < nc / 2; ++kk) {
+          uint32_t qv[4], b[4];
+          ldsm4(qv, qa + kk * 32);
+          ldsm4(b, base + (kr * nc + place(kk * 2 + kcl, kr, krot)) * 16);
+          mma16(sc[0], qv, b[0], b[1]);
+          mma16(sc[1], qv, b[2], b[3]);
+        }
+        uint32_t wh[4], wl[4];
+        float now[2], back[2];
+        bool moved = false;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          float m = -INFINITY;
+#pragma unroll
+          for (int n8 = 0; n8 < 2; ++n8)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const int j = j0 + n8 * 8 + (lane & 3) * 2 + e;
+              float& s = sc[n8][2 * i + e];
+              s = j <= pos[i] && pos[i] - j < a.window ? s * a.scale2 : -INFINITY;   // (a select: stale bytes may be anything)
+              m = fmaxf(m, s);
+            }
+          m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
+          m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
+          now[i] = fmaxf(mx[i], m);
+          moved |= now[i] > mx[i];
+          const float ref = now[i] == -INFINITY ? 0.f : now[i];
+          back[i] = exp2f(mx[i] - ref);
+          mx[i] = now[i];
+          float w[4], ws = 0.f;
+#pragma unroll
+          for (int n8 = 0; n8 < 2; ++n8) {
+            w[2 * n8] = exp2f(sc[n8][2 * i] - ref), w[2 * n8 + 1] = exp2f(sc[n8][2 * i + 1] - ref);
+            ws += w[2 * n8] + w[2 * n8 + 1];
+            split2(w[2 * n8], w[2 * n8 + 1], wh[n8 * 2 + i], wl[n8 * 2 + i]);
+          }
+          sum[i] = sum[i] * back[i] + ws;                  // (this lane's keys; added over the quad at the end)
+        }
+        if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+          for (int nd = 0; nd < OD / 8; ++nd) o[nd][0] *= back[0], o[nd][1] *= back[0], o[nd][2] *= back[1], o[nd][3] *= back[1];
+        }
+#pragma unroll
+        for (int nd = 0; nd < OD / 8; nd += 2) {
+          if (nd < vch) {
+            uint32_t b[4];
+            ldsm4t(b, base + (vr * nc + place(vc0 + nd + vcl, vr, vrot)) * 16);
+            mma16(o[nd], wh, b[0], b[1]);
+            mma16(o[nd + 1], wh, b[2], b[3]);
+            mma16(o[nd], wl, b[0], b[1]);
+            mma16(o[nd + 1], wl, b[2], b[3]);
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar_a + 32u + 8u * st) : "memory");
+      if (++st == a.n_stages) st = 0, ph ^= 1u;
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
+      sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+      if (half == 0 && (lane & 3) == 0) s_m[kw][(lane >> 2) + 8 * i] = mx[i], s_l[kw][(lane >> 2) + 8 * i] = sum[i];
+    }
+  }
+  __syncthreads();
+  pdl_trigger();
+  if (!s_ok) {                                              // copies may still be in flight towards this block
+    const long long t_begin = clock64();
+    while (clock64() - t_begin < 2000000LL) {
+    }
+  }
+  // the four warps saw different keys: merge them in order, through the (idle) ring
+  float* so = reinterpret_cast<float*>(ring);               // [4][16][kv]
+  if (warp < NW) {
+    const int vc0 = half * (OD / 8), vch = min(OD / 8, a.vch - vc0), r = lane >> 2;
+#pragma unroll
+    for (int nd = 0; nd < OD / 8; ++nd) {
+      if (nd < vch) {
+        const int d = (vc0 + nd) * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(so + (size_t)(kw * 16 + r) * kv + d) = make_float2(o[nd][0], o[nd][1]);
+        *reinterpret_cast<float2*>(so + (size_t)(kw * 16 + r + 8) * kv + d) = make_float2(o[nd][2], o[nd][3]);
+      }
+    }
+  }
+  __syncthreads();
+  for (int x = threadIdx.x; x < rows * (kv / 4); x += THREADS) {
+    const int r = x / (kv / 4), d = (x % (kv / 4)) * 4, row = row0 + r;
+    const float m = fmaxf(fmaxf(s_m[0][r], s_m[1][r]), fmaxf(s_m[2][r], s_m[3][r])), ref = m == -INFINITY ? 0.f : m;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    float l = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float f = exp2f(s_m[k][r] - ref);
+      const float4 y = *reinterpret_cast<const float4*>(so + (size_t)(k * 16 + r) * kv + d);
+      v.x = fmaf(f, y.x, v.x), v.y = fmaf(f, y.y, v.y), v.z = fmaf(f, y.z, v.z), v.w = fmaf(f, y.w, v.w);
+      l = fmaf(f, s_l[k][r], l);
+    }
+    const size_t at = ((size_t)(q0 + row / a.heads) * a.heads + row % a.heads) * a.n_splits + split;
+    *reinterpret_cast<float4*>(a.part + at * kv + d) = v;
+    if (d == 0) a.ml[at] = make_float2(m, l);
+  }
+}
+
+// grid (head, TT tokens, shares of the value rows), 256 threads
+template <int TT>
+__global__ void __launch_bounds__(256)
+latent_out_kernel(const float* part, const float2* ml, int n_splits, const bf16* __restrict__ uv, int kv, int dv, const bf16* gate, int ldp,
+                  bf16* out, int n_out, const int* seq_ids, const int* q_start, const int* q_len, const int* positions, int T, int heads,
+                  int window, int max_len) {
+  extern __shared__ float s_oc[];                        // [TT][kv]
+  __shared__ int s_in[TT];
+  pdl_launch_dependents(46);
+  pdl_wait();
+  const int h = blockIdx.x, t0 = blockIdx.y * TT, n = min(TT, T - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int rows = (dv + gridDim.z - 1) / gridDim.z, d0 = blockIdx.z * rows, d1 = min(dv, d0 + rows);
+  bool any = false;
+#pragma unroll
+  for (int i = 0; i < TT; ++i) {
+    const int t = t0 + i;
+    bool in = i < n;
+    int seq = 0, len = 0, q0 = 0;
+    if (in) seq = seq_ids[t], len = q_len[seq], q0 = q_start[seq], in = len <= max_len && t - q0 < len;
+    if (tid == 0) s_in[i] = in;
+    any |= in;
+    if (!in) {
+      for (int c = tid; c < kv; c += 256) s_oc[i * kv + c] = 0.f;
+      continue;
+    }
+    const int n_rows = len * heads, row0 = ((t - q0) * heads + h) / 16 * 16;
+    int page0, stages;
+    tile_range(positions[q0 + row0 / heads], positions[q0 + (min(row0 + 16, n_rows) - 1) / heads], window, page0, stages);
+    const int sps = stages_per_split(stages, n_splits), used = (stages + sps - 1) / sps;
+    const size_t at = ((size_t)t * heads + h) * n_splits;
+    float m = -INFINITY;
+    for (int s = 0; s < used; ++s) m = fmaxf(m, ml[at + s].x);
+    float l = 0.f;
+    for (int s = 0; s < used; ++s) l += exp2f(ml[at + s].x - m) * ml[at + s].y;
+    for (int c = tid; c < kv; c += 256) {
+      float v = 0.f;
+      for (int s = 0; s < used; ++s) v = fmaf(exp2f(ml[at + s].x - m), part[(at + s) * kv + c], v);
+      s_oc[i * kv + c] = v / l;
+    }
+  }
+  if (!any) return;
+  __syncthreads();
+  for (int d = d0 + warp; d < d1; d += 8) {
+    const uint4* w = reinterpret_cast<const uint4*>(uv + ((size_t)h * dv + d) * kv);
+    float acc[TT];
+#pragma unroll
+    for (int i = 0; i < TT; ++i) acc[i] = 0.f;
+    for (int c = lane; c < kv / 8; c += 32) {
+      float f[8];
+      Chunk<bf16>::get(w[c], f);
+#pragma unroll
+      for (int i = 0; i < TT; ++i) {
+        const float4 a0 = *reinterpret_cast<const float4*>(s_oc + i * kv + c * 8), a1 = *reinterpret_cast<const float4*>(s_oc + i * kv + c * 8 + 4);
+        acc[i] += f[0] * a0.x + f[1] * a0.y + f[2] * a0.z + f[3] * a0.w + f[4] * a1.x + f[5] * a1.y + f[6] * a1.z + f[7] * a1.w;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TT; ++i) {
+      const float v = warp_sum(acc[i]);
+      if (lane == 0 && s_in[i])
+        out[(size_t)(t0 + i) * n_out + h * dv + d] = __float2bfloat16(v * sigmoid_x(__bfloat162float(gate[(size_t)(t0 + i) * ldp + h * dv + d])));
+    }
+  }
+  if (h == 0 && blockIdx.z == 0)
+    for (int i = 0; i < n; ++i)
+      if (s_in[i])
+        for (int c = heads * dv + tid; c < n_out; c += 256) out[(size_t)(t0 + i) * n_out + c] = __float2bfloat16(0.f);
+}
+
+// grid (positions lo .. of one sequence): cached rows -> c [n, kv], kr [n, rd]
+__global__ void __launch_bounds__(64)
+latent_gather_kernel(const unsigned char* pages, int n_blocks, const int* table, int lo, int kch, int vch, bf16* c, bf16* kr) {
+  pdl_launch_dependents(47);
+  pdl_wait();
+  const int j = lo + blockIdx.x, r = j % KVB;
+  const uint4* row = reinterpret_cast<const uint4*>(pages + (size_t)trl_checked(table[j / KVB], n_blocks, 12) * KVB * kch * 16) + r * kch;
+  uint4* cd = reinterpret_cast<uint4*>(c) + (size_t)blockIdx.x * vch;
+  uint4* kd = reinterpret_cast<uint4*>(kr) + (size_t)blockIdx.x * (kch - vch);
+  for (int x = threadIdx.x; x < kch; x += 64) {
+    const uint4 v = row[page_chunk(x, r, kch)];
+    if (x < vch) cd[x] = v;
+    else kd[x - vch] = v;
+  }
+}
+
+struct PromptArgs {
+  const bf16 *q, *kvx, *kr, *gate;     // query heads [T, heads, dq]; expanded [keys, ldkv]: heads x dk, heads x dv; [keys, rd]
+  bf16* out;
+  const int* positions;                // of the sequence's first query token on
+  int n, lo, n_keys, heads, dq, dk, rd, dv, ldkv, ldp, n_out, window;
+  float scale2;
+};
+
+// one block = (128 query tokens, head); a warp owns 16 of them
+template <int DQ, int DV>
+__global__ void __launch_bounds__(256) latent_prompt_kernel(const PromptArgs a) {
+  constexpr int QROW = DQ * 2, VROW = DV * 2;
+  extern __shared__ unsigned char lp_raw[];
+  const uint32_t raw_a = (uint32_t)__cvta_generic_to_shared(lp_raw), q_a = (raw_a + 127u) & ~127u;
+  const uint32_t k_a = q_a + 128 * QROW, v_a = k_a + 2 * TILE * QROW;
+  pdl_launch_dependents(48);
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, row0 = blockIdx.x * 128;
+  const int rows = min(128, a.n - row0);
+  auto off = [](int r, int c, int rowb) { return (uint32_t)(r * rowb + ((c ^ (r & 7)) << 4)); };
+  auto zcp = [](uint32_t dst, const void* src, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
+  };
+  const int first = a.positions[row0], last = a.positions[row0 + rows - 1];
+  const int j_lo = max(a.lo, first - a.window + 1), n_tiles = (last - j_lo) / TILE + 1;
+  for (int x = tid; x < 128 * (DQ / 8); x += 256) {
+    const int r = x / (DQ / 8), c = x % (DQ / 8);
+    const bool in = r < rows && c * 8 < a.dq;
+    zcp(q_a + off(r, c, QROW), a.q + (in ? ((size_t)(row0 + r) * a.heads + h) * a.dq + c * 8 : 0), in);
+  }
+  auto stage = [&](int kt, int b) {
+    const int j0 = j_lo + kt * TILE - a.lo;                 // row of the expanded keys
+    for (int x = tid; x < TILE * (DQ / 8); x += 256) {
+      const int r = x / (DQ / 8), c = x % (DQ / 8);
+      const bool in = j0 + r < a.n_keys && c * 8 < a.dq;
+      const bf16* src = c * 8 < a.dk ? a.kvx + (size_t)(in ? j0 + r : 0) * a.ldkv + h * a.dk + c * 8
+                                     : a.kr + (in ? (size_t)(j0 + r) * a.rd + c * 8 - a.dk : 0);
+      zcp(k_a + b * TILE * QROW + off(r, c, QROW), src, in);
+    }
+    for (int x = tid; x < TILE * (DV / 8); x += 256) {
+      const int r = x / (DV / 8), c = x % (DV / 8);
+      const bool in = j0 + r < a.n_keys && c * 8 < a.dv;
+      zcp(v_a + b * TILE * VROW + off(r, c, VROW), a.kvx + (in ? (size_t)(j0 + r) * a.ldkv + a.heads * a.dk + h * a.dv + c * 8 : 0), in);
+    }
+    cp_commit();
+  };
+  stage(0, 0);
+  float o[DV / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  int pos[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = warp * 16 + (lane >> 2) + 8 * i;
+    pos[i] = r < rows ? a.positions[row0 + r] : -1;
+  }
+  const bool live = warp * 16 < rows;
+  const int w_first = live ? a.positions[row0 + warp * 16] : 0, w_last = live ? a.positions[row0 + min(rows, warp * 16 + 16) - 1] : -1;
+  const int lrow = (lane & 7) + ((lane >> 3) & 1) * 8, lch = lane >> 4, brow = (lane & 7) + (lane >> 4) * 8, bch = (lane >> 3) & 1;
+  const int nk = a.dq / 16, nv = a.dv / 8;
+  for (int kt = 0; kt < n_tiles; ++kt) {
+    const int b = kt & 1;
+    cp_wait<0>();
+    __syncthreads();                                        // tile kt is in, the other buffer is free
+    if (kt + 1 < n_tiles) stage(kt + 1, b ^ 1);
+    const int j0 = j_lo + kt * TILE;
+    if (j0 > w_last || j0 + TILE - 1 <= w_first - a.window) continue;
+    float sc[4][2][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int n8 = 0; n8 < 2; ++n8) sc[j][n8][0] = sc[j][n8][1] = sc[j][n8][2] = sc[j][n8][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < DQ / 16; ++kk) {
+      if (kk < nk) {
+        uint32_t qf[4];
+        ldsm4(qf, q_a + off(warp * 16 + lrow, kk * 2 + lch, QROW));
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          uint32_t kf[4];
+          ldsm4(kf, k_a + b * TILE * QROW + off(16 * j + brow, kk * 2 + bch, QROW));
+          mma16(sc[j][0], qf, kf[0], kf[1]);
+          mma16(sc[j][1], qf, kf[2], kf[3]);
+        }
+      }
+    }
+    const bool edge = j0 + TILE - 1 > w_first || j0 <= w_last - a.window;      // some row does not see all of this tile
+    float back[2];
+    bool moved = false;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      float m = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int n8 = 0; n8 < 2; ++n8)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            float& s = sc[j][n8][2 * i + e];
+            s *= a.scale2;
+            if (edge) {
+              const int key = j0 + 16 * j + 8 * n8 + (lane & 3) * 2 + e;
+              s = key <= pos[i] && pos[i] - key < a.window ? s : -INFINITY;
+            }
+            m = fmaxf(m, s);
+          }
+      m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
+      m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
+      const float now = fmaxf(mx[i], m), ref = now == -INFINITY ? 0.f : now;
+      moved |= now > mx[i];
+      back[i] = exp2f(mx[i] - ref);
+      mx[i] = now;
+      float ws = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int n8 = 0; n8 < 2; ++n8)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            float& s = sc[j][n8][2 * i + e];
+            s = exp2f(s - ref);
+            ws += s;
+          }
+      sum[i] = sum[i] * back[i] + ws;
+    }
+    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+      for (int nd = 0; nd < DV / 8; ++nd) o[nd][0] *= back[0], o[nd][1] *= back[0], o[nd][2] *= back[1], o[nd][3] *= back[1];
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      uint32_t wh[4], wl[4];
+#pragma unroll
+      for (int n8 = 0; n8 < 2; ++n8)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) split2(sc[j][n8][2 * i], sc[j][n8][2 * i + 1], wh[n8 * 2 + i], wl[n8 * 2 + i]);
+#pragma unroll
+      for (int nd = 0; nd < DV / 8; nd += 2) {
+        if (nd < nv) {
+          uint32_t f[4];
+          ldsm4t(f, v_a + b * TILE * VROW + off(16 * j + lrow, nd + lch, VROW));
+          mma16(o[nd], wh, f[0], f[1]);
+          mma16(o[nd + 1], wh, f[2], f[3]);
+          mma16(o[nd], wl, f[0], f[1]);
+          mma16(o[nd + 1], wl, f[2], f[3]);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
+    sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+    const int r = warp * 16 + (lane >> 2) + 8 * i;
+    if (r >= rows) continue;
+    const float f = 1.f / sum[i];
+    const bf16* g = a.gate + (size_t)(row0 + r) * a.ldp + h * a.dv;
+    bf16* dst = a.out + (size_t)(row0 + r) * a.n_out + h * a.dv;
+#pragma unroll
+    for (int nd = 0; nd < DV / 8; ++nd) {
+      if (nd < nv) {
+        const int d = nd * 8 + (lane & 3) * 2;
+        const float2 gg = bf162_bits_to_f2(*reinterpret_cast<const uint32_t*>(g + d));
+        *reinterpret_cast<uint32_t*>(dst + d) = f2_to_bf162_bits(o[nd][2 * i] * f * sigmoid_f(gg.x), o[nd][2 * i + 1] * f * sigmoid_f(gg.y));
+      }
+    }
+  }
+  if (h == 0)
+    for (int x = tid; x < rows * (a.n_out - a.heads * a.dv); x += 256) {
+      const int w = a.n_out - a.heads * a.dv;
+      a.out[(size_t)(row0 + x / w) * a.n_out + a.heads * a.dv + x % w] = __float2bfloat16(0.f);
+    }
+}
+
+template <int OD, int HALVES> cudaError_t decode_launch(DecArgs a, int tiles, int B, cudaStream_t st) {
+  const size_t q_bytes = (size_t)(16 * (a.kch * 16 + 16) + 127) / 128 * 128, stage = (size_t)TILE * a.kch * 16;
+  const size_t merge = (size_t)4 * 16 * a.vch * 8 * sizeof(float);
+  int stages = 4;
+  while (stages > 2 && q_bytes + stages * stage > 104 * 1024) --stages;          // two blocks on an SM where three stages allow it
+  if (stages < 3 && q_bytes + 3 * stage <= (size_t)LD_SMEM) stages = 3;
+  const size_t smem = q_bytes + (stages * stage > merge ? stages * stage : merge) + 128;
+  if (smem > (size_t)LD_SMEM + 128) return cudaErrorInvalidValue;
+  a.n_stages = stages;
+  auto k = latent_decode_kernel<OD, HALVES>;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM + 128);
+    if (e != cudaSuccess) return e;
+    cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
+    configured = true;
+  }
+  return trl_launch(k, dim3(tiles * a.n_splits, B), dim3((4 * HALVES + 1) * 32), smem, st, a);
+}
+
+template <int DQ, int DV> cudaError_t prompt_launch(const PromptArgs& a, cudaStream_t st) {
+  constexpr int smem = 128 * DQ * 2 + 2 * TILE * (DQ + DV) * 2 + 128;
+  auto k = latent_prompt_kernel<DQ, DV>;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    configured = true;
+  }
+  return trl_launch(k, dim3((a.n + 127) / 128, a.heads), dim3(256), smem, st, a);
+}
+
+}  // namespace
+
+// 1 when the tensor-core forms take heads of these (padded) sizes.
+TRL_API int trl_latent_mma_ok(int dk, int rd, int dv, int kv) {
+  const size_t row = (size_t)(kv + rd) * 2, q = (size_t)16 * (row + 16) + 128, merge = (size_t)4 * 16 * kv * 4;
+  return dk + rd <= 256 && dv <= 256 && kv <= 512 && q + (2 * TILE * row > merge ? 2 * TILE * row : merge) <= (size_t)LD_SMEM;
+}
+
+// Sequences of min_len..max_len tokens in the absorbed form.  q: [T, heads, dq]; up: [heads * dk key rows ; heads * dv value rows][kv];
+// ql: [T, heads, kv + rd]; part: fp32 [T, heads, n_splits, kv]; ml: [T, heads, n_splits] pairs; tiles: 16-row tiles of the longest
+// sequence; gate: gate columns of the fused projection rows.
+TRL_API int trl_latent_decode(const void* q, int dq, int dk, int rd, const void* up, int kv, int dv, void* ql, const void* pages, int n_blocks,
+                              const void* table, int max_blocks, const void* q_start, const void* q_len, const void* positions,
+                              const void* seq_ids, void* part, void* ml, const void* gate, int ldp, void* out, int n_out, int T, int B,
+                              int tiles, int heads, int n_splits, int window, int min_len, int max_len, float scale, void* stream) {
+  if (T <= 0 || B <= 0 || tiles <= 0 || heads <= 0 || dk % 16 || rd % 16 || dv % 16 || kv % 16 || dk + rd != dq || n_splits < 1 || window < 1 ||
+      n_blocks <= 0 || n_out < heads * dv || !trl_latent_mma_ok(dk, rd, dv, kv) || ((uintptr_t)pages & 15) || ((uintptr_t)q & 15))
+    return (int)cudaErrorInvalidValue;
+  cudaStream_t st = (cudaStream_t)stream;
+  const bf16 *uk = (const bf16*)up, *uv = uk + (size_t)heads * dk * kv;
+  const int tt = T >= 8 ? 4 : 1, groups = (T + tt - 1) / tt;
+  const size_t sm1 = (size_t)(tt * dk + 8 * tt * 128) * sizeof(float);
+  cudaError_t e;
+  if (tt == 4)
+    e = trl_launch(latent_absorb_kernel<4>, dim3(heads, (kv + 127) / 128, groups), dim3(128), sm1, st, (const bf16*)q, dq, dk, rd, uk, kv,
+                   (const int*)seq_ids, (const int*)q_len, max_len, (bf16*)ql, T, heads);
+  else
+    e = trl_launch(latent_absorb_kernel<1>, dim3(heads, (kv + 127) / 128, groups), dim3(128), sm1, st, (const bf16*)q, dq, dk, rd, uk, kv,
+                   (const int*)seq_ids, (const int*)q_len, max_len, (bf16*)ql, T, heads);
+  if (e != cudaSuccess) return (int)e;
+  DecArgs a;
+  a.ql = (const bf16*)ql, a.pages = (const unsigned char*)pages, a.kch = (kv + rd) / 8, a.vch = kv / 8, a.n_blocks = n_blocks;
+  a.table = (const int*)table, a.max_blocks = max_blocks, a.q_start = (const int*)q_start, a.q_len = (const int*)q_len;
+  a.positions = (const int*)positions, a.part = (float*)part, a.ml = (float2*)ml, a.heads = heads, a.n_splits = n_splits, a.n_stages = 2;
+  a.window = window, a.min_len = min_len, a.max_len = max_len, a.scale2 = scale * LOG2E;
+  if (kv <= 128) e = decode_launch<128, 1>(a, tiles, B, st);
+  else if (kv <= 256) e = decode_launch<256, 1>(a, tiles, B, st);
+  else e = decode_launch<256, 2>(a, tiles, B, st);
+  if (e != cudaSuccess) return (int)e;
+  const int z = groups * heads < 148 ? min(4, (dv + 15) / 16) : 1;
+  const size_t sm2 = (size_t)tt * kv * sizeof(float);
+#define OUT(TTT)                                                                                                               \
+  return (int)trl_launch(latent_out_kernel<TTT>, dim3(heads, groups, z), dim3(256), sm2, st, (const float*)part, (const float2*)ml, \
+                         n_splits, uv, kv, dv, (const bf16*)gate, ldp, (bf16*)out, n_out, (const int*)seq_ids, (const int*)q_start,  \
+                         (const int*)q_len, (const int*)positions, T, heads, window, max_len)
+  if (tt == 4) OUT(4);
+  OUT(1);
+#undef OUT
+}
+
+// Cached rows of positions lo .. lo + n - 1 of one sequence (table: its row of the block table).
+TRL_API int trl_latent_gather(const void* pages, int n_blocks, const void* table, int lo, int n, int kv, int rd, void* c, void* kr, void* stream) {
+  if (n <= 0 || lo < 0 || kv % 16 || rd % 16 || n_blocks <= 0) return (int)cudaErrorInvalidValue;
+  return (int)trl_launch(latent_gather_kernel, dim3(n), dim3(64), 0, (cudaStream_t)stream, (const unsigned char*)pages, n_blocks,
+                         (const int*)table, lo, (kv + rd) / 8, kv / 8, (bf16*)c, (bf16*)kr);
+}
+
+// One sequence's n query tokens (pointers at its first token) against expanded keys of positions lo .. lo + n_keys - 1.
+TRL_API int trl_latent_prompt(const void* q, int dq, int dk, int rd, int dv, const void* kvx, int ldkv, const void* kr, const void* gate, int ldp,
+                              void* out, int n_out, const void* positions, int n, int lo, int n_keys, int heads, int window, float scale,
+                              void* stream) {
+  if (n <= 0 || n_keys <= 0 || heads <= 0 || dk % 16 || rd % 16 || dv % 16 || dk + rd != dq || dq > 256 || dv > 256 || ldkv % 8 || ldp % 2 ||
+      ldkv < heads * (dk + dv) || n_out < heads * dv || window < 1 || ((uintptr_t)q & 15) || ((uintptr_t)kvx & 15) || ((uintptr_t)kr & 15))
+    return (int)cudaErrorInvalidValue;
+  PromptArgs a;
+  a.q = (const bf16*)q, a.kvx = (const bf16*)kvx, a.kr = (const bf16*)kr, a.gate = (const bf16*)gate, a.out = (bf16*)out;
+  a.positions = (const int*)positions, a.n = n, a.lo = lo, a.n_keys = n_keys, a.heads = heads, a.dq = dq, a.dk = dk, a.rd = rd, a.dv = dv;
+  a.ldkv = ldkv, a.ldp = ldp, a.n_out = n_out, a.window = window, a.scale2 = scale * LOG2E;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (dv <= 128 && dq <= 128) return (int)prompt_launch<128, 128>(a, st);
+  if (dv <= 128 && dq <= 192) return (int)prompt_launch<192, 128>(a, st);
+  return (int)prompt_launch<256, 256>(a, st);
+}

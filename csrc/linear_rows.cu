@@ -2,6 +2,8 @@
 //
 //   y[m, n] (store bf16 | store fp32 | += fp32) = sum_k x'[m, k] * W[n, k]
 //
+// or, in the epilogue, rows n >= n_split stored in fp32 beside the bf16 ones (gates of a recurrence), pairs of rows (gate, up)
+// joined to g sigmoid(1.702 g) (u + 1) with clamps, or gelu(y) times a token's side-embedding row.
 // x' is the row itself (bf16) or rms(x) * norm_w of an fp32 stream row, rounded to bf16.  The weights are streamed
 // once: a warp owns 16 weight rows and a share of K, and every lane copies the 16-byte pieces it will itself feed to
 // mma.sync (8 consecutive k of rows g and g + 8 per 32-wide step) into its own slots of a shared-memory ring, so no
@@ -12,14 +14,23 @@
 // order, so a run repeats bit for bit.  A block stages the activations once and walks its row tiles; the ring runs on
 // across tiles, and its first fill is issued before the dependency wait: weights are constants of the tick.
 // Reference parity: it projects out of a bf16 residual (no counterpart).
-#include "common.cuh"
+#include "packed.cuh"
 
 namespace {
 
 constexpr int LR_THREADS = 256, LR_WARPS = LR_THREADS / 32, LR_U = 4, LR_PAD = 32;
 constexpr int LR_SLOT = LR_U * 2 * 512;                        // bytes of a ring stage of one warp
 constexpr int LR_SMEM = 216 * 1024;
-enum { LR_STORE = 0, LR_STORE_F32 = 1, LR_ADD_F32 = 2 };
+enum { LR_STORE = 0, LR_STORE_F32 = 1, LR_ADD_F32 = 2, LR_GLU = 3, LR_SIDE = 4 };
+struct LrExtra {
+  float* y2;                                                   // LR_STORE: fp32 rows n >= n_split
+  int ldy2, n_split;
+  float limit;                                                 // LR_GLU
+  const int* ids;                                              // LR_SIDE: side[id * ld_side + off + n] for n < dim, 0 past it
+  const bf16* side;
+  long ld_side;
+  int off, dim, vocab;
+};
 
 __device__ __forceinline__ void lr_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -39,7 +50,7 @@ __device__ __forceinline__ uint4 lr_lds(uint32_t a) {
 template <bool NORM, int NT, int EPI, int DEPTH>
 __global__ void __launch_bounds__(LR_THREADS)
 linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const float* __restrict__ norm_w, float eps, int n_norm,
-                   void* y, int ldy, int M, int N, int K, int KW, int n_tiles) {
+                   void* y, int ldy, int M, int N, int K, int KW, int n_tiles, const LrExtra ex) {
   extern __shared__ __align__(16) unsigned char lr_smem[];
   __shared__ float red[32];
   __shared__ float s_r[16];
@@ -140,12 +151,27 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
       for (int e = 0; e < 4; ++e)
         s_part[(warp * NT * 8 + i * 8 + 2 * t + (e & 1)) * 16 + g + (e >> 1) * 8] = acc[i][e];
     __syncthreads();
-    for (int x = threadIdx.x; x < RW * 16 * M; x += LR_THREADS) {
-      const int m = x / (RW * 16), c = x % (RW * 16), n = tile * RW * 16 + c;
-      if (n >= N) continue;
+    auto total = [&](int m, int c) {
       float v = 0.f;
       for (int k = 0; k < KW; ++k) v += s_part[(((c >> 4) * KW + k) * NT * 8 + m) * 16 + (c & 15)];
-      if (EPI == LR_STORE) reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(v);
+      return v;
+    };
+    constexpr int PER = EPI == LR_GLU ? 8 : 16;                // outputs of a row tile
+    for (int x = threadIdx.x; x < RW * PER * M; x += LR_THREADS) {
+      const int m = x / (RW * PER), c = x % (RW * PER) * (16 / PER), n = tile * RW * 16 + c;
+      if (n >= N) continue;
+      const float v = total(m, c);
+      if (EPI == LR_GLU) {
+        const float g = fminf(v, ex.limit), u = fminf(fmaxf(total(m, c + 1), -ex.limit), ex.limit);
+        reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n / 2] = __float2bfloat16(g * sigmoid_f(1.702f * g) * (u + 1.f));
+      } else if (EPI == LR_SIDE) {
+        const int id = ex.ids[m];
+        float o = 0.f;
+        if (n < ex.dim && id >= 0 && id < ex.vocab) o = gelu_tanh_x(v) * __bfloat162float(ex.side[(size_t)id * ex.ld_side + ex.off + n]);
+        reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(o);
+      } else if (EPI == LR_STORE && n >= ex.n_split) {
+        ex.y2[(size_t)m * ex.ldy2 + n - ex.n_split] = v;
+      } else if (EPI == LR_STORE) reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(v);
       else if (EPI == LR_STORE_F32) reinterpret_cast<float*>(y)[(size_t)m * ldy + n] = v;
       else reinterpret_cast<float*>(y)[(size_t)m * ldy + n] += v;
     }
@@ -173,9 +199,9 @@ TRL_API int trl_linear_rows_max(int K) {
 
 // x: bf16 [M, ldx], or the fp32 stream when norm_w is given (its row norm counts n_norm columns).  w: bf16 [N, K],
 // K a multiple of 64.  epi: 0 store bf16, 1 store fp32, 2 add to fp32.  M <= trl_linear_rows_max(K).
-TRL_API int trl_linear_rows(const void* x, int ldx, const void* w, const void* norm_w, float eps, int n_norm, void* y, int ldy,
-                            int M, int N, int K, int epi, void* stream) {
-  if (M < 1 || N < 1 || K < 64 || K % 64 || M > trl_linear_rows_max(K) || ldx % 8 || epi < 0 || epi > 2 ||
+static int lr_launch(const void* x, int ldx, const void* w, const void* norm_w, float eps, int n_norm, void* y, int ldy,
+                     int M, int N, int K, int epi, const LrExtra& ex, void* stream) {
+  if (M < 1 || N < 1 || K < 64 || K % 64 || M > trl_linear_rows_max(K) || ldx % 8 || epi < 0 || epi > 4 ||
       (norm_w && n_norm < 1) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return (int)cudaErrorInvalidValue;
   const int groups = (N + 15) / 16;
@@ -198,13 +224,48 @@ TRL_API int trl_linear_rows(const void* x, int ldx, const void* w, const void* n
       configured = true;                                                                                                \
     }                                                                                                                   \
     e = trl_launch(kern, dim3(grid), dim3(LR_THREADS), smem, (cudaStream_t)stream, x, ldx, (const bf16*)w,              \
-                   (const float*)norm_w, eps, n_norm, y, ldy, M, N, K, KW, n_tiles);                                    \
+                   (const float*)norm_w, eps, n_norm, y, ldy, M, N, K, KW, n_tiles, ex);                                    \
   }
 #define LR_BOTH(NO, NTT, EP) LR_CASE(NO, NTT, EP, 2) LR_CASE(NO, NTT, EP, 4)
   LR_BOTH(true, 1, LR_STORE) LR_BOTH(true, 1, LR_STORE_F32) LR_BOTH(true, 2, LR_STORE) LR_BOTH(true, 2, LR_STORE_F32)
   LR_BOTH(false, 1, LR_STORE) LR_BOTH(false, 1, LR_STORE_F32) LR_BOTH(false, 1, LR_ADD_F32)
   LR_BOTH(false, 2, LR_STORE) LR_BOTH(false, 2, LR_STORE_F32) LR_BOTH(false, 2, LR_ADD_F32)
+  LR_BOTH(false, 1, LR_GLU) LR_BOTH(false, 2, LR_GLU) LR_BOTH(false, 1, LR_SIDE) LR_BOTH(false, 2, LR_SIDE)
 #undef LR_BOTH
 #undef LR_CASE
   return (int)e;
+}
+
+TRL_API int trl_linear_rows(const void* x, int ldx, const void* w, const void* norm_w, float eps, int n_norm, void* y, int ldy,
+                            int M, int N, int K, int epi, void* stream) {
+  if (epi > 2) return (int)cudaErrorInvalidValue;
+  LrExtra ex = {};
+  ex.n_split = 1 << 30;
+  return lr_launch(x, ldx, w, norm_w, eps, n_norm, y, ldy, M, N, K, epi, ex, stream);
+}
+
+// Rows n < n_split as bf16 into y, the others as fp32 into y2 (both row-major, their own leading dimensions).
+TRL_API int trl_linear_rows_split(const void* x, int ldx, const void* w, void* y, int ldy, int n_split, void* y2, int ldy2, int M, int N,
+                                  int K, void* stream) {
+  if (!y2 || n_split < 0) return (int)cudaErrorInvalidValue;
+  LrExtra ex = {};
+  ex.y2 = (float*)y2, ex.ldy2 = ldy2, ex.n_split = n_split;
+  return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_STORE, ex, stream);
+}
+
+// w: rows 2j = gate_j, 2j + 1 = up_j; y: bf16 [M, N / 2].
+TRL_API int trl_linear_rows_glu(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, float limit, void* stream) {
+  if (N % 2) return (int)cudaErrorInvalidValue;
+  LrExtra ex = {};
+  ex.limit = limit;
+  return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_GLU, ex, stream);
+}
+
+// y[m, n] = gelu(x W^T) * side[ids[m], off + n] for n < dim, 0 past it.
+TRL_API int trl_linear_rows_side(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, const void* ids, const void* side,
+                                 long ld_side, int off, int dim, int vocab, void* stream) {
+  if (!ids || !side || dim > N || off < 0 || off + dim > ld_side) return (int)cudaErrorInvalidValue;
+  LrExtra ex = {};
+  ex.ids = (const int*)ids, ex.side = (const bf16*)side, ex.ld_side = ld_side, ex.off = off, ex.dim = dim, ex.vocab = vocab;
+  return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_SIDE, ex, stream);
 }

@@ -8,7 +8,7 @@ import pytest
 import torch
 
 import fetotar_oracle as oracle
-from fetotar_cases import (BACKENDS, CONFIGS, TOL, attn, backends, build, feed_all, needle_model, random_weights, rel_err, rot, tokens,
+from fetotar_cases import (BACKENDS, CONFIGS, TOL, attn, backends, build, close, feed_all, needle_model, random_weights, rel_err, rot, tokens,
                            want_logits)
 from tilerl_b200.config import FetotarConfig, config_from_dir, get_config
 from tilerl_b200.engine import SamplingParams, StepLimits
@@ -176,7 +176,7 @@ def test_whole_prompt_matches_the_oracle(backend, name):
     eng = build(cfg, w, backend)
     for n in (1, 2, 15, 17, 64, 65, 150):
         toks = tokens(cfg, n, seed=n)
-        assert rel_err(feed_all(eng, "a", toks, [n]), want_logits(cfg, w, toks)) < TOL[backend], n
+        assert close(feed_all(eng, "a", toks, [n]), want_logits(cfg, w, toks), backend), n
     assert eng.kv.used_blocks == 0 and eng.states.free_slots == 4
 
 
@@ -188,7 +188,7 @@ def test_portions_and_token_by_token_match_the_oracle(backend, name, cuts):
     w = random_weights(cfg, seed=3)
     toks = tokens(cfg, 147, seed=7)
     got = feed_all(build(cfg, w, backend), "a", toks, cuts)
-    assert rel_err(got, want_logits(cfg, w, toks)) < TOL[backend]
+    assert close(got, want_logits(cfg, w, toks), backend)
 
 
 @backends
@@ -203,7 +203,7 @@ def test_layer_outputs_match_the_oracle(backend):
     _, x, taps = eng.model.forward(batch, eng.ops, eng.kv, eng.states, aux_layers=tuple(range(cfg.n_layers)))
     for layer, t in taps.items():
         want = states[layer].float()
-        assert float((t.cpu().float() - want).abs().max() / want.abs().max()) < TOL[backend], layer
+        assert float((t.cpu().float() - want).abs().max() / want.abs().max()) < 3 * TOL[backend], layer
     assert torch.equal(x, taps[cfg.n_layers - 1])
 
 
@@ -241,7 +241,7 @@ def test_mixed_batches_of_unequal_requests_equal_each_alone(backend, name):
             got[k].append(out[o:o + len(t)])
             o += len(t)
     for k in lens:
-        assert rel_err(torch.cat(got[k]), want_logits(cfg, w, toks[k])) < TOL[backend], k
+        assert close(torch.cat(got[k]), want_logits(cfg, w, toks[k]), backend), k
     assert eng.kv.used_blocks == 0 and eng.states.free_slots == 4
 
 
@@ -256,7 +256,7 @@ def test_freed_pages_and_slots_carry_nothing_over(backend):
         eng.states.states.fill_(math.nan), eng.states.ring.fill_(math.nan)
         eng.states.cur.fill_(0)
         toks = tokens(cfg, n, seed=20 + i)
-        assert rel_err(feed_all(eng, i, toks, [50, 1, 1, 3, 16, 1]), want_logits(cfg, w, toks)) < TOL[backend]
+        assert close(feed_all(eng, i, toks, [50, 1, 1, 3, 16, 1]), want_logits(cfg, w, toks), backend)
 
 
 @backends
@@ -284,7 +284,7 @@ def test_window_edges(backend, decode, window, turned):
             if cut:
                 eng.feed([("a", toks[:cut], [])])
             got = eng.feed([("a", toks[cut:], [n - 1 - cut])], ["a"])
-            assert rel_err(got, want) < TOL[backend], (at, cut)
+            assert close(got, want, backend), (at, cut)
 
 
 @backends
@@ -298,7 +298,7 @@ def test_the_first_tokens_of_a_sequence(backend):
     for n in range(1, 9):
         got = eng.feed([("a", toks[:n], list(range(n)))]).clone()
         rest = eng.feed([("a", toks[n:], list(range(30 - n)))], ["a"])
-        assert rel_err(torch.cat([got, rest]), want) < TOL[backend], n
+        assert close(torch.cat([got, rest]), want, backend), n
 
 
 @backends
@@ -321,7 +321,7 @@ def test_a_state_remembers_a_far_token(backend, name):
     eng = build(cfg, w, backend)
     for cuts in ([n], [64, 64, 64, 3], [37, 100, 1, 2, 100], [200, 1]):
         got, moved = feed_all(eng, "a", toks, cuts), feed_all(eng, "b", other, cuts)
-        assert rel_err(got, want) < TOL[backend] and rel_err(moved, changed) < TOL[backend], cuts
+        assert close(got, want, backend) and close(moved, changed, backend), cuts
         d = (moved[-1] - got[-1]).float().cpu()
         assert rel_err(d[None], (changed - want)[-1:]) < (0.02 if "bf16" not in backend else 1.5), cuts
 
@@ -332,7 +332,7 @@ def test_long_decoding_through_cache_and_state(backend):
     w = random_weights(cfg, seed=8)
     toks = tokens(cfg, 300, seed=40)
     eng = build(cfg, w, backend)
-    assert rel_err(feed_all(eng, "a", toks, [20, 1]), want_logits(cfg, w, toks)) < TOL[backend]
+    assert close(feed_all(eng, "a", toks, [20, 1]), want_logits(cfg, w, toks), backend)
     if eng.graph is not None and eng.graph.enabled:
         assert eng.counters["graph_ticks"] == 280              # decoded in captured ticks
 
@@ -464,4 +464,4 @@ def test_trace_replay_program(backend, tmp_path):
     la, lb = want_logits(cfg, w, ta), want_logits(cfg, w, tb)
     for n, want in ((0, la[[3, 19]]), (2, torch.stack([lb[8], la[29], la[20]]))):
         got = torch.from_numpy(np.fromfile(str(tmp_path / f"{n}.f32"), dtype="<f4").reshape(-1, cfg.vocab).copy())
-        assert rel_err(got, want) < TOL[backend]
+        assert close(got, want, backend)

@@ -11,9 +11,14 @@ import ctypes
 import torch
 
 from . import native as N
-from .cuda_stream import EPI_STORE_F32
+from .cuda_stream import EPI_STORE, EPI_STORE_F32
 
 MAMBA2, MLSTM = 0, 1
+MIX_ROWS_MAX = 16       # rows the weight-streaming projection serves
+LATENT_SHORT = 32       # tokens of a sequence up to which attention runs in the latent (absorbed) form
+SCAN_SHORT = 16         # tokens of a sequence up to which a scan goes token by token
+CHUNK_DK = 128          # state rows the chunked scan takes
+PART_BYTES = 1 << 28    # most fp32 partial sums of split attention
 
 
 class ScanArgs(ctypes.Structure):
@@ -34,6 +39,10 @@ def _norm_kind(norm) -> int:
 
 
 class MixerOps:
+    def _streams_mix(self, rows: int, w) -> bool:
+        """This many rows go through the weight-streaming projection, whose epilogues save a launch each."""
+        return w.dtype == torch.bfloat16 and rows <= MIX_ROWS_MAX and rows <= self.lib.trl_linear_rows_max(w.shape[1])
+
     # ---- stream ----------------------------------------------------------------------
     def _join(self, x, y, post, nxt, h, table, ids, scale, eps, n):
         t, ld = x.shape
@@ -65,6 +74,11 @@ class MixerOps:
         t, ng = h.shape[0], w.shape[0] - n_in
         proj = self.ws.get(f"block_proj_{w.dtype}", (t, n_in), w.dtype)
         gates = self.ws.get("mix_gates", (t, max(ng, 1)), torch.float32)
+        if self._streams_mix(t, w):
+            N.check(self.lib.trl_linear_rows_split(h.data_ptr(), h.stride(0), w.data_ptr(), proj.data_ptr(), n_in, n_in, gates.data_ptr(),
+                                                   max(ng, 1), t, w.shape[0], w.shape[1], N.stream()), "linear_rows_split")
+            N.count()
+            return proj, gates
         self._mm(h, w[:n_in], proj)
         if ng:
             self._mm(h, w[n_in:], gates)
@@ -72,7 +86,7 @@ class MixerOps:
 
     def project_f32(self, a, w):
         y = self.ws.get("branch", (a.shape[0], w.shape[0]), torch.float32)
-        if self._streams(a.shape[0], w):
+        if self._streams_mix(a.shape[0], w):
             self._linear_rows(a, w, y, EPI_STORE_F32)
             return y
         return self._mm(a, w, y)
@@ -80,7 +94,7 @@ class MixerOps:
     def project_logits(self, h, w):
         logits = self.ws.get("logits", (h.shape[0], w.shape[0]), torch.float32)
         h = h.contiguous()
-        if self._streams(h.shape[0], w):
+        if self._streams_mix(h.shape[0], w):
             self._linear_rows(h, w, logits, EPI_STORE_F32)
             return logits
         return self._mm(h, w, logits)
@@ -88,6 +102,11 @@ class MixerOps:
     def clamped_glu(self, h, w, limit):
         t, n = h.shape[0], w.shape[0]
         out = self.ws.get(f"glu_{w.dtype}", (t, n // 2), w.dtype)
+        if self._streams_mix(t, w):
+            N.check(self.lib.trl_linear_rows_glu(h.data_ptr(), h.stride(0), w.data_ptr(), out.data_ptr(), n // 2, t, n, w.shape[1], limit,
+                                                 N.stream()), "linear_rows_glu")
+            N.count()
+            return out
         gu = self._mm(h, w, self.ws.get(f"gate_up_{w.dtype}", (t, n), w.dtype))
         N.check(self.lib.trl_clamped_glu(gu.data_ptr(), out.data_ptr(), out.numel(), limit, _f32(w), N.stream()), "clamped_glu")
         N.count()
@@ -95,10 +114,15 @@ class MixerOps:
 
     def side_input(self, h, w, table, ids, layer, dim):
         t, n = h.shape[0], w.shape[0]
-        out = self.ws.get(f"side_{w.dtype}", (t, n), w.dtype)
+        out, off = self.ws.get(f"side_{w.dtype}", (t, n), w.dtype), layer * ((dim + 7) // 8 * 8)
+        if self._streams_mix(t, w):
+            N.check(self.lib.trl_linear_rows_side(h.data_ptr(), h.stride(0), w.data_ptr(), out.data_ptr(), n, t, n, w.shape[1], ids.data_ptr(),
+                                                  table.data_ptr(), table.shape[1], off, dim, table.shape[0], N.stream()), "linear_rows_side")
+            N.count()
+            return out
         z = self._mm(h, w, self.ws.get(f"side_z_{w.dtype}", (t, n), w.dtype))
         N.check(self.lib.trl_side_input(z.data_ptr(), table.data_ptr(), ids.data_ptr(), out.data_ptr(), t, n, dim, table.shape[1],
-                                        layer * ((dim + 7) // 8 * 8), table.shape[0], _f32(w), N.stream()), "side_input")
+                                        off, table.shape[0], _f32(w), N.stream()), "side_input")
         N.count()
         return out
 
@@ -110,13 +134,19 @@ class MixerOps:
             proj.data_ptr(), proj.stride(0), q_norm.data_ptr(), kv_norm.data_ptr(), freqs.data_ptr(), batch.positions.data_ptr(),
             batch.slot_mapping.data_ptr(), cq.data_ptr(), cache.data_ptr(), cache.shape[0], t, l.c0, l.kr0, l.q_rank, l.kv_rank, l.kv,
             l.rd, freqs.numel(), rot.amplitude, eps, _f32(proj), st), "latent_prep")
-        q = self._mm(cq, uq, self.ws.get(f"latent_q_{proj.dtype}", (t, uq.shape[0]), proj.dtype))
+        q = self.ws.get(f"latent_q_{proj.dtype}", (t, uq.shape[0]), proj.dtype)
+        if self._streams_mix(t, uq):
+            self._linear_rows(cq, uq, q, EPI_STORE)
+        else:
+            self._mm(cq, uq, q)
         N.check(self.lib.trl_latent_rope(q.data_ptr(), freqs.data_ptr(), batch.positions.data_ptr(), t, l.heads, l.dq, l.dk, freqs.numel(),
                                          rot.amplitude, _f32(q), st), "latent_rope")
         N.count(2)
         return q.view(t, l.heads, l.dq)
 
     def latent_attention(self, q, proj, up, l, batch, pool, idx):
+        if proj.dtype == torch.bfloat16 and self.lib.trl_latent_mma_ok(l.dk, l.rd, l.dv, l.kv):
+            return self._latent_mma(q, proj, up, l, batch, pool, idx)
         t, cache, table, dt, st = proj.shape[0], pool.layer(idx), batch.block_table, proj.dtype, N.stream()
         uk, uv = up[:l.heads * l.dk].view(l.heads, l.dk, l.kv), up[l.heads * l.dk:].view(l.heads, l.dv, l.kv)
         ql = self.ws.get(f"latent_ql_{dt}", (l.heads, t, l.kv), dt)
@@ -134,7 +164,69 @@ class MixerOps:
         N.count(2)
         return out
 
+    def _latent_mma(self, q, proj, up, l, batch, pool, idx):
+        """Short sequences in the absorbed form (one pass over the cached latents for all heads), prompts over expanded
+        keys and values."""
+        t, cache, table, st = proj.shape[0], pool.layer(idx), batch.block_table, N.stream()
+        lens, kvs, bf = batch.host_q_len, batch.host_kv_len, torch.bfloat16
+        out = self.ws.get(f"mix_out_{bf}", (t, l.n_out), bf)
+        starts = [0]
+        for n in lens:
+            starts.append(starts[-1] + n)
+        short = [i for i, n in enumerate(lens) if n <= LATENT_SHORT]
+        prompts = [i for i, n in enumerate(lens) if n > LATENT_SHORT]
+        if short:
+            ts = max(starts[i + 1] for i in short)                           # tokens up to the last short sequence's
+            blocks = sum((lens[i] * l.heads + 15) // 16 for i in short)
+            keys = min(l.window + LATENT_SHORT, table.shape[1] * 16 if self.attn_splits else max(kvs[i] for i in short))
+            splits = max(1, min(16, (keys + 127) // 128, self.sms // blocks, PART_BYTES // (ts * l.heads * l.kv * 4)))
+            ql = self.ws.get("latent_rows", (ts, l.heads, l.row), bf)
+            part = self.ws.get("attn_part", (ts * l.heads * splits * l.kv,), torch.float32)
+            ml = self.ws.get("attn_part_ml", (ts * l.heads * splits * 2,), torch.float32)
+            N.check(self.lib.trl_latent_decode(
+                q.data_ptr(), l.dq, l.dk, l.rd, up.data_ptr(), l.kv, l.dv, ql.data_ptr(), cache.data_ptr(), cache.shape[0], table.data_ptr(),
+                table.stride(0), batch.q_start.data_ptr(), batch.q_len.data_ptr(), batch.positions.data_ptr(), batch.seq_ids.data_ptr(),
+                part.data_ptr(), ml.data_ptr(), proj[:, l.g0:].data_ptr(), proj.stride(0), out.data_ptr(), l.n_out, ts, batch.n_seqs,
+                max((lens[i] * l.heads + 15) // 16 for i in short), l.heads, splits, l.window, 1, LATENT_SHORT if prompts else 1 << 30, l.scale,
+                st), "latent_decode")
+            N.count(3)
+        if prompts:
+            los = [max(0, kvs[i] - lens[i] - l.window + 1) for i in prompts]
+            n_keys = [kvs[i] - lo for i, lo in zip(prompts, los)]
+            total, ldkv = sum(n_keys), l.heads * (l.dk + l.dv)
+            c, kr = self.ws.get("latent_c", (total, l.kv), bf), self.ws.get("latent_kr", (total, l.rd), bf)
+            o = 0
+            for i, lo, n in zip(prompts, los, n_keys):
+                N.check(self.lib.trl_latent_gather(cache.data_ptr(), cache.shape[0], table[i].data_ptr(), lo, n, l.kv, l.rd, c[o:].data_ptr(),
+                                                   kr[o:].data_ptr(), st), "latent_gather")
+                o += n
+            kvx = self._mm(c, up, self.ws.get("latent_kvx", (total, ldkv), bf))
+            o = 0
+            for i, lo, n in zip(prompts, los, n_keys):
+                q0 = starts[i]
+                N.check(self.lib.trl_latent_prompt(
+                    q[q0:].data_ptr(), l.dq, l.dk, l.rd, l.dv, kvx[o:].data_ptr(), ldkv, kr[o:].data_ptr(), proj[q0:, l.g0:].data_ptr(),
+                    proj.stride(0), out[q0:].data_ptr(), l.n_out, batch.positions[q0:].data_ptr(), lens[i], lo, n, l.heads, l.window, l.scale,
+                    st), "latent_prompt")
+                o += n
+            N.count(2 * len(prompts))
+        return out
+
     # ---- recurrent mixers ------------------------------------------------------------------
+    def _scan(self, a: ScanArgs, batch, kind: int, dt, st) -> None:
+        """Prompts chunk by chunk on tensor cores, everything else token by token."""
+        chunked = dt == torch.bfloat16 and a.dk <= CHUNK_DK and not a.keep_flags
+        prompts = sum(n > SCAN_SHORT for n in batch.host_q_len) if chunked else 0
+        if prompts:
+            a.min_len = SCAN_SHORT + 1 if prompts < batch.n_seqs else 1
+            narrow = int(prompts * a.heads * ((a.dv + 63) // 64) < self.sms)
+            N.check(self.lib.trl_scan_chunk(ctypes.byref(a), batch.n_seqs, kind, narrow, st), "scan_chunk")
+            N.count()
+        if prompts < batch.n_seqs:
+            a.min_len, a.max_len = 1, SCAN_SHORT if prompts else 1 << 30
+            N.check(self.lib.trl_scan_serial(ctypes.byref(a), batch.n_seqs, kind, int(dt == torch.float32), st), "scan_serial")
+            N.count()
+
     def recurrent_mix(self, proj, gates, w, l, batch, pool, idx, eps):
         t, dt, st = proj.shape[0], proj.dtype, N.stream()
         kind = MAMBA2 if l.kind == "mamba2" else MLSTM
@@ -158,12 +250,12 @@ class MixerOps:
         a.cur, a.keep_flags = pool.cur.data_ptr(), N.ptr(batch.keep_flags) if batch.keep_steps else None
         a.q_start, a.q_len, a.slots = batch.q_start.data_ptr(), batch.q_len.data_ptr(), batch.state_slots.data_ptr()
         a.o, a.heads, a.dk, a.dv, a.min_len, a.max_len = o.data_ptr(), l.heads, l.dk, l.dv, 1, 1 << 30
-        N.check(self.lib.trl_scan_serial(ctypes.byref(a), batch.n_seqs, kind, _f32(proj), st), "scan_serial")
+        self._scan(a, batch, kind, dt, st)
         out = self.ws.get(f"mix_out_{dt}", (t, l.n_out), dt)
         N.check(self.lib.trl_scan_norm(
             o.data_ptr(), proj[:, l.g0:].data_ptr(), proj.stride(0), w["norm"].data_ptr(), out.data_ptr(), l.n_out, t, l.heads, l.vdim, l.dv,
             l.norm_groups, eps, proj.data_ptr(), N.ptr(ring), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1), l.conv_c,
             batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(), batch.q_len.data_ptr(),
             batch.state_slots.data_ptr(), kind, _f32(proj), st), "scan_norm")
-        N.count(2)
+        N.count()
         return out

@@ -10,6 +10,7 @@ JSON line:
   command profiler captures of single kernels are taken on;
 * ``zinutar`` (:mod:`.zinutar`): the Zinutar design beside the hybrid's attention-only form at equal size,
   whole models and single kernels;
+* ``fetotar`` (:mod:`.fetotar`): the Fetotar design beside the hybrid with Gated-DeltaNet layers, likewise;
 * ``grpo`` (:mod:`.grpo`): one-GPU GRPO step with LoRA adapters, split rollout / train;
 * ``grpo-zero3`` (:mod:`.grpo_zero3`, started under ``torchrun``): GRPO step with ZeRO-3 training
   and a tensor-parallel NVFP4 rollout engine on the same GPUs.
@@ -28,6 +29,7 @@ SUITES = {
     "sparse": ("serve", ["--what", "sparse"]),
     "tick": ("tick", []),
     "zinutar": ("zinutar", []),
+    "fetotar": ("fetotar", []),
     "grpo": ("grpo", []),
     "grpo-zero3": ("grpo_zero3", []),
 }
