@@ -14,20 +14,6 @@ namespace {
 
 enum { NORM_NONE = 0, NORM_RMS = 1, NORM_LAYER = 2 };
 
-template <typename T> __device__ __forceinline__ void store4(T* p, float a, float b, float c, float d);
-template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float a, float b, float c, float d) {
-  *reinterpret_cast<uint2*>(p) = make_uint2(f2_to_bf162_bits(a, b), f2_to_bf162_bits(c, d));
-}
-template <> __device__ __forceinline__ void store4<float>(float* p, float a, float b, float c, float d) {
-  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
-}
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const bf16* p) {
-  const uint2 v = *reinterpret_cast<const uint2*>(p);
-  const float2 a = bf162_bits_to_f2(v.x), b = bf162_bits_to_f2(v.y);
-  return make_float4(a.x, a.y, b.x, b.y);
-}
-
 // (mean, 1 / deviation) of the row's first n values, or (0, 1 / rms)
 template <int R>
 __device__ __forceinline__ float2 row_stats(const float4 (&v)[R], int kind, int n, float eps, float* red) {

@@ -18,13 +18,6 @@
 
 namespace {
 
-__device__ __forceinline__ void pair_angle(int pos, double freq, float amp, float& c, float& s) {
-  const double a = (double)pos * freq;
-  const double turns = rint(a * 0.15915494309189535);
-  sincosf((float)fma(-turns, 6.283185307179586, a), &s, &c);
-  c *= amp, s *= amp;
-}
-
 struct PrepArgs {
   int ldp, c0, kr0, q_rank, kv_rank, kv, rd, n_pairs, n_blocks;
   float amp, eps;

@@ -19,68 +19,76 @@ namespace {
 
 constexpr int TILE = 64, TPAGES = TILE / KVB;
 constexpr long long LD_WAIT_CYCLES = 4000000000LL;
-constexpr int LD_SMEM = 216 * 1024;
+constexpr int LD_SMEM = 216 * 1024, MAX_SPLITS = 32;
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ bool in_class(int n, int lo, int hi) { return n >= lo && n <= hi; }
 
-// grid (head, 128 latent columns, TT tokens), 128 threads: 16 column groups of 8 x 8 groups of query dimensions
-template <int TT>
-__global__ void __launch_bounds__(128)
-latent_absorb_kernel(const bf16* q, int dq, int dk, int rd, const bf16* __restrict__ uk, int kv, const int* seq_ids, const int* q_len,
-                     int max_len, bf16* ql, int T, int heads) {
-  extern __shared__ float s_ab[];                      // [TT][dk], then [8][TT][128]
-  pdl_launch_dependents(44);
-  const int h = blockIdx.x, c0 = blockIdx.y * 128, t0 = blockIdx.z * TT, n = min(TT, T - t0), tid = threadIdx.x;
-  pdl_wait();
-  bool any = false;
-  for (int t = 0; t < n; ++t) any |= q_len[seq_ids[t0 + t]] <= max_len;
-  if (!any) return;
-  const int D = kv + rd;
-  for (int x = tid; x < TT * dk; x += 128) {
-    const int t = x / dk, d = x % dk;
-    s_ab[x] = t < n ? __bfloat162float(q[((size_t)(t0 + t) * heads + h) * dq + d]) : 0.f;
-  }
-  if (blockIdx.y == 0)                                 // the rotated part as it is
-    for (int x = tid; x < n * (rd / 8); x += 128) {
-      const int t = x / (rd / 8), c = x % (rd / 8);
-      *reinterpret_cast<uint4*>(ql + ((size_t)(t0 + t) * heads + h) * D + kv + c * 8) =
-          *reinterpret_cast<const uint4*>(q + ((size_t)(t0 + t) * heads + h) * dq + dk + c * 8);
-    }
-  __syncthreads();
-  const int c = (tid & 15) * 8, g = tid >> 4;
-  float acc[TT][8];
-#pragma unroll
-  for (int t = 0; t < TT; ++t)
-#pragma unroll
-    for (int e = 0; e < 8; ++e) acc[t][e] = 0.f;
-  if (c0 + c < kv) {
-    const bf16* w = uk + (size_t)h * dk * kv + c0 + c;
+// acc += 16 weight rows x 8 token columns over K (a multiple of 16): wa, wb point at rows g and g + 8 of the tile (g = lane / 4)
+// plus 8 (lane % 4); xs at token g's row of the activations in shared memory plus the same.  The 8 values a lane loads of a
+// row serve two MMAs under a permutation of k that the activations share.
+template <bool TWO>
+__device__ __forceinline__ void rows16(float (&acc)[4], const bf16* __restrict__ wa, const bf16* __restrict__ wb, const bf16* xs, const bf16* xl,
+                                       int K, int t4) {
 #pragma unroll 4
-    for (int d = g; d < dk; d += 8) {
-      float f[8];
-      Chunk<bf16>::get(*reinterpret_cast<const uint4*>(w + (size_t)d * kv), f);
-#pragma unroll
-      for (int t = 0; t < TT; ++t) {
-        const float x = s_ab[t * dk + d];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[t][e] = fmaf(x, f[e], acc[t][e]);
-      }
+  for (int k = 0; k < K; k += 32) {
+    uint4 a = make_uint4(0u, 0u, 0u, 0u), b = a, x = a, y = a;
+    if (k + t4 * 8 < K) {
+      a = *reinterpret_cast<const uint4*>(wa + k), b = *reinterpret_cast<const uint4*>(wb + k);
+      x = *reinterpret_cast<const uint4*>(xs + k);
+      if (TWO) y = *reinterpret_cast<const uint4*>(xl + k);
     }
+    const uint32_t f0[4] = {a.x, b.x, a.y, b.y}, f1[4] = {a.z, b.z, a.w, b.w};
+    mma16(acc, f0, x.x, x.y);
+    mma16(acc, f1, x.z, x.w);
+    if (TWO) mma16(acc, f0, y.x, y.y), mma16(acc, f1, y.z, y.w);
   }
-  float* part = s_ab + TT * dk;
-#pragma unroll
-  for (int t = 0; t < TT; ++t)
-#pragma unroll
-    for (int e = 0; e < 8; ++e) part[(g * TT + t) * 128 + c + e] = acc[t][e];
+}
+
+// grid (head, 128 latent columns, 8 tokens), 256 threads: a warp forms 16 columns of 8 tokens.  ukt: [heads][kv][dk].
+__global__ void __launch_bounds__(256)
+latent_absorb_kernel(const bf16* q, int dq, int dk, int rd, const bf16* __restrict__ ukt, int kv, const double* __restrict__ freqs, int n_pairs,
+                     float amp, const int* positions, const int* seq_ids, const int* q_len, int max_len, bf16* ql, int T, int heads) {
+  extern __shared__ __align__(16) unsigned char ab_raw[];
+  __shared__ bf16 s_o[8][128];
+  bf16* xs = reinterpret_cast<bf16*>(ab_raw);            // [8][dk + 8]
+  pdl_launch_dependents(44);
+  const int h = blockIdx.x, c0 = blockIdx.y * 128, t0 = blockIdx.z * 8, n = min(8, T - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int ldx = dk + 8, D = kv + rd;
+  pdl_wait();
+  const bool in = tid < n && q_len[seq_ids[t0 + tid]] <= max_len;
+  if (!__syncthreads_or(in)) return;
+  for (int x = tid; x < 8 * (dk / 8); x += 256) {
+    const int t = x / (dk / 8), c = x % (dk / 8);
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (t < n) v = *reinterpret_cast<const uint4*>(q + ((size_t)(t0 + t) * heads + h) * dq + c * 8);
+    *reinterpret_cast<uint4*>(xs + t * ldx + c * 8) = v;
+  }
+  if (blockIdx.y == 0)                                   // the rotated part, turned unless it already is (n_pairs 0)
+    for (int x = tid; x < n * (rd / 2); x += 256) {
+      const int t = x / (rd / 2), p = x % (rd / 2);
+      float2 v = bf162_bits_to_f2(*reinterpret_cast<const uint32_t*>(q + ((size_t)(t0 + t) * heads + h) * dq + dk + 2 * p));
+      if (p < n_pairs) {
+        float cs, sn;
+        pair_angle(positions[t0 + t], freqs[p], amp, cs, sn);
+        v = make_float2(v.x * cs - v.y * sn, v.y * cs + v.x * sn);
+      }
+      *reinterpret_cast<uint32_t*>(ql + ((size_t)(t0 + t) * heads + h) * D + kv + 2 * p) = f2_to_bf162_bits(v.x, v.y);
+    }
   __syncthreads();
-  for (int x = tid; x < n * 128; x += 128) {
-    const int t = x >> 7, cc = x & 127;
-    if (c0 + cc >= kv) continue;
-    float v = 0.f;
+  const int g = lane >> 2, t4 = lane & 3, r0 = c0 + warp * 16;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  if (r0 < kv) {                                         // (kv is a multiple of 16)
+    const bf16* w = ukt + ((size_t)h * kv + r0 + g) * dk + t4 * 8;
+    rows16<false>(acc, w, w + (size_t)8 * dk, xs + g * ldx + t4 * 8, nullptr, dk, t4);
+  }
 #pragma unroll
-    for (int k = 0; k < 8; ++k) v += part[(k * TT + t) * 128 + cc];
-    ql[((size_t)(t0 + t) * heads + h) * D + c0 + cc] = __float2bfloat16(v);
+  for (int e = 0; e < 4; ++e) s_o[2 * t4 + (e & 1)][warp * 16 + g + (e >> 1) * 8] = __float2bfloat16(acc[e]);
+  __syncthreads();
+  for (int x = tid; x < n * 16; x += 256) {
+    const int t = x >> 4, c = (x & 15) * 8;
+    if (c0 + c < kv)
+      *reinterpret_cast<uint4*>(ql + ((size_t)(t0 + t) * heads + h) * D + c0 + c) = *reinterpret_cast<const uint4*>(&s_o[t][c]);
   }
 }
 
@@ -103,7 +111,7 @@ __device__ __forceinline__ void tile_range(int p_first, int p_last, int window, 
   stages = (p_last / KVB - page0) / TPAGES + 1;
 }
 __device__ __forceinline__ int stages_per_split(int stages, int n_splits) {
-  const int want = max(1, min(n_splits, (stages + 1) / 2));        // at least 128 keys each
+  const int want = max(1, min(n_splits, stages));
   return (stages + want - 1) / want;
 }
 __device__ __forceinline__ uint32_t ld_try_wait(uint32_t bar, uint32_t parity) {
@@ -119,8 +127,9 @@ template <int OD, int HALVES>
 __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(const DecArgs a) {
   constexpr int NW = 4 * HALVES, THREADS = (NW + 1) * 32;
   extern __shared__ unsigned char ld_raw[];
-  __shared__ __align__(8) uint64_t s_bar[8];               // full[4], empty[4]
+  __shared__ __align__(8) uint64_t s_bar[12];              // full[4], empty[4], pair[4]
   __shared__ float s_m[4][16], s_l[4][16];
+  __shared__ float4 s_x[HALVES == 2 ? 2 : 1][HALVES == 2 ? 8 : 1][32];     // scores the two warps of a page exchange
   __shared__ volatile int s_ok;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const uint32_t raw_a = (uint32_t)__cvta_generic_to_shared(ld_raw);
@@ -131,6 +140,7 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
       asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(bar_a + 8u * st));
       asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar_a + 32u + 8u * st), "r"(NW));
     }
+    for (int k = 0; k < 4; ++k) asm volatile("mbarrier.init.shared::cta.b64 [%0], 2;" ::"r"(bar_a + 64u + 8u * k));
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     s_ok = 1;
   }
@@ -231,20 +241,52 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
     };
     const int vc0 = half * (OD / 8), vch = min(OD / 8, a.vch - vc0);      // this warp's output chunks
     int st = 0;
-    uint32_t ph = 0;
+    uint32_t ph = 0, xp = 0;                               // xp: parity and buffer of the exchange
     for (int k = s0; k < s1; ++k) {
       if (!bounded_wait(bar_a + 8u * st, ph, 520 + st)) break;
       const int j0 = (page0 + k * TPAGES + kw) * KVB;
       if (j0 < hi) {
         const uint32_t base = ring_a + st * stage_b + kw * page_b;
         float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        if constexpr (HALVES == 1) {
 #pragma unroll 4
-        for (int kk = 0; kk < nc / 2; ++kk) {
-          uint32_t qv[4], b[4];
-          ldsm4(qv, qa + kk * 32);
-          ldsm4(b, base + (kr * nc + place(kk * 2 + kcl, kr, krot)) * 16);
-          mma16(sc[0], qv, b[0], b[1]);
-          mma16(sc[1], qv, b[2], b[3]);
+          for (int kk = 0; kk < nc / 2; ++kk) {
+            uint32_t qv[4], b[4];
+            ldsm4(qv, qa + kk * 32);
+            ldsm4(b, base + (kr * nc + place(kk * 2 + kcl, kr, krot)) * 16);
+            mma16(sc[0], qv, b[0], b[1]);
+            mma16(sc[1], qv, b[2], b[3]);
+          }
+        } else {
+          // each of the page's two warps scores 8 of its keys (two k-steps an iteration, in two sums) and hands them over
+          float s2[4] = {0.f, 0.f, 0.f, 0.f};
+          const int r8 = half * 8 + (lane & 7), rot8 = r8 % nc, c8 = lane >> 3;
+#pragma unroll 2
+          for (int kk = 0; kk < nc / 4; ++kk) {
+            uint32_t q0v[4], q1v[4], b[4];
+            ldsm4(q0v, qa + kk * 64);
+            ldsm4(q1v, qa + kk * 64 + 32);
+            ldsm4(b, base + (r8 * nc + place(kk * 4 + c8, r8, rot8)) * 16);
+            mma16(sc[0], q0v, b[0], b[1]);
+            mma16(s2, q1v, b[2], b[3]);
+          }
+          if (nc & 2) {                                    // an odd number of k-steps: the last one alone
+            uint32_t q0v[4], b[4];
+            ldsm4(q0v, qa + (nc / 2 - 1) * 32);
+            ldsm4(b, base + (r8 * nc + place(nc - 2 + (c8 & 1), r8, rot8)) * 16);
+            mma16(sc[0], q0v, b[0], b[1]);
+          }
+          const float4 mine = make_float4(sc[0][0] + s2[0], sc[0][1] + s2[1], sc[0][2] + s2[2], sc[0][3] + s2[3]);
+          const uint32_t pair = bar_a + 64u + 8u * kw;
+          s_x[xp][warp][lane] = mine;
+          __syncwarp();
+          if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(pair) : "memory");
+          if (!bounded_wait(pair, xp, 540 + kw)) break;
+          const float4 other = s_x[xp][warp ^ 4][lane];
+          xp ^= 1u;
+          const float4 lo4 = half ? other : mine, hi4 = half ? mine : other;
+          sc[0][0] = lo4.x, sc[0][1] = lo4.y, sc[0][2] = lo4.z, sc[0][3] = lo4.w;
+          sc[1][0] = hi4.x, sc[1][1] = hi4.y, sc[1][2] = hi4.z, sc[1][3] = hi4.w;
         }
         uint32_t wh[4], wl[4];
         float now[2], back[2];
@@ -343,72 +385,70 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
   }
 }
 
-// grid (head, TT tokens, shares of the value rows), 256 threads
-template <int TT>
+// grid (head, 8 tokens, shares of the value rows), 256 threads
 __global__ void __launch_bounds__(256)
 latent_out_kernel(const float* part, const float2* ml, int n_splits, const bf16* __restrict__ uv, int kv, int dv, const bf16* gate, int ldp,
                   bf16* out, int n_out, const int* seq_ids, const int* q_start, const int* q_len, const int* positions, int T, int heads,
                   int window, int max_len) {
-  extern __shared__ float s_oc[];                        // [TT][kv]
-  __shared__ int s_in[TT];
+  extern __shared__ __align__(16) unsigned char oc_raw[];
+  __shared__ float s_f[8][MAX_SPLITS];                   // factor of every share
+  __shared__ int s_used[8];                              // shares of a token's row; 0: not this launch's
+  const int ldx = kv + 8;
+  bf16 *hi = reinterpret_cast<bf16*>(oc_raw), *lo = hi + 8 * ldx;       // [8][kv + 8] each
   pdl_launch_dependents(46);
   pdl_wait();
-  const int h = blockIdx.x, t0 = blockIdx.y * TT, n = min(TT, T - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int rows = (dv + gridDim.z - 1) / gridDim.z, d0 = blockIdx.z * rows, d1 = min(dv, d0 + rows);
-  bool any = false;
-#pragma unroll
-  for (int i = 0; i < TT; ++i) {
-    const int t = t0 + i;
-    bool in = i < n;
-    int seq = 0, len = 0, q0 = 0;
-    if (in) seq = seq_ids[t], len = q_len[seq], q0 = q_start[seq], in = len <= max_len && t - q0 < len;
-    if (tid == 0) s_in[i] = in;
-    any |= in;
-    if (!in) {
-      for (int c = tid; c < kv; c += 256) s_oc[i * kv + c] = 0.f;
-      continue;
-    }
-    const int n_rows = len * heads, row0 = ((t - q0) * heads + h) / 16 * 16;
-    int page0, stages;
-    tile_range(positions[q0 + row0 / heads], positions[q0 + (min(row0 + 16, n_rows) - 1) / heads], window, page0, stages);
-    const int sps = stages_per_split(stages, n_splits), used = (stages + sps - 1) / sps;
-    const size_t at = ((size_t)t * heads + h) * n_splits;
-    float m = -INFINITY;
-    for (int s = 0; s < used; ++s) m = fmaxf(m, ml[at + s].x);
-    float l = 0.f;
-    for (int s = 0; s < used; ++s) l += exp2f(ml[at + s].x - m) * ml[at + s].y;
-    for (int c = tid; c < kv; c += 256) {
-      float v = 0.f;
-      for (int s = 0; s < used; ++s) v = fmaf(exp2f(ml[at + s].x - m), part[(at + s) * kv + c], v);
-      s_oc[i * kv + c] = v / l;
-    }
-  }
-  if (!any) return;
-  __syncthreads();
-  for (int d = d0 + warp; d < d1; d += 8) {
-    const uint4* w = reinterpret_cast<const uint4*>(uv + ((size_t)h * dv + d) * kv);
-    float acc[TT];
-#pragma unroll
-    for (int i = 0; i < TT; ++i) acc[i] = 0.f;
-    for (int c = lane; c < kv / 8; c += 32) {
-      float f[8];
-      Chunk<bf16>::get(w[c], f);
-#pragma unroll
-      for (int i = 0; i < TT; ++i) {
-        const float4 a0 = *reinterpret_cast<const float4*>(s_oc + i * kv + c * 8), a1 = *reinterpret_cast<const float4*>(s_oc + i * kv + c * 8 + 4);
-        acc[i] += f[0] * a0.x + f[1] * a0.y + f[2] * a0.z + f[3] * a0.w + f[4] * a1.x + f[5] * a1.y + f[6] * a1.z + f[7] * a1.w;
+  const int h = blockIdx.x, t0 = blockIdx.y * 8, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  {
+    const int t = t0 + warp;                             // a warp per token: maxima and sums of its shares
+    int used = 0;
+    if (t < T) {
+      const int seq = seq_ids[t], len = q_len[seq], q0 = q_start[seq];
+      if (len <= max_len && t - q0 < len) {
+        const int n_rows = len * heads, row0 = ((t - q0) * heads + h) / 16 * 16;
+        int page0, stages;
+        tile_range(positions[q0 + row0 / heads], positions[q0 + (min(row0 + 16, n_rows) - 1) / heads], window, page0, stages);
+        const int sps = stages_per_split(stages, n_splits);
+        used = (stages + sps - 1) / sps;
+        const size_t at = ((size_t)t * heads + h) * n_splits;
+        const float2 v = lane < used ? ml[at + lane] : make_float2(-INFINITY, 0.f);
+        const float m = warp_max(v.x), f = exp2f(v.x - m), l = warp_sum(f * v.y);
+        if (lane < used) s_f[warp][lane] = f / l;
       }
     }
+    if (lane == 0) s_used[warp] = used;
+    if (!__syncthreads_or(used > 0)) return;
+  }
+  for (int x = tid; x < 8 * (kv / 4); x += 256) {
+    const int t = x / (kv / 4), d = x % (kv / 4) * 4, used = s_used[t];
+    const float* p = part + ((size_t)(t0 + t) * heads + h) * n_splits * kv + d;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < used; ++s) {
+      const float f = s_f[t][s];
+      const float4 y = *reinterpret_cast<const float4*>(p + (size_t)s * kv);
+      v.x = fmaf(f, y.x, v.x), v.y = fmaf(f, y.y, v.y), v.z = fmaf(f, y.z, v.z), v.w = fmaf(f, y.w, v.w);
+    }
+    uint2 a, b;
+    split2(v.x, v.y, a.x, b.x), split2(v.z, v.w, a.y, b.y);
+    *reinterpret_cast<uint2*>(hi + t * ldx + d) = a;
+    *reinterpret_cast<uint2*>(lo + t * ldx + d) = b;
+  }
+  __syncthreads();
+  const int g = lane >> 2, t4 = lane & 3;
+  for (int tile = blockIdx.z * 8 + warp; tile * 16 < dv; tile += gridDim.z * 8) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    const bf16* w = uv + ((size_t)h * dv + tile * 16 + g) * kv + t4 * 8;
+    rows16<true>(acc, w, w + (size_t)8 * kv, hi + g * ldx + t4 * 8, lo + g * ldx + t4 * 8, kv, t4);
 #pragma unroll
-    for (int i = 0; i < TT; ++i) {
-      const float v = warp_sum(acc[i]);
-      if (lane == 0 && s_in[i])
-        out[(size_t)(t0 + i) * n_out + h * dv + d] = __float2bfloat16(v * sigmoid_x(__bfloat162float(gate[(size_t)(t0 + i) * ldp + h * dv + d])));
+    for (int e = 0; e < 4; ++e) {
+      const int t = 2 * t4 + (e & 1), d = h * dv + tile * 16 + g + (e >> 1) * 8;
+      if (s_used[t])
+        out[(size_t)(t0 + t) * n_out + d] = __float2bfloat16(acc[e] * sigmoid_x(__bfloat162float(gate[(size_t)(t0 + t) * ldp + d])));
     }
   }
   if (h == 0 && blockIdx.z == 0)
-    for (int i = 0; i < n; ++i)
-      if (s_in[i])
+    for (int i = 0; i < 8; ++i)
+      if (s_used[i])
         for (int c = heads * dv + tid; c < n_out; c += 256) out[(size_t)(t0 + i) * n_out + c] = __float2bfloat16(0.f);
 }
 
@@ -642,27 +682,23 @@ TRL_API int trl_latent_mma_ok(int dk, int rd, int dv, int kv) {
   return dk + rd <= 256 && dv <= 256 && kv <= 512 && q + (2 * TILE * row > merge ? 2 * TILE * row : merge) <= (size_t)LD_SMEM;
 }
 
-// Sequences of min_len..max_len tokens in the absorbed form.  q: [T, heads, dq]; up: [heads * dk key rows ; heads * dv value rows][kv];
-// ql: [T, heads, kv + rd]; part: fp32 [T, heads, n_splits, kv]; ml: [T, heads, n_splits] pairs; tiles: 16-row tiles of the longest
-// sequence; gate: gate columns of the fused projection rows.
-TRL_API int trl_latent_decode(const void* q, int dq, int dk, int rd, const void* up, int kv, int dv, void* ql, const void* pages, int n_blocks,
-                              const void* table, int max_blocks, const void* q_start, const void* q_len, const void* positions,
-                              const void* seq_ids, void* part, void* ml, const void* gate, int ldp, void* out, int n_out, int T, int B,
-                              int tiles, int heads, int n_splits, int window, int min_len, int max_len, float scale, void* stream) {
-  if (T <= 0 || B <= 0 || tiles <= 0 || heads <= 0 || dk % 16 || rd % 16 || dv % 16 || kv % 16 || dk + rd != dq || n_splits < 1 || window < 1 ||
-      n_blocks <= 0 || n_out < heads * dv || !trl_latent_mma_ok(dk, rd, dv, kv) || ((uintptr_t)pages & 15) || ((uintptr_t)q & 15))
+// Sequences of min_len..max_len tokens in the absorbed form.  q: [T, heads, dq], whose rotated part is turned here (n_pairs 0: it
+// already is); ukt: [heads][kv][dk]; uv: [heads * dv, kv]; ql: [T, heads, kv + rd]; part: fp32 [T, heads, n_splits, kv]; ml:
+// [T, heads, n_splits] pairs; tiles: 16-row tiles of the longest sequence; gate: gate columns of the fused projection rows.
+TRL_API int trl_latent_decode(const void* q, int dq, int dk, int rd, const void* ukt, const void* uv, int kv, int dv, const void* freqs,
+                              int n_pairs, float amp, void* ql, const void* pages, int n_blocks, const void* table, int max_blocks,
+                              const void* q_start, const void* q_len, const void* positions, const void* seq_ids, void* part, void* ml,
+                              const void* gate, int ldp, void* out, int n_out, int T, int B, int tiles, int heads, int n_splits, int window,
+                              int min_len, int max_len, float scale, void* stream) {
+  if (T <= 0 || B <= 0 || tiles <= 0 || heads <= 0 || dk % 16 || rd % 16 || dv % 16 || kv % 16 || dk + rd != dq || n_splits < 1 ||
+      n_splits > MAX_SPLITS || window < 1 || n_blocks <= 0 || n_out < heads * dv || 2 * n_pairs > rd || !trl_latent_mma_ok(dk, rd, dv, kv) ||
+      ((uintptr_t)pages & 15) || ((uintptr_t)q & 15) || ((uintptr_t)ukt & 15) || ((uintptr_t)uv & 15))
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
-  const bf16 *uk = (const bf16*)up, *uv = uk + (size_t)heads * dk * kv;
-  const int tt = T >= 8 ? 4 : 1, groups = (T + tt - 1) / tt;
-  const size_t sm1 = (size_t)(tt * dk + 8 * tt * 128) * sizeof(float);
-  cudaError_t e;
-  if (tt == 4)
-    e = trl_launch(latent_absorb_kernel<4>, dim3(heads, (kv + 127) / 128, groups), dim3(128), sm1, st, (const bf16*)q, dq, dk, rd, uk, kv,
-                   (const int*)seq_ids, (const int*)q_len, max_len, (bf16*)ql, T, heads);
-  else
-    e = trl_launch(latent_absorb_kernel<1>, dim3(heads, (kv + 127) / 128, groups), dim3(128), sm1, st, (const bf16*)q, dq, dk, rd, uk, kv,
-                   (const int*)seq_ids, (const int*)q_len, max_len, (bf16*)ql, T, heads);
+  const int groups = (T + 7) / 8;
+  cudaError_t e = trl_launch(latent_absorb_kernel, dim3(heads, (kv + 127) / 128, groups), dim3(256), (size_t)8 * (dk + 8) * sizeof(bf16), st,
+                             (const bf16*)q, dq, dk, rd, (const bf16*)ukt, kv, (const double*)freqs, n_pairs, amp, (const int*)positions,
+                             (const int*)seq_ids, (const int*)q_len, max_len, (bf16*)ql, T, heads);
   if (e != cudaSuccess) return (int)e;
   DecArgs a;
   a.ql = (const bf16*)ql, a.pages = (const unsigned char*)pages, a.kch = (kv + rd) / 8, a.vch = kv / 8, a.n_blocks = n_blocks;
@@ -673,15 +709,10 @@ TRL_API int trl_latent_decode(const void* q, int dq, int dk, int rd, const void*
   else if (kv <= 256) e = decode_launch<256, 1>(a, tiles, B, st);
   else e = decode_launch<256, 2>(a, tiles, B, st);
   if (e != cudaSuccess) return (int)e;
-  const int z = groups * heads < 148 ? min(4, (dv + 15) / 16) : 1;
-  const size_t sm2 = (size_t)tt * kv * sizeof(float);
-#define OUT(TTT)                                                                                                               \
-  return (int)trl_launch(latent_out_kernel<TTT>, dim3(heads, groups, z), dim3(256), sm2, st, (const float*)part, (const float2*)ml, \
-                         n_splits, uv, kv, dv, (const bf16*)gate, ldp, (bf16*)out, n_out, (const int*)seq_ids, (const int*)q_start,  \
-                         (const int*)q_len, (const int*)positions, T, heads, window, max_len)
-  if (tt == 4) OUT(4);
-  OUT(1);
-#undef OUT
+  const int z = groups * heads >= 148 ? 1 : (dv > 128 ? 2 : 1);
+  return (int)trl_launch(latent_out_kernel, dim3(heads, groups, z), dim3(256), (size_t)2 * 8 * (kv + 8) * sizeof(bf16), st, (const float*)part,
+                         (const float2*)ml, n_splits, (const bf16*)uv, kv, dv, (const bf16*)gate, ldp, (bf16*)out, n_out, (const int*)seq_ids,
+                         (const int*)q_start, (const int*)q_len, (const int*)positions, T, heads, window, max_len);
 }
 
 // Cached rows of positions lo .. lo + n - 1 of one sequence (table: its row of the block table).

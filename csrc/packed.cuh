@@ -40,12 +40,35 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16(v); }
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 
+// four activations <-> fp32
+template <typename T> __device__ __forceinline__ void store4(T* p, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float a, float b, float c, float d) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(f2_to_bf162_bits(a, b), f2_to_bf162_bits(c, d));
+}
+template <> __device__ __forceinline__ void store4<float>(float* p, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = bf162_bits_to_f2(v.x), b = bf162_bits_to_f2(v.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 __device__ __forceinline__ float inv_rms(float ss, int n, float eps) { return 1.f / sqrtf(ss / (float)n + eps); }
 // (full-precision forms: what feeds a recurrence or a gate is computed in 32 bits)
 __device__ __forceinline__ float sigmoid_x(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_x(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float gelu_tanh_x(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+// cos and sin of position x frequency, times amp; the angle is formed and reduced in fp64
+__device__ __forceinline__ void pair_angle(int pos, double freq, float amp, float& c, float& s) {
+  const double a = (double)pos * freq;
+  const double turns = rint(a * 0.15915494309189535);
+  sincosf((float)fma(-turns, 6.283185307179586, a), &s, &c);
+  c *= amp, s *= amp;
 }
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {

@@ -57,19 +57,23 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
   *reinterpret_cast<uint4*>(out + (size_t)t * channels + c) = Chunk<T>::put(acc);
 }
 
-// grid (heads * column slices, sequences), 256 threads: lane = column, warp = dk / 8 state rows.
+// grid (heads * column slices, sequences), 256 threads: lane = column, warp = dk / 8 state rows.  CONV: one token per
+// sequence whose rows still have to pass the convolution.  The state is fetched before the dependency wait: its last writer
+// is the previous tick, and every tick has launches in between that let their dependents in only after their own wait.
 constexpr int SS_TB = 16;
-template <typename T, int KIND, int RMAX>
+template <typename T, int KIND, int RMAX, bool CONV>
 __global__ void __launch_bounds__(256) scan_serial_kernel(const ScanArgs a) {
   constexpr int DK = RMAX * 8;
   __shared__ float s_q[SS_TB][DK], s_k[SS_TB][DK], s_v[SS_TB][32];
   __shared__ float s_keep[SS_TB], s_add[SS_TB], s_floor[SS_TB], s_m;
   __shared__ float s_part[2][8][32], s_den[2][8];
   pdl_launch_dependents(41);
-  pdl_wait();
   const int n_sl = (a.dv + 31) / 32, h = blockIdx.x / n_sl, col0 = (blockIdx.x % n_sl) * 32, seq = blockIdx.y;
   const int T_ = a.q_len[seq], t0 = a.q_start[seq];
-  if (T_ < a.min_len || T_ > a.max_len) return;
+  if (T_ < a.min_len || T_ > a.max_len) {
+    pdl_wait();                              // (a launch ends no sooner than those before it)
+    return;
+  }
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, R = a.dk / 8, col = col0 + lane;
   const int slot = a.slots[seq], plane = a.cur[slot];
   const bool keep_all = a.keep_flags && a.keep_flags[seq];
@@ -88,6 +92,7 @@ __global__ void __launch_bounds__(256) scan_serial_kernel(const ScanArgs a) {
       if (tid == 0) s_m = src[m_off];
     }
   }
+  pdl_wait();
   auto save = [&](int pl) {
     float* dst = rec + (size_t)pl * a.plane_stride;
 #pragma unroll
@@ -99,13 +104,35 @@ __global__ void __launch_bounds__(256) scan_serial_kernel(const ScanArgs a) {
   for (int i0 = 0; i0 < T_; i0 += SS_TB) {
     const int nb = min(SS_TB, T_ - i0);
     __syncthreads();
-    for (int x = tid; x < nb * a.dk; x += 256) {
+    if constexpr (CONV) {
+      const int pos = a.positions[t0];
+      const T* row = base + (size_t)t0 * a.ld;
+      const T* rg = reinterpret_cast<const T*>(a.ring) + (size_t)slot * a.ring_slot;
+      for (int x = tid; x < 2 * a.dk + 32; x += 256) {
+        const int d = x < a.dk ? x : x < 2 * a.dk ? x - a.dk : x - 2 * a.dk;
+        const int c = (x < a.dk ? a.q0 : a.k0) + (h / a.per) * a.dk + d, cc = x < 2 * a.dk ? c : a.v0 + h * a.dv + col0 + d;
+        float v = 0.f;
+        if (x < 2 * a.dk || col0 + d < a.dv) {
+          v = a.conv_b[cc];
+          for (int j = 0; j < a.taps; ++j) {
+            const int back = a.taps - 1 - j;
+            if (back <= pos)
+              v = fmaf(to_f(back ? rg[(size_t)((pos - back) % a.ring_rows) * a.ring_ld + cc] : row[cc]), a.conv_w[(size_t)j * a.channels + cc], v);
+          }
+          v = to_f(from_f<T>(v * sigmoid_x(v)));
+        }
+        if (x < a.dk) s_q[0][d] = v * a.q_scale;
+        else if (x < 2 * a.dk) s_k[0][d] = v;
+        else s_v[0][d] = v;
+      }
+    }
+    for (int x = tid; x < (CONV ? 0 : nb * a.dk); x += 256) {
       const int j = x / a.dk, d = x % a.dk;
       const T* row = base + (size_t)(t0 + i0 + j) * a.ld;
       s_q[j][d] = to_f(row[a.q0 + (h / a.per) * a.dk + d]) * a.q_scale;
       s_k[j][d] = to_f(row[a.k0 + (h / a.per) * a.dk + d]);
     }
-    for (int x = tid; x < nb * 32; x += 256)
+    for (int x = tid; x < (CONV ? 0 : nb * 32); x += 256)
       s_v[x >> 5][x & 31] = col0 + (x & 31) < a.dv ? to_f(base[(size_t)(t0 + i0 + (x >> 5)) * a.ld + a.v0 + h * a.dv + col0 + (x & 31)]) : 0.f;
     if (tid < nb) {
       float g0, g1;
@@ -185,6 +212,7 @@ struct NormArgs {
 };
 
 // one block per token
+constexpr int NORM_R = 8;
 template <typename T, int KIND>
 __global__ void __launch_bounds__(256) scan_norm_kernel(const NormArgs a) {
   extern __shared__ float s_y[];               // [heads * vdim], true columns only
@@ -203,6 +231,40 @@ __global__ void __launch_bounds__(256) scan_norm_kernel(const NormArgs a) {
                                             (size_t)(a.positions[t] % a.ring_rows) * a.ring_ld);
       for (int c = tid; c < a.channels / C; c += 256) dst[c] = src[c];
     }
+  }
+  T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.n_out;
+  if (a.vdim == a.dv && inner % 1024 == 0 && inner <= NORM_R * 1024 && (inner / a.groups) % 128 == 0) {
+    // unpadded heads, groups of whole warps of four columns a thread: everything stays in registers
+    float4 v[NORM_R], z[NORM_R];
+    const int nr = inner / 1024;
+#pragma unroll
+    for (int i = 0; i < NORM_R; ++i)
+      if (i < nr) v[i] = *reinterpret_cast<const float4*>(o + (i * 256 + tid) * 4), z[i] = load4(gate + (i * 256 + tid) * 4);
+#pragma unroll
+    for (int i = 0; i < NORM_R; ++i)
+      if (i < nr) {
+        const float4 s = make_float4(sigmoid_x(z[i].x), sigmoid_x(z[i].y), sigmoid_x(z[i].z), sigmoid_x(z[i].w));
+        if (KIND == SCAN_MAMBA2) v[i].x *= z[i].x * s.x, v[i].y *= z[i].y * s.y, v[i].z *= z[i].z * s.z, v[i].w *= z[i].w * s.w;
+        z[i] = s;
+        const float ss = warp_sum(v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w);
+        if (lane == 0) s_y[i * 8 + warp] = ss;             // sums of 128 columns each
+      }
+    __syncthreads();
+    const int per = inner / a.groups / 128;
+#pragma unroll
+    for (int i = 0; i < NORM_R; ++i)
+      if (i < nr) {
+        const int g = (i * 8 + warp) / per, p = (i * 256 + tid) * 4;
+        float ss = 0.f;
+        for (int k = 0; k < per; ++k) ss += s_y[g * per + k];
+        const float r = inv_rms(ss, per * 128, a.eps);
+        const float4 w = *reinterpret_cast<const float4*>(a.w + p);
+        float4 y = make_float4(v[i].x * r * w.x, v[i].y * r * w.y, v[i].z * r * w.z, v[i].w * r * w.w);
+        if (KIND == SCAN_MLSTM) y.x *= z[i].x, y.y *= z[i].y, y.z *= z[i].z, y.w *= z[i].w;
+        store4<T>(out + p, y.x, y.y, y.z, y.w);
+      }
+    for (int p = inner + tid; p < a.n_out; p += 256) out[p] = from_f<T>(0.f);
+    return;
   }
   for (int x = tid; x < inner; x += 256) {
     const int p = x / a.vdim * a.dv + x % a.vdim;
@@ -231,7 +293,6 @@ __global__ void __launch_bounds__(256) scan_norm_kernel(const NormArgs a) {
     }
   }
   __syncthreads();
-  T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.n_out;
   for (int p = tid; p < a.n_out; p += 256) {
     const int h = p / a.dv, d = p % a.dv;
     float v = 0.f;
@@ -243,13 +304,13 @@ __global__ void __launch_bounds__(256) scan_norm_kernel(const NormArgs a) {
   }
 }
 
-template <typename T, int KIND>
+template <typename T, int KIND, bool CONV>
 cudaError_t serial_launch(const ScanArgs& a, int B, cudaStream_t st) {
   const dim3 grid(a.heads * ((a.dv + 31) / 32), B);
-  if (a.dk <= 32) return trl_launch(scan_serial_kernel<T, KIND, 4>, grid, dim3(256), 0, st, a);
-  if (a.dk <= 64) return trl_launch(scan_serial_kernel<T, KIND, 8>, grid, dim3(256), 0, st, a);
-  if (a.dk <= 128) return trl_launch(scan_serial_kernel<T, KIND, 16>, grid, dim3(256), 0, st, a);
-  return trl_launch(scan_serial_kernel<T, KIND, 32>, grid, dim3(256), 0, st, a);
+  if (a.dk <= 32) return trl_launch(scan_serial_kernel<T, KIND, 4, CONV>, grid, dim3(256), 0, st, a);
+  if (a.dk <= 64) return trl_launch(scan_serial_kernel<T, KIND, 8, CONV>, grid, dim3(256), 0, st, a);
+  if (a.dk <= 128) return trl_launch(scan_serial_kernel<T, KIND, 16, CONV>, grid, dim3(256), 0, st, a);
+  return trl_launch(scan_serial_kernel<T, KIND, 32, CONV>, grid, dim3(256), 0, st, a);
 }
 
 }  // namespace
@@ -274,10 +335,15 @@ TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* 
 
 // kind 0: Mamba-2, 1: mLSTM.  args: a ScanArgs (scan.cuh) filled by the caller.  Serves sequences of min_len..max_len tokens.
 TRL_API int trl_scan_serial(const ScanArgs* a, int B, int kind, int f32, void* stream) {
-  if (B <= 0 || scan_args_bad(*a, kind)) return (int)cudaErrorInvalidValue;
+  if (B <= 0 || scan_args_bad(*a, kind) || (a->taps && (kind != SCAN_MAMBA2 || a->taps > a->ring_rows || !a->conv_w || !a->conv_b || !a->ring ||
+                                                        !a->positions || a->keep_flags)))
+    return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
-  if (kind == SCAN_MAMBA2) return (int)(f32 ? serial_launch<float, SCAN_MAMBA2>(*a, B, st) : serial_launch<bf16, SCAN_MAMBA2>(*a, B, st));
-  return (int)(f32 ? serial_launch<float, SCAN_MLSTM>(*a, B, st) : serial_launch<bf16, SCAN_MLSTM>(*a, B, st));
+  if (kind == SCAN_MAMBA2 && a->taps)
+    return (int)(f32 ? serial_launch<float, SCAN_MAMBA2, true>(*a, B, st) : serial_launch<bf16, SCAN_MAMBA2, true>(*a, B, st));
+  if (kind == SCAN_MAMBA2)
+    return (int)(f32 ? serial_launch<float, SCAN_MAMBA2, false>(*a, B, st) : serial_launch<bf16, SCAN_MAMBA2, false>(*a, B, st));
+  return (int)(f32 ? serial_launch<float, SCAN_MLSTM, false>(*a, B, st) : serial_launch<bf16, SCAN_MLSTM, false>(*a, B, st));
 }
 
 // o: fp32 [T, heads * dv]; gate, conv_in: columns of the fused projection rows (ldp wide); out: [T, n_out].

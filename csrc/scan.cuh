@@ -17,6 +17,12 @@ struct ScanArgs {
   int heads, per, dk, dv;              // per: heads that share q and k
   int min_len, max_len;
   float cap, q_scale;
+  // decode ticks of Mamba-2: rows are not convolved yet, scan_serial_kernel does it (taps 0: they are)
+  int taps, channels, ring_rows, ring_ld;
+  const float *conv_w, *conv_b;        // [taps, channels], [channels]
+  const void* ring;                    // the layer's first column of slot 0
+  long ring_slot;
+  const int* positions;
 };
 
 inline bool scan_args_bad(const ScanArgs& a, int kind) {

@@ -7,7 +7,7 @@ import torch
 
 import fetotar_oracle as oracle
 from tilerl_b200.fetotar_layout import layout_of, pad
-from tilerl_b200.mixers import LatentAttnSpec, Mamba2Spec, MlstmSpec, RotarySpec
+from tilerl_b200.mixers import LatentAttnSpec, Mamba2Spec, MlstmSpec, RotarySpec, YarnSpec
 
 pytestmark = pytest.mark.gpu
 
@@ -190,13 +190,17 @@ def test_latent_attention_forms(ops, shape, lens):
         pages = (pg,)
         layer = staticmethod(lambda i: cache)
     assert ops.lib.trl_latent_mma_ok(l.dk, l.rd, l.dv, l.kv)
-    out = ops.latent_attention(q, proj, up, l, batch, Pool, 0).clone()
+    ukt = up[:heads * l.dk].view(heads, l.dk, l.kv).transpose(1, 2).contiguous()
+    rot = RotarySpec(rd, 1e4, YarnSpec(4.0, 64.0, 8.0, 1.0))
+    freqs = torch.tensor(rot.frequencies(), dtype=torch.float64, device="cuda")
+    turned = torch.cat([q[:, :, :l.dk].double(), oracle.rotate(q[:, :, l.dk:].double().cpu(), batch.positions.tolist(), rot.to_json()).cuda()], -1)
+    out = ops.latent_attention(q, proj, up, ukt, l, freqs, rot, batch, Pool, 0).clone()
     uk, uv = up.double()[:heads * l.dk].view(heads, l.dk, l.kv), up.double()[heads * l.dk:].view(heads, l.dv, l.kv)
     o = 0
     for (n, ctx), r in zip(lens, rows):
         r = r.double()
         k = torch.cat([torch.einsum("nc,hdc->hnd", r[:, :l.kv], uk), r[None, :, l.kv:].expand(heads, -1, -1)], -1)
-        s = torch.einsum("thd,hnd->htn", q[o:o + n].double(), k) * l.scale
+        s = torch.einsum("thd,hnd->htn", turned[o:o + n], k) * l.scale
         back = torch.arange(ctx - n, ctx, device="cuda")[:, None] - torch.arange(ctx, device="cuda")[None, :]
         p = torch.softmax(s.masked_fill((back < 0) | (back >= window), -math.inf), -1)
         want = torch.einsum("htn,hnd->thd", p, torch.einsum("nc,hdc->hnd", r[:, :l.kv], uv)).reshape(n, -1)

@@ -167,6 +167,9 @@ class FetotarModel:
         # radians per position of every rotated pair (fp64: angles are reduced before they are rounded)
         self.freqs = [None if b.mixer.recurrent else
                       torch.tensor(b.mixer.rot.frequencies(), dtype=torch.float64, device=params["embed"].device) for b in cfg.layers]
+        # the key maps once more, transposed per head [heads, latent, dim]: rows of the map of queries into the latent
+        self.ukt = [None if l.kind != "latent" else
+                    params[f"L{i}.up"][:l.heads * l.dk].view(l.heads, l.dk, l.kv).transpose(1, 2).contiguous() for i, l in enumerate(self.layouts)]
         self.lora: Dict[str, object] = {}
         self.weights_version = 0
         if params["lm_head"].is_cuda:      # library products accumulate in fp32 and read fp32 operands whole
@@ -206,7 +209,7 @@ class FetotarModel:
         if l.kind == "latent":
             rot = self.cfg.layers[i].mixer.rot
             q = ops.latent_prep(proj, l, P[p + "q_norm"], P[p + "kv_norm"], P[p + "uq"], self.freqs[i], rot, batch, kv_pool, c, eps)
-            return ops.latent_attention(q, proj, P[p + "up"], l, batch, kv_pool, c)
+            return ops.latent_attention(q, proj, P[p + "up"], self.ukt[i], l, self.freqs[i], rot, batch, kv_pool, c)
         w = {k: P.get(p + k) for k in ("norm", "gate_b", "conv", "conv_b", "a_log", "skip")}
         return ops.recurrent_mix(proj, gates, w, l, batch, state_pool, c, eps)
 

@@ -14,10 +14,11 @@ from . import native as N
 from .cuda_stream import EPI_STORE, EPI_STORE_F32
 
 MAMBA2, MLSTM = 0, 1
-MIX_ROWS_MAX = 16       # rows the weight-streaming projection serves
+MIX_ROWS_MAX = 8        # rows the weight-streaming projection serves
 LATENT_SHORT = 32       # tokens of a sequence up to which attention runs in the latent (absorbed) form
 SCAN_SHORT = 16         # tokens of a sequence up to which a scan goes token by token
 CHUNK_DK = 128          # state rows the chunked scan takes
+MAX_SPLITS = 32         # shares of a window its keys are split into (a warp merges them)
 PART_BYTES = 1 << 28    # most fp32 partial sums of split attention
 
 
@@ -27,7 +28,9 @@ class ScanArgs(ctypes.Structure):
                                                 "q_start", "q_len", "slots", "o")]
                 + [(n, ctypes.c_long) for n in ("slot_stride", "plane_stride")]
                 + [(n, ctypes.c_int) for n in ("ld", "q0", "k0", "v0", "ldg", "heads", "per", "dk", "dv", "min_len", "max_len")]
-                + [(n, ctypes.c_float) for n in ("cap", "q_scale")])
+                + [(n, ctypes.c_float) for n in ("cap", "q_scale")]
+                + [(n, ctypes.c_int) for n in ("taps", "channels", "ring_rows", "ring_ld")]
+                + [(n, ctypes.c_void_p) for n in ("conv_w", "conv_b", "ring")] + [("ring_slot", ctypes.c_long), ("positions", ctypes.c_void_p)])
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -139,14 +142,18 @@ class MixerOps:
             self._linear_rows(cq, uq, q, EPI_STORE)
         else:
             self._mm(cq, uq, q)
-        N.check(self.lib.trl_latent_rope(q.data_ptr(), freqs.data_ptr(), batch.positions.data_ptr(), t, l.heads, l.dq, l.dk, freqs.numel(),
-                                         rot.amplitude, _f32(q), st), "latent_rope")
-        N.count(2)
+        N.count()
         return q.view(t, l.heads, l.dq)
 
-    def latent_attention(self, q, proj, up, l, batch, pool, idx):
+    def _latent_rope(self, q, l, freqs, rot, positions) -> None:
+        N.check(self.lib.trl_latent_rope(q.data_ptr(), freqs.data_ptr(), positions.data_ptr(), q.shape[0], l.heads, l.dq, l.dk, freqs.numel(),
+                                         rot.amplitude, _f32(q), N.stream()), "latent_rope")
+        N.count()
+
+    def latent_attention(self, q, proj, up, ukt, l, freqs, rot, batch, pool, idx):
         if proj.dtype == torch.bfloat16 and self.lib.trl_latent_mma_ok(l.dk, l.rd, l.dv, l.kv):
-            return self._latent_mma(q, proj, up, l, batch, pool, idx)
+            return self._latent_mma(q, proj, up, ukt, l, freqs, rot, batch, pool, idx)
+        self._latent_rope(q, l, freqs, rot, batch.positions)
         t, cache, table, dt, st = proj.shape[0], pool.layer(idx), batch.block_table, proj.dtype, N.stream()
         uk, uv = up[:l.heads * l.dk].view(l.heads, l.dk, l.kv), up[l.heads * l.dk:].view(l.heads, l.dv, l.kv)
         ql = self.ws.get(f"latent_ql_{dt}", (l.heads, t, l.kv), dt)
@@ -164,7 +171,7 @@ class MixerOps:
         N.count(2)
         return out
 
-    def _latent_mma(self, q, proj, up, l, batch, pool, idx):
+    def _latent_mma(self, q, proj, up, ukt, l, freqs, rot, batch, pool, idx):
         """Short sequences in the absorbed form (one pass over the cached latents for all heads), prompts over expanded
         keys and values."""
         t, cache, table, st = proj.shape[0], pool.layer(idx), batch.block_table, N.stream()
@@ -175,16 +182,19 @@ class MixerOps:
             starts.append(starts[-1] + n)
         short = [i for i, n in enumerate(lens) if n <= LATENT_SHORT]
         prompts = [i for i, n in enumerate(lens) if n > LATENT_SHORT]
+        if prompts:
+            self._latent_rope(q, l, freqs, rot, batch.positions)
         if short:
             ts = max(starts[i + 1] for i in short)                           # tokens up to the last short sequence's
             blocks = sum((lens[i] * l.heads + 15) // 16 for i in short)
             keys = min(l.window + LATENT_SHORT, table.shape[1] * 16 if self.attn_splits else max(kvs[i] for i in short))
-            splits = max(1, min(16, (keys + 127) // 128, self.sms // blocks, PART_BYTES // (ts * l.heads * l.kv * 4)))
+            splits = max(1, min(MAX_SPLITS, (keys + 63) // 64 + 1, self.sms // blocks, PART_BYTES // (ts * l.heads * l.kv * 4)))
             ql = self.ws.get("latent_rows", (ts, l.heads, l.row), bf)
             part = self.ws.get("attn_part", (ts * l.heads * splits * l.kv,), torch.float32)
             ml = self.ws.get("attn_part_ml", (ts * l.heads * splits * 2,), torch.float32)
             N.check(self.lib.trl_latent_decode(
-                q.data_ptr(), l.dq, l.dk, l.rd, up.data_ptr(), l.kv, l.dv, ql.data_ptr(), cache.data_ptr(), cache.shape[0], table.data_ptr(),
+                q.data_ptr(), l.dq, l.dk, l.rd, ukt.data_ptr(), up[l.heads * l.dk:].data_ptr(), l.kv, l.dv, freqs.data_ptr(),
+                0 if prompts else freqs.numel(), rot.amplitude, ql.data_ptr(), cache.data_ptr(), cache.shape[0], table.data_ptr(),
                 table.stride(0), batch.q_start.data_ptr(), batch.q_len.data_ptr(), batch.positions.data_ptr(), batch.seq_ids.data_ptr(),
                 part.data_ptr(), ml.data_ptr(), proj[:, l.g0:].data_ptr(), proj.stride(0), out.data_ptr(), l.n_out, ts, batch.n_seqs,
                 max((lens[i] * l.heads + 15) // 16 for i in short), l.heads, splits, l.window, 1, LATENT_SHORT if prompts else 1 << 30, l.scale,
@@ -233,13 +243,20 @@ class MixerOps:
         ring = pool.ring_view(idx, 0) if kind == MAMBA2 else None
         o = self.ws.get("scan_o", (t, l.heads * l.dv), torch.float32)
         a = ScanArgs()
-        if kind == MAMBA2:
+        if kind == MAMBA2 and batch.max_q_len == 1 and not batch.keep_steps:
+            # a decode tick: the scan convolves its own columns
+            rows = proj
+            a.taps, a.channels, a.conv_w, a.conv_b = l.taps, l.conv_c, w["conv"].data_ptr(), w["conv_b"].data_ptr()
+            a.ring, a.ring_slot, a.ring_rows, a.ring_ld = ring.data_ptr(), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1)
+            a.positions = batch.positions.data_ptr()
+        elif kind == MAMBA2:
             rows = self.ws.get(f"scan_conv_{dt}", (t, l.conv_c), dt)
             N.check(self.lib.trl_scan_conv(
                 proj.data_ptr(), proj.stride(0), w["conv"].data_ptr(), w["conv_b"].data_ptr(), ring.data_ptr(), pool.ring.stride(0),
                 pool.ring_rows, pool.ring.stride(1), batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(),
                 batch.state_slots.data_ptr(), rows.data_ptr(), t, l.conv_c, l.taps, _f32(proj), st), "scan_conv")
             N.count()
+        if kind == MAMBA2:
             a.q0, a.k0, a.v0, a.per, a.q_scale, a.cap = l.q0, l.k0, 0, l.heads // l.groups, 1.0, 1.0
         else:
             rows = proj

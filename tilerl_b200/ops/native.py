@@ -96,7 +96,7 @@ _SIGS = {
     "trl_linear_rows_glu": [P, I, P, P, I, I, I, I, F, P],
     "trl_linear_rows_side": [P, I, P, P, I, I, I, I, P, P, L, I, I, I, P],
     "trl_latent_mma_ok": [I, I, I, I],
-    "trl_latent_decode": [P, I, I, I, P, I, I, P, P, I, P, I, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, F, P],
+    "trl_latent_decode": [P, I, I, I, P, P, I, I, P, I, F, P, P, I, P, I, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, F, P],
     "trl_latent_gather": [P, I, P, I, I, I, I, P, P, P],
     "trl_latent_prompt": [P, I, I, I, I, P, I, P, P, I, P, I, P, I, I, I, I, I, F, P],
     "trl_scan_chunk": [P, I, I, I, P],

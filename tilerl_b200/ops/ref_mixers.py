@@ -148,8 +148,8 @@ class RefMixers:
 
     # ---- latent attention ----------------------------------------------------------------
     def latent_prep(self, proj, l, q_norm, kv_norm, uq, freqs, rot, batch, pool, idx, eps):
-        """Normed latents and the rotated shared key into the cache; returns the query heads ``[T, heads, dk + rd]`` with
-        their rotated part turned."""
+        """Normed latents and the rotated shared key into the cache; returns the query heads ``[T, heads, dk + rd]``, not
+        turned yet."""
         t = proj.shape[0]
         cq = proj[:, :l.c0].float()
         cq = (cq * ref.rms_factor(cq, l.q_rank, eps)[:, None] * q_norm).to(self.act_dtype)
@@ -157,16 +157,15 @@ class RefMixers:
         c = c * ref.rms_factor(c, l.kv_rank, eps)[:, None] * kv_norm
         kr = rotate_pairs(proj[:, l.kr0:l.g0].float(), batch.positions, freqs, rot.amplitude)
         latent_write(pool.layer(idx), pool.pages[idx], torch.cat([c, kr], 1).to(pool.dtype), batch.slot_mapping)
-        q = ref.linear(cq, uq).view(t, l.heads, l.dq)
-        q[:, :, l.dk:] = rotate_pairs(q[:, :, l.dk:], batch.positions, freqs, rot.amplitude)
-        return q.to(self.act_dtype)
+        return ref.linear(cq, uq).view(t, l.heads, l.dq).to(self.act_dtype)
 
-    def latent_attention(self, q, proj, up, l, batch, pool, idx):
+    def latent_attention(self, q, proj, up, ukt, l, freqs, rot, batch, pool, idx):
         """Gated attention output, padded to the output projection's columns."""
         t = proj.shape[0]
         uk, uv = up.float().split([l.heads * l.dk, l.heads * l.dv])
         uk, uv = uk.view(l.heads, l.dk, l.kv), uv.view(l.heads, l.dv, l.kv)
-        ql = torch.cat([torch.einsum("thd,hdc->thc", q[:, :, :l.dk].float(), uk), q[:, :, l.dk:].float()], -1)
+        qr = rotate_pairs(q[:, :, l.dk:].float(), batch.positions, freqs, rot.amplitude)
+        ql = torch.cat([torch.einsum("thd,hdc->thc", q[:, :, :l.dk].float(), uk), qr], -1)
         out = torch.zeros(t, l.n_out, dtype=self.act_dtype, device=proj.device)
         for i in range(t):
             p = int(batch.positions[i])

@@ -50,7 +50,7 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
     ops, dev = make_ops("cuda"), "cuda"
     model = build_model(cf, dev, seed=0, ops=ops)
     lm, la, lb = model.layouts
-    P, eps = model.params, cf.norm_eps
+    P, eps, rot = model.params, cf.norm_eps, cf.layers[1].mixer.rot
     bf = lambda *s: (torch.randn(*s, device=dev) * 0.5).to(torch.bfloat16)
     flush = torch.empty(1 << 28, dtype=torch.uint8, device=dev)
     rows = []
@@ -120,7 +120,7 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
         # cached rows and the maps read once, queries and gates read, output written; scores and sums over expanded heads
         by = keys * la.row * 2 + P["L1.up"].numel() * 2 + t * la.heads * (la.dq + 2 * la.dv) * 2
         fl = 2.0 * seen * la.heads * (la.dq + la.dv) + 2.0 * t * P["L1.up"].numel()
-        row(f"attention {what}", "fetotar", lambda: ops.latent_attention(q, proj, P["L1.up"], la, batch, kv, 0), by, fl)
+        row(f"attention {what}", "fetotar", lambda: ops.latent_attention(q, proj, P["L1.up"], model.ukt[1], la, model.freqs[1], rot, batch, kv, 0), by, fl)
         pa = make_kv_pool(replace(ch, layer_types=(ATTN,)), b * per + 1, dev)
         pa.k.normal_(), pa.v.normal_()
         qkv = bf(t, ch.qkv_rows)
