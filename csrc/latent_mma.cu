@@ -4,8 +4,8 @@
 // same cached rows, so a page is fetched once for all heads.
 //   latent_absorb_kernel  q W_uk per head, and the rotated part beside it: query rows [kv | rd] of every (token, head).
 //   latent_decode_kernel  one block = 16 (token, head) rows of a sequence and a share of the window's keys.  Pages come
-//                         through a ring of stages (one bulk copy each, from a producing warp); each of four warps (eight,
-//                         for latents above 256) owns one page of a stage and keeps its own softmax, merged at the end.
+//                         through a ring of stages (one bulk copy each, from a producing warp).  Of a stage's 64 keys each of eight
+//                         warps scores eight; every warp then forms all weights and sums an eighth of the latent's columns.
 //   latent_out_kernel     merges the shares, maps the sum back (W_uv) and applies the output gate.
 // Prompts: keys and values of the window are expanded once for all query tokens.
 //   latent_gather_kernel  cached rows of a range of positions, dense; the expansion itself is one library product.
@@ -123,13 +123,12 @@ __device__ __forceinline__ uint32_t ld_try_wait(uint32_t bar, uint32_t parity) {
   return ok;
 }
 
-template <int OD, int HALVES>
-__global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(const DecArgs a) {
-  constexpr int NW = 4 * HALVES, THREADS = (NW + 1) * 32;
+template <int CW>
+__global__ void __launch_bounds__(288) latent_decode_kernel(const DecArgs a) {
+  constexpr int NW = 8, SX = 72, THREADS = (NW + 1) * 32;
   extern __shared__ unsigned char ld_raw[];
-  __shared__ __align__(8) uint64_t s_bar[12];              // full[4], empty[4], pair[4]
-  __shared__ float s_m[4][16], s_l[4][16];
-  __shared__ float4 s_x[HALVES == 2 ? 2 : 1][HALVES == 2 ? 8 : 1][32];     // scores the two warps of a page exchange
+  __shared__ __align__(8) uint64_t s_bar[9];               // full[4], empty[4], scores
+  __shared__ __align__(16) float s_x[2][16][SX];           // scores of a stage's 64 keys
   __shared__ volatile int s_ok;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const uint32_t raw_a = (uint32_t)__cvta_generic_to_shared(ld_raw);
@@ -140,7 +139,7 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
       asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(bar_a + 8u * st));
       asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar_a + 32u + 8u * st), "r"(NW));
     }
-    for (int k = 0; k < 4; ++k) asm volatile("mbarrier.init.shared::cta.b64 [%0], 2;" ::"r"(bar_a + 64u + 8u * k));
+    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar_a + 64u), "r"(NW));
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     s_ok = 1;
   }
@@ -195,10 +194,9 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
     }
     return true;
   };
-  const int kw = warp & 3, half = warp >> 2;               // key page of a stage, column half
-  float o[OD / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
+  float o[CW / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
 #pragma unroll
-  for (int i = 0; i < OD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int i = 0; i < CW / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   if (warp == NW) {
     // ---------------- producer ----------------
     const int* table = a.table + (size_t)seq * a.max_blocks;
@@ -231,107 +229,108 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
       pos[i] = r < rows ? a.positions[q0 + (row0 + r) / a.heads] : -1;
     }
     const uint32_t qa = smem_a + ((lane & 7) + ((lane >> 3) & 1) * 8) * qld + (lane >> 4) * 16;
-    const int kr = (lane & 7) + (lane >> 4) * 8, kcl = (lane >> 3) & 1;
     const int vr = (lane & 7) + ((lane >> 3) & 1) * 8, vcl = lane >> 4;
-    const int krot = kr % a.kch, vrot = vr % a.kch, nc = a.kch;
+    const int page = warp >> 1, r8 = (warp & 1) * 8 + (lane & 7), c8 = lane >> 3;      // this warp scores 8 keys of a page
+    const int nc = a.kch, rot8 = r8 % nc, vrot = vr % nc, g = lane >> 2, t4 = lane & 3;
     const bool xored = nc % 8 == 0;
     auto place = [&](int c, int r, int rot) {              // page_chunk without a division (rot = r % nc)
       const int x = c + rot;
       return xored ? c ^ (r & 7) : (x >= nc ? x - nc : x);
     };
-    const int vc0 = half * (OD / 8), vch = min(OD / 8, a.vch - vc0);      // this warp's output chunks
+    const int vc0 = warp * (CW / 8), vch = min(CW / 8, a.vch - vc0);      // this warp's output chunks (none: it only scores)
     int st = 0;
-    uint32_t ph = 0, xp = 0;                               // xp: parity and buffer of the exchange
+    uint32_t ph = 0, xp = 0;                               // xp: parity and buffer of the scores
     for (int k = s0; k < s1; ++k) {
       if (!bounded_wait(bar_a + 8u * st, ph, 520 + st)) break;
-      const int j0 = (page0 + k * TPAGES + kw) * KVB;
-      if (j0 < hi) {
-        const uint32_t base = ring_a + st * stage_b + kw * page_b;
-        float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        if constexpr (HALVES == 1) {
-#pragma unroll 4
-          for (int kk = 0; kk < nc / 2; ++kk) {
-            uint32_t qv[4], b[4];
-            ldsm4(qv, qa + kk * 32);
-            ldsm4(b, base + (kr * nc + place(kk * 2 + kcl, kr, krot)) * 16);
-            mma16(sc[0], qv, b[0], b[1]);
-            mma16(sc[1], qv, b[2], b[3]);
-          }
-        } else {
-          // each of the page's two warps scores 8 of its keys (two k-steps an iteration, in two sums) and hands them over
-          float s2[4] = {0.f, 0.f, 0.f, 0.f};
-          const int r8 = half * 8 + (lane & 7), rot8 = r8 % nc, c8 = lane >> 3;
-#pragma unroll 2
-          for (int kk = 0; kk < nc / 4; ++kk) {
-            uint32_t q0v[4], q1v[4], b[4];
-            ldsm4(q0v, qa + kk * 64);
-            ldsm4(q1v, qa + kk * 64 + 32);
-            ldsm4(b, base + (r8 * nc + place(kk * 4 + c8, r8, rot8)) * 16);
-            mma16(sc[0], q0v, b[0], b[1]);
-            mma16(s2, q1v, b[2], b[3]);
-          }
-          if (nc & 2) {                                    // an odd number of k-steps: the last one alone
-            uint32_t q0v[4], b[4];
-            ldsm4(q0v, qa + (nc / 2 - 1) * 32);
-            ldsm4(b, base + (r8 * nc + place(nc - 2 + (c8 & 1), r8, rot8)) * 16);
-            mma16(sc[0], q0v, b[0], b[1]);
-          }
-          const float4 mine = make_float4(sc[0][0] + s2[0], sc[0][1] + s2[1], sc[0][2] + s2[2], sc[0][3] + s2[3]);
-          const uint32_t pair = bar_a + 64u + 8u * kw;
-          s_x[xp][warp][lane] = mine;
-          __syncwarp();
-          if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(pair) : "memory");
-          if (!bounded_wait(pair, xp, 540 + kw)) break;
-          const float4 other = s_x[xp][warp ^ 4][lane];
-          xp ^= 1u;
-          const float4 lo4 = half ? other : mine, hi4 = half ? mine : other;
-          sc[0][0] = lo4.x, sc[0][1] = lo4.y, sc[0][2] = lo4.z, sc[0][3] = lo4.w;
-          sc[1][0] = hi4.x, sc[1][1] = hi4.y, sc[1][2] = hi4.z, sc[1][3] = hi4.w;
-        }
-        uint32_t wh[4], wl[4];
-        float now[2], back[2];
-        bool moved = false;
+      const int j0 = (page0 + k * TPAGES) * KVB;
+      const uint32_t stage = ring_a + st * stage_b;
+      if (j0 + page * KVB < hi) {
+        const uint32_t base = stage + page * page_b + r8 * row_b;
+        float sc[4][4];
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          float m = -INFINITY;
+        for (int i = 0; i < 4; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+        int kk = 0;                                        // groups of 4 chunks: two k-steps
+#pragma unroll 2
+        for (; kk + 2 <= nc / 4; kk += 2) {
+          uint32_t q[4][4], b[2][4];
+          ldsm4(b[0], base + place(kk * 4 + c8, r8, rot8) * 16);
+          ldsm4(b[1], base + place(kk * 4 + 4 + c8, r8, rot8) * 16);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) ldsm4(q[i], qa + kk * 64 + i * 32);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) mma16(sc[i], q[i], b[i >> 1][(i & 1) * 2], b[i >> 1][(i & 1) * 2 + 1]);
+        }
+        for (int c = kk * 4; c < nc; c += 2) {             // what is left, k-step by k-step
+          uint32_t q[4], b[4];
+          ldsm4(q, qa + c * 16);
+          ldsm4(b, base + place(c + (c8 & 1), r8, rot8) * 16);
+          mma16(sc[0], q, b[0], b[1]);
+        }
+        float* dst = &s_x[xp][g][warp * 8 + 2 * t4];
+        *reinterpret_cast<float2*>(dst) = make_float2((sc[0][0] + sc[1][0]) + (sc[2][0] + sc[3][0]), (sc[0][1] + sc[1][1]) + (sc[2][1] + sc[3][1]));
+        *reinterpret_cast<float2*>(dst + 8 * SX) = make_float2((sc[0][2] + sc[1][2]) + (sc[2][2] + sc[3][2]), (sc[0][3] + sc[1][3]) + (sc[2][3] + sc[3][3]));
+      }
+      __syncwarp();
+      if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar_a + 64u) : "memory");
+      if (!bounded_wait(bar_a + 64u, xp, 540)) break;
+      // every warp forms the weights of all 64 keys (it needs them as operands), then sums its columns
+      float w[TPAGES][2][4], back[2];
+      bool moved = false;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        float m = -INFINITY;
+#pragma unroll
+        for (int p = 0; p < TPAGES; ++p)
+#pragma unroll
+          for (int n8 = 0; n8 < 2; ++n8) {
+            const float2 v = *reinterpret_cast<const float2*>(&s_x[xp][g + 8 * i][p * 16 + n8 * 8 + 2 * t4]);
+            const int j = j0 + p * 16 + n8 * 8 + 2 * t4;   // (selects: scores past the range may be anything)
+            w[p][n8][2 * i] = j <= pos[i] && pos[i] - j < a.window ? v.x * a.scale2 : -INFINITY;
+            w[p][n8][2 * i + 1] = j + 1 <= pos[i] && pos[i] - j - 1 < a.window ? v.y * a.scale2 : -INFINITY;
+            m = fmaxf(m, fmaxf(w[p][n8][2 * i], w[p][n8][2 * i + 1]));
+          }
+        m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
+        m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
+        const float now = fmaxf(mx[i], m), ref = now == -INFINITY ? 0.f : now;
+        moved |= now > mx[i];
+        back[i] = exp2f(mx[i] - ref);
+        mx[i] = now;
+        float ws = 0.f;
+#pragma unroll
+        for (int p = 0; p < TPAGES; ++p)
 #pragma unroll
           for (int n8 = 0; n8 < 2; ++n8)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-              const int j = j0 + n8 * 8 + (lane & 3) * 2 + e;
-              float& s = sc[n8][2 * i + e];
-              s = j <= pos[i] && pos[i] - j < a.window ? s * a.scale2 : -INFINITY;   // (a select: stale bytes may be anything)
-              m = fmaxf(m, s);
+              float& x = w[p][n8][2 * i + e];
+              x = exp2f(x - ref);
+              ws += x;
             }
-          m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
-          m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
-          now[i] = fmaxf(mx[i], m);
-          moved |= now[i] > mx[i];
-          const float ref = now[i] == -INFINITY ? 0.f : now[i];
-          back[i] = exp2f(mx[i] - ref);
-          mx[i] = now[i];
-          float w[4], ws = 0.f;
+        sum[i] = sum[i] * back[i] + ws;                    // (this lane's keys; added over the quad at the end)
+      }
+      xp ^= 1u;
+      if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
-          for (int n8 = 0; n8 < 2; ++n8) {
-            w[2 * n8] = exp2f(sc[n8][2 * i] - ref), w[2 * n8 + 1] = exp2f(sc[n8][2 * i + 1] - ref);
-            ws += w[2 * n8] + w[2 * n8 + 1];
-            split2(w[2 * n8], w[2 * n8 + 1], wh[n8 * 2 + i], wl[n8 * 2 + i]);
-          }
-          sum[i] = sum[i] * back[i] + ws;                  // (this lane's keys; added over the quad at the end)
-        }
-        if (__any_sync(0xffffffffu, moved)) {
+        for (int nd = 0; nd < CW / 8; ++nd) o[nd][0] *= back[0], o[nd][1] *= back[0], o[nd][2] *= back[1], o[nd][3] *= back[1];
+      }
 #pragma unroll
-          for (int nd = 0; nd < OD / 8; ++nd) o[nd][0] *= back[0], o[nd][1] *= back[0], o[nd][2] *= back[1], o[nd][3] *= back[1];
-        }
+      for (int p = 0; p < TPAGES; ++p) {
+        if (j0 + p * KVB < hi) {
+          uint32_t wh[4], wl[4];
 #pragma unroll
-        for (int nd = 0; nd < OD / 8; nd += 2) {
-          if (nd < vch) {
-            uint32_t b[4];
-            ldsm4t(b, base + (vr * nc + place(vc0 + nd + vcl, vr, vrot)) * 16);
-            mma16(o[nd], wh, b[0], b[1]);
-            mma16(o[nd + 1], wh, b[2], b[3]);
-            mma16(o[nd], wl, b[0], b[1]);
-            mma16(o[nd + 1], wl, b[2], b[3]);
+          for (int n8 = 0; n8 < 2; ++n8)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) split2(w[p][n8][2 * i], w[p][n8][2 * i + 1], wh[n8 * 2 + i], wl[n8 * 2 + i]);
+#pragma unroll
+          for (int nd = 0; nd < CW / 8; nd += 2) {
+            if (nd < vch) {
+              uint32_t b[4];
+              ldsm4t(b, stage + p * page_b + (vr * nc + place(vc0 + nd + vcl, vr, vrot)) * 16);
+              mma16(o[nd], wh, b[0], b[1]);
+              mma16(o[nd + 1], wh, b[2], b[3]);
+              mma16(o[nd], wl, b[0], b[1]);
+              mma16(o[nd + 1], wl, b[2], b[3]);
+            }
           }
         }
       }
@@ -343,7 +342,13 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
     for (int i = 0; i < 2; ++i) {
       sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
       sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
-      if (half == 0 && (lane & 3) == 0) s_m[kw][(lane >> 2) + 8 * i] = mx[i], s_l[kw][(lane >> 2) + 8 * i] = sum[i];
+      const int r = g + 8 * i, row = row0 + r;
+      if (r >= rows) continue;
+      const size_t at = ((size_t)(q0 + row / a.heads) * a.heads + row % a.heads) * a.n_splits + split;
+      if (warp == 0 && t4 == 0) a.ml[at] = make_float2(mx[i], sum[i]);
+#pragma unroll
+      for (int nd = 0; nd < CW / 8; ++nd)
+        if (nd < vch) *reinterpret_cast<float2*>(a.part + at * kv + (vc0 + nd) * 8 + 2 * t4) = make_float2(o[nd][2 * i], o[nd][2 * i + 1]);
     }
   }
   __syncthreads();
@@ -352,36 +357,6 @@ __global__ void __launch_bounds__((4 * HALVES + 1) * 32) latent_decode_kernel(co
     const long long t_begin = clock64();
     while (clock64() - t_begin < 2000000LL) {
     }
-  }
-  // the four warps saw different keys: merge them in order, through the (idle) ring
-  float* so = reinterpret_cast<float*>(ring);               // [4][16][kv]
-  if (warp < NW) {
-    const int vc0 = half * (OD / 8), vch = min(OD / 8, a.vch - vc0), r = lane >> 2;
-#pragma unroll
-    for (int nd = 0; nd < OD / 8; ++nd) {
-      if (nd < vch) {
-        const int d = (vc0 + nd) * 8 + (lane & 3) * 2;
-        *reinterpret_cast<float2*>(so + (size_t)(kw * 16 + r) * kv + d) = make_float2(o[nd][0], o[nd][1]);
-        *reinterpret_cast<float2*>(so + (size_t)(kw * 16 + r + 8) * kv + d) = make_float2(o[nd][2], o[nd][3]);
-      }
-    }
-  }
-  __syncthreads();
-  for (int x = threadIdx.x; x < rows * (kv / 4); x += THREADS) {
-    const int r = x / (kv / 4), d = (x % (kv / 4)) * 4, row = row0 + r;
-    const float m = fmaxf(fmaxf(s_m[0][r], s_m[1][r]), fmaxf(s_m[2][r], s_m[3][r])), ref = m == -INFINITY ? 0.f : m;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    float l = 0.f;
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const float f = exp2f(s_m[k][r] - ref);
-      const float4 y = *reinterpret_cast<const float4*>(so + (size_t)(k * 16 + r) * kv + d);
-      v.x = fmaf(f, y.x, v.x), v.y = fmaf(f, y.y, v.y), v.z = fmaf(f, y.z, v.z), v.w = fmaf(f, y.w, v.w);
-      l = fmaf(f, s_l[k][r], l);
-    }
-    const size_t at = ((size_t)(q0 + row / a.heads) * a.heads + row % a.heads) * a.n_splits + split;
-    *reinterpret_cast<float4*>(a.part + at * kv + d) = v;
-    if (d == 0) a.ml[at] = make_float2(m, l);
   }
 }
 
@@ -642,16 +617,15 @@ __global__ void __launch_bounds__(256) latent_prompt_kernel(const PromptArgs a) 
     }
 }
 
-template <int OD, int HALVES> cudaError_t decode_launch(DecArgs a, int tiles, int B, cudaStream_t st) {
+template <int CW> cudaError_t decode_launch(DecArgs a, int tiles, int B, cudaStream_t st) {
   const size_t q_bytes = (size_t)(16 * (a.kch * 16 + 16) + 127) / 128 * 128, stage = (size_t)TILE * a.kch * 16;
-  const size_t merge = (size_t)4 * 16 * a.vch * 8 * sizeof(float);
   int stages = 4;
-  while (stages > 2 && q_bytes + stages * stage > 104 * 1024) --stages;          // two blocks on an SM where three stages allow it
+  while (stages > 2 && q_bytes + stages * stage > 100 * 1024) --stages;          // two blocks on an SM where three stages allow it
   if (stages < 3 && q_bytes + 3 * stage <= (size_t)LD_SMEM) stages = 3;
-  const size_t smem = q_bytes + (stages * stage > merge ? stages * stage : merge) + 128;
+  const size_t smem = q_bytes + stages * stage + 128;
   if (smem > (size_t)LD_SMEM + 128) return cudaErrorInvalidValue;
   a.n_stages = stages;
-  auto k = latent_decode_kernel<OD, HALVES>;
+  auto k = latent_decode_kernel<CW>;
   static bool configured = false;
   if (!configured) {
     const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM + 128);
@@ -659,7 +633,7 @@ template <int OD, int HALVES> cudaError_t decode_launch(DecArgs a, int tiles, in
     cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     configured = true;
   }
-  return trl_launch(k, dim3(tiles * a.n_splits, B), dim3((4 * HALVES + 1) * 32), smem, st, a);
+  return trl_launch(k, dim3(tiles * a.n_splits, B), dim3(288), smem, st, a);
 }
 
 template <int DQ, int DV> cudaError_t prompt_launch(const PromptArgs& a, cudaStream_t st) {
@@ -678,8 +652,8 @@ template <int DQ, int DV> cudaError_t prompt_launch(const PromptArgs& a, cudaStr
 
 // 1 when the tensor-core forms take heads of these (padded) sizes.
 TRL_API int trl_latent_mma_ok(int dk, int rd, int dv, int kv) {
-  const size_t row = (size_t)(kv + rd) * 2, q = (size_t)16 * (row + 16) + 128, merge = (size_t)4 * 16 * kv * 4;
-  return dk + rd <= 256 && dv <= 256 && kv <= 512 && q + (2 * TILE * row > merge ? 2 * TILE * row : merge) <= (size_t)LD_SMEM;
+  const size_t row = (size_t)(kv + rd) * 2;
+  return dk + rd <= 256 && dv <= 256 && kv <= 512 && 16 * (row + 16) + 128 + 2 * TILE * row <= (size_t)LD_SMEM;
 }
 
 // Sequences of min_len..max_len tokens in the absorbed form.  q: [T, heads, dq], whose rotated part is turned here (n_pairs 0: it
@@ -705,9 +679,9 @@ TRL_API int trl_latent_decode(const void* q, int dq, int dk, int rd, const void*
   a.table = (const int*)table, a.max_blocks = max_blocks, a.q_start = (const int*)q_start, a.q_len = (const int*)q_len;
   a.positions = (const int*)positions, a.part = (float*)part, a.ml = (float2*)ml, a.heads = heads, a.n_splits = n_splits, a.n_stages = 2;
   a.window = window, a.min_len = min_len, a.max_len = max_len, a.scale2 = scale * LOG2E;
-  if (kv <= 128) e = decode_launch<128, 1>(a, tiles, B, st);
-  else if (kv <= 256) e = decode_launch<256, 1>(a, tiles, B, st);
-  else e = decode_launch<256, 2>(a, tiles, B, st);
+  if (kv <= 128) e = decode_launch<16>(a, tiles, B, st);
+  else if (kv <= 256) e = decode_launch<32>(a, tiles, B, st);
+  else e = decode_launch<64>(a, tiles, B, st);
   if (e != cudaSuccess) return (int)e;
   const int z = groups * heads >= 148 ? 1 : (dv > 128 ? 2 : 1);
   return (int)trl_launch(latent_out_kernel, dim3(heads, groups, z), dim3(256), (size_t)2 * 8 * (kv + 8) * sizeof(bf16), st, (const float*)part,

@@ -114,6 +114,7 @@ __global__ void __launch_bounds__(256) scan_serial_kernel(const ScanArgs a) {
         float v = 0.f;
         if (x < 2 * a.dk || col0 + d < a.dv) {
           v = a.conv_b[cc];
+#pragma unroll 4
           for (int j = 0; j < a.taps; ++j) {
             const int back = a.taps - 1 - j;
             if (back <= pos)

@@ -17,6 +17,7 @@ MAMBA2, MLSTM = 0, 1
 MIX_ROWS_MAX = 8        # rows the weight-streaming projection serves
 LATENT_SHORT = 32       # tokens of a sequence up to which attention runs in the latent (absorbed) form
 SCAN_SHORT = 16         # tokens of a sequence up to which a scan goes token by token
+CONV_FUSED = 2          # sequences of a decode tick up to which the scan convolves its columns itself
 CHUNK_DK = 128          # state rows the chunked scan takes
 MAX_SPLITS = 32         # shares of a window its keys are split into (a warp merges them)
 PART_BYTES = 1 << 28    # most fp32 partial sums of split attention
@@ -243,8 +244,8 @@ class MixerOps:
         ring = pool.ring_view(idx, 0) if kind == MAMBA2 else None
         o = self.ws.get("scan_o", (t, l.heads * l.dv), torch.float32)
         a = ScanArgs()
-        if kind == MAMBA2 and batch.max_q_len == 1 and not batch.keep_steps:
-            # a decode tick: the scan convolves its own columns
+        if kind == MAMBA2 and batch.max_q_len == 1 and batch.n_seqs <= CONV_FUSED and not batch.keep_steps:
+            # a small decode tick: the scan convolves its own columns (every slice of a head its keys anew)
             rows = proj
             a.taps, a.channels, a.conv_w, a.conv_b = l.taps, l.conv_c, w["conv"].data_ptr(), w["conv_b"].data_ptr()
             a.ring, a.ring_slot, a.ring_rows, a.ring_ld = ring.data_ptr(), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1)

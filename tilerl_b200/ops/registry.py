@@ -85,6 +85,12 @@ register("any", "cpu", {op: Kernel(fn, _REF) for op, fn in {
     "page_bounds": "page_bounds", "select_pages": "select_pages", "sigmoid_attention": "sigmoid_attention",
     "polynorm": "polynorm", "packed_kv_write": "packed_kv_write",
 }.items()})
+_MIX = "tilerl_b200/ops/ref_mixers.py"
+register("any", "cpu", {op: Kernel(fn, _MIX) for op, fn in {
+    "join": "stream_norm", "clamped_glu": "clamped_glu", "side_input": "gelu_tanh", "latent_prep": "latent_write",
+    "latent_attention_decode": "latent_attention", "latent_attention_prefill": "latent_attention", "latent_attention_plain": "latent_attention",
+    "scan_decode": "mlstm_step", "scan_prefill": "mamba2_step",
+}.items()})
 register("any", "cpu", {
     "quantize_nvfp4": Kernel("quantize_nvfp4", "tilerl_b200/formats.py"),
     "dequantize_nvfp4": Kernel("dequantize_nvfp4", "tilerl_b200/formats.py"),
@@ -162,6 +168,18 @@ register("any", "sm100", {
     "block_mid": Kernel("block_mid_kernel", "csrc/stream.cu", "trl_block_mid", note="packed K / V write + PolyNorm"),
     "sigmoid_attention": Kernel("sig_attn_kernel + sig_combine_kernel", "csrc/attn_sigmoid.cu", "trl_sigmoid_attn",
                                 note="bf16 packed pool; narrow row tiles for decoding, wide ones for prompts, key splits"),
+    "join": Kernel("join_kernel", "csrc/join.cu", "trl_join", note="branch norm + stream addition + next norm; bf16 or fp32 rows"),
+    "clamped_glu": Kernel("glu_kernel", "csrc/join.cu", "trl_clamped_glu", note="few rows: epilogue of linear_rows_kernel"),
+    "side_input": Kernel("side_kernel", "csrc/join.cu", "trl_side_input", note="few rows: epilogue of linear_rows_kernel"),
+    "latent_prep": Kernel("latent_prep_kernel", "csrc/latent.cu", "trl_latent_prep", note="normed latents and rotated key into packed pages"),
+    "latent_attention_decode": Kernel("latent_absorb_kernel + latent_decode_kernel + latent_out_kernel", "csrc/latent_mma.cu", "trl_latent_decode",
+                                      note="absorbed form: all heads share the cached latents; maps in and out on tensor cores"),
+    "latent_attention_prefill": Kernel("latent_gather_kernel + latent_prompt_kernel", "csrc/latent_mma.cu", "trl_latent_prompt",
+                                       note="expanded keys / values, windowed, output gate in the epilogue"),
+    "latent_attention_plain": Kernel("latent_attn_kernel", "csrc/latent.cu", "trl_latent_attn", note="fp32 models, sizes without a tensor-core form"),
+    "scan_decode": Kernel("scan_serial_kernel + scan_norm_kernel", "csrc/scan.cu", "trl_scan_serial", note="Mamba-2 / mLSTM, token by token, fp32 state"),
+    "scan_prefill": Kernel("scan_conv_kernel + scan_chunk_kernel + scan_norm_kernel", "csrc/scan_mma.cu", "trl_scan_chunk",
+                           note="64-token chunks on tensor cores, fp32 state"),
     "batch_fill": Kernel("trl_batch_fill", "csrc/runtime.cpp", "trl_batch_fill", note="host runtime"),
     "pager": Kernel("trl_pager_*", "csrc/runtime.cpp", "trl_pager_alloc", note="host runtime"),
 })
