@@ -62,7 +62,7 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
 // is the previous tick, and every tick has launches in between that let their dependents in only after their own wait.
 constexpr int SS_TB = 16;
 template <typename T, int KIND, int RMAX, bool CONV>
-__global__ void __launch_bounds__(256) scan_serial_kernel(const ScanArgs a) {
+__global__ void __launch_bounds__(256, RMAX <= 16 ? 4 : 2) scan_serial_kernel(const ScanArgs a) {
   constexpr int DK = RMAX * 8;
   __shared__ float s_q[SS_TB][DK], s_k[SS_TB][DK], s_v[SS_TB][32];
   __shared__ float s_keep[SS_TB], s_add[SS_TB], s_floor[SS_TB], s_m;
