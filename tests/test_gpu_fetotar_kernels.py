@@ -155,7 +155,7 @@ def test_scans_against_the_recurrence(ops, spec, form):
 
 
 # ---- latent attention ----------------------------------------------------------------------------------------
-LATENTS = [(3, 16, 16, 16, 32, 19), (6, 64, 32, 64, 96, 40), (16, 128, 64, 128, 512, 300), (5, 48, 16, 80, 240, 64), (1, 192, 64, 256, 128, 1),
+LATENTS = [(3, 16, 16, 16, 32, 19), (7, 80, 32, 64, 112, 45), (16, 128, 64, 128, 512, 300), (5, 48, 16, 80, 240, 64), (1, 192, 64, 256, 128, 1),
            (40, 32, 16, 32, 48, 129), (2, 128, 16, 96, 400, 5000)]
 
 

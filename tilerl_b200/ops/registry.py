@@ -89,7 +89,7 @@ _MIX = "tilerl_b200/ops/ref_mixers.py"
 register("any", "cpu", {op: Kernel(fn, _MIX) for op, fn in {
     "join": "stream_norm", "clamped_glu": "clamped_glu", "side_input": "gelu_tanh", "latent_prep": "latent_write",
     "latent_attention_decode": "latent_attention", "latent_attention_prefill": "latent_attention", "latent_attention_plain": "latent_attention",
-    "scan_decode": "mlstm_step", "scan_prefill": "mamba2_step",
+    "scan_conv": "conv_rows", "scan_decode": "mlstm_step", "scan_prefill": "mamba2_step",
 }.items()})
 register("any", "cpu", {
     "quantize_nvfp4": Kernel("quantize_nvfp4", "tilerl_b200/formats.py"),
@@ -178,7 +178,8 @@ register("any", "sm100", {
                                        note="expanded keys / values, windowed, output gate in the epilogue"),
     "latent_attention_plain": Kernel("latent_attn_kernel", "csrc/latent.cu", "trl_latent_attn", note="fp32 models, sizes without a tensor-core form"),
     "scan_decode": Kernel("scan_serial_kernel + scan_norm_kernel", "csrc/scan.cu", "trl_scan_serial", note="Mamba-2 / mLSTM, token by token, fp32 state"),
-    "scan_prefill": Kernel("scan_conv_kernel + scan_chunk_kernel + scan_norm_kernel", "csrc/scan_mma.cu", "trl_scan_chunk",
+    "scan_conv": Kernel("scan_conv_kernel", "csrc/scan.cu", "trl_scan_conv", note="causal convolution + silu of a tick's rows"),
+    "scan_prefill": Kernel("scan_chunk_kernel", "csrc/scan_mma.cu", "trl_scan_chunk",
                            note="64-token chunks on tensor cores, fp32 state"),
     "batch_fill": Kernel("trl_batch_fill", "csrc/runtime.cpp", "trl_batch_fill", note="host runtime"),
     "pager": Kernel("trl_pager_*", "csrc/runtime.cpp", "trl_pager_alloc", note="host runtime"),
