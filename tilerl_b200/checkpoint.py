@@ -37,13 +37,14 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import ATTN, ModelConfig, StreamDesign, ZinutarConfig
+from .config import ATTN, DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig
 from .formats import (FP8BlockTensor, NVFP4Tensor, dequantize_fp8_block, dequantize_nvfp4,
                       quantize_nvfp4)
 from .models.hybrid import HybridModel, linear_names, quantize_weight
+from .models.deluvik import DeluvikModel
 from .models.fetotar import FetotarModel
 from .models.zinutar import ZinutarModel
-from . import fetotar_layout, zinutar_layout
+from . import deluvik_layout, fetotar_layout, zinutar_layout
 
 
 class CheckpointError(ValueError):
@@ -258,9 +259,13 @@ def assemble_master(cfg: ModelConfig, reader: _Reader) -> Dict[str, torch.Tensor
     return out
 
 
+STREAM_DESIGNS = {ZinutarConfig: (ZinutarModel, zinutar_layout), FetotarConfig: (FetotarModel, fetotar_layout),
+                  DeluvikConfig: (DeluvikModel, deluvik_layout)}
+
+
 def load_stream_design(cfg: StreamDesign, path: str, device="cpu", dtype: Optional[torch.dtype] = None):
     """Dense checkpoint of a stream design (tensor names and shapes: ``tensor_shapes`` of its layout module)."""
-    model, layout = (ZinutarModel, zinutar_layout) if isinstance(cfg, ZinutarConfig) else (FetotarModel, fetotar_layout)
+    model, layout = STREAM_DESIGNS[type(cfg)]
     reader = _Reader(path)
     lacks = [n for n in layout.tensor_shapes(cfg) if not reader.has(n)]
     if lacks:

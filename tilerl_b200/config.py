@@ -1,7 +1,9 @@
 """Model configurations: the hybrid (gated-GQA attention + Gated-DeltaNet) decoder, and the stream designs
 (:class:`StreamDesign`: an fp32 residual stream, served in bf16 or fp32 on one GPU per process; no counterpart in the
-reference): Zinutar (:class:`ZinutarConfig`, a looped decoder of parallel blocks) and Fetotar (:class:`FetotarConfig`,
-sandwich-normed layers of latent attention, Mamba-2 and mLSTM with a per-layer token input).
+reference): Zinutar (:class:`ZinutarConfig`, a looped decoder of parallel blocks), Fetotar (:class:`FetotarConfig`,
+sandwich-normed layers of latent attention, Mamba-2 and mLSTM with a per-layer token input) and Deluvik
+(:class:`DeluvikConfig`, softmax attention with sinks, shared keys and short convolutions, a gated linear recurrence beside
+windowed attention, mixtures of experts, norms on every branch's output).
 
 One frozen dataclass describes every shape the kernels, the KV pools, the
 tensor-parallel shard tables and the cost model derive from.  Layer kinds are
@@ -14,11 +16,14 @@ Parity: reference ``src/tilerl/config.py:11`` (``ModelConfig``), ``:114``
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import dataclass, replace
+from importlib import import_module
 from typing import Dict, Optional, Tuple
 
-from .mixers import MIXERS, ClampedGluSpec, LatentAttnSpec, LayerSpec, Mamba2Spec, MlstmSpec, RotarySpec, YarnSpec, take
+from .mixers import (MIXERS, BandScalingSpec, ClampedGluSpec, GluSpec, LatentAttnSpec, LayerSpec, LruSpec, Mamba2Spec, MlstmSpec, MoeSpec,
+                     ParallelSpec, RotarySpec, SoftmaxAttnSpec, YarnSpec, take)
 
 ATTN = "attn"
 GDN = "gdn"
@@ -224,6 +229,12 @@ class StreamDesign:
     # no Gated-DeltaNet layers: recurrent state, where a design has any, lives in a RecurrentPool
     n_gdn_layers = 0
     gdn_k_heads = gdn_v_heads = gdn_head_dim = gdn_conv_dim = 0
+
+
+    @property
+    def layout(self):
+        """The module with the shapes and memory layout of the design's parameters."""
+        return import_module(f"..{self.architecture.lower()}_layout", __name__)
 
 
 # ---- Zinutar: looped parallel-block decoder with sigmoid-weighted attention ------------------------
@@ -516,9 +527,168 @@ def fetotar_small() -> FetotarConfig:
     return fetotar_uniform("fetotar-small", hidden=2048, vocab=32768, ff=6144, heads=16, repeats=1, window=1024, q_rank=768)
 
 
-ARCHITECTURES = {c.architecture: c for c in (ZinutarConfig, FetotarConfig)}
+# ---- Deluvik: attention beside a gated linear recurrence, shared keys, mixtures of experts ----------------------
+# which optional parts the design's attention mixers have
+_DELUVIK_ATTN = {"attention": dict(norm="all", half=True, capped=True, sink=True, tied=True),
+                 "attention_2": dict(norm="all", half=True, conv=True, sink=True)}
+_DELUVIK_LEFT = dict(norm="head", half=False, windowed=True)
+
+
+def _deluvik_mixer(kind: str, m: Dict, where: str):
+    if kind in _DELUVIK_ATTN:
+        return SoftmaxAttnSpec.from_json(m, where, **_DELUVIK_ATTN[kind])
+    if kind != "parallel":
+        raise ValueError(f"{where}: unknown mixer type {kind!r}")
+    take(m, ("left", "right", "left_scale", "right_scale"), where)
+    return ParallelSpec(SoftmaxAttnSpec.from_json(m["left"], where + " left", **_DELUVIK_LEFT), LruSpec.from_json(m["right"], where + " right"),
+                        float(m["left_scale"]), float(m["right_scale"]))
+
+
+def _deluvik_mixer_json(m) -> Tuple[str, Dict]:
+    if isinstance(m, ParallelSpec):
+        return "parallel", {"left": m.left.to_json(), "right": m.right.to_json(), "left_scale": m.left_scale, "right_scale": m.right_scale}
+    return ("attention" if m.tied else "attention_2"), m.to_json()
+
+
+@dataclass(frozen=True)
+class DeluvikConfig(StreamDesign):
+    """Sizes and constants of a Deluvik model.  Every layer has its own mixer and feed-forward; a layer that reads another
+    layer's keys and values (``kv_from``) has no KV cache of its own."""
+    name: str
+    hidden: int
+    vocab: int
+    layers: Tuple[LayerSpec, ...]
+    logit_cap: float
+    norm_eps: float = 1e-5
+    max_ctx: int = 1 << 20
+
+    architecture = "Deluvik"
+
+    def __post_init__(self) -> None:
+        object.__setattr__(self, "layers", tuple(self.layers))
+        if self.hidden <= 0 or self.vocab <= 0 or not self.layers or self.logit_cap <= 0:
+            raise ValueError("a model needs positive sizes, a positive cap on its logits and at least one layer")
+        for i, l in enumerate(self.layers):
+            a = self.attn(i)
+            if a.kv_from is None:
+                continue
+            src = self.layers[a.kv_from].mixer if 0 <= a.kv_from < i else None
+            if not isinstance(src, SoftmaxAttnSpec) or src.kv_from is not None or src.tied != a.tied or not a.same_keys(src):
+                raise ValueError(f"layer {i} cannot read the keys of layer {a.kv_from}")
+
+    def attn(self, layer: int) -> SoftmaxAttnSpec:
+        """The attention of a layer (every layer has one)."""
+        m = self.layers[layer].mixer
+        return m.left if isinstance(m, ParallelSpec) else m
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def cache_owners(self) -> Tuple[int, ...]:
+        """Layers with a KV cache, in the order of the caches."""
+        return tuple(i for i in range(self.n_layers) if self.attn(i).kv_from is None)
+
+    def cache_index(self, layer: int) -> int:
+        """Number of the KV cache that the layer reads."""
+        src = self.attn(layer).kv_from
+        return self.cache_owners.index(layer if src is None else src)
+
+    @property
+    def n_attn_layers(self) -> int:
+        return len(self.cache_owners)
+
+    @property
+    def n_q_heads(self) -> int:
+        return max(self.attn(i).heads for i in range(self.n_layers))
+
+    @property
+    def n_kv_heads(self) -> int:
+        return max(self.attn(i).kv_heads for i in range(self.n_layers))
+
+    def n_params(self) -> int:
+        from .deluvik_layout import tensor_shapes
+        return sum(math.prod(s) for s in tensor_shapes(self).values())
+
+    # ---- config.json -----------------------------------------------------------------------
+    @classmethod
+    def from_json(cls, j: Dict, name: str = "deluvik", max_ctx: Optional[int] = None) -> "DeluvikConfig":
+        take(j, ("architecture", "width", "vocab", "norm", "logit_softcap", "layers"), "configuration")
+        take(j["norm"], ("eps",), "norm")
+        layers = []
+        for i, l in enumerate(j["layers"]):
+            l = take({"mlp": None, **l}, ("type", "mixer", "mlp"), f"layer {i}")
+            f = l["mlp"]
+            if f is not None:
+                if f.get("kind") not in ("dense", "moe"):
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {f.get('kind')!r}")
+                f = GluSpec.from_json(f, f"layer {i} mlp", "gelu") if f["kind"] == "dense" else MoeSpec.from_json(f, f"layer {i} mlp")
+            layers.append(LayerSpec(_deluvik_mixer(l["type"], l["mixer"], f"layer {i} mixer"), f))
+        return cls(name=name, hidden=int(j["width"]), vocab=int(j["vocab"]), layers=tuple(layers), logit_cap=float(j["logit_softcap"]),
+                   norm_eps=float(j["norm"]["eps"]), **({} if max_ctx is None else {"max_ctx": max_ctx}))
+
+    def to_json(self) -> Dict:
+        layers = []
+        for l in self.layers:
+            kind, mixer = _deluvik_mixer_json(l.mixer)
+            layers.append({"type": kind, "mixer": mixer, "mlp": None if l.mlp is None else l.mlp.to_json()})
+        return {"architecture": self.architecture, "width": self.hidden, "vocab": self.vocab, "norm": {"eps": self.norm_eps},
+                "logit_softcap": self.logit_cap, "layers": layers}
+
+
+def deluvik_attention(heads, kv_heads, dim, scale, cap, rot) -> SoftmaxAttnSpec:
+    """Mixer whose values are its keys: capped scores and a sink."""
+    return SoftmaxAttnSpec(heads, kv_heads, dim, dim, scale, replace(rot, half=True), "all", None, cap, True, 0, True)
+
+
+def deluvik_conv_attention(heads, kv_heads, dim, vdim, scale, conv, rot, kv_from=None) -> SoftmaxAttnSpec:
+    """Mixer whose projections pass a short convolution, with a sink."""
+    return SoftmaxAttnSpec(heads, kv_heads, dim, vdim, scale, replace(rot, half=True), "all", None, None, True, conv, False, kv_from)
+
+
+def deluvik_parallel(left_scale, right_scale, right: LruSpec, heads, kv_heads, dim, vdim, scale, window, rot) -> ParallelSpec:
+    """Windowed attention beside a gated linear recurrence."""
+    return ParallelSpec(SoftmaxAttnSpec(heads, kv_heads, dim, vdim, scale, rot, "head", window), right, left_scale, right_scale)
+
+
+def deluvik_tiny() -> DeluvikConfig:
+    """Smoke model: every mixer, shared keys, both feed-forwards and none, byte vocabulary of 320."""
+    rot, scaled = RotarySpec(16, 10000.0), RotarySpec(24, 5000.0, BandScalingSpec(4.0, 1.0, 4.0, 64.0))
+    moe = MoeSpec(40, 6, 2, 56)
+    return DeluvikConfig(
+        name="deluvik-tiny", hidden=72, vocab=320, logit_cap=25.0, norm_eps=1e-5, max_ctx=4096,
+        layers=(LayerSpec(deluvik_parallel(0.8, 1.1, LruSpec(60, 3, 4), 4, 2, 24, 32, 0.2, 24, rot), moe),
+                LayerSpec(deluvik_attention(5, 1, 24, 0.2, 30.0, scaled), GluSpec(100, "gelu")),
+                LayerSpec(deluvik_conv_attention(4, 2, 32, 16, 0.18, 3, rot), None),
+                LayerSpec(deluvik_conv_attention(4, 2, 32, 16, 0.18, 3, rot, kv_from=2), moe)))
+
+
+def deluvik_uniform(name: str, *, hidden: int, vocab: int, ff: int, expert_ff: int, experts: int, top: int, heads: int, kv_heads: int,
+                    repeats: int, window: int, dim: int = 128, lru_blocks: int = 16, **kw) -> DeluvikConfig:
+    """A model of ``repeats`` x (parallel, attention with a convolution, the same over the keys of the one before, attention over
+    tied keys) layers of one width; the last of the four has a dense feed-forward, the others experts and a shared one."""
+    rot, moe, layers = RotarySpec(dim, 500000.0), MoeSpec(expert_ff, experts, top, expert_ff), []
+    for _ in range(repeats):
+        n = len(layers)
+        layers += [LayerSpec(deluvik_parallel(1.0, 1.0, LruSpec(hidden, lru_blocks, 4), heads, kv_heads, dim, dim, dim ** -0.5, window, rot), moe),
+                   LayerSpec(deluvik_conv_attention(heads, kv_heads, dim, dim, dim ** -0.5, 4, rot), moe),
+                   LayerSpec(deluvik_conv_attention(heads, kv_heads, dim, dim, dim ** -0.5, 4, rot, kv_from=n + 1), moe),
+                   LayerSpec(deluvik_attention(heads, kv_heads, dim, dim ** -0.5, 50.0, replace(rot, scaling=BandScalingSpec(8.0, 1.0, 4.0, 8192.0))),
+                             GluSpec(ff, "gelu"))]
+    return DeluvikConfig(name=name, hidden=hidden, vocab=vocab, layers=tuple(layers), logit_cap=30.0, **kw)
+
+
+def deluvik_small() -> DeluvikConfig:
+    """Four layers of a 1B-class width; profiler captures and GPU engine tests."""
+    return deluvik_uniform("deluvik-small", hidden=2048, vocab=32768, ff=6144, expert_ff=768, experts=32, top=4, heads=16, kv_heads=4,
+                           repeats=1, window=1024)
+
+
+ARCHITECTURES = {c.architecture: c for c in (ZinutarConfig, FetotarConfig, DeluvikConfig)}
 
 _REGISTRY = {
+    "deluvik-tiny": deluvik_tiny, "deluvik-small": deluvik_small,
     "fetotar-tiny": fetotar_tiny, "fetotar-small": fetotar_small,
     "zinutar-tiny": zinutar_tiny, "zinutar-small": zinutar_small, "zinutar-8b": zinutar_8b,
     "qwen38-27b": qwen38_27b, "qwen36-27b": qwen36_27b, "tiny": tiny,

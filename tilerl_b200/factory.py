@@ -20,10 +20,11 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig, get_config
+from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig, get_config
 from .engine import Engine, StepLimits
 from .formats import NVFP4Tensor
 from .kv import NoPrefixStore, PrefixStore, kv_pages, make_kv_pool, make_state_pool
+from .models.deluvik import DeluvikModel
 from .models.fetotar import FetotarModel
 from .models.hybrid import HybridModel, linear_names, param_shapes, quantize_weight
 from .models.zinutar import ZinutarModel
@@ -31,7 +32,7 @@ from .ops.backend import RefOps
 from .ops.ref import KV_BLOCK
 
 
-STREAM_MODELS = {ZinutarConfig: ZinutarModel, FetotarConfig: FetotarModel}
+STREAM_MODELS = {ZinutarConfig: ZinutarModel, FetotarConfig: FetotarModel, DeluvikConfig: DeluvikModel}
 
 
 def _seed_for(name: str, seed: int) -> int:

@@ -252,13 +252,9 @@ def weight_specs(cfg) -> Dict[str, Tuple[Tuple[int, ...], str]]:
     """Every served tensor -> (shape, format name).  The cost model, the memory
     planner and the dry-run ledger all read this one table.
     Reference ``precision.py:103`` (``weight_specs``)."""
-    from .config import ATTN, FetotarConfig, StreamDesign
+    from .config import ATTN, StreamDesign
     if isinstance(cfg, StreamDesign):
-        if isinstance(cfg, FetotarConfig):
-            from .fetotar_layout import param_shapes
-        else:
-            from .zinutar_layout import param_shapes
-        return {n: (s, "bf16" if k == "w" else "f32") for n, (s, k) in param_shapes(cfg).items()}
+        return {n: (s, "bf16" if k == "w" else "f32") for n, (s, k) in cfg.layout.param_shapes(cfg).items()}
     q = cfg.quant
     lin = {"nvfp4": "nvfp4", "fp8": "fp8_block", "bf16": "bf16"}[q]
     h = cfg.hidden

@@ -11,8 +11,8 @@
   ``cur[slot]`` names the live plane, so adopting "the state after n accepted
   tokens" is one int32 write instead of a 144 MiB copy, and the conv window
   needs no rollback at all because the ring is addressed by absolute position.
-* :class:`RecurrentPool` -- the same slots and planes for layers whose state differs in form and size (decayed scans);
-  no counterpart in the reference.
+* :class:`RecurrentPool` -- the same slots and planes for layers whose state differs in form and size (decayed scans,
+  linear recurrences, inputs of short convolutions); no counterpart in the reference.
 * :class:`PrefixStore` -- rolling-hash cache of whole 16-token blocks; an entry
   owns refcounted block ids *and* a GDN snapshot taken at the same boundary
   (a hybrid model needs both to resume).
@@ -31,8 +31,9 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from .config import FetotarConfig, ModelConfig, StreamDesign
-from .fetotar_layout import LatentLayout, layout_of, state_layouts
+from . import deluvik_layout, fetotar_layout
+from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign
+from .fetotar_layout import LatentLayout, layout_of
 from .ops.ref import KV_BLOCK
 
 RING = 16  # conv ring rows; >= spec width + conv taps
@@ -191,8 +192,8 @@ def _page_index(width: int, chunks: int, base: int, itemsize: int) -> torch.Tens
 @dataclass(frozen=True)
 class KvPage:
     """Byte layout of one page of one KV head in a :class:`PackedKvPool`: 16 K rows, the 16 fp32 reciprocal
-    root mean squares of those rows (64 bytes, and 64 unused ones), 16 V rows, back to back, so that one bulk copy
-    brings a page whole.
+    root mean squares of those rows (64 bytes, and 64 unused ones; without ``factors`` K is kept normalised and there are
+    none), 16 V rows, back to back, so that one bulk copy brings a page whole.
 
     Rows are made of 16-byte chunks whose order depends on the row, so that eight rows read at one chunk index fall
     into different shared-memory banks: chunk ``c`` of row ``r`` sits at ``c ^ (r % 8)`` when a row is a multiple of
@@ -201,6 +202,7 @@ class KvPage:
     dim: int
     vdim: int
     itemsize: int
+    factors: bool = True
 
     @staticmethod
     def pad(n: int) -> int:
@@ -220,7 +222,7 @@ class KvPage:
 
     @property
     def v_offset(self) -> int:
-        return self.rms_offset + RMS_BYTES
+        return self.rms_offset + (RMS_BYTES if self.factors else 0)
 
     @property
     def nbytes(self) -> int:
@@ -271,14 +273,16 @@ def kv_pages(cfg, itemsize: int) -> Tuple[object, ...]:
     """Page layout of every KV cache of a design whose layers differ in size (one per execution of an attention layer)."""
     if isinstance(cfg, FetotarConfig):
         return tuple(LatentPage.of(layout_of(m), itemsize) for m in cfg.attn_mixers)
+    if isinstance(cfg, DeluvikConfig):
+        return tuple(KvPage(a.kv_heads, a.dim, a.vdim, itemsize, False) for a in map(cfg.attn, cfg.cache_owners))
     return tuple(KvPage(a.kv_heads, a.dim, a.vdim, itemsize)
                  for a in (cfg.layers[run.layer].mixer for run in cfg.runs))
 
 
 class PackedKvPool(PagedKvPool):
     """Paged pool whose caches may differ in head count and widths: cache ``i`` is a contiguous
-    ``[blocks, kv heads, page bytes]`` slice of one byte buffer (layout: :class:`KvPage`).  K is stored as
-    projected, with the norm's reciprocal root mean square beside it.  Allocator, reference counts and tier
+    ``[blocks, kv heads, page bytes]`` slice of one byte buffer (layouts: :class:`KvPage`, which may hold K as
+    projected with the norm's reciprocal root mean square beside it, and :class:`LatentPage`).  Allocator, reference counts and tier
     hooks are the parent's."""
     fp8 = False
 
@@ -385,10 +389,15 @@ class GdnStatePool:
         self.ring[slot].copy_(snap[1])
 
 
+def state_layouts(cfg) -> Tuple[object, ...]:
+    """What a design's layers keep per sequence beside keys and values, in the order of the states."""
+    return (deluvik_layout if isinstance(cfg, DeluvikConfig) else fetotar_layout).state_layouts(cfg)
+
+
 class RecurrentPool:
-    """State slots of decayed-scan layers that differ in form and size: ``states [slots, planes, floats]`` fp32, every
-    layer's record at a fixed offset (``fetotar_layout``: ``S [heads, dk, dv]``, then an mLSTM's key sum and running
-    maximum), and a ring ``[slots, rows, channels]`` of convolution inputs indexed by ``position % rows``.  ``planes`` and
+    """State slots of layers that differ in form and size: ``states [slots, planes, floats]`` fp32, every layer's record
+    at a fixed offset (``fetotar_layout``: ``S [heads, dk, dv]``, then an mLSTM's key sum and running maximum;
+    ``deluvik_layout``: a vector, or nothing where only a convolution's inputs are kept), and a ring ``[slots, rows, channels]`` of convolution inputs indexed by ``position % rows``.  ``planes`` and
     ``cur`` work as in :class:`GdnStatePool`."""
 
     def __init__(self, cfg: FetotarConfig, num_slots: int, device="cpu", planes: int = 1, ring_dtype=torch.bfloat16):
@@ -429,9 +438,11 @@ class RecurrentPool:
         return self.states[0].numel() * 4 + self.ring[0].numel() * self.ring.element_size()
 
     def view(self, idx: int, slot: int, plane: int) -> List[torch.Tensor]:
-        """The parts of one layer's state: ``S`` and, for an mLSTM, the copies of ``n`` and ``m``."""
+        """The parts of one layer's state: ``S`` and, for an mLSTM, the copies of ``n`` and ``m``; a vector for a linear recurrence."""
         l, o = self.layouts[idx], self.offsets[idx]
         rec = self.states[slot, plane, o:o + l.state_floats]
+        if l.kind == "lru":
+            return l.parts(rec)
         k = l.heads * l.dk * l.dv
         parts = [rec[:k].view(l.heads, l.dk, l.dv)]
         if l.kind == "mlstm":
@@ -458,7 +469,7 @@ class RecurrentPool:
 def make_state_pool(cfg, num_slots: int, device="cpu", *, planes: int = 1, ring_dtype=torch.bfloat16,
                     n_v_heads: Optional[int] = None, n_k_heads: Optional[int] = None):
     """The pool a configuration's recurrent layers keep their state in (it also hands out the slots of designs without any)."""
-    if isinstance(cfg, FetotarConfig):
+    if isinstance(cfg, (FetotarConfig, DeluvikConfig)):
         return RecurrentPool(cfg, num_slots, device, planes=planes, ring_dtype=ring_dtype)
     return GdnStatePool(cfg, num_slots, device, planes=planes, ring_dtype=ring_dtype, n_v_heads=n_v_heads, n_k_heads=n_k_heads)
 

@@ -17,7 +17,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
-from .config import FetotarConfig, ModelConfig, StreamDesign
+from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign
 from .formats import nbytes, weight_specs
 from .parallel.mesh import is_sharded, tp_dims
 
@@ -61,8 +61,8 @@ def kv_block_bytes(cfg: ModelConfig, tp: int = 1, fp8: bool = False) -> int:
 
 
 def state_slot_bytes(cfg: ModelConfig, tp: int = 1, planes: int = 1) -> int:
-    if isinstance(cfg, FetotarConfig):
-        from .fetotar_layout import state_layouts
+    if isinstance(cfg, (FetotarConfig, DeluvikConfig)):
+        from .kv import state_layouts
         return sum(planes * l.state_floats * 4 + 16 * l.conv_c * 2 for l in state_layouts(cfg))
     if not cfg.n_gdn_layers:
         return 0
@@ -106,6 +106,17 @@ def workspace_bytes(cfg: ModelConfig, tokens: int, tp: int = 1) -> int:
         per = stream_width(cfg) * (4 + 4 + 2) + 2 * max(l.n_in for l in ls) + 2 * max(l.n_out for l in ls) + 6 * glu + 2 * side_width(cfg)
         per += max([2 * l.heads * (l.dq + l.row + 2 * l.kv + l.dk + l.dv) for l in ls if l.kind == "latent"] + [0])
         per += max([4 * l.heads * l.dv + 2 * l.conv_c for l in ls if l.kind != "latent"] + [0])
+        return tokens * per + head_rows(cfg) * 4 * 64
+    if isinstance(cfg, DeluvikConfig):
+        from .deluvik_layout import MoeLayout, head_rows, layouts, pad, stream_width
+        from .mixers import MoeSpec
+        ls, w = layouts(cfg), stream_width(cfg)
+        moe = [MoeLayout(b.mlp) for b in cfg.layers if isinstance(b.mlp, MoeSpec)]
+        glu = max([pad(b.mlp.ff, 64) for b in cfg.layers if b.mlp is not None and not isinstance(b.mlp, MoeSpec)] + [0])
+        # fp32 stream and branch output, bf16 rounded row, fused projection rows, queries, mixer output, feed-forward; a
+        # recurrence's convolved rows and fp32 gates; of every used expert: the input row, the gated row, the fp32 output row
+        per = w * (4 + 4 + 2) + 2 * max(l.n_in for l in ls) + 2 * max(l.attn.k0 for l in ls) + 2 * max(l.n_out for l in ls) + 6 * glu
+        per += max([10 * l.lru.width for l in ls if l.lru] + [0]) + max([m.slots * (w * 6 + m.ff * 2) + 4 * m.router_rows for m in moe] + [0])
         return tokens * per + head_rows(cfg) * 4 * 64
     if isinstance(cfg, StreamDesign):
         from .zinutar_layout import BlockLayout, head_rows, stream_width

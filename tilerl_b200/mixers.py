@@ -6,7 +6,7 @@ dictionaries of a ``config.json``; a design's configuration lists them layer by 
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
+from dataclasses import asdict, dataclass, fields
 from typing import Dict, Optional, Tuple
 
 
@@ -41,11 +41,38 @@ class YarnSpec:
 
 
 @dataclass(frozen=True)
+class BandScalingSpec:
+    """Frequency scaling by wavelength bands: pairs that turn more than ``high`` times over ``original`` tokens keep their
+    frequency, those that turn less than ``low`` times are slowed down by ``factor``, a linear blend in the number of turns in
+    between."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def __post_init__(self) -> None:
+        _positive("rotary scaling", self.factor, self.low, self.high, self.original)
+        if self.high < self.low:
+            raise ValueError(f"rotary scaling: the bands overlap: {self}")
+
+    def apply(self, f: float) -> float:
+        turns = self.original * f / (2.0 * math.pi)
+        if turns > self.high:
+            return f
+        if turns < self.low:
+            return f / self.factor
+        keep = (turns - self.low) / (self.high - self.low) if self.high > self.low else 1.0
+        return (1.0 - keep) * f / self.factor + keep * f
+
+
+@dataclass(frozen=True)
 class RotarySpec:
-    """Rotation of the first ``dims`` dimensions in neighbouring pairs (2i, 2i + 1)."""
+    """Rotation of the first ``dims`` dimensions: in neighbouring pairs (2i, 2i + 1), or, with ``half``, of dimension i with
+    dimension i + dims / 2."""
     dims: int
     base: float
-    scaling: Optional[YarnSpec] = None
+    scaling: Optional[object] = None       # YarnSpec or BandScalingSpec
+    half: bool = False
 
     def __post_init__(self) -> None:
         if self.dims <= 0 or self.dims % 2 or self.base <= 1.0:
@@ -57,6 +84,8 @@ class RotarySpec:
         s = self.scaling
         if s is None:
             return tuple(plain)
+        if isinstance(s, BandScalingSpec):
+            return tuple(s.apply(f) for f in plain)
 
         def dim_of(turns: float) -> float:      # (real-valued) dimension whose pair turns this often over `original`
             return self.dims * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
@@ -69,24 +98,24 @@ class RotarySpec:
 
     @property
     def amplitude(self) -> float:
-        return 1.0 if self.scaling is None else 0.1 * math.log(self.scaling.factor) + 1.0
+        return 0.1 * math.log(self.scaling.factor) + 1.0 if isinstance(self.scaling, YarnSpec) else 1.0
 
     @classmethod
-    def from_json(cls, d: Dict, where: str) -> "RotarySpec":
+    def from_json(cls, d: Dict, where: str, scaling=YarnSpec, half: bool = False) -> "RotarySpec":
+        """``scaling``: the class of the design's frequency scaling (used where the dictionary has one)."""
         if "scaling" not in d or d["scaling"] is None:
             d = {k: v for k, v in d.items() if k != "scaling"}
             take(d, ("dims", "base"), where)
-            return cls(int(d["dims"]), float(d["base"]))
+            return cls(int(d["dims"]), float(d["base"]), None, half)
         take(d, ("dims", "base", "scaling"), where)
-        s = take(d["scaling"], ("factor", "original", "fast", "slow"), where + " scaling")
-        return cls(int(d["dims"]), float(d["base"]),
-                   YarnSpec(float(s["factor"]), float(s["original"]), float(s["fast"]), float(s["slow"])))
+        names = [f.name for f in fields(scaling)]
+        s = take(d["scaling"], names, where + " scaling")
+        return cls(int(d["dims"]), float(d["base"]), scaling(*(float(s[n]) for n in names)), half)
 
     def to_json(self) -> Dict:
         out: Dict = {"dims": self.dims, "base": self.base}
         if self.scaling is not None:
-            s = self.scaling
-            out["scaling"] = {"factor": s.factor, "original": s.original, "fast": s.fast, "slow": s.slow}
+            out["scaling"] = asdict(self.scaling)
         return out
 
 
@@ -190,6 +219,107 @@ class MlstmSpec:
 MIXERS = {c.type: c for c in (LatentAttnSpec, Mamba2Spec, MlstmSpec)}
 
 
+@dataclass(frozen=True)
+class SoftmaxAttnSpec:
+    """Causal softmax attention of ``heads`` query heads over ``kv_heads`` key / value heads (contiguous groups).  Queries and
+    keys are RMS-normalised with a weight, over the whole projection (``norm`` "all") or per head ("head"), then rotated.
+    Optional: a ``window`` (a query sees itself and the ``window - 1`` tokens before it), a soft cap on scores (``cap``), a
+    learned ``sink`` per head in the denominator, a short convolution of ``conv`` taps on every projection, values that are
+    the projected keys (``tied``), keys and values of an earlier layer (``kv_from``)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotarySpec
+    norm: str = "all"
+    window: Optional[int] = None
+    cap: Optional[float] = None
+    sink: bool = False
+    conv: int = 0
+    tied: bool = False
+    kv_from: Optional[int] = None
+
+    def __post_init__(self) -> None:
+        _positive("attention", self.heads, self.kv_heads, self.dim, self.vdim)
+        if self.heads % self.kv_heads:
+            raise ValueError(f"attention needs heads a multiple of kv_heads: {self}")
+        if self.rot.dims > self.dim:
+            raise ValueError("more rotated dimensions than a head has")
+        if self.norm not in ("all", "head") or self.conv < 0 or (self.window is not None and self.window < 1) or \
+                (self.cap is not None and self.cap <= 0):
+            raise ValueError(f"attention: {self}")
+        if self.tied and (self.dim != self.vdim or self.kv_from is not None):
+            raise ValueError("values that are the keys have their size and their layer")
+
+    @property
+    def channels(self) -> int:
+        """Columns of the layer's projections."""
+        own = 0 if self.kv_from is not None else self.kv_heads * (self.dim + (0 if self.tied else self.vdim))
+        return self.heads * self.dim + own
+
+    def same_keys(self, other: "SoftmaxAttnSpec") -> bool:
+        """The keys and values that ``other`` caches are what this layer reads."""
+        return (self.heads, self.kv_heads, self.dim, self.vdim, self.rot) == (other.heads, other.kv_heads, other.dim, other.vdim, other.rot)
+
+    @classmethod
+    def from_json(cls, m: Dict, where: str, *, norm: str, half: bool, capped: bool = False, windowed: bool = False, conv: bool = False,
+                  sink: bool = False, tied: bool = False) -> "SoftmaxAttnSpec":
+        """The keyword arguments say which of the optional parts the design's mixer has."""
+        m = dict(m)
+        source = m.pop("kv_from", None) if conv else None
+        take(m, ("heads", "kv_heads", "dim", "vdim", "scale", "rot") + capped * ("softcap",) + windowed * ("mask",) + conv * ("conv",), where)
+        if windowed:
+            take(m["mask"], ("size",), where + " mask")
+        return cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                   RotarySpec.from_json(m["rot"], where + " rot", BandScalingSpec, half), norm, int(m["mask"]["size"]) if windowed else None,
+                   float(m["softcap"]) if capped else None, sink, int(m["conv"]) if conv else 0, tied, None if source is None else int(source))
+
+    def to_json(self) -> Dict:
+        out: Dict = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale,
+                     "rot": self.rot.to_json()}
+        for name, value in (("softcap", self.cap), ("conv", self.conv or None), ("kv_from", self.kv_from),
+                            ("mask", None if self.window is None else {"size": self.window})):
+            if value is not None:
+                out[name] = value
+        return out
+
+
+@dataclass(frozen=True)
+class LruSpec:
+    """Gated linear recurrence of ``width`` channels (De et al., Griffin): a branch through a short convolution of ``conv``
+    taps whose two gates are block-diagonal maps (``blocks`` equal parts), times a gelu branch."""
+    width: int
+    blocks: int
+    conv: int
+
+    def __post_init__(self) -> None:
+        _positive("linear recurrence", self.width, self.blocks, self.conv)
+        if self.width % self.blocks:
+            raise ValueError(f"linear recurrence: the width must divide into the blocks: {self}")
+
+    @property
+    def part(self) -> int:
+        return self.width // self.blocks
+
+    @classmethod
+    def from_json(cls, m: Dict, where: str) -> "LruSpec":
+        take(m, ("width", "blocks", "conv"), where)
+        return cls(int(m["width"]), int(m["blocks"]), int(m["conv"]))
+
+    def to_json(self) -> Dict:
+        return asdict(self)
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same row: ``left_scale`` attention + ``right_scale`` recurrence."""
+    left: SoftmaxAttnSpec
+    right: LruSpec
+    left_scale: float
+    right_scale: float
+
+
 # ---- feed-forwards -----------------------------------------------------------------------------------------
 @dataclass(frozen=True)
 class ClampedGluSpec:
@@ -214,7 +344,60 @@ class ClampedGluSpec:
 
 
 @dataclass(frozen=True)
+class GluSpec:
+    """``W_down (act(W_gate h) * (W_up h))``."""
+    ff: int
+    act: str                  # "gelu" (its tanh form) or "silu"
+    kind = "dense"
+
+    def __post_init__(self) -> None:
+        _positive("feed-forward", self.ff)
+        if self.act not in ("gelu", "silu"):
+            raise ValueError(f"unknown activation {self.act!r}")
+
+    @classmethod
+    def from_json(cls, f: Dict, where: str, act: str) -> "GluSpec":
+        take(f, ("ff", "kind"), where)
+        return cls(int(f["ff"]), act)
+
+    def to_json(self) -> Dict:
+        return {"kind": self.kind, "ff": self.ff}
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    """``experts`` gated feed-forwards of width ``ff``, of which a token uses the ``top`` with the largest router logits, weighted
+    by the softmax over those; ``shared`` (0: none) is the width of one that every token uses."""
+    ff: int
+    experts: int
+    top: int
+    shared: int = 0
+    act: str = "silu"
+    kind = "moe"
+
+    def __post_init__(self) -> None:
+        _positive("experts", self.ff, self.experts, self.top)
+        if self.top > self.experts or self.shared < 0 or self.act not in ("gelu", "silu"):
+            raise ValueError(f"experts: {self}")
+
+    @classmethod
+    def from_json(cls, f: Dict, where: str) -> "MoeSpec":
+        f = take({"shared": None, **f}, ("kind", "expert", "router", "shared"), where)
+        take(f["expert"], ("ff",), where + " expert"), take(f["router"], ("experts", "top"), where + " router")
+        if f["shared"] is not None:
+            take(f["shared"], ("ff",), where + " shared")
+        return cls(int(f["expert"]["ff"]), int(f["router"]["experts"]), int(f["router"]["top"]),
+                   0 if f["shared"] is None else int(f["shared"]["ff"]))
+
+    def to_json(self) -> Dict:
+        out: Dict = {"kind": self.kind, "expert": {"ff": self.ff}, "router": {"experts": self.experts, "top": self.top}}
+        if self.shared:
+            out["shared"] = {"ff": self.shared}
+        return out
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One layer: a mixer and, unless ``mlp`` is None, a feed-forward after it."""
     mixer: object
-    mlp: Optional[ClampedGluSpec] = None
+    mlp: Optional[object] = None

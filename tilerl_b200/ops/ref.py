@@ -211,11 +211,12 @@ def rms_factor(x, n: int, eps: float):
 
 def packed_kv_write(cache, page, k, v, slot_mapping, eps: float):
     """Write rows ``k [T, hkv, dk]`` / ``v [T, hkv, dv]`` (padded widths) into a packed cache
-    ``[blocks, hkv, page bytes]``: K unnormalised with its reciprocal root mean square beside it."""
+    ``[blocks, hkv, page bytes]``: K unnormalised with its reciprocal root mean square beside it, or, in pages without
+    factors, as given."""
     el = cache.view(k.dtype)
     f32 = cache.view(torch.float32)
     ki, vi, ri = page.k_index().to(k.device), page.v_index().to(k.device), page.rms_index().to(k.device)
-    fac = rms_factor(k, page.dim, eps)
+    fac = rms_factor(k, page.dim, eps) if page.factors else None
     for t in range(k.shape[0]):
         s = int(slot_mapping[t])
         if s < 0:
@@ -223,7 +224,8 @@ def packed_kv_write(cache, page, k, v, slot_mapping, eps: float):
         b, o = divmod(s, KV_BLOCK)
         el[b][:, ki[o]] = k[t]
         el[b][:, vi[o]] = v[t]
-        f32[b, :, ri[o]] = fac[t]
+        if page.factors:
+            f32[b, :, ri[o]] = fac[t]
 
 
 def packed_kv_gather(cache, page, dtype, block_row, length: int):
@@ -233,8 +235,10 @@ def packed_kv_gather(cache, page, dtype, block_row, length: int):
     el, dev = pages.view(dtype), cache.device
     k = _f(el[..., page.k_index().to(dev)])                           # [nb, hkv, 16, dk]
     v = _f(el[..., page.v_index().to(dev)])
-    r = pages.view(torch.float32)[..., page.rms_index().to(dev)]      # [nb, hkv, 16]
     flat = lambda a: a.transpose(1, 2).reshape(nb * KV_BLOCK, a.shape[1], *a.shape[3:])[:length]
+    if not page.factors:
+        return flat(k), flat(v)
+    r = pages.view(torch.float32)[..., page.rms_index().to(dev)]      # [nb, hkv, 16]
     return flat(k) * flat(r)[..., None], flat(v)
 
 

@@ -1,6 +1,7 @@
-"""fp32 torch form of the stream designs' mechanisms (latent attention, decayed scans, norms, gates) and, on top of
-them, the op surface :class:`RefMixers` that ``models/fetotar.py`` calls; mixed into
-:class:`~tilerl_b200.ops.backend.RefOps`.  The CUDA twin is :mod:`tilerl_b200.ops.cuda_mixers`.  No counterpart in the
+"""fp32 torch form of the stream designs' mechanisms (latent and softmax attention, decayed scans, linear recurrence, experts,
+norms, gates) and, on top of them, the op surface :class:`RefMixers` that ``models/fetotar.py`` and ``models/deluvik.py`` call;
+mixed into :class:`~tilerl_b200.ops.backend.RefOps`.  The CUDA twins are :mod:`tilerl_b200.ops.cuda_mixers` and
+:mod:`tilerl_b200.ops.cuda_blocks`.  No counterpart in the
 reference.
 """
 from __future__ import annotations
@@ -50,6 +51,16 @@ def rotate_pairs(x, positions, freqs, amplitude: float):
     return out
 
 
+def rotate_halves(x, positions, freqs):
+    """Turn column i of ``x [T, ..., width]`` with column ``i + len(freqs)``; columns past ``2 len(freqs)`` stay."""
+    n = freqs.numel()
+    ang = positions.to(torch.float64)[:, None] * freqs.to(positions.device)[None, :]
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [n]
+    c, s = ang.cos().float().view(shape), ang.sin().float().view(shape)
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
 def latent_write(cache, page, rows, slot_mapping):
     """Cached rows ``[T, width]`` into ``cache [blocks, 1, page bytes]``."""
     el, idx = cache.view(rows.dtype), page.index().to(rows.device)
@@ -71,6 +82,47 @@ def latent_attention(q, rows, kv: int, scale: float):
     """One query token over the rows it sees: ``q [heads, kv + rd]`` (the unrotated part already mapped into the latent),
     ``rows [n, kv + rd]``; softmax-weighted sum of the latents ``[heads, kv]``."""
     return torch.softmax(q @ rows.t() * scale, dim=-1) @ rows[:, :kv]
+
+
+# ---- softmax attention over packed pages ----------------------------------------------------------------
+def soft_cap(z, cap: float):
+    return cap * torch.tanh(z / cap)
+
+
+def softmax_attention(q, k, v, scale: float, cap=None, sink=None):
+    """One query token over the keys it sees: ``q [heads, dk]``, ``k [n, kv_heads, dk]``, ``v [n, kv_heads, dv]``; ``sink
+    [heads]`` counts in the denominator only."""
+    hq, hkv = q.shape[0], k.shape[1]
+    s = torch.einsum("hgd,nhd->hgn", q.view(hkv, hq // hkv, -1), k) * scale
+    s = s if cap is None else soft_cap(s, cap)
+    if sink is not None:
+        s = torch.cat([s, sink.float().view(hkv, -1, 1)], -1)
+    p = torch.softmax(s, dim=-1)[..., :k.shape[0]]
+    return torch.einsum("hgn,nhd->hgd", p, v).reshape(hq, -1)
+
+
+def weighted_norm(x, heads: int, d: int, weight, whole: bool, eps: float):
+    """RMS norm of ``x [T, heads, dp]`` (``d`` true columns per head), over all heads at once or per head, times ``weight``."""
+    n = heads * d if whole else d
+    ss = x.pow(2).sum((-2, -1), keepdim=True) if whole else x.pow(2).sum(-1, keepdim=True)
+    return x * torch.rsqrt(ss / n + eps) * (weight.view(heads, -1) if whole else weight)
+
+
+# ---- linear recurrence, experts ---------------------------------------------------------------------------
+def lru_step(state, u, r, i, lam):
+    """``state, u [width]``, gate pre-activations ``r, i`` -> new state."""
+    log_a = -8.0 * torch.sigmoid(r) * F.softplus(lam)
+    return torch.exp(log_a) * state + torch.sqrt(-torch.expm1(2.0 * log_a)) * torch.sigmoid(i) * u
+
+
+def activate(z, act: str):
+    return gelu_tanh(z) if act == "gelu" else F.silu(z)
+
+
+def choose(logits, top: int):
+    """(experts ``[T, top]``, their weights): the largest logits (the first of equal ones), softmax over those."""
+    best, idx = torch.sort(logits, dim=1, descending=True, stable=True)
+    return idx[:, :top], torch.softmax(best[:, :top], dim=1)
 
 
 # ---- decayed scans ---------------------------------------------------------------------------------------
@@ -132,8 +184,17 @@ class RefMixers:
     def project_f32(self, a, w):
         return ref.linear(a, w)
 
-    def project_logits(self, h, w):
-        return ref.linear(h, w)
+    def project_logits(self, h, w, cap=0.0):
+        z = ref.linear(h, w)
+        return soft_cap(z, cap) if cap else z
+
+    def project(self, h, w):
+        return ref.linear(h, w).to(self.act_dtype)
+
+    def glu(self, h, w, act):
+        """Rows ``2j`` = gate, ``2j + 1`` = up of ``w``: ``act(gate) * up``."""
+        gu = ref.linear(h, w)
+        return (activate(gu[:, 0::2], act) * gu[:, 1::2]).to(self.act_dtype)
 
     def clamped_glu(self, h, w, limit):
         return clamped_glu(ref.linear(h, w), limit).to(self.act_dtype)
@@ -174,6 +235,84 @@ class RefMixers:
             o = torch.einsum("hc,hdc->hd", latent_attention(ql[i], rows, l.kv, l.scale), uv).reshape(-1)
             out[i, :l.heads * l.dv] = (o * torch.sigmoid(proj[i, l.g0:l.n_in].float())).to(self.act_dtype)
         return out
+
+    # ---- softmax attention ---------------------------------------------------------------
+    def _conv_inputs(self, row, ring, pos: int, taps: int):
+        """The last ``taps`` inputs (oldest first) of one sequence's convolution, ``row`` included; it goes into the ring."""
+        ring[pos % ring.shape[0]] = row.to(ring.dtype)
+        zero = torch.zeros_like(row, dtype=torch.float32)
+        return torch.stack([ring[(pos - j) % ring.shape[0]].float() if pos >= j else zero for j in range(taps - 1, -1, -1)])
+
+    def attn_prep(self, proj, l, w, freqs, batch, pool, idx, spool, sidx, eps):
+        """Convolved, normed and turned queries ``[T, heads, dk]``; keys and values of layers that have their own into the
+        cache.  Also the (zeroed) input of the layer's output projection."""
+        a, s, t = l.attn, l.attn.spec, proj.shape[0]
+        rows = proj[:, :a.n_in].float()
+        if s.conv:
+            rows = torch.stack([(self._conv_inputs(proj[i, :a.n_in], spool.ring_view(sidx, int(batch.state_slots[int(batch.seq_ids[i])])),
+                                                   int(batch.positions[i]), s.conv) * w["conv"]).sum(0) for i in range(t)])
+        turn = rotate_halves if s.rot.half else lambda x, p, f: rotate_pairs(x, p, f, 1.0)
+        q = weighted_norm(rows[:, :a.k0].view(t, s.heads, a.dk), s.heads, s.dim, w["q_norm"], s.norm == "all", eps)
+        if a.own:
+            k = rows[:, a.k0:a.k0 + s.kv_heads * a.dk].view(t, s.kv_heads, a.dk)
+            v = rows[:, a.v0:a.v0 + s.kv_heads * a.dv].view(t, s.kv_heads, a.dv)
+            k = turn(weighted_norm(k, s.kv_heads, s.dim, w["k_norm"], s.norm == "all", eps), batch.positions, freqs)
+            ref.packed_kv_write(pool.layer(idx), pool.pages[idx], k.to(pool.dtype), v.to(pool.dtype), batch.slot_mapping, eps)
+        return turn(q, batch.positions, freqs).to(self.act_dtype), torch.zeros(t, l.n_out, dtype=self.act_dtype, device=proj.device)
+
+    def softmax_attention(self, q, mid, a, sink, factor, batch, pool, idx):
+        """Attention output of every token, times ``factor``, into the first columns of ``mid``."""
+        s = a.spec
+        for i in range(q.shape[0]):
+            p = int(batch.positions[i])
+            k, v = ref.packed_kv_gather(pool.layer(idx), pool.pages[idx], pool.dtype, batch.block_table[int(batch.seq_ids[i])], p + 1)
+            lo = 0 if s.window is None else max(0, p + 1 - s.window)
+            o = softmax_attention(q[i].float(), k[lo:], v[lo:], s.scale, s.cap, sink)
+            mid[i, :a.n_out] = (o * factor).reshape(-1).to(self.act_dtype)
+
+    # ---- gated linear recurrence -----------------------------------------------------------
+    def lru_mix(self, proj, mid, l, w, batch, spool, sidx):
+        """Recurrence x gelu branch, times the layer's factor, into the columns of ``mid`` behind the attention's."""
+        r, t, y0 = l.lru, proj.shape[0], l.attn.n_in
+        y = gelu_tanh(proj[:, y0:y0 + r.width].float() + w["y_b"])
+        for q in range(batch.n_seqs):
+            s0, n, slot = int(batch.q_start[q]), int(batch.q_len[q]), int(batch.state_slots[q])
+            if n == 0:
+                continue
+            keep = bool(batch.keep_steps) and batch.keep_rows[q]
+            live = spool.view(sidx, slot, int(spool.cur[slot]))[0]
+            state = live.clone()
+            for i in range(s0, s0 + n):
+                pos = int(batch.positions[i])
+                rows = self._conv_inputs(proj[i, y0 + r.width:y0 + 2 * r.width], spool.ring_view(sidx, slot), pos, r.spec.conv)
+                rows[max(0, r.spec.conv - 1 - pos):] += w["x_b"]         # zeros before the start carry no bias
+                u = ((rows * w["lru_conv"]).sum(0) + w["lru_conv_b"]).to(self.act_dtype).float()
+                z = torch.einsum("bk,bjk->bj", u.view(r.spec.blocks, r.pp), w["gates"].float()) + w["gates_b"]
+                state = lru_step(state, u, z[:, :r.pp].reshape(-1), z[:, r.pp:].reshape(-1), w["lam"])
+                mid[i, l.attn.n_out:l.n_mid] = (state * y[i] * l.lru_scale).to(self.act_dtype)
+                if keep:
+                    spool.view(sidx, slot, i - s0)[0].copy_(state)
+            if not keep:
+                live.copy_(state)
+
+    # ---- experts -----------------------------------------------------------------------------
+    def experts(self, h, router, router_b, gate_up, down, m):
+        """Weighted sum of the experts' outputs (the CUDA backend leaves the sum to :meth:`join_experts`)."""
+        z = (ref.linear(h, router) + router_b)[:, :m.spec.experts]
+        idx, weight = choose(z, m.spec.top)
+        y = torch.zeros(h.shape[0], down.shape[1], dtype=torch.float32, device=h.device)
+        for e in range(m.n):
+            if e < m.spec.experts:
+                rows, place = torch.nonzero(idx == e, as_tuple=True)
+                scale = weight[rows, place][:, None]
+            else:
+                rows, scale = torch.arange(h.shape[0], device=h.device), 1.0
+            if len(rows):
+                y[rows] += scale * ref.linear(self.glu(h[rows], gate_up[e], m.spec.act), down[e])
+        return y
+
+    def join_experts(self, x, y, post, nxt, eps, n):
+        return self.join(x, y, post, nxt, eps, n)
 
     # ---- recurrent mixers ------------------------------------------------------------------
     def recurrent_mix(self, proj, gates, w, l, batch, pool, idx, eps):
