@@ -48,7 +48,8 @@ __device__ __forceinline__ void trl_set_error(int code, int a, int b, int c) {
 // compiles to the bare index.  Sites: 1 KV slot of a token (attn_prep), 2 block-table entry in decode
 // attention, 3 block-table entry in prefill attention, 4 KV slot in the one-launch decode attention, 5 KV slot in the
 // block middle of packed pools, 6 / 7 block-table entry in sigmoid attention (bf16 / fp32), 8 token id of a stream start, 9 KV slot of a
-// cached latent, 10 / 11 / 12 block-table entry in latent attention (plain, decode, gather of a prompt).
+// cached latent, 10 / 11 / 12 block-table entry in latent attention (plain, decode, gather of a prompt), 13 KV slot in the
+// preparation of softmax attention, 14 / 15 its block-table entry (tensor cores, CUDA cores).
 #ifdef TRL_DEBUG_BOUNDS
 __device__ __forceinline__ int trl_checked(int i, int n, int site) {
   if ((unsigned)i >= (unsigned)n) {

@@ -3,7 +3,10 @@
 //   join_kernel       x += norm_post(y) and h = norm_next(x) in the next projection's input type, a row per block; each
 //                     norm is a layer norm (weight and bias), an RMS norm (weight) or, for h, nothing but the rounding.
 //                     With a table it starts the stream instead: x = table[id] * scale.
-//   glu_kernel        g sigmoid(1.702 g) (u + 1) over interleaved (gate, up) columns, gate bounded above, up on both sides.
+//                     The branch may also come as the rows of a token's experts, summed with their weights.
+//   glu_kernel        act(g) u over interleaved (gate, up) columns: silu, gelu (tanh form), or g sigmoid(1.702 g) (u + 1) with
+//                     the gate bounded above, up on both sides.
+//   cap_kernel        cap tanh(x / cap), in place.
 //   side_kernel       gelu(z) * side[token, layer].
 //
 // Rows are `ld` wide (a multiple of 64) with zeros past the model width `n`: weights and biases are zero there.
@@ -50,7 +53,8 @@ __device__ __forceinline__ float4 apply_norm(const float4& v, const float2& st, 
 template <typename T, int R>
 __global__ void __launch_bounds__(512)
 join_kernel(float* x, const float* y, const float* __restrict__ post, int post_kind, const float* __restrict__ next, int next_kind,
-            T* h, const T* __restrict__ table, const int* ids, float scale, int V, int ld, int n, float eps) {
+            T* h, const T* __restrict__ table, const int* ids, float scale, int V, int ld, int n, float eps, const int* place,
+            const float* weight, int slots) {
   __shared__ float red[32];
   pdl_launch_dependents(30);
   pdl_wait();
@@ -74,13 +78,25 @@ join_kernel(float* x, const float* y, const float* __restrict__ post, int post_k
       }
     }
   } else {
-    const float* yr = y + (size_t)t * ld;
     float4 xv[R];
+    const int parts = slots ? slots : 1;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       const int k = (threadIdx.x + i * blockDim.x) * 4;
       v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (k < ld) v[i] = load4(yr + k), xv[i] = load4(xr + k);
+      if (k < ld) xv[i] = load4(xr + k);
+    }
+    for (int j = 0; j < parts; ++j) {        // rows y[place[t, j]], weighted; without slots the token's own row
+      const float wj = slots ? weight[(size_t)t * slots + j] : 1.f;
+      const float* yr = y + (size_t)(slots ? place[(size_t)t * slots + j] : t) * ld;
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int k = (threadIdx.x + i * blockDim.x) * 4;
+        if (k < ld) {
+          const float4 a = load4(yr + k);
+          v[i].x = fmaf(wj, a.x, v[i].x), v[i].y = fmaf(wj, a.y, v[i].y), v[i].z = fmaf(wj, a.z, v[i].z), v[i].w = fmaf(wj, a.w, v[i].w);
+        }
+      }
     }
     const float2 st = row_stats<R>(v, post_kind, n, eps, red);
 #pragma unroll
@@ -107,7 +123,7 @@ join_kernel(float* x, const float* y, const float* __restrict__ post, int post_k
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) glu_kernel(const T* gu, T* out, long n4, float limit) {
+__global__ void __launch_bounds__(256) glu_kernel(const T* gu, T* out, long n4, int act, float limit) {
   pdl_launch_dependents(31);
   pdl_wait();
   for (long i = blockIdx.x * 256L + threadIdx.x; i < n4; i += (long)gridDim.x * 256) {      // 4 outputs from 8 inputs
@@ -115,11 +131,18 @@ __global__ void __launch_bounds__(256) glu_kernel(const T* gu, T* out, long n4, 
     const float g[4] = {a.x, a.z, b.x, b.z}, u[4] = {a.y, a.w, b.y, b.w};
     float o[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float gg = fminf(g[e], limit), uu = fminf(fmaxf(u[e], -limit), limit);
-      o[e] = gg * sigmoid_f(1.702f * gg) * (uu + 1.f);
-    }
+    for (int e = 0; e < 4; ++e) o[e] = glu_x(g[e], u[e], act, limit);
     store4<T>(out + i * 4, o[0], o[1], o[2], o[3]);
+  }
+}
+
+__global__ void __launch_bounds__(256) cap_kernel(float4* x, long n4, float cap) {
+  pdl_launch_dependents(33);
+  pdl_wait();
+  for (long i = blockIdx.x * 256L + threadIdx.x; i < n4; i += (long)gridDim.x * 256) {
+    float4 v = x[i];
+    v.x = cap * tanhf(v.x / cap), v.y = cap * tanhf(v.y / cap), v.z = cap * tanhf(v.z / cap), v.w = cap * tanhf(v.w / cap);
+    x[i] = v;
   }
 }
 
@@ -139,11 +162,13 @@ side_kernel(const T* z, const T* __restrict__ side, const int* ids, T* out, int 
 
 template <typename T>
 cudaError_t join_launch(void* x, const void* y, const void* post, int pk, const void* next, int nk, void* h, const void* table,
-                        const void* ids, float scale, int V, int T_, int ld, int n, float eps, cudaStream_t st) {
+                        const void* ids, float scale, int V, int T_, int ld, int n, float eps, const void* place, const void* weight,
+                        int slots, cudaStream_t st) {
   const int thr = ld >= 2048 ? 512 : (ld >= 1024 ? 256 : 128), need = (ld / 4 + thr - 1) / thr;
 #define JOIN(R)                                                                                                            \
   return trl_launch(join_kernel<T, R>, dim3(T_), dim3(thr), 0, st, (float*)x, (const float*)y, (const float*)post, pk,     \
-                    (const float*)next, nk, (T*)h, (const T*)table, (const int*)ids, scale, V, ld, n, eps)
+                    (const float*)next, nk, (T*)h, (const T*)table, (const int*)ids, scale, V, ld, n, eps,                 \
+                    (const int*)place, (const float*)weight, slots)
   if (need <= 1) JOIN(1);
   if (need <= 2) JOIN(2);
   if (need <= 4) JOIN(4);
@@ -162,17 +187,34 @@ TRL_API int trl_join(void* x, const void* y, const void* post, int post_kind, co
       next_kind < 0 || next_kind > 2 || (next_kind && !next) || (table && !ids))
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
-  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, st)
-                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, st));
+  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, st)
+                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, st));
 }
 
-// gu: rows of 2 ff interleaved (gate, up) columns; out: rows of ff; n_out = rows * ff, a multiple of 4.
-TRL_API int trl_clamped_glu(const void* gu, void* out, long n_out, float limit, int f32, void* stream) {
-  if (n_out <= 0 || n_out % 4) return (int)cudaErrorInvalidValue;
+// The same with the branch of token t given as sum_j weight[t, j] y[place[t, j]] over `slots` rows.
+TRL_API int trl_join_experts(void* x, const void* y, const void* place, const void* weight, int slots, const void* post, int post_kind,
+                             const void* next, int next_kind, void* h, int T, int ld, int n, float eps, int f32, void* stream) {
+  if (T <= 0 || ld % 64 || ld > 16384 || n <= 0 || n > ld || !y || !post || !place || !weight || slots <= 0 || post_kind < 1 || post_kind > 2 ||
+      next_kind < 0 || next_kind > 2 || (next_kind && !next))
+    return (int)cudaErrorInvalidValue;
+  cudaStream_t st = (cudaStream_t)stream;
+  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, st)
+                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, st));
+}
+
+// x: n fp32 values, n a multiple of 4.
+TRL_API int trl_soft_cap(void* x, long n, float cap, void* stream) {
+  if (n <= 0 || n % 4 || !(cap > 0.f)) return (int)cudaErrorInvalidValue;
+  return (int)trl_launch(cap_kernel, dim3((int)min((n / 4 + 255) / 256, 148L * 16)), dim3(256), 0, (cudaStream_t)stream, (float4*)x, n / 4, cap);
+}
+
+// gu: rows of 2 ff interleaved (gate, up) columns; out: rows of ff; n_out = rows * ff, a multiple of 4.  act: GLU_* of packed.cuh.
+TRL_API int trl_glu(const void* gu, void* out, long n_out, int act, float limit, int f32, void* stream) {
+  if (n_out <= 0 || n_out % 4 || act < GLU_CLAMPED || act > GLU_GELU) return (int)cudaErrorInvalidValue;
   const int grid = (int)min((n_out / 4 + 255) / 256, 148L * 16);
   if (f32)
-    return (int)trl_launch(glu_kernel<float>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, (const float*)gu, (float*)out, n_out / 4, limit);
-  return (int)trl_launch(glu_kernel<bf16>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, (const bf16*)gu, (bf16*)out, n_out / 4, limit);
+    return (int)trl_launch(glu_kernel<float>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, (const float*)gu, (float*)out, n_out / 4, act, limit);
+  return (int)trl_launch(glu_kernel<bf16>, dim3(grid), dim3(256), 0, (cudaStream_t)stream, (const bf16*)gu, (bf16*)out, n_out / 4, act, limit);
 }
 
 // z, out: [T, width]; side: [V, ld_side], the layer's share in columns off .. off + dim - 1.

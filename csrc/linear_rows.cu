@@ -3,7 +3,7 @@
 //   y[m, n] (store bf16 | store fp32 | += fp32) = sum_k x'[m, k] * W[n, k]
 //
 // or, in the epilogue, rows n >= n_split stored in fp32 beside the bf16 ones (gates of a recurrence), pairs of rows (gate, up)
-// joined to g sigmoid(1.702 g) (u + 1) with clamps, or gelu(y) times a token's side-embedding row.
+// joined by a gated activation, the soft cap of logits, or gelu(y) times a token's side-embedding row.
 // x' is the row itself (bf16) or rms(x) * norm_w of an fp32 stream row, rounded to bf16.  The weights are streamed
 // once: a warp owns 16 weight rows and a share of K, and every lane copies the 16-byte pieces it will itself feed to
 // mma.sync (8 consecutive k of rows g and g + 8 per 32-wide step) into its own slots of a shared-memory ring, so no
@@ -25,7 +25,9 @@ enum { LR_STORE = 0, LR_STORE_F32 = 1, LR_ADD_F32 = 2, LR_GLU = 3, LR_SIDE = 4 }
 struct LrExtra {
   float* y2;                                                   // LR_STORE: fp32 rows n >= n_split
   int ldy2, n_split;
-  float limit;                                                 // LR_GLU
+  int act;                                                     // LR_GLU
+  float limit;
+  float cap;                                                   // LR_STORE_F32: cap tanh(y / cap) (0: y)
   const int* ids;                                              // LR_SIDE: side[id * ld_side + off + n] for n < dim, 0 past it
   const bf16* side;
   long ld_side;
@@ -162,8 +164,7 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
       if (n >= N) continue;
       const float v = total(m, c);
       if (EPI == LR_GLU) {
-        const float g = fminf(v, ex.limit), u = fminf(fmaxf(total(m, c + 1), -ex.limit), ex.limit);
-        reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n / 2] = __float2bfloat16(g * sigmoid_f(1.702f * g) * (u + 1.f));
+        reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n / 2] = __float2bfloat16(glu_x(v, total(m, c + 1), ex.act, ex.limit));
       } else if (EPI == LR_SIDE) {
         const int id = ex.ids[m];
         float o = 0.f;
@@ -172,7 +173,7 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
       } else if (EPI == LR_STORE && n >= ex.n_split) {
         ex.y2[(size_t)m * ex.ldy2 + n - ex.n_split] = v;
       } else if (EPI == LR_STORE) reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(v);
-      else if (EPI == LR_STORE_F32) reinterpret_cast<float*>(y)[(size_t)m * ldy + n] = v;
+      else if (EPI == LR_STORE_F32) reinterpret_cast<float*>(y)[(size_t)m * ldy + n] = ex.cap > 0.f ? ex.cap * tanhf(v / ex.cap) : v;
       else reinterpret_cast<float*>(y)[(size_t)m * ldy + n] += v;
     }
     __syncthreads();
@@ -253,11 +254,20 @@ TRL_API int trl_linear_rows_split(const void* x, int ldx, const void* w, void* y
   return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_STORE, ex, stream);
 }
 
-// w: rows 2j = gate_j, 2j + 1 = up_j; y: bf16 [M, N / 2].
-TRL_API int trl_linear_rows_glu(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, float limit, void* stream) {
-  if (N % 2) return (int)cudaErrorInvalidValue;
+// y[m, n] = cap tanh((x W^T) / cap) in fp32.
+TRL_API int trl_linear_rows_cap(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, float cap, void* stream) {
+  if (!(cap > 0.f)) return (int)cudaErrorInvalidValue;
   LrExtra ex = {};
-  ex.limit = limit;
+  ex.cap = cap;
+  return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_STORE_F32, ex, stream);
+}
+
+// w: rows 2j = gate_j, 2j + 1 = up_j; y: bf16 [M, N / 2].  act: GLU_* of packed.cuh.
+TRL_API int trl_linear_rows_glu(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int act, float limit,
+                                void* stream) {
+  if (N % 2 || act < GLU_CLAMPED || act > GLU_GELU) return (int)cudaErrorInvalidValue;
+  LrExtra ex = {};
+  ex.act = act, ex.limit = limit;
   return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_GLU, ex, stream);
 }
 

@@ -1,0 +1,8 @@
+// What the expert kernels share (moe.cu, moe_tc.cu).
+#pragma once
+#include "packed.cuh"
+
+// One tile of rows of an expert: rows [row0, row0 + n) of the list ordered by expert.
+struct MoeItem {
+  int expert, row0, n, pad;
+};

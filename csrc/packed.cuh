@@ -63,6 +63,15 @@ __device__ __forceinline__ float gelu_tanh_x(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+// gated feed-forwards: act(g) combined with u
+enum { GLU_CLAMPED = 0, GLU_SILU = 1, GLU_GELU = 2 };
+__device__ __forceinline__ float glu_x(float g, float u, int act, float limit) {
+  if (act == GLU_SILU) return g * sigmoid_f(g) * u;
+  if (act == GLU_GELU) return gelu_tanh_x(g) * u;
+  const float gg = fminf(g, limit), uu = fminf(fmaxf(u, -limit), limit);
+  return gg * sigmoid_f(1.702f * gg) * (uu + 1.f);
+}
+
 // cos and sin of position x frequency, times amp; the angle is formed and reduced in fp64
 __device__ __forceinline__ void pair_angle(int pos, double freq, float amp, float& c, float& s) {
   const double a = (double)pos * freq;

@@ -6,7 +6,9 @@
 //             m_t = max(f + m_(t-1), i), keep = exp(f + m_(t-1) - m_t), add = exp(i - m_t); beside S the sum n of the keys,
 //             and o is divided by max(|n . q|, exp(-m)) + 1e-6; then RMS norm per head, weight, sigmoid gate.
 //
-//   scan_conv_kernel    convolution + silu of a tick's rows; rows before the tick's first token come from the slot's ring.
+//   scan_conv_kernel    convolution of a tick's rows (with or without silu, inputs with or without a bias); rows before the tick's
+//                       first token come from the slot's ring.
+//   ring_store_kernel   a tick's last convolution inputs into the ring.
 //   scan_serial_kernel  token after token, 32 value columns of a head per block, the state in registers: decoding, windows of
 //                       kept states, short portions, and fp32 models.
 //   scan_norm_kernel    the norm and gates behind the scan; puts the tick's last convolution inputs into the ring.
@@ -23,9 +25,9 @@ namespace {
 // thread = one chunk of channels of one token
 template <typename T>
 __global__ void __launch_bounds__(128)
-scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const float* __restrict__ bias, const T* ring, long ring_slot,
-                 int ring_rows, int ring_ld, const int* positions, const int* seq_ids, const int* q_start, const int* slots, T* out,
-                 int channels, int taps) {
+scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ pre,
+                 const T* ring, long ring_slot, int ring_rows, int ring_ld, const int* positions, const int* seq_ids,
+                 const int* q_start, const int* slots, T* out, int channels, int taps, int silu) {
   constexpr int C = Chunk<T>::N;
   pdl_launch_dependents(40);
   pdl_wait();
@@ -45,6 +47,10 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
     const T* src = t - back >= t0 ? proj + (size_t)(t - back) * ldp + c : rg + (size_t)((pos - back) % ring_rows) * ring_ld + c;
     float f[C];
     Chunk<T>::get(*reinterpret_cast<const uint4*>(src), f);
+    if (pre) {
+#pragma unroll
+      for (int e = 0; e < C; ++e) f[e] += pre[c + e];
+    }
 #pragma unroll
     for (int e = 0; e < C; e += 4) {
       const float4 b = *reinterpret_cast<const float4*>(w + (size_t)j * channels + c + e);
@@ -52,9 +58,24 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
       acc[e + 2] = fmaf(f[e + 2], b.z, acc[e + 2]), acc[e + 3] = fmaf(f[e + 3], b.w, acc[e + 3]);
     }
   }
+  if (silu) {
 #pragma unroll
-  for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
+    for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
+  }
   *reinterpret_cast<uint4*>(out + (size_t)t * channels + c) = Chunk<T>::put(acc);
+}
+
+// one block per token: its row into the ring unless later ones of the tick would overwrite it
+__global__ void __launch_bounds__(128)
+ring_store_kernel(const unsigned char* rows, long ld, unsigned char* ring, long ring_slot, int ring_rows, long ring_ld, int chunks,
+                  const int* positions, const int* seq_ids, const int* q_start, const int* q_len, const int* slots) {
+  pdl_launch_dependents(43);
+  pdl_wait();
+  const int t = blockIdx.x, seq = seq_ids[t], left = q_start[seq] + q_len[seq] - 1 - t;
+  if (left < 0 || left >= ring_rows) return;
+  const uint4* src = reinterpret_cast<const uint4*>(rows + (size_t)t * ld);
+  uint4* dst = reinterpret_cast<uint4*>(ring + (size_t)slots[seq] * ring_slot + (size_t)(positions[t] % ring_rows) * ring_ld);
+  for (int c = threadIdx.x; c < chunks; c += 128) dst[c] = src[c];
 }
 
 // grid (heads * column slices, sequences), 256 threads: lane = column, warp = dk / 8 state rows.  CONV: one token per
@@ -316,10 +337,23 @@ cudaError_t serial_launch(const ScanArgs& a, int B, cudaStream_t st) {
 
 }  // namespace
 
-// proj: rows whose first `channels` columns are convolved; w: [taps, channels]; ring: the layer's first column of slot 0.
-TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* bias, const void* ring, long ring_slot, int ring_rows,
-                          int ring_ld, const void* positions, const void* seq_ids, const void* q_start, const void* slots, void* out,
-                          int T, int channels, int taps, int f32, void* stream) {
+// The last rows of every sequence's tick into its ring: `channels` columns from rows (leading dimension ld, bytes per value: item).
+TRL_API int trl_ring_store(const void* rows, int ld, void* ring, long ring_slot, int ring_rows, int ring_ld, int channels, const void* positions,
+                           const void* seq_ids, const void* q_start, const void* q_len, const void* slots, int T, int f32, void* stream) {
+  const int item = f32 ? 4 : 2, per = 16 / item;
+  if (T <= 0 || channels <= 0 || channels % per || ld % per || ring_ld % per || ring_slot % per || ring_rows <= 0 || ((uintptr_t)ring & 15) ||
+      ((uintptr_t)rows & 15))
+    return (int)cudaErrorInvalidValue;
+  return (int)trl_launch(ring_store_kernel, dim3(T), dim3(128), 0, (cudaStream_t)stream, (const unsigned char*)rows, (long)ld * item,
+                         (unsigned char*)ring, ring_slot * item, ring_rows, (long)ring_ld * item, channels / per, (const int*)positions,
+                         (const int*)seq_ids, (const int*)q_start, (const int*)q_len, (const int*)slots);
+}
+
+// proj: rows whose first `channels` columns are convolved; w: [taps, channels]; pre (or null): bias of the inputs, which zeros before
+// a sequence's start do not get; ring: the layer's first column of slot 0.
+TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* bias, const void* pre, const void* ring, long ring_slot,
+                          int ring_rows, int ring_ld, const void* positions, const void* seq_ids, const void* q_start, const void* slots,
+                          void* out, int T, int channels, int taps, int silu, int f32, void* stream) {
   const int per = f32 ? 4 : 8;
   if (T <= 0 || channels <= 0 || channels % 16 || taps < 1 || taps > ring_rows || ldp % per || ring_ld % per || ring_slot % per ||
       ((uintptr_t)ring & 15) || ((uintptr_t)proj & 15))
@@ -327,11 +361,11 @@ TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* 
   const dim3 grid(T, (channels / per + 127) / 128);
   if (f32)
     return (int)trl_launch(scan_conv_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, (const float*)proj, ldp, (const float*)w,
-                           (const float*)bias, (const float*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,
-                           (const int*)seq_ids, (const int*)q_start, (const int*)slots, (float*)out, channels, taps);
+                           (const float*)bias, (const float*)pre, (const float*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,
+                           (const int*)seq_ids, (const int*)q_start, (const int*)slots, (float*)out, channels, taps, silu);
   return (int)trl_launch(scan_conv_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, (const bf16*)proj, ldp, (const float*)w,
-                         (const float*)bias, (const bf16*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,
-                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (bf16*)out, channels, taps);
+                         (const float*)bias, (const float*)pre, (const bf16*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,
+                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (bf16*)out, channels, taps, silu);
 }
 
 // kind 0: Mamba-2, 1: mLSTM.  args: a ScanArgs (scan.cuh) filled by the caller.  Serves sequences of min_len..max_len tokens.

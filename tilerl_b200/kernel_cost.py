@@ -15,7 +15,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Dict, List, Optional
 
-from .config import ATTN, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig
+from .config import ATTN, DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig
 from .formats import FORMATS, nbytes
 from .parallel.mesh import tp_dims
 
@@ -101,12 +101,45 @@ def _fetotar_rows(cfg: FetotarConfig, m: int, ctx: int, n_seqs: int, head_rows_m
     return rows
 
 
+def _deluvik_rows(cfg: DeluvikConfig, m: int, ctx: int, n_seqs: int, head_rows_m: int) -> List[Row]:
+    """One forward of ``m`` tokens in ``n_seqs`` sequences that end at ``ctx`` tokens each."""
+    from .deluvik_layout import MoeLayout, head_rows, layouts, pad, stream_width
+    from .mixers import MoeSpec
+    w, q = stream_width(cfg), m // n_seqs
+    lin = lambda name, n, k, out=2: Row(name, 1, n * k * 2 + m * (k * 2 + n * out), 2.0 * m * n * k)
+    rows = [Row("embedding", 1, m * w * (2 + 4 + 2), 0)]
+    for i, (b, l) in enumerate(zip(cfg.layers, layouts(cfg))):
+        a, s = l.attn, l.attn.spec
+        win = s.window or ctx
+        seen = sum(min(p + 1, win) for p in range(ctx - q, ctx))                 # (query, key) pairs of one sequence
+        keys = min(ctx, q + win - 1)
+        rows += [lin(f"L{i} in", l.n_in, w), Row(f"L{i} attn.prep (norm, rotation, cache)", 1, m * a.n_in * 4.0, 0),
+                 Row(f"L{i} attn.softmax", 1, n_seqs * keys * s.kv_heads * (a.dk + a.dv) * 2 + m * s.heads * (a.dk + a.dv) * 2.0,
+                     2.0 * n_seqs * seen * s.heads * (a.dk + a.dv))]
+        if l.lru is not None:
+            r = l.lru
+            gates = r.spec.blocks * 2 * r.pp * r.pp
+            rows.append(Row(f"L{i} lru (gates, scan)", 1, gates * 2 + n_seqs * r.width * 8 + m * r.width * 6.0, 2.0 * m * gates))
+        rows += [lin(f"L{i} o", w, l.n_out, 4), Row(f"L{i} joins", 1 + (b.mlp is not None), m * w * (4 + 8 + 2.0), 0)]
+        if isinstance(b.mlp, MoeSpec):
+            e = MoeLayout(b.mlp)
+            used = e.pieces + e.spec.experts * (1.0 - (1.0 - e.spec.top / e.spec.experts) ** m)     # experts some token chooses
+            rows.append(lin(f"L{i} router", e.router_rows, w, 4))
+            for name, n, k, out in (("up", 2 * e.ff, w, 1), ("down", w, e.ff, 4)):
+                rows.append(Row(f"L{i} experts {name}", 1, used * n * k * 2 + m * e.slots * (k * 2 + n * out), 2.0 * m * e.slots * n * k))
+        elif b.mlp is not None:
+            ff = pad(b.mlp.ff, 64)
+            rows += [lin(f"L{i} gate_up", 2 * ff, w), lin(f"L{i} down", w, ff, 4)]
+    rows.append(Row("lm_head", 1, head_rows(cfg) * w * 2 + head_rows_m * (w * 2 + head_rows(cfg) * 4), 2.0 * head_rows_m * head_rows(cfg) * w))
+    return rows
+
+
 def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
     """One decode (or verify) tick on one TP rank."""
     if isinstance(cfg, StreamDesign):
         b, c = s.batch, s.ctx
-        if isinstance(cfg, FetotarConfig):
-            return _fetotar_rows(cfg, b * s.width, c, b, b * s.width)
+        if isinstance(cfg, (FetotarConfig, DeluvikConfig)):
+            return (_fetotar_rows if isinstance(cfg, FetotarConfig) else _deluvik_rows)(cfg, b * s.width, c, b, b * s.width)
         return _zinutar_rows(cfg, b * s.width, b * s.width * c, b * c, b * s.width)
     d = tp_dims(cfg, s.tp)
     m = s.batch * s.width
@@ -144,6 +177,8 @@ def prefill_rows(cfg: ModelConfig, tokens: int, tp: int = 1, terms: int = 2) -> 
     activation terms per token multiply the tensor-core work."""
     if isinstance(cfg, FetotarConfig):
         return _fetotar_rows(cfg, tokens, tokens, 1, 1)
+    if isinstance(cfg, DeluvikConfig):
+        return _deluvik_rows(cfg, tokens, tokens, 1, 1)
     if isinstance(cfg, StreamDesign):
         return _zinutar_rows(cfg, tokens, tokens * (tokens + 1) / 2, tokens, 1)
     d = tp_dims(cfg, tp)

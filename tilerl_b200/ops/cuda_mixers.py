@@ -14,6 +14,8 @@ from . import native as N
 from .cuda_stream import EPI_STORE, EPI_STORE_F32
 
 MAMBA2, MLSTM = 0, 1
+GLU_CLAMPED = 0
+GLU_ACTS = {"silu": 1, "gelu": 2}
 MIX_ROWS_MAX = 8        # rows the weight-streaming projection serves
 LATENT_SHORT = 32       # tokens of a sequence up to which attention runs in the latent (absorbed) form
 SCAN_SHORT = 16         # tokens of a sequence up to which a scan goes token by token
@@ -88,6 +90,14 @@ class MixerOps:
             self._mm(h, w[n_in:], gates)
         return proj, gates
 
+    def project(self, h, w):
+        """Projection rows in the compute type."""
+        y = self.ws.get(f"block_proj_{w.dtype}", (h.shape[0], w.shape[0]), w.dtype)
+        if self._streams_mix(h.shape[0], w):
+            self._linear_rows(h, w, y, EPI_STORE)
+            return y
+        return self._mm(h, w, y)
+
     def project_f32(self, a, w):
         y = self.ws.get("branch", (a.shape[0], w.shape[0]), torch.float32)
         if self._streams_mix(a.shape[0], w):
@@ -95,24 +105,41 @@ class MixerOps:
             return y
         return self._mm(a, w, y)
 
-    def project_logits(self, h, w):
+    def project_logits(self, h, w, cap=0.0):
+        """``cap``: logits are soft-capped there (0: not)."""
         logits = self.ws.get("logits", (h.shape[0], w.shape[0]), torch.float32)
         h = h.contiguous()
         if self._streams_mix(h.shape[0], w):
-            self._linear_rows(h, w, logits, EPI_STORE_F32)
+            if cap:
+                N.check(self.lib.trl_linear_rows_cap(h.data_ptr(), h.stride(0), w.data_ptr(), logits.data_ptr(), logits.stride(0), h.shape[0],
+                                                     w.shape[0], w.shape[1], cap, N.stream()), "linear_rows_cap")
+                N.count()
+            else:
+                self._linear_rows(h, w, logits, EPI_STORE_F32)
             return logits
-        return self._mm(h, w, logits)
+        self._mm(h, w, logits)
+        if cap:
+            N.check(self.lib.trl_soft_cap(logits.data_ptr(), logits.numel(), cap, N.stream()), "soft_cap")
+            N.count()
+        return logits
 
     def clamped_glu(self, h, w, limit):
+        return self._glu(h, w, GLU_CLAMPED, limit)
+
+    def glu(self, h, w, act):
+        """Rows ``2j`` = gate, ``2j + 1`` = up of ``w``: ``act(gate) * up``."""
+        return self._glu(h, w, GLU_ACTS[act], 0.0)
+
+    def _glu(self, h, w, act: int, limit: float):
         t, n = h.shape[0], w.shape[0]
         out = self.ws.get(f"glu_{w.dtype}", (t, n // 2), w.dtype)
         if self._streams_mix(t, w):
-            N.check(self.lib.trl_linear_rows_glu(h.data_ptr(), h.stride(0), w.data_ptr(), out.data_ptr(), n // 2, t, n, w.shape[1], limit,
+            N.check(self.lib.trl_linear_rows_glu(h.data_ptr(), h.stride(0), w.data_ptr(), out.data_ptr(), n // 2, t, n, w.shape[1], act, limit,
                                                  N.stream()), "linear_rows_glu")
             N.count()
             return out
         gu = self._mm(h, w, self.ws.get(f"gate_up_{w.dtype}", (t, n), w.dtype))
-        N.check(self.lib.trl_clamped_glu(gu.data_ptr(), out.data_ptr(), out.numel(), limit, _f32(w), N.stream()), "clamped_glu")
+        N.check(self.lib.trl_glu(gu.data_ptr(), out.data_ptr(), out.numel(), act, limit, _f32(w), N.stream()), "glu")
         N.count()
         return out
 
@@ -253,9 +280,9 @@ class MixerOps:
         elif kind == MAMBA2:
             rows = self.ws.get(f"scan_conv_{dt}", (t, l.conv_c), dt)
             N.check(self.lib.trl_scan_conv(
-                proj.data_ptr(), proj.stride(0), w["conv"].data_ptr(), w["conv_b"].data_ptr(), ring.data_ptr(), pool.ring.stride(0),
+                proj.data_ptr(), proj.stride(0), w["conv"].data_ptr(), w["conv_b"].data_ptr(), None, ring.data_ptr(), pool.ring.stride(0),
                 pool.ring_rows, pool.ring.stride(1), batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(),
-                batch.state_slots.data_ptr(), rows.data_ptr(), t, l.conv_c, l.taps, _f32(proj), st), "scan_conv")
+                batch.state_slots.data_ptr(), rows.data_ptr(), t, l.conv_c, l.taps, 1, _f32(proj), st), "scan_conv")
             N.count()
         if kind == MAMBA2:
             a.q0, a.k0, a.v0, a.per, a.q_scale, a.cap = l.q0, l.k0, 0, l.heads // l.groups, 1.0, 1.0

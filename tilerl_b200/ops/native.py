@@ -86,23 +86,35 @@ _SIGS = {
     "trl_sigmoid_attn_f32": [P, I, P, I, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, F, F, P],
     # sandwich-normed layers: joins, latent attention, decayed scans (csrc/join.cu, latent.cu, scan.cu)
     "trl_join": [P, P, P, I, P, I, P, P, P, F, I, I, I, I, F, I, P],
-    "trl_clamped_glu": [P, P, L, F, I, P],
+    "trl_glu": [P, P, L, I, F, I, P],
+    "trl_join_experts": [P, P, P, P, I, P, I, P, I, P, I, I, I, F, I, P],
+    "trl_soft_cap": [P, L, F, P],
+    "trl_linear_rows_cap": [P, I, P, P, I, I, I, I, F, P],
+    "trl_ring_store": [P, I, P, L, I, I, I, P, P, P, P, P, I, I, P],
     "trl_side_input": [P, P, P, P, I, I, I, L, I, I, I, P],
     "trl_latent_prep": [P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, F, I, P],
     "trl_latent_rope": [P, P, P, I, I, I, I, I, F, I, P],
     "trl_latent_gate": [P, P, I, P, I, I, I, I, I, P],
     "trl_latent_attn": [P, L, L, P, I, I, P, I, I, I, P, I, P, P, P, P, L, L, I, I, I, I, F, I, P],
     "trl_linear_rows_split": [P, I, P, P, I, I, P, I, I, I, I, P],
-    "trl_linear_rows_glu": [P, I, P, P, I, I, I, I, F, P],
+    "trl_linear_rows_glu": [P, I, P, P, I, I, I, I, I, F, P],
     "trl_linear_rows_side": [P, I, P, P, I, I, I, I, P, P, L, I, I, I, P],
     "trl_latent_mma_ok": [I, I, I, I],
     "trl_latent_decode": [P, I, I, I, P, P, I, I, P, I, F, P, P, I, P, I, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, F, P],
     "trl_latent_gather": [P, I, P, I, I, I, I, P, P, P],
     "trl_latent_prompt": [P, I, I, I, I, P, I, P, P, I, P, I, P, I, I, I, I, I, F, P],
     "trl_scan_chunk": [P, I, I, I, P],
-    "trl_scan_conv": [P, I, P, P, P, L, I, I, P, P, P, P, P, I, I, I, I, P],
+    "trl_scan_conv": [P, I, P, P, P, P, L, I, I, P, P, P, P, P, I, I, I, I, I, P],
     "trl_scan_serial": [P, I, I, I, P],
     "trl_scan_norm": [P, P, I, P, P, I, I, I, I, I, I, F, P, P, L, I, I, I, P, P, P, P, P, I, I, P],
+    # softmax attention on packed pages, linear recurrence, experts (csrc/attn_softmax.cu, lru.cu, moe.cu)
+    "trl_qkv_prep": [P, I, I, P],
+    "trl_softmax_attn": [P, P, I, P, I, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, F, I, P],
+    "trl_softmax_attn_rows": [I, I], "trl_softmax_attn_ok": [I, I],
+    "trl_lru_scan": [P, I, I, P], "trl_lru_step": [P, I, I, P],
+    "trl_moe_plan": [P, P],
+    "trl_moe_rows": [P, I, P, P, I, P, P, P, I, I, I, I, I, I, P],
+    "trl_moe_gather": [P, I, P, P, I, I, P],
     "trl_decode_advance": [P, P, P, P, P, P, I, I, P, I, P, P],
 }
 

@@ -169,7 +169,7 @@ register("any", "sm100", {
     "sigmoid_attention": Kernel("sig_attn_kernel + sig_combine_kernel", "csrc/attn_sigmoid.cu", "trl_sigmoid_attn",
                                 note="bf16 packed pool; narrow row tiles for decoding, wide ones for prompts, key splits"),
     "join": Kernel("join_kernel", "csrc/join.cu", "trl_join", note="branch norm + stream addition + next norm; bf16 or fp32 rows"),
-    "clamped_glu": Kernel("glu_kernel", "csrc/join.cu", "trl_clamped_glu", note="few rows: epilogue of linear_rows_kernel"),
+    "clamped_glu": Kernel("glu_kernel", "csrc/join.cu", "trl_glu", note="few rows: epilogue of linear_rows_kernel"),
     "side_input": Kernel("side_kernel", "csrc/join.cu", "trl_side_input", note="few rows: epilogue of linear_rows_kernel"),
     "latent_prep": Kernel("latent_prep_kernel", "csrc/latent.cu", "trl_latent_prep", note="normed latents and rotated key into packed pages"),
     "latent_attention_decode": Kernel("latent_absorb_kernel + latent_decode_kernel + latent_out_kernel", "csrc/latent_mma.cu", "trl_latent_decode",
