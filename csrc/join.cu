@@ -54,7 +54,7 @@ template <typename T, int R>
 __global__ void __launch_bounds__(512)
 join_kernel(float* x, const float* y, const float* __restrict__ post, int post_kind, const float* __restrict__ next, int next_kind,
             T* h, const T* __restrict__ table, const int* ids, float scale, int V, int ld, int n, float eps, const int* place,
-            const float* weight, int slots) {
+            const float* weight, int slots, int y_bf16) {
   __shared__ float red[32];
   pdl_launch_dependents(30);
   pdl_wait();
@@ -88,12 +88,12 @@ join_kernel(float* x, const float* y, const float* __restrict__ post, int post_k
     }
     for (int j = 0; j < parts; ++j) {        // rows y[place[t, j]], weighted; without slots the token's own row
       const float wj = slots ? weight[(size_t)t * slots + j] : 1.f;
-      const float* yr = y + (size_t)(slots ? place[(size_t)t * slots + j] : t) * ld;
+      const size_t yr = (size_t)(slots ? place[(size_t)t * slots + j] : t) * ld;
 #pragma unroll
       for (int i = 0; i < R; ++i) {
         const int k = (threadIdx.x + i * blockDim.x) * 4;
         if (k < ld) {
-          const float4 a = load4(yr + k);
+          const float4 a = y_bf16 ? load4(reinterpret_cast<const bf16*>(y) + yr + k) : load4(y + yr + k);
           v[i].x = fmaf(wj, a.x, v[i].x), v[i].y = fmaf(wj, a.y, v[i].y), v[i].z = fmaf(wj, a.z, v[i].z), v[i].w = fmaf(wj, a.w, v[i].w);
         }
       }
@@ -163,12 +163,12 @@ side_kernel(const T* z, const T* __restrict__ side, const int* ids, T* out, int 
 template <typename T>
 cudaError_t join_launch(void* x, const void* y, const void* post, int pk, const void* next, int nk, void* h, const void* table,
                         const void* ids, float scale, int V, int T_, int ld, int n, float eps, const void* place, const void* weight,
-                        int slots, cudaStream_t st) {
+                        int slots, int y_bf16, cudaStream_t st) {
   const int thr = ld >= 2048 ? 512 : (ld >= 1024 ? 256 : 128), need = (ld / 4 + thr - 1) / thr;
 #define JOIN(R)                                                                                                            \
   return trl_launch(join_kernel<T, R>, dim3(T_), dim3(thr), 0, st, (float*)x, (const float*)y, (const float*)post, pk,     \
                     (const float*)next, nk, (T*)h, (const T*)table, (const int*)ids, scale, V, ld, n, eps,                 \
-                    (const int*)place, (const float*)weight, slots)
+                    (const int*)place, (const float*)weight, slots, y_bf16)
   if (need <= 1) JOIN(1);
   if (need <= 2) JOIN(2);
   if (need <= 4) JOIN(4);
@@ -187,19 +187,19 @@ TRL_API int trl_join(void* x, const void* y, const void* post, int post_kind, co
       next_kind < 0 || next_kind > 2 || (next_kind && !next) || (table && !ids))
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
-  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, st)
-                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, st));
+  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, 0, st)
+                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, 0, st));
 }
 
-// The same with the branch of token t given as sum_j weight[t, j] y[place[t, j]] over `slots` rows.
-TRL_API int trl_join_experts(void* x, const void* y, const void* place, const void* weight, int slots, const void* post, int post_kind,
+// The same with the branch of token t given as sum_j weight[t, j] y[place[t, j]] over `slots` rows, fp32 or bf16.
+TRL_API int trl_join_experts(void* x, const void* y, int y_bf16, const void* place, const void* weight, int slots, const void* post, int post_kind,
                              const void* next, int next_kind, void* h, int T, int ld, int n, float eps, int f32, void* stream) {
   if (T <= 0 || ld % 64 || ld > 16384 || n <= 0 || n > ld || !y || !post || !place || !weight || slots <= 0 || post_kind < 1 || post_kind > 2 ||
       next_kind < 0 || next_kind > 2 || (next_kind && !next))
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
-  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, st)
-                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, st));
+  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, y_bf16, st)
+                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, y_bf16, st));
 }
 
 // x: n fp32 values, n a multiple of 4.

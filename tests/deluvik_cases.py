@@ -81,8 +81,38 @@ def random_weights(cfg, seed=0):
             t = 1.2 * t
         else:
             t = t * (1.3 / shape[-1] ** 0.5)
-        out[name] = t.to(torch.bfloat16).float()           # representable in every compute dtype
-    return out
+        out[name] = t
+    _clear_choices(cfg, out, g)
+    return {n: t.to(torch.bfloat16).float() for n, t in out.items()}      # representable in every compute dtype
+
+
+def _clear_choices(cfg, w, g, share=0.05, margin=1.2):
+    """Routers without close calls, which rounding would turn round: a few columns of the stream that no branch writes to (their norm
+    weights are zero) carry what mostly decides, drawn for every token until the last expert chosen stands clear of the next one."""
+    moe = [(i, l.mlp) for i, l in enumerate(cfg.layers) if isinstance(l.mlp, MoeSpec)]
+    if not moe:
+        return
+    r = 12
+    for i, l in enumerate(cfg.layers):
+        for n in (f"l{i}.norm1", f"l{i}.norm2"):
+            if n in w:
+                w[n][-r:] = 0.0
+    for i, m in moe:
+        t = w[f"l{i}.mlp.router"]
+        t[:, :-r] *= share
+        t[:, -r:] = torch.randn(t.shape[0], r, generator=g) * 4.0 / r ** 0.5
+    open_ = torch.arange(cfg.vocab)
+    for _ in range(4000):
+        w["embed"][open_, -r:] = 1.2 * torch.randn(len(open_), r, generator=g)
+        clear = torch.ones(len(open_), dtype=torch.bool)
+        for i, m in moe:
+            if m.top < m.experts:
+                z = (w["embed"][open_, -r:] @ w[f"l{i}.mlp.router"][:, -r:].T + w[f"l{i}.mlp.router.b"]).sort(dim=1, descending=True).values
+                clear &= z[:, m.top - 1] - z[:, m.top] > margin
+        open_ = open_[~clear]
+        if not len(open_):
+            return
+    raise AssertionError("no clear choice found")
 
 
 def build(cfg, weights, backend, *, max_tokens=1024, slots=4, graph=True, **kw):

@@ -15,6 +15,7 @@ from .cuda_mixers import GLU_ACTS, _f32
 from .cuda_stream import EPI_STORE_F32, SHORT_ROWS
 
 P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_long, ctypes.c_float
+MOE_TC_MIN = 16         # tokens from which on experts run as tensor-core tiles
 MOE_TILE = 8            # rows of a tile of the weight-streaming expert projections
 
 
@@ -184,6 +185,8 @@ class BlockOps:
         """Outputs of a tick's experts, ordered by expert, with the place and weight of every token's
         (:meth:`join_experts` sums them)."""
         pairs, dt, act = h.shape[0] * m.slots, h.dtype, GLU_ACTS[m.spec.act]
+        if dt == torch.bfloat16 and h.shape[0] >= MOE_TC_MIN:
+            return self._experts_tc(h, router, router_b, gate_up, down, m, act)
         plan, place, weight = self._moe_plan(h, router, router_b, m, MOE_TILE)
         mid = self.ws.get(f"moe_mid_{dt}", (pairs, m.ff), dt)
         y = self.ws.get("moe_out", (pairs, down.shape[1]), torch.float32)
@@ -191,12 +194,24 @@ class BlockOps:
         self._moe_rows(mid, down, y, plan, 1, act, m)
         return y, place, weight
 
+    def _experts_tc(self, h, router, router_b, gate_up, down, m, act: int):
+        """Many rows: tensor-core tiles of each expert's rows, gathered in order first; output rows in bf16."""
+        pairs, w, bf, lib, st = h.shape[0] * m.slots, h.shape[1], torch.bfloat16, self.lib, N.stream()
+        plan, place, weight = self._moe_plan(h, router, router_b, m, lib.trl_moe_tc_tile())
+        rows, mid, y = (self.ws.get(n, (pairs, k), bf) for n, k in (("moe_rows", w), ("moe_mid_tc", m.ff), ("moe_out_tc", down.shape[1])))
+        N.check(lib.trl_moe_gather(h.data_ptr(), h.stride(0), plan.token, rows.data_ptr(), pairs, w, st), "moe_gather")
+        for x, wt, out, kind in ((rows, gate_up, mid, 0), (mid, down, y, 1)):
+            N.check(lib.trl_moe_tc(x.data_ptr(), wt.data_ptr(), out.data_ptr(), out.stride(0), plan.items, plan.n_items, pairs, wt.shape[0],
+                                   wt.shape[1], wt.shape[2], kind, act, st), "moe_tc")
+        N.count(3)
+        return y, place, weight
+
     def join_experts(self, x, branch, post, nxt, eps, n):
         """:meth:`join` with the weighted sum over a token's experts as the branch."""
         y, place, weight = branch
         t, ld = x.shape
         h = self.ws.get(f"join_h_{self._join_dtype}", (t, ld), self._join_dtype)
-        N.check(self.lib.trl_join_experts(x.data_ptr(), y.data_ptr(), place.data_ptr(), weight.data_ptr(), weight.shape[1], post.data_ptr(),
+        N.check(self.lib.trl_join_experts(x.data_ptr(), y.data_ptr(), int(y.dtype == torch.bfloat16), place.data_ptr(), weight.data_ptr(), weight.shape[1], post.data_ptr(),
                                           post.shape[0], N.ptr(nxt), 0 if nxt is None else nxt.shape[0], h.data_ptr(), t, ld, n, eps, _f32(h),
                                           N.stream()), "join_experts")
         N.count()

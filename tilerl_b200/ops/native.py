@@ -87,7 +87,7 @@ _SIGS = {
     # sandwich-normed layers: joins, latent attention, decayed scans (csrc/join.cu, latent.cu, scan.cu)
     "trl_join": [P, P, P, I, P, I, P, P, P, F, I, I, I, I, F, I, P],
     "trl_glu": [P, P, L, I, F, I, P],
-    "trl_join_experts": [P, P, P, P, I, P, I, P, I, P, I, I, I, F, I, P],
+    "trl_join_experts": [P, P, I, P, P, I, P, I, P, I, P, I, I, I, F, I, P],
     "trl_soft_cap": [P, L, F, P],
     "trl_linear_rows_cap": [P, I, P, P, I, I, I, I, F, P],
     "trl_ring_store": [P, I, P, L, I, I, I, P, P, P, P, P, I, I, P],
@@ -114,6 +114,7 @@ _SIGS = {
     "trl_lru_scan": [P, I, I, P], "trl_lru_step": [P, I, I, P],
     "trl_moe_plan": [P, P],
     "trl_moe_rows": [P, I, P, P, I, P, P, P, I, I, I, I, I, I, P],
+    "trl_moe_tc": [P, P, P, I, P, P, I, I, I, I, I, I, P], "trl_moe_tc_tile": [],
     "trl_moe_gather": [P, I, P, P, I, I, P],
     "trl_decode_advance": [P, P, P, P, P, P, I, I, P, I, P, P],
 }

@@ -11,6 +11,7 @@ JSON line:
 * ``zinutar`` (:mod:`.zinutar`): the Zinutar design beside the hybrid's attention-only form at equal size,
   whole models and single kernels;
 * ``fetotar`` (:mod:`.fetotar`): the Fetotar design beside the hybrid with Gated-DeltaNet layers, likewise;
+* ``deluvik`` (:mod:`.deluvik`): the Deluvik design beside the hybrid with mostly attention layers, likewise;
 * ``grpo`` (:mod:`.grpo`): one-GPU GRPO step with LoRA adapters, split rollout / train;
 * ``grpo-zero3`` (:mod:`.grpo_zero3`, started under ``torchrun``): GRPO step with ZeRO-3 training
   and a tensor-parallel NVFP4 rollout engine on the same GPUs.
@@ -30,6 +31,7 @@ SUITES = {
     "tick": ("tick", []),
     "zinutar": ("zinutar", []),
     "fetotar": ("fetotar", []),
+    "deluvik": ("deluvik", []),
     "grpo": ("grpo", []),
     "grpo-zero3": ("grpo_zero3", []),
 }
