@@ -3,7 +3,7 @@
 //
 //   qkv_prep_kernel             fused projection rows -> queries and cached keys / values of a token: an optional short convolution
 //                               (earlier rows from the slot's ring), RMS norm with a weight over the whole projection or per head,
-//                               rotation in halves or neighbouring pairs; one block per token.  Everything between the projection's
+//                               rotation in halves or neighbouring pairs; two blocks per token.  Everything between the projection's
 //                               rounding and the final one is fp32.
 //   sm_attn_kernel<D, WM, WN>   tensor cores (mma.sync m16n8k16 bf16).  One block = (16 WM query rows, kv head, sequence, key split); a
 //                               row is a (token, head of the group) pair.  Keys come 64 at a time (four pages) into a ring of stages,
@@ -58,107 +58,148 @@ struct PrepArgs {
   int ldm, pad0;
 };
 
+// grid (token, part): part 0 = queries, part 1 = keys and values.  Weights of a tick take the read-only path (they are constants).
 template <typename T>
 __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
   constexpr int C = Chunk<T>::N;
-  extern __shared__ __align__(16) float s_row[];           // [n_in], then cos and sin, then a factor per head
+  extern __shared__ __align__(16) float s_row[];           // the part's columns, then cos and sin, then a factor per head
   __shared__ float red[32];
-  float* s_cs = s_row + a.n_in;
-  float* s_fac = s_cs + 2 * a.n_pairs;
   pdl_launch_dependents(50);
-  pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nt = blockDim.x, nw = nt >> 5;
+  const bool is_q = blockIdx.y == 0;
+  const int base = is_q ? 0 : a.k0, cols = is_q ? a.k0 : a.n_in - a.k0, heads = is_q ? a.heads : a.kv_heads;
+  float* s_cs = s_row + cols;
+  float* s_fac = s_cs + 2 * a.n_pairs;
+  pdl_wait();
   const int pos = a.positions[t], seq = a.seq_ids[t];
-  const T* row = reinterpret_cast<const T*>(a.proj) + (size_t)t * a.ldp;
-  for (int i = tid; i < a.n_pairs; i += nt) pair_angle(pos, a.freqs[i], 1.f, s_cs[2 * i], s_cs[2 * i + 1]);
-  T* ring = reinterpret_cast<T*>(a.ring) + (a.taps ? (size_t)a.slots[seq] * a.ring_slot : 0);
+  const T* row = reinterpret_cast<const T*>(a.proj) + (size_t)t * a.ldp + base;
+  T* ring = reinterpret_cast<T*>(a.ring) + (a.taps ? (size_t)a.slots[seq] * a.ring_slot + base : 0);
   const int t0 = a.q_start[seq];
-  for (int c = tid * C; c < a.n_in; c += nt * C) {
+  for (int i = tid; i < a.n_pairs; i += nt) pair_angle(pos, __ldg(a.freqs + i), 1.f, s_cs[2 * i], s_cs[2 * i + 1]);
+  for (int c = tid * C; c < cols; c += nt * C) {
     const uint4 own = *reinterpret_cast<const uint4*>(row + c);
     float f[C];
     Chunk<T>::get(own, f);
     if (a.taps) {
+      const float* w = a.conv + base + c;
       float acc[C];
 #pragma unroll
-      for (int e = 0; e < C; ++e) acc[e] = f[e] * a.conv[(size_t)(a.taps - 1) * a.n_in + c + e];
-      for (int back = 1; back < a.taps && back <= pos; ++back) {
-        const T* src = t - back >= t0 ? row - (size_t)back * a.ldp + c : ring + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + c;
-        Chunk<T>::get(*reinterpret_cast<const uint4*>(src), f);
+      for (int e = 0; e < C; ++e) acc[e] = 0.f;
+      for (int back = 0; back < a.taps && back <= pos; ++back) {
+        if (back) {
+          const T* src = t - back >= t0 ? row - (size_t)back * a.ldp + c : ring + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + c;
+          Chunk<T>::get(*reinterpret_cast<const uint4*>(src), f);
+        }
 #pragma unroll
-        for (int e = 0; e < C; ++e) acc[e] = fmaf(f[e], a.conv[(size_t)(a.taps - 1 - back) * a.n_in + c + e], acc[e]);
+        for (int e = 0; e < C; e += 4) {
+          const float4 k = __ldg(reinterpret_cast<const float4*>(w + (size_t)(a.taps - 1 - back) * a.n_in + e));
+          acc[e] = fmaf(f[e], k.x, acc[e]), acc[e + 1] = fmaf(f[e + 1], k.y, acc[e + 1]);
+          acc[e + 2] = fmaf(f[e + 2], k.z, acc[e + 2]), acc[e + 3] = fmaf(f[e + 3], k.w, acc[e + 3]);
+        }
       }
 #pragma unroll
       for (int e = 0; e < C; ++e) f[e] = acc[e];
       if (a.write_ring) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.ring_rows) * a.ring_ld + c) = own;
     }
 #pragma unroll
-    for (int e = 0; e < C; ++e) s_row[c + e] = f[e];
+    for (int e = 0; e < C; e += 4) *reinterpret_cast<float4*>(s_row + c + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
   }
-  if (a.mid)
+  if (a.mid && is_q)
     for (int c = a.pad0 + tid; c < a.ldm; c += nt) reinterpret_cast<T*>(a.mid)[(size_t)t * a.ldm + c] = from_f<T>(0.f);
   __syncthreads();
   // ---- norm factors (padding columns hold zeros)
-  const int n_heads = a.heads + (a.own ? a.kv_heads : 0);
   if (a.norm_all) {
-    float sq = 0.f, sk = 0.f;
-    for (int c = tid; c < a.k0; c += nt) sq += s_row[c] * s_row[c];
-    if (a.own)
-      for (int c = tid; c < a.kv_heads * a.dk; c += nt) sk += s_row[a.k0 + c] * s_row[a.k0 + c];
-    sq = block_sum(sq, red);
-    if (tid == 0) s_fac[0] = inv_rms(sq, a.heads * a.dim, a.eps);
-    if (a.own) {
-      sk = block_sum(sk, red);
-      if (tid == 0) s_fac[1] = inv_rms(sk, a.kv_heads * a.dim, a.eps);
+    float ss = 0.f;
+    for (int c = tid * 4; c < heads * a.dk; c += nt * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(s_row + c);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
+    ss = block_sum(ss, red);
+    if (tid == 0) s_fac[0] = inv_rms(ss, heads * a.dim, a.eps);
   } else {
-    for (int h = warp; h < n_heads; h += nw) {
+    for (int h = warp; h < heads; h += nw) {
       float ss = 0.f;
-      for (int d = lane; d < a.dk; d += 32) ss += s_row[h * a.dk + d] * s_row[h * a.dk + d];     // key heads follow the query heads
+      for (int d = lane * 4; d < a.dk; d += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(s_row + h * a.dk + d);
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      }
       ss = warp_sum(ss);
       if (lane == 0) s_fac[h] = inv_rms(ss, a.dim, a.eps);
     }
   }
   __syncthreads();
   // ---- turned rows, in chunks
-  int slot = a.own ? a.slot_mapping[t] : -1;
-  if (slot >= 0) slot = trl_checked(slot, a.n_blocks * KVB, 13);
+  int slot = is_q ? 0 : a.slot_mapping[t];
+  if (slot < 0) return;
+  if (!is_q) slot = trl_checked(slot, a.n_blocks * KVB, 13);
   const int kch = a.dk / C, vch = a.dv / C, page_bytes = KVB * (kch + vch) * 16, r = slot & (KVB - 1);
-  unsigned char* page0 = slot >= 0 ? a.pages + (size_t)(slot / KVB) * a.kv_heads * page_bytes : nullptr;
-  for (int x = tid; x < n_heads * kch; x += nt) {
-    const int h = x / kch, d0 = (x % kch) * C;
-    const bool is_q = h < a.heads;
-    if (!is_q && slot < 0) continue;
-    const float* src = s_row + h * a.dk;
-    const float* w = is_q ? a.q_norm + (a.norm_all ? h * a.dk : 0) : a.k_norm + (a.norm_all ? (h - a.heads) * a.dk : 0);
-    const float fac = s_fac[a.norm_all ? !is_q : h];
-    float o[C];
+  unsigned char* page0 = is_q ? nullptr : a.pages + (size_t)(slot / KVB) * a.kv_heads * page_bytes;
+  const float* norm = is_q ? a.q_norm : a.k_norm;
+  auto scaled = [&](const float* src, const float* w, float fac, int d, float (&o)[C]) {
 #pragma unroll
-    for (int e = 0; e < C; ++e) {
-      const int d = d0 + e;
-      const float v = src[d] * fac * w[d];
-      o[e] = v;
-      if (d < 2 * a.n_pairs) {
-        const bool second = a.half ? d >= a.n_pairs : d & 1;
-        const int p = a.half ? (second ? d - a.n_pairs : d) : d >> 1;
-        const int m = a.half ? (second ? d - a.n_pairs : d + a.n_pairs) : d ^ 1;
-        const float u = src[m] * fac * w[m], c = s_cs[2 * p], s = s_cs[2 * p + 1];
-        o[e] = second ? fmaf(v, c, u * s) : fmaf(v, c, -u * s);
+    for (int e = 0; e < C; e += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(src + d + e), g = __ldg(reinterpret_cast<const float4*>(w + d + e));
+      o[e] = v.x * fac * g.x, o[e + 1] = v.y * fac * g.y, o[e + 2] = v.z * fac * g.z, o[e + 3] = v.w * fac * g.w;
+    }
+  };
+  for (int x = tid; x < heads * kch; x += nt) {
+    const int h = x / kch, ci = x - h * kch, d0 = ci * C;
+    const float* src = s_row + h * a.dk;
+    const float* w = norm + (a.norm_all ? h * a.dk : 0);
+    const float fac = s_fac[a.norm_all ? 0 : h];
+    float o[C];
+    scaled(src, w, fac, d0, o);
+    if (d0 < 2 * a.n_pairs) {
+      if (!a.half) {
+#pragma unroll
+        for (int e = 0; e < C; e += 2) {
+          if (d0 + e < 2 * a.n_pairs) {
+            const float2 cs = *reinterpret_cast<const float2*>(s_cs + d0 + e);
+            const float u = o[e], v = o[e + 1];
+            o[e] = fmaf(u, cs.x, -v * cs.y), o[e + 1] = fmaf(v, cs.x, u * cs.y);
+          }
+        }
+      } else if (a.n_pairs % C == 0) {                      // a chunk turns with one other chunk
+        const bool second = d0 >= a.n_pairs;
+        const int p0 = second ? d0 - a.n_pairs : d0;
+        float m[C];
+        scaled(src, w, fac, second ? p0 : d0 + a.n_pairs, m);
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+          const float2 cs = *reinterpret_cast<const float2*>(s_cs + 2 * (p0 + e));
+          o[e] = second ? fmaf(o[e], cs.x, m[e] * cs.y) : fmaf(o[e], cs.x, -m[e] * cs.y);
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+          const int d = d0 + e;
+          if (d < 2 * a.n_pairs) {
+            const bool second = d >= a.n_pairs;
+            const int p = second ? d - a.n_pairs : d, m = second ? p : d + a.n_pairs;
+            const float u = src[m] * fac * w[m], c = s_cs[2 * p], s = s_cs[2 * p + 1];
+            o[e] = second ? fmaf(o[e], c, u * s) : fmaf(o[e], c, -u * s);
+          }
+        }
       }
     }
     const uint4 out = Chunk<T>::put(o);
     if (is_q) {
       *reinterpret_cast<uint4*>(reinterpret_cast<T*>(a.q) + (size_t)t * a.k0 + h * a.dk + d0) = out;
     } else {
-      uint4* kd = reinterpret_cast<uint4*>(page0 + (size_t)(h - a.heads) * page_bytes);
-      kd[r * kch + page_chunk(d0 / C, r, kch)] = out;
+      uint4* kd = reinterpret_cast<uint4*>(page0 + (size_t)h * page_bytes);
+      kd[r * kch + page_chunk(ci, r, kch)] = out;
     }
   }
-  if (slot < 0) return;
+  if (is_q) return;
   for (int x = tid; x < a.kv_heads * vch; x += nt) {
-    const int h = x / vch, c = x % vch;
+    const int h = x / vch, c = x - h * vch;
+    const float* src = s_row + a.v0 - a.k0 + h * a.dv + c * C;
     float o[C];
 #pragma unroll
-    for (int e = 0; e < C; ++e) o[e] = s_row[a.v0 + h * a.dv + c * C + e];
+    for (int e = 0; e < C; e += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(src + e);
+      o[e] = v.x, o[e + 1] = v.y, o[e + 2] = v.z, o[e + 3] = v.w;
+    }
     uint4* vd = reinterpret_cast<uint4*>(page0 + (size_t)h * page_bytes + KVB * kch * 16);
     vd[r * vch + page_chunk(c, r, vch)] = Chunk<T>::put(o);
   }
@@ -683,7 +724,8 @@ cudaError_t sm_launch(const SmArgs& a, int tiles, int B, const int* seq_ids, int
 TRL_API int trl_qkv_prep(const PrepArgs* args, int T, int f32, void* stream) {
   const PrepArgs& a = *args;
   const int per = f32 ? 4 : 8;
-  const size_t smem = (size_t)(a.n_in + 2 * a.n_pairs + a.heads + a.kv_heads + 2) * sizeof(float);
+  const int widest = max(a.k0, a.n_in - a.k0);
+  const size_t smem = (size_t)(widest + 2 * a.n_pairs + max(a.heads, a.kv_heads) + 2) * sizeof(float);
   if (T <= 0 || a.ldp % per || a.n_in % 16 || a.n_in > a.ldp || a.dk % 16 || a.dv % 16 || a.heads <= 0 || a.kv_heads <= 0 || a.dim > a.dk ||
       2 * a.n_pairs > a.dim || a.k0 != a.heads * a.dk || a.n_in != (a.own ? a.v0 + a.kv_heads * a.dv : a.k0) || smem > 200 * 1024 ||
       ((uintptr_t)a.proj & 15) || !a.q || !a.q_norm || (a.own && (!a.pages || !a.k_norm || ((uintptr_t)a.pages & 15))) ||
@@ -697,9 +739,10 @@ TRL_API int trl_qkv_prep(const PrepArgs* args, int T, int f32, void* stream) {
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const int threads = T <= 148 && a.n_in >= 2048 ? 512 : 256;
-  if (f32) return (int)trl_launch(qkv_prep_kernel<float>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, a);
-  return (int)trl_launch(qkv_prep_kernel<bf16>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, a);
+  const int threads = T <= 148 && widest >= 2048 ? 512 : (widest >= 1024 ? 256 : 128);
+  const dim3 grid(T, a.own ? 2 : 1);
+  if (f32) return (int)trl_launch(qkv_prep_kernel<float>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
+  return (int)trl_launch(qkv_prep_kernel<bf16>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
 }
 
 // Rows of a wide row tile: 128, or 112 for the widest heads (a ninth warp would leave 168 registers a thread).

@@ -3,13 +3,13 @@
 //   r = sigmoid(R u + b_r), i = sigmoid(I u + b_i)      R, I block-diagonal, u the convolved branch
 //   log a = -8 r softplus(lam),  S_t = a S_(t-1) + sqrt(1 - a^2) i u,  out = S_t gelu(y) factor
 //
-//   lru_scan_kernel   gate pre-activations given (library product): 32 channels of a sequence per block, 128 tokens at a time; a
-//                     warp scans 16 of them from zero, the carries meet in shared memory.  Any length, verify windows (a state
-//                     plane per token) included.
-//   lru_step_kernel   one token per sequence (decode ticks): convolution, gates and recurrence in one launch; a block owns 16
-//                     channels and streams their rows of R and I once for up to 8 sequences.
+//   lru_scan_kernel   gate pre-activations given (library product): 32 (16) channels of a sequence per block, 128 (256) tokens at a
+//                     time; runs of 8 tokens are scanned from zero, the carries meet in shared memory.  Any length, verify windows
+//                     (a state plane per token) included.
+//   lru_step_kernel   one token per sequence (decode ticks): convolution, gates (mma.sync in bf16) and recurrence in one launch; a
+//                     block owns 16 or 64 channels and streams their rows of R and I once for up to 8 sequences.
 //
-// Everything behind u is fp32; sqrt(1 - a^2) is formed from expm1 of the exponent.
+// Everything behind u is fp32.
 // Reference parity: the reference's recurrence is Gated DeltaNet only (no counterpart).
 #include "packed.cuh"
 
@@ -34,19 +34,39 @@ struct LruArgs {
 
 namespace {
 
-// (a, input factor) of the recurrence from the gates' pre-activations
+constexpr float LRU_LOG2E = 1.4426950408889634f;
+__device__ __forceinline__ float lru_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float lru_sigmoid(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + lru_ex2(-LRU_LOG2E * x)));
+  return y;
+}
+// the tanh form of gelu: z / 2 (1 + tanh(t)) = z sigmoid(2 t)
+__device__ __forceinline__ float lru_gelu(float z) { return z * lru_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
+// (a, input factor) of the recurrence from the gates' pre-activations; sp: softplus(lam)
 __device__ __forceinline__ float2 lru_decay(float zr, float zi, float sp) {
-  const float la = -8.f * sigmoid_x(zr) * sp;
-  return make_float2(expf(la), sqrtf(-expm1f(2.f * la)) * sigmoid_x(zi));
+  const float la = -8.f * lru_sigmoid(zr) * sp, a = lru_ex2(LRU_LOG2E * la), t = 2.f * la;
+  // 1 - a^2 = 1 - e^t; near t = 0 by the exponential series, whose first omitted term is t^6 / 5040 of the sum
+  const float near = -t * fmaf(t * (1.f / 2.f), fmaf(t * (1.f / 3.f), fmaf(t * (1.f / 4.f), fmaf(t * (1.f / 5.f), fmaf(t, 1.f / 6.f, 1.f), 1.f), 1.f), 1.f), 1.f);
+  const float left = t > -0.25f ? near : fmaf(-a, a, 1.f);
+  float root;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(root) : "f"(left));
+  return make_float2(a, root * lru_sigmoid(zi));
 }
 
-constexpr int LS_WARPS = 8, LS_L = 16, LS_TILE = LS_WARPS * LS_L;
-template <typename T>
+// CH channels a block; a warp holds 32 / CH runs of LS_L consecutive tokens, one channel a lane.
+constexpr int LS_WARPS = 16, LS_L = 8;
+template <typename T, int CH>
 __global__ void __launch_bounds__(LS_WARPS * 32) lru_scan_kernel(const LruArgs a) {
-  __shared__ float s_a[2][LS_WARPS][32], s_s[2][LS_WARPS][32];
+  constexpr int RUNS = LS_WARPS * (32 / CH), TILE = RUNS * LS_L;
+  __shared__ float s_a[2][RUNS][CH], s_s[2][RUNS][CH];
   pdl_launch_dependents(54);
   pdl_wait();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, seq = blockIdx.y, ch = blockIdx.x * 32 + lane;
+  const int lane = threadIdx.x % CH, run = threadIdx.x / CH, seq = blockIdx.y, ch = blockIdx.x * CH + lane;
   const int n = a.q_len[seq], t0 = a.q_start[seq], slot = a.slots[seq];
   if (n <= 0) return;
   const bool in = ch < a.width, keep = a.keep_flags && a.keep_flags[seq];
@@ -59,131 +79,163 @@ __global__ void __launch_bounds__(LS_WARPS * 32) lru_scan_kernel(const LruArgs a
   const T* y = reinterpret_cast<const T*>(a.y) + (size_t)t0 * a.ldp + c;
   T* out = reinterpret_cast<T*>(a.out) + (size_t)t0 * a.ldo + c;
   float carry = rec[plane];
-  int buf = 0;
-  for (int i0 = 0; i0 < n; i0 += LS_TILE, buf ^= 1) {
-    const int f = i0 + warp * LS_L, m = min(LS_L, n - f);          // this warp's tokens (m <= 0: none)
-    float pa[LS_L], ps[LS_L];                                       // product of decays and state from zero, up to each token
-    {
-      float zr[LS_L], zi[LS_L], uu[LS_L];
+  float zr[LS_L], zi[LS_L];
+  T uu[LS_L], yy[LS_L];
+  auto load = [&](int f) {                                          // (tokens past the end repeat the last one: never used)
 #pragma unroll
-      for (int k = 0; k < LS_L; ++k) {
-        const bool ok = k < m;
-        zr[k] = ok ? z[(size_t)(f + k) * 2 * a.pp] : 0.f;
-        zi[k] = ok ? z[(size_t)(f + k) * 2 * a.pp + a.pp] : 0.f;
-        uu[k] = ok ? to_f(u[(size_t)(f + k) * a.width]) : 0.f;
-      }
-      float A = 1.f, S = 0.f;
-#pragma unroll
-      for (int k = 0; k < LS_L; ++k) {
-        if (k < m) {
-          const float2 d = lru_decay(zr[k] + br, zi[k] + bi, sp);
-          A *= d.x, S = fmaf(d.x, S, d.y * uu[k]);
-        }
-        pa[k] = A, ps[k] = S;
-      }
+    for (int k = 0; k < LS_L; ++k) {
+      const int t = min(f + k, n - 1);
+      zr[k] = z[(size_t)t * 2 * a.pp], zi[k] = z[(size_t)t * 2 * a.pp + a.pp];
+      uu[k] = u[(size_t)t * a.width], yy[k] = y[(size_t)t * a.ldp];
     }
-    s_a[buf][warp][lane] = pa[LS_L - 1], s_s[buf][warp][lane] = ps[LS_L - 1];
+  };
+  load(run * LS_L);
+  int buf = 0;
+  for (int i0 = 0; i0 < n; i0 += TILE, buf ^= 1) {
+    const int f = i0 + run * LS_L, m = n - f;                       // this run's first token; tokens left (<= 0: none)
+    float pa[LS_L], ps[LS_L], g[LS_L];                              // product of decays and state from zero up to each token
+    float A = 1.f, S = 0.f;
+#pragma unroll
+    for (int k = 0; k < LS_L; ++k) {
+      const float2 d = lru_decay(zr[k] + br, zi[k] + bi, sp);
+      if (k < m) A *= d.x, S = fmaf(d.x, S, d.y * to_f(uu[k]));
+      pa[k] = A, ps[k] = S;
+      g[k] = lru_gelu(to_f(yy[k]) + yb) * a.factor;
+    }
+    s_a[buf][run][lane] = A, s_s[buf][run][lane] = S;
+    if (i0 + TILE < n) load(f + TILE);                              // the next tile's rows travel while the carries meet
     __syncthreads();
     float from = carry;
 #pragma unroll
-    for (int w = 0; w < LS_WARPS; ++w) {
-      if (w == warp) from = carry;
+    for (int w = 0; w < RUNS; ++w) {
+      if (w == run) from = carry;
       carry = fmaf(s_a[buf][w][lane], carry, s_s[buf][w][lane]);
     }
 #pragma unroll
     for (int k = 0; k < LS_L; ++k) {
       if (k < m && in) {
-        const float S = fmaf(pa[k], from, ps[k]);
-        out[(size_t)(f + k) * a.ldo] = from_f<T>(S * gelu_tanh_x(to_f(y[(size_t)(f + k) * a.ldp]) + yb) * a.factor);
-        if (keep) rec[(size_t)(f + k) * a.plane_stride] = S;
+        const float now = fmaf(pa[k], from, ps[k]);
+        out[(size_t)(f + k) * a.ldo] = from_f<T>(now * g[k]);
+        if (keep) rec[(size_t)(f + k) * a.plane_stride] = now;
       }
     }
   }
-  if (!keep && warp == 0 && in) rec[plane] = carry;
+  if (!keep && run == 0 && in) rec[plane] = carry;
 }
 
-// grid (channel groups of 16 within a part, groups of NB sequences), 8 warps of two channels each
-constexpr int LT_CH = 16;
-template <typename T, int NB>
+// grid (groups of CH channels within a part, groups of 8 sequences).  bf16: the gates' rows times the convolved rows on tensor cores,
+// K split over the warps; fp32: two channels a warp at a time.
+constexpr int LT_NB = 8, LT_PAD = 16;
+template <typename T, int CH>
 __global__ void __launch_bounds__(256) lru_step_kernel(const LruArgs a, int B) {
   constexpr int C = Chunk<T>::N;
-  extern __shared__ __align__(16) float s_u[];              // [NB][pp]
+  constexpr bool MMA = sizeof(T) == 2;
+  extern __shared__ __align__(16) unsigned char lt_smem[];
+  T* s_u = reinterpret_cast<T*>(lt_smem);                   // [8][ldu] convolved rows
+  const int ldu = (a.pp + 31) / 32 * 32 + LT_PAD;
+  float* s_z = reinterpret_cast<float*>(lt_smem + (size_t)LT_NB * ldu * sizeof(T));      // MMA: [8 warps][2][CH][8]; else [2][CH][8]
   pdl_launch_dependents(55);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, groups = (a.pp + CH - 1) / CH;
+  const int b = blockIdx.x / groups, g0 = (blockIdx.x % groups) * CH, m0 = blockIdx.y * LT_NB, nb = min(LT_NB, B - m0);
+  const int chans = min(CH, a.pp - g0);
   pdl_wait();
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, groups = a.pp / LT_CH;
-  const int b = blockIdx.x / groups, g0 = (blockIdx.x % groups) * LT_CH, m0 = blockIdx.y * NB, nb = min(NB, B - m0);
-  for (int x = tid; x < NB * a.pp; x += 256) {
-    const int m = x / a.pp, j = x % a.pp, c = b * a.pp + j;
-    float v = 0.f;
-    if (m < nb) {
+  for (int x = tid; x < LT_NB * (ldu / C); x += 256) {
+    const int m = x / (ldu / C), j = x % (ldu / C) * C, c = b * a.pp + j;
+    float v[C];
+#pragma unroll
+    for (int e = 0; e < C; ++e) v[e] = 0.f;
+    if (m < nb && j < a.pp) {
       const int t = a.q_start[m0 + m], pos = a.positions[t];
       T* rg = reinterpret_cast<T*>(a.ring) + (size_t)a.slots[m0 + m] * a.ring_slot + c;
-      const T own = reinterpret_cast<const T*>(a.u)[(size_t)t * a.ldp + c];
-      v = fmaf(to_f(own) + a.x_b[c], a.conv[(size_t)(a.taps - 1) * a.width + c], a.conv_b[c]);
-      for (int back = 1; back < a.taps && back <= pos; ++back)
-        v = fmaf(to_f(rg[(size_t)((pos - back) % a.ring_rows) * a.ring_ld]) + a.x_b[c], a.conv[(size_t)(a.taps - 1 - back) * a.width + c], v);
-      v = to_f(from_f<T>(v));
-      if (j >= g0 && j < g0 + LT_CH) rg[(size_t)(pos % a.ring_rows) * a.ring_ld] = own;
+      const uint4 own = *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(a.u) + (size_t)t * a.ldp + c);
+#pragma unroll
+      for (int e = 0; e < C; ++e) v[e] = a.conv_b[c + e];
+      for (int back = 0; back < a.taps && back <= pos; ++back) {
+        float f[C];
+        Chunk<T>::get(back ? *reinterpret_cast<const uint4*>(rg + (size_t)((pos - back) % a.ring_rows) * a.ring_ld) : own, f);
+#pragma unroll
+        for (int e = 0; e < C; ++e) v[e] = fmaf(f[e] + a.x_b[c + e], a.conv[(size_t)(a.taps - 1 - back) * a.width + c + e], v[e]);
+      }
+      if (j >= g0 && j < g0 + CH) *reinterpret_cast<uint4*>(rg + (size_t)(pos % a.ring_rows) * a.ring_ld) = own;
     }
-    s_u[x] = v;
+    *reinterpret_cast<uint4*>(s_u + (size_t)m * ldu + j) = Chunk<T>::put(v);
   }
   __syncthreads();
+  const T* wg = reinterpret_cast<const T*>(a.gates) + ((size_t)b * 2 * a.pp + g0) * a.pp;
+  if constexpr (MMA) {
+    // a lane feeds 8 consecutive k of rows g and g + 8 to two MMAs under a permutation of k that both operands share
+    const int g = lane >> 2, t = lane & 3;
+    float acc[2 * (CH / 16)][4];
 #pragma unroll
-  for (int i = 0; i < LT_CH / 8; ++i) {
-    const int j = g0 + warp * (LT_CH / 8) + i, c = b * a.pp + j;
-    const T* wr = reinterpret_cast<const T*>(a.gates) + ((size_t)b * 2 * a.pp + j) * a.pp;
-    const T* wi = wr + (size_t)a.pp * a.pp;
-    float zr[NB], zi[NB];
+    for (int i = 0; i < 2 * (CH / 16); ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int k0 = warp * 32; k0 < a.pp; k0 += 8 * 32) {
+      const int k = k0 + t * 8;
+      const uint4 xv = *reinterpret_cast<const uint4*>(s_u + (size_t)g * ldu + k);
 #pragma unroll
-    for (int m = 0; m < NB; ++m) zr[m] = zi[m] = 0.f;
-    for (int k = lane * C; k < a.pp; k += 32 * C) {
-      float fr[C], fi[C];
-      Chunk<T>::get(*reinterpret_cast<const uint4*>(wr + k), fr);
-      Chunk<T>::get(*reinterpret_cast<const uint4*>(wi + k), fi);
-#pragma unroll
-      for (int m = 0; m < NB; ++m)
-#pragma unroll
-        for (int e = 0; e < C; ++e) {
-          const float v = s_u[m * a.pp + k + e];
-          zr[m] = fmaf(fr[e], v, zr[m]), zi[m] = fmaf(fi[e], v, zi[m]);
+      for (int i = 0; i < 2 * (CH / 16); ++i) {
+        const int r = (i & 1) * a.pp + (i >> 1) * 16 + g;            // row of the recurrence gate, then of the input gate
+        uint4 va = make_uint4(0u, 0u, 0u, 0u), vb = va;
+        if (k < a.pp && (i >> 1) * 16 < chans) {
+          va = ldg_stream_16(wg + (size_t)r * a.pp + k);
+          vb = ldg_stream_16(wg + (size_t)(r + 8) * a.pp + k);
         }
+        const uint32_t a0[4] = {va.x, vb.x, va.y, vb.y}, a1[4] = {va.z, vb.z, va.w, vb.w};
+        mma16(acc[i], a0, xv.x, xv.y);
+        mma16(acc[i], a1, xv.z, xv.w);
+      }
     }
-    float r = 0.f, q = 0.f;                                  // lane m: the sums of sequence m
+    // accumulator e: channel g + 8 (e / 2) of its tile, sequence 2 t + e % 2
 #pragma unroll
-    for (int m = 0; m < NB; ++m) {
-      const float sr = warp_sum(zr[m]), si = warp_sum(zi[m]);
-      if (lane == m) r = sr, q = si;
+    for (int i = 0; i < 2 * (CH / 16); ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s_z[((warp * 2 + (i & 1)) * CH + (i >> 1) * 16 + g + (e >> 1) * 8) * LT_NB + 2 * t + (e & 1)] = acc[i][e];
+  } else {
+    for (int i = warp; i < 2 * chans; i += 8) {
+      const int gate = i / chans, j = i % chans;
+      const T* w = wg + ((size_t)gate * a.pp + j) * a.pp;
+      float acc[LT_NB];
+#pragma unroll
+      for (int m = 0; m < LT_NB; ++m) acc[m] = 0.f;
+      for (int k = lane; k < a.pp; k += 32) {
+        const float f = to_f(w[k]);
+#pragma unroll
+        for (int m = 0; m < LT_NB; ++m) acc[m] = fmaf(f, to_f(s_u[(size_t)m * ldu + k]), acc[m]);
+      }
+#pragma unroll
+      for (int m = 0; m < LT_NB; ++m) {
+        const float v = warp_sum(acc[m]);
+        if (lane == 0) s_z[(gate * CH + j) * LT_NB + m] = v;
+      }
     }
-    if (lane < nb) {
-      const int seq = m0 + lane, t = a.q_start[seq], slot = a.slots[seq];
-      float* st = a.states + (size_t)slot * a.slot_stride + (size_t)a.cur[slot] * a.plane_stride + c;
-      const float2 d = lru_decay(r + a.gates_b[(size_t)b * 2 * a.pp + j], q + a.gates_b[(size_t)b * 2 * a.pp + a.pp + j], softplus_x(a.lam[c]));
-      const float S = fmaf(d.x, *st, d.y * s_u[lane * a.pp + j]);
-      *st = S;
-      const float yv = to_f(reinterpret_cast<const T*>(a.y)[(size_t)t * a.ldp + c]) + a.y_b[c];
-      reinterpret_cast<T*>(a.out)[(size_t)t * a.ldo + c] = from_f<T>(S * gelu_tanh_x(yv) * a.factor);
-    }
+  }
+  __syncthreads();
+  for (int x = tid; x < chans * nb; x += 256) {
+    const int m = x / chans, j = x % chans, c = b * a.pp + g0 + j, seq = m0 + m, t = a.q_start[seq], slot = a.slots[seq];
+    float zr = 0.f, zi = 0.f;
+#pragma unroll
+    for (int k = 0; k < (MMA ? 8 : 1); ++k) zr += s_z[((k * 2) * CH + j) * LT_NB + m], zi += s_z[((k * 2 + 1) * CH + j) * LT_NB + m];
+    float* st = a.states + (size_t)slot * a.slot_stride + (size_t)a.cur[slot] * a.plane_stride + c;
+    const size_t gb = (size_t)b * 2 * a.pp + g0 + j;
+    const float2 d = lru_decay(zr + a.gates_b[gb], zi + a.gates_b[gb + a.pp], softplus_x(a.lam[c]));
+    const float S = fmaf(d.x, *st, d.y * to_f(s_u[(size_t)m * ldu + g0 + j]));
+    *st = S;
+    const float yv = to_f(reinterpret_cast<const T*>(a.y)[(size_t)t * a.ldp + c]) + a.y_b[c];
+    reinterpret_cast<T*>(a.out)[(size_t)t * a.ldo + c] = from_f<T>(S * lru_gelu(yv) * a.factor);
   }
 }
 
-template <typename T>
+template <typename T, int CH>
 cudaError_t step_launch(const LruArgs& a, int B, cudaStream_t st) {
-#define LRU_STEP(NB)                                                                                                       \
-  {                                                                                                                        \
-    auto k = lru_step_kernel<T, NB>;                                                                                       \
-    static bool configured = false;                                                                                        \
-    if (!configured) {                                                                                                     \
-      const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);              \
-      if (e != cudaSuccess) return e;                                                                                      \
-      configured = true;                                                                                                   \
-    }                                                                                                                      \
-    return trl_launch(k, dim3(a.width / LT_CH, (B + NB - 1) / NB), dim3(256), (size_t)NB * a.pp * sizeof(float), st, a, B); \
+  auto k = lru_step_kernel<T, CH>;
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return e;
+    configured = true;
   }
-  if (B == 1) LRU_STEP(1)
-  if (B == 2) LRU_STEP(2)
-  if (B <= 4 || a.pp > 4096) LRU_STEP(4)
-  LRU_STEP(8)
-#undef LRU_STEP
+  const size_t smem = (size_t)LT_NB * ((a.pp + 31) / 32 * 32 + LT_PAD) * sizeof(T) + (size_t)(sizeof(T) == 2 ? 8 : 1) * 2 * CH * LT_NB * sizeof(float);
+  if (smem > 200 * 1024) return cudaErrorInvalidValue;
+  return trl_launch(k, dim3(a.width / a.pp * ((a.pp + CH - 1) / CH), (B + LT_NB - 1) / LT_NB), dim3(256), smem, st, a, B);
 }
 
 bool lru_bad(const LruArgs& a) {
@@ -195,15 +247,21 @@ bool lru_bad(const LruArgs& a) {
 
 TRL_API int trl_lru_scan(const LruArgs* a, int B, int f32, void* stream) {
   if (B <= 0 || lru_bad(*a) || !a->z) return (int)cudaErrorInvalidValue;
-  const dim3 grid((a->width + 31) / 32, B);
-  if (f32) return (int)trl_launch(lru_scan_kernel<float>, grid, dim3(LS_WARPS * 32), 0, (cudaStream_t)stream, *a);
-  return (int)trl_launch(lru_scan_kernel<bf16>, grid, dim3(LS_WARPS * 32), 0, (cudaStream_t)stream, *a);
+  cudaStream_t st = (cudaStream_t)stream;
+  const bool narrow = (a->width + 31) / 32 * B < 128;             // too few blocks of 32 channels to fill the GPU
+  const dim3 grid((a->width + (narrow ? 15 : 31)) / (narrow ? 16 : 32), B), thr(LS_WARPS * 32);
+  if (f32) return (int)trl_launch(lru_scan_kernel<float, 32>, dim3((a->width + 31) / 32, B), thr, 0, st, *a);
+  if (narrow) return (int)trl_launch(lru_scan_kernel<bf16, 16>, grid, thr, 0, st, *a);
+  return (int)trl_launch(lru_scan_kernel<bf16, 32>, grid, thr, 0, st, *a);
 }
 
 // Every sequence of the batch has one token.
 TRL_API int trl_lru_step(const LruArgs* a, int B, int f32, void* stream) {
+  const int per = f32 ? 4 : 8;
   if (B <= 0 || lru_bad(*a) || !a->gates || !a->conv || !a->conv_b || !a->x_b || !a->ring || a->taps < 1 || a->taps > a->ring_rows ||
-      a->pp > 8192 || ((uintptr_t)a->gates & 15))
+      a->ldp % per || a->ring_ld % per || a->ring_slot % per || ((uintptr_t)a->gates & 15) || ((uintptr_t)a->u & 15) || ((uintptr_t)a->ring & 15))
     return (int)cudaErrorInvalidValue;
-  return (int)(f32 ? step_launch<float>(*a, B, (cudaStream_t)stream) : step_launch<bf16>(*a, B, (cudaStream_t)stream));
+  cudaStream_t st = (cudaStream_t)stream;
+  if (f32) return (int)step_launch<float, 16>(*a, B, st);
+  return (int)(B > 2 * LT_NB ? step_launch<bf16, 64>(*a, B, st) : step_launch<bf16, 16>(*a, B, st));
 }

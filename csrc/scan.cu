@@ -8,6 +8,7 @@
 //
 //   scan_conv_kernel    convolution of a tick's rows (with or without silu, inputs with or without a bias); rows before the tick's
 //                       first token come from the slot's ring.
+//   conv_run_kernel     the same for prompts (up to 4 taps).
 //   ring_store_kernel   a tick's last convolution inputs into the ring.
 //   scan_serial_kernel  token after token, 32 value columns of a head per block, the state in registers: decoding, windows of
 //                       kept states, short portions, and fp32 models.
@@ -63,6 +64,68 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
     for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
   }
   *reinterpret_cast<uint4*>(out + (size_t)t * channels + c) = Chunk<T>::put(acc);
+}
+
+// The same for prompts: thread = one chunk of channels of CR_RUN consecutive tokens; weights and the last inputs stay in registers.
+constexpr int CR_RUN = 16;
+template <typename T, int K>
+__global__ void __launch_bounds__(128)
+conv_run_kernel(const T* proj, int ldp, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ pre,
+                const T* ring, long ring_slot, int ring_rows, int ring_ld, const int* positions, const int* seq_ids,
+                const int* q_start, const int* slots, T* out, int n_tok, int channels, int taps, int silu) {
+  constexpr int C = Chunk<T>::N;
+  pdl_launch_dependents(44);
+  const int c = (blockIdx.y * 128 + threadIdx.x) * C, first = blockIdx.x * CR_RUN, end = min(n_tok, first + CR_RUN);
+  if (c >= channels) {
+    pdl_wait();
+    return;
+  }
+  float wt[K][C], b[C], p[C], h[K][C];       // weight and input of `k` tokens back (inputs with their bias)
+#pragma unroll
+  for (int e = 0; e < C; ++e) b[e] = bias[c + e], p[e] = pre ? pre[c + e] : 0.f;
+#pragma unroll
+  for (int k = 0; k < K; ++k)
+#pragma unroll
+    for (int e = 0; e < C; ++e) wt[k][e] = k < taps ? w[(size_t)(taps - 1 - k) * channels + c + e] : 0.f, h[k][e] = 0.f;
+  pdl_wait();
+  int seq = -1;
+#pragma unroll 4
+  for (int t = first; t < end; ++t) {
+    const uint4 own = *reinterpret_cast<const uint4*>(proj + (size_t)t * ldp + c);
+    if (seq_ids[t] != seq) {                 // another sequence (or the run's first token): inputs before this token
+      seq = seq_ids[t];
+      const int pos = positions[t], t0 = q_start[seq];
+      const T* rg = ring + (size_t)slots[seq] * ring_slot + c;
+#pragma unroll
+      for (int k = 1; k < K; ++k) {
+        const bool there = k < taps && k <= pos;
+        float f[C];
+        if (there) Chunk<T>::get(*reinterpret_cast<const uint4*>(t - k >= t0 ? proj + (size_t)(t - k) * ldp + c : rg + (size_t)((pos - k) % ring_rows) * ring_ld), f);
+#pragma unroll
+        for (int e = 0; e < C; ++e) h[k][e] = there ? f[e] + p[e] : 0.f;
+      }
+    }
+    Chunk<T>::get(own, h[0]);
+    float acc[C];
+#pragma unroll
+    for (int e = 0; e < C; ++e) {
+      h[0][e] += p[e];
+      acc[e] = b[e];
+    }
+#pragma unroll
+    for (int k = K - 1; k >= 0; --k)
+#pragma unroll
+      for (int e = 0; e < C; ++e) acc[e] = fmaf(h[k][e], wt[k][e], acc[e]);
+#pragma unroll
+    for (int k = K - 1; k > 0; --k)
+#pragma unroll
+      for (int e = 0; e < C; ++e) h[k][e] = h[k - 1][e];
+    if (silu) {
+#pragma unroll
+      for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)t * channels + c) = Chunk<T>::put(acc);
+  }
 }
 
 // one block per token: its row into the ring unless later ones of the tick would overwrite it
@@ -359,6 +422,16 @@ TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* 
       ((uintptr_t)ring & 15) || ((uintptr_t)proj & 15))
     return (int)cudaErrorInvalidValue;
   const dim3 grid(T, (channels / per + 127) / 128);
+  if (T >= 512 && taps <= 4) {
+    const dim3 runs((T + CR_RUN - 1) / CR_RUN, grid.y);
+#define CONV_RUN(TT)                                                                                                               \
+  return (int)trl_launch(conv_run_kernel<TT, 4>, runs, dim3(128), 0, (cudaStream_t)stream, (const TT*)proj, ldp, (const float*)w,  \
+                         (const float*)bias, (const float*)pre, (const TT*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions, \
+                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (TT*)out, T, channels, taps, silu)
+    if (f32) CONV_RUN(float);
+    CONV_RUN(bf16);
+#undef CONV_RUN
+  }
   if (f32)
     return (int)trl_launch(scan_conv_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, (const float*)proj, ldp, (const float*)w,
                            (const float*)bias, (const float*)pre, (const float*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,

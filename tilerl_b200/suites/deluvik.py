@@ -66,6 +66,7 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
     from ..config import ATTN, GDN
     from ..factory import build_model, make_ops
     from ..kv import make_kv_pool, make_state_pool
+    from ..ops import native as N
     cd, ch = configs(size)["deluvik"], configs(size)["hybrid"]
     cd = replace(cd, layers=cd.layers[:4])
     h, heads, kvh, ff, eff, n_exp, top, _, window = SIZES[size]
@@ -87,7 +88,7 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
             r.add(f"in projection {m} rows", "hybrid", lambda: ops.norm_linear(hb, norm, w_in, eps), by, fl)
             by, fl = w_gu.numel() * 2 + m * (h + ff) * 2, 2.0 * m * w_gu.numel()
             r.add(f"dense gate / up {m} rows", "deluvik", lambda: ops.glu(hb, w_gu, "gelu"), by, fl)
-            r.add(f"dense gate / up {m} rows", "hybrid", lambda: ops.norm_linear_swiglu(hb, norm, w_gu, eps), by, fl)
+            r.add(f"dense gate / up {m} rows (without activation)", "hybrid", lambda: ops.norm_linear(hb, norm, w_gu, eps), by + m * ff * 2, fl)
             by, fl = w_dn.numel() * 2 + m * (ff * 2 + h * 4), 2.0 * m * w_dn.numel()
             r.add(f"dense down {m} rows", "deluvik", lambda: ops.project_f32(a, w_dn), by, fl)
             r.add(f"dense down {m} rows", "hybrid", lambda: ops.linear_residual(a, w_dn, hb), by, fl)
@@ -97,8 +98,8 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
         per = 2 * moe.ff * h + h * moe.ff
         by, fl = used * per * 2 + m * h * 2 + m * moe.slots * (moe.ff * 2 + h * 2), 2.0 * m * moe.slots * per
         r.add(f"experts {m} rows (router to weighted rows)", "deluvik", lambda: ops.experts(hb, P["L1.router"], P["L1.router_b"], P["L1.gate_up"], P["L1.down"], moe), by, fl)
-        r.add(f"experts {m} rows: dense feed-forward", "hybrid",
-              lambda: ops.linear_residual(ops.norm_linear_swiglu(hb, norm, w_gu, eps), w_dn, hb), (w_gu.numel() + w_dn.numel()) * 2 + m * (2 * h + ff) * 2,
+        r.add(f"experts {m} rows: dense gate / up and down (without activation)", "hybrid",
+              lambda: (ops.norm_linear(hb, norm, w_gu, eps), ops.linear_residual(a, w_dn, hb)), (w_gu.numel() + w_dn.numel()) * 2 + m * (2 * h + 3 * ff) * 2,
               2.0 * m * (w_gu.numel() + w_dn.numel()))
         branch = ops.experts(hb, P["L1.router"], P["L1.router_b"], P["L1.gate_up"], P["L1.down"], moe)
         r.add(f"join {m} rows", "deluvik", lambda: ops.join(x, y, P["L1.norm1"], None, eps, h), m * h * (4 + 8 + 2))
@@ -110,7 +111,6 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
             plan, _, _ = ops._moe_plan(hb, P["L1.router"], P["L1.router_b"], moe, tile)
             pairs = m * moe.slots
             xs, mid, out = bf(pairs, h), bf(pairs, moe.ff), bf(pairs, h)
-            from ..ops import native as N
             for what, x_, w_, o_, kind in (("up", xs, P["L1.gate_up"], mid, 0), ("down", mid, P["L1.down"], out, 1)):
                 def go():
                     N.check(ops.lib.trl_moe_tc(x_.data_ptr(), w_.data_ptr(), o_.data_ptr(), o_.stride(0), plan.items, plan.n_items, pairs, w_.shape[0],
@@ -159,6 +159,13 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
         pa = make_kv_pool(replace(ch, layer_types=(ATTN,)), b * pages + 1, dev)
         pa.k.normal_(), pa.v.normal_()
         qkv = bf(t, ch.qkv_rows)
+        qb, (kc, vc) = bf(t, nq * 256), pa.layer(0)
+
+        def prep():
+            N.check(ops.lib.trl_attn_prep(qkv.data_ptr(), qkv.stride(0), alp["q_norm"].data_ptr(), alp["k_norm"].data_ptr(), batch.positions.data_ptr(),
+                                          batch.slot_mapping.data_ptr(), qb.data_ptr(), kc.data_ptr(), vc.data_ptr(), t, nq, nkv, 256, ch.rotary_dim,
+                                          ch.rope_theta, eps, 0, kc.shape[0], N.stream()))
+        r.add(f"preparation {what}", "hybrid", prep, t * (2 * ch.qkv_rows) * 2)
         pairs = b * sum(range(ctx - n + 1, ctx + 1))
         r.add(f"attention {what}: with preparation", "hybrid", lambda: ops.attention(qkv, alp, batch, pa, 0, ch, nq, nkv),
               b * ctx * nkv * 256 * 4 + t * nq * 256 * 6, 4.0 * pairs * nq * 256)
