@@ -577,7 +577,10 @@ sm_attn_kernel(const SmArgs a) {
 }
 
 // grid (token, head): merges the partial rows of a launch whose row tiles were `rows` tall
-__global__ void __launch_bounds__(128) sm_combine_kernel(const SmArgs a, const int* seq_ids, int rows) {
+constexpr int CB_THREADS = 256;
+__global__ void __launch_bounds__(CB_THREADS) sm_combine_kernel(const SmArgs a, const int* seq_ids, int rows) {
+  __shared__ float s_w[64];                                 // weight of each split
+  __shared__ float2 s_v[CB_THREADS];
   pdl_launch_dependents(52);
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y, seq = seq_ids[t], T = a.q_len[seq];
@@ -591,21 +594,29 @@ __global__ void __launch_bounds__(128) sm_combine_kernel(const SmArgs a, const i
   const size_t cell = (size_t)t * a.n_q + h;
   const float2* ml = a.ml + cell * a.n_splits;
   const float* p = a.part + cell * a.n_splits * dv;
-  float top = -INFINITY, l = 0.f;
-  for (int s = 0; s < used; ++s) top = fmaxf(top, ml[s].x);
-  for (int s = 0; s < used; ++s) l = fmaf(ml[s].y, rel_weight(ml[s].x, top), l);
-  const float2 f = with_sink(top, l, a.sink, h);
+  // every warp on its own: all splits' maxima and sums (at most 64), two a lane
+  const int lane = threadIdx.x & 31;
+  const float2 none = make_float2(-INFINITY, 0.f), m0 = lane < used ? ml[lane] : none, m1 = lane + 32 < used ? ml[lane + 32] : none;
+  const float top = warp_max(fmaxf(m0.x, m1.x)), w0 = rel_weight(m0.x, top), w1 = rel_weight(m1.x, top);
+  const float2 f = with_sink(top, warp_sum(fmaf(m0.y, w0, m1.y * w1)), a.sink, h);
   const float g = f.x / f.y * a.factor;
-  for (int d = threadIdx.x * 2; d < dv; d += 256) {
-    float2 v = make_float2(0.f, 0.f);
-#pragma unroll 8
-    for (int s = 0; s < used; ++s) {
+  if (threadIdx.x < 32) s_w[lane] = w0, s_w[lane + 32] = w1;
+  __syncthreads();
+  // a thread: two columns of every n_g-th split; then the n_g sums of a column in order
+  const int pairs = dv / 2, n_g = CB_THREADS / pairs, grp = threadIdx.x / pairs, d = threadIdx.x % pairs * 2;
+  float2 v = make_float2(0.f, 0.f);
+  if (grp < n_g) {
+#pragma unroll 4
+    for (int s = grp; s < used; s += n_g) {
       const float2 x = *reinterpret_cast<const float2*>(p + (size_t)s * dv + d);
-      const float e = rel_weight(ml[s].x, top);
-      v.x = fmaf(x.x, e, v.x), v.y = fmaf(x.y, e, v.y);
+      v.x = fmaf(x.x, s_w[s], v.x), v.y = fmaf(x.y, s_w[s], v.y);
     }
-    *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(a.out) + (size_t)t * a.ldo + (size_t)h * dv + d) = f2_to_bf162_bits(v.x * g, v.y * g);
   }
+  s_v[threadIdx.x] = v;
+  __syncthreads();
+  if (grp) return;
+  for (int k = 1; k < n_g; ++k) v.x += s_v[k * pairs + threadIdx.x].x, v.y += s_v[k * pairs + threadIdx.x].y;
+  *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(a.out) + (size_t)t * a.ldo + (size_t)h * dv + d) = f2_to_bf162_bits(v.x * g, v.y * g);
 }
 
 // CUDA cores: one block = (16 query rows, kv head, sequence), a page of keys at a time; thread (r, c) forms the score of
@@ -708,7 +719,7 @@ cudaError_t sm_launch_as(SmArgs a, int tiles, int B, const int* seq_ids, int n_t
   }
   cudaError_t e = trl_launch(kern, dim3(tiles * a.n_splits, a.n_kv, B), dim3((WM * WN + 1) * 32), smem + 128, st, a);
   if (e == cudaSuccess && a.n_splits > 1)
-    e = trl_launch(sm_combine_kernel, dim3(n_tok, a.n_q), dim3(128), 0, st, a, seq_ids, ROWS);
+    e = trl_launch(sm_combine_kernel, dim3(n_tok, a.n_q), dim3(CB_THREADS), 0, st, a, seq_ids, ROWS);
   return e;
 }
 
@@ -760,7 +771,7 @@ TRL_API int trl_softmax_attn(const void* q, const void* pages, int n_blocks, con
                              int wide, int window, float scale, float cap, float factor, int f32, void* stream) {
   const int per = f32 ? 4 : 8;
   if (T <= 0 || B <= 0 || tiles <= 0 || n_kv <= 0 || n_q % n_kv || dk % 16 || dv % 16 || dk > F_MAXD || dv > F_MAXD || dk <= 0 || dv <= 0 ||
-      n_splits < 1 || (n_splits > 1 && (!part || !ml)) || ldo % per || n_blocks <= 0 || window < 0 || cap < 0.f || ((uintptr_t)pages & 15) ||
+      n_splits < 1 || n_splits > 64 || (n_splits > 1 && (!part || !ml)) || ldo % per || n_blocks <= 0 || window < 0 || cap < 0.f || ((uintptr_t)pages & 15) ||
       ((uintptr_t)q & 15) || ((uintptr_t)out & 15) || (wide != 2 && (f32 || dk > 256 || dv > 256)))
     return (int)cudaErrorInvalidValue;
   SmArgs a;

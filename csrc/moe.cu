@@ -2,7 +2,7 @@
 // the softmax over those, and `pieces` experts that all tokens share (weight one).
 //
 //   moe_topk_kernel    router logits -> expert numbers and weights of every token, one warp per token.
-//   moe_plan_kernel    one block: orders the (token, expert) pairs by expert and cuts every expert's rows into tiles.  Ticks of few
+//   moe_plan_kernel    (moe_plan_small_kernel for a few pairs) one block: orders the (token, expert) pairs by expert and cuts every expert's rows into tiles.  Ticks of few
 //                      tokens choose their experts in here, too.  The place of a row among its expert's is arbitrary; its values are not.
 //   moe_rows_kernel    few rows: gated up projection / down projection of every tile (up to 8 rows), weights streamed as in
 //                      linear_rows.cu: a warp owns 16 weight rows and a share of K in its own slots of a ring.
@@ -114,6 +114,34 @@ __global__ void __launch_bounds__(MP_THREADS) moe_plan_kernel(const MoePlanArgs 
   }
 }
 
+// The same for a few pairs: a thread a pair, ranks by counting.
+constexpr int MQ_MAX = 256;
+__global__ void __launch_bounds__(MQ_MAX) moe_plan_small_kernel(const MoePlanArgs a) {
+  __shared__ int s_e[MQ_MAX], s_tiles[MQ_MAX];
+  pdl_launch_dependents(61);
+  pdl_wait();
+  const int tid = threadIdx.x, slots = a.top + a.pieces, P = a.T * slots;
+  for (int t = tid >> 5; t < a.T; t += blockDim.x >> 5) choose_experts(a, t);
+  __syncthreads();
+  const int e = tid < P ? a.ids[tid] : 0;
+  s_e[tid] = e;
+  __syncthreads();
+  int row = 0, rank = 0, cnt = 0, item = 0, total = 0;          // rows before, rank among the expert's, its rows, tiles before it
+  for (int q = 0; q < P; ++q) {
+    const int o = s_e[q];
+    row += o < e || (o == e && q < tid), rank += o == e && q < tid, cnt += o == e;
+  }
+  s_tiles[tid] = rank ? 0 : (cnt + a.tile - 1) / a.tile;        // an expert's tiles count, and are written, at its first pair
+  __syncthreads();
+  if (tid >= P) return;
+  a.place[tid] = row, a.token[row] = tid / slots;
+  if (rank) return;
+  for (int q = 0; q < P; ++q) total += s_tiles[q], item += s_e[q] < e ? s_tiles[q] : 0;
+  for (int i = 0; i * a.tile < cnt; ++i)
+    if (item + i < a.max_items) a.items[item + i] = MoeItem{e, row + i * a.tile, min(a.tile, cnt - i * a.tile), 0};
+  if (row == 0) *a.n_items = min(total, a.max_items);
+}
+
 // ---- few rows -----------------------------------------------------------------------------------------------
 constexpr int MR_THREADS = 256, MR_WARPS = MR_THREADS / 32, MR_U = 4, MR_PAD = 32, MR_ROWS = 8;
 constexpr int MR_SLOT = MR_U * 2 * 512;                        // bytes of a ring stage of one warp
@@ -138,7 +166,7 @@ __global__ void __launch_bounds__(MR_THREADS)
 moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int ldy, const MoeItem* items, const int* n_items, const int* token,
                 int N, int K, int KW, int per_item, int act) {
   extern __shared__ __align__(16) unsigned char mr_smem[];
-  __shared__ float s_part[MR_WARPS * 16 * MR_ROWS];
+  __shared__ float s_part[2][MR_WARPS * 16 * MR_ROWS];           // one barrier a tile: the sums of a tile are formed under the next one
   bf16* xs = reinterpret_cast<bf16*>(mr_smem + MR_WARPS * DEPTH * MR_SLOT);     // [8][K + MR_PAD]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
   const int RW = MR_WARPS / KW, wr = warp / KW, wk = warp % KW, ldxs = K + MR_PAD;
@@ -149,17 +177,15 @@ moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int
   const long total = (long)*n_items * per_item;
   const int first = (int)(total * blockIdx.x / gridDim.x), end = (int)(total * (blockIdx.x + 1) / gridDim.x);
   // fetch cursor: runs DEPTH - 1 blocks of MR_U steps ahead of the products, across row tiles and items
-  int f_tile = first, f_j = jb, f_slot = 0, f_item = -1;
-  const bf16* f_w = w;
+  int f_tile = first, f_j = jb, f_slot = 0, f_item = first / per_item, f_in = first - f_item * per_item;
+  const bf16 *f_w = w, *wa = w, *wb = w;
+  auto aim = [&]() {                                           // rows of the tile the cursor is on
+    const int r0 = (f_in * RW + wr) * 16;
+    wa = f_w + (size_t)min(r0 + g, N - 1) * K + (t << 3), wb = f_w + (size_t)min(r0 + g + 8, N - 1) * K + (t << 3);
+  };
+  if (first < end) f_w = w + (size_t)items[f_item].expert * N * K, aim();
   auto fetch = [&]() {
     if (f_tile < end && jb < je) {
-      if (f_tile / per_item != f_item) {
-        f_item = f_tile / per_item;
-        f_w = w + (size_t)items[f_item].expert * N * K;
-      }
-      const int r0 = (f_tile % per_item * RW + wr) * 16;
-      const bf16* wa = f_w + (size_t)min(r0 + g, N - 1) * K + (t << 3);
-      const bf16* wb = f_w + (size_t)min(r0 + g + 8, N - 1) * K + (t << 3);
 #pragma unroll
       for (int u = 0; u < MR_U; ++u) {
         if (f_j + u < je) {
@@ -169,19 +195,28 @@ moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int
         }
       }
       f_j += MR_U;
-      if (f_j >= je) f_j = jb, ++f_tile;
+      if (f_j >= je) {
+        f_j = jb, ++f_tile;
+        if (++f_in == per_item) {
+          f_in = 0, ++f_item;
+          if (f_tile < end) f_w = w + (size_t)items[f_item].expert * N * K;
+        }
+        aim();
+      }
     }
     f_slot = f_slot + 1 == DEPTH ? 0 : f_slot + 1;
     cp_commit();
   };
 #pragma unroll
   for (int i = 0; i < DEPTH - 1; ++i) fetch();
-  int slot = 0, now = -1;
+  int slot = 0, item = first / per_item, in = first - item * per_item, buf = 0;
+  bool fresh = true;
   MoeItem it = {0, 0, 0, 0};
-  for (int tile = first; tile < end; ++tile) {
-    if (tile / per_item != now) {
-      now = tile / per_item;
-      it = items[now];
+  for (int tile = first; tile < end; ++tile, ++in, buf ^= 1) {
+    if (in == per_item) in = 0, ++item, fresh = true;
+    if (fresh) {
+      fresh = false;
+      it = items[item];
       __syncthreads();
       for (int m = 0; m < it.n; ++m) {
         const bf16* src = x + (size_t)(KIND == MOE_UP ? token[it.row0 + m] : it.row0 + m) * ldx;
@@ -214,22 +249,21 @@ moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int
     }
     // accumulator e: weight row g + 8 (e / 2), activation row 2 t + e % 2
 #pragma unroll
-    for (int e = 0; e < 4; ++e) s_part[(warp * MR_ROWS + 2 * t + (e & 1)) * 16 + g + (e >> 1) * 8] = acc[e];
+    for (int e = 0; e < 4; ++e) s_part[buf][(warp * MR_ROWS + 2 * t + (e & 1)) * 16 + g + (e >> 1) * 8] = acc[e];
     __syncthreads();
     auto total_of = [&](int m, int c) {
       float v = 0.f;
-      for (int k = 0; k < KW; ++k) v += s_part[(((c >> 4) * KW + k) * MR_ROWS + m) * 16 + (c & 15)];
+      for (int k = 0; k < KW; ++k) v += s_part[buf][(((c >> 4) * KW + k) * MR_ROWS + m) * 16 + (c & 15)];
       return v;
     };
     constexpr int PER = KIND == MOE_UP ? 8 : 16;               // outputs of 16 weight rows
     for (int i = threadIdx.x; i < RW * PER * it.n; i += MR_THREADS) {
-      const int m = i / (RW * PER), c = i % (RW * PER) * (16 / PER), n = tile % per_item * RW * 16 + c;
+      const int m = i / (RW * PER), c = i % (RW * PER) * (16 / PER), n = in * RW * 16 + c;
       if (n >= N) continue;
       const float v = total_of(m, c);
       if (KIND == MOE_UP) reinterpret_cast<bf16*>(y)[(size_t)(it.row0 + m) * ldy + n / 2] = __float2bfloat16(glu_x(v, total_of(m, c + 1), act, 0.f));
       else reinterpret_cast<float*>(y)[(size_t)(it.row0 + m) * ldy + n] = v;
     }
-    __syncthreads();
   }
   asm volatile("cp.async.wait_all;" ::: "memory");
 }
@@ -303,9 +337,10 @@ int mr_sms() {
 template <int KIND, int DEPTH>
 cudaError_t rows_launch(const void* x, int ldx, const void* w, void* y, int ldy, const void* items, const void* n_items, const void* token,
                         int groups, int likely, int N, int K, int act, size_t smem, cudaStream_t st) {
-  // split K over the warps of a block: shares of at least 16 steps, more splits where there are few tiles
+  // split K over the warps of a block: shares of at least 16 steps, more splits where a block would get fewer than eight tiles
+  // (the blocks' tile counts differ by one)
   int KW = 1;
-  while (KW < MR_WARPS && (K / 32 / (2 * KW) >= 16 || (long)groups * likely * KW < 2L * mr_sms() * MR_WARPS)) KW *= 2;
+  while (KW < MR_WARPS && (K / 32 / (2 * KW) >= 16 || (long)groups * likely * KW < 8L * mr_sms() * MR_WARPS)) KW *= 2;
   const int RW = MR_WARPS / KW, per_item = (groups + RW - 1) / RW;
   auto kern = moe_rows_kernel<KIND, DEPTH>;
   static bool configured = false;
@@ -331,6 +366,8 @@ TRL_API int trl_moe_plan(const MoePlanArgs* args, void* stream) {
   const int choose = a.T <= 64;
   cudaStream_t st = (cudaStream_t)stream;
   cudaError_t e = cudaSuccess;
+  const int pairs = a.T * (a.top + a.pieces);
+  if (pairs <= MQ_MAX && a.T <= 32) return (int)trl_launch(moe_plan_small_kernel, dim3(1), dim3(pairs <= 64 && a.T <= 2 ? 64 : MQ_MAX), 0, st, a);
   if (!choose) e = trl_launch(moe_topk_kernel, dim3((a.T + 7) / 8), dim3(256), 0, st, a);
   if (e == cudaSuccess) e = trl_launch(moe_plan_kernel, dim3(1), dim3(MP_THREADS), 0, st, a, choose);
   return (int)e;
