@@ -14,7 +14,7 @@
 //   sm_attn_plain_kernel        the same attention on CUDA cores: fp32 pools and heads beyond the tensor-core tiles.
 //
 // Scores, maxima, weights and sums are fp32; weights go into the value product as a bf16 pair (high part + rest).
-// Reference parity: the reference's attention has no sink, cap, window or differing widths (csrc/attn.cu is its counterpart).
+// Reference parity: the reference's attention has no sink, cap, window or differing widths (no counterpart).
 #include "packed.cuh"
 
 namespace {

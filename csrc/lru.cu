@@ -263,5 +263,5 @@ TRL_API int trl_lru_step(const LruArgs* a, int B, int f32, void* stream) {
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
   if (f32) return (int)step_launch<float, 16>(*a, B, st);
-  return (int)(B > 2 * LT_NB ? step_launch<bf16, 64>(*a, B, st) : step_launch<bf16, 16>(*a, B, st));
+  return (int)(B > LT_NB ? step_launch<bf16, 64>(*a, B, st) : step_launch<bf16, 16>(*a, B, st));
 }

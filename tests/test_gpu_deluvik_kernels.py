@@ -229,6 +229,33 @@ def test_recurrence_in_portions(ops, dtype, tol, spec):
         assert _rel(spool.states[10 - i, 0].view(b, r.pp)[:, :k].reshape(-1), s[-1]) < (1e-5 if dtype == torch.float32 else 2e-2)
 
 
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-6), (torch.bfloat16, 6e-3)])
+@pytest.mark.parametrize("taps,silu,biased", [(4, False, True), (3, True, False), (1, False, True), (6, False, False)])
+def test_convolution_of_long_prompts(ops, dtype, tol, taps, silu, biased):
+    """Sequences of unequal length whose borders fall anywhere, with and without earlier inputs."""
+    from tilerl_b200.batch import Batch
+    from tilerl_b200.ops import native as N
+    ch, rows = 272, 16
+    lens, starts = (333, 1, 2, 400, 17), (0, 5, 0, 2, 40)
+    batch = Batch.build([dict(tokens=[1] * n, start=s, blocks=[0] * 40, slot=i) for i, (n, s) in enumerate(zip(lens, starts))], "cuda")
+    t = sum(lens)
+    w, b, pre = _randn(taps, ch, seed=1), _randn(ch, seed=2), _randn(ch, seed=3)
+    proj, ring, out = torch.zeros(t, ch + 16, dtype=dtype, device="cuda"), torch.full((5, rows, ch), math.nan, dtype=dtype, device="cuda"), torch.zeros(t, ch, dtype=dtype, device="cuda")
+    want, o = [], 0
+    for i, (n, s) in enumerate(zip(lens, starts)):
+        x = _randn(n + s, ch, seed=10 + i).to(dtype)
+        proj[o:o + n, :ch], o = x[s:], o + n
+        for p in range(max(0, s - rows), s):
+            ring[i, p % rows] = x[p]
+        x = x.double().cpu() + (pre.double().cpu() if biased else 0.0)
+        y = (oracle.causal_conv(x, w.double().cpu().T) + b.double().cpu())[s:]
+        want.append(oracle.silu(y) if silu else y)
+    N.check(ops.lib.trl_scan_conv(proj.data_ptr(), proj.stride(0), w.data_ptr(), b.data_ptr(), pre.data_ptr() if biased else None, ring.data_ptr(), ring.stride(0),
+                                  rows, ring.stride(1), batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(),
+                                  batch.state_slots.data_ptr(), out.data_ptr(), t, ch, taps, int(silu), int(dtype == torch.float32), N.stream()))
+    assert _rel(out, torch.cat(want)) < tol
+
+
 # ---- experts ----------------------------------------------------------------------------------------------------
 MOES = [MoeSpec(24, 5, 2, 40), MoeSpec(64, 8, 8, 0), MoeSpec(192, 40, 6, 192), MoeSpec(100, 3, 1, 300), MoeSpec(256, 64, 4, 256)]
 

@@ -169,7 +169,7 @@ register("any", "sm100", {
     "sigmoid_attention": Kernel("sig_attn_kernel + sig_combine_kernel", "csrc/attn_sigmoid.cu", "trl_sigmoid_attn",
                                 note="bf16 packed pool; narrow row tiles for decoding, wide ones for prompts, key splits"),
     "join": Kernel("join_kernel", "csrc/join.cu", "trl_join", note="branch norm + stream addition + next norm; bf16 or fp32 rows"),
-    "clamped_glu": Kernel("glu_kernel", "csrc/join.cu", "trl_glu", note="few rows: epilogue of linear_rows_kernel"),
+    "glu": Kernel("glu_kernel", "csrc/join.cu", "trl_glu", note="few rows: epilogue of linear_rows_kernel"),
     "side_input": Kernel("side_kernel", "csrc/join.cu", "trl_side_input", note="few rows: epilogue of linear_rows_kernel"),
     "latent_prep": Kernel("latent_prep_kernel", "csrc/latent.cu", "trl_latent_prep", note="normed latents and rotated key into packed pages"),
     "latent_attention_decode": Kernel("latent_absorb_kernel + latent_decode_kernel + latent_out_kernel", "csrc/latent_mma.cu", "trl_latent_decode",
@@ -181,6 +181,18 @@ register("any", "sm100", {
     "scan_conv": Kernel("scan_conv_kernel", "csrc/scan.cu", "trl_scan_conv", note="causal convolution + silu of a tick's rows"),
     "scan_prefill": Kernel("scan_chunk_kernel", "csrc/scan_mma.cu", "trl_scan_chunk",
                            note="64-token chunks on tensor cores, fp32 state"),
+    "qkv_prep": Kernel("qkv_prep_kernel", "csrc/attn_softmax.cu", "trl_qkv_prep", note="short convolution, weighted norm, rotation, packed K / V write; bf16 or fp32"),
+    "softmax_attention": Kernel("sm_attn_kernel + sm_combine_kernel", "csrc/attn_softmax.cu", "trl_softmax_attn",
+                                note="window, score cap, sinks; narrow row tiles for decoding, wide ones for prompts, key splits; fp32: sm_attn_plain_kernel"),
+    "lru_decode": Kernel("lru_step_kernel", "csrc/lru.cu", "trl_lru_step", note="convolution, block-diagonal gates and recurrence of one token per sequence"),
+    "lru_prefill": Kernel("lru_scan_kernel", "csrc/lru.cu", "trl_lru_scan", note="gates from a library product; runs of tokens scanned from zero"),
+    "ring_store": Kernel("ring_store_kernel", "csrc/scan.cu", "trl_ring_store", note="last convolution inputs of a tick"),
+    "moe_plan": Kernel("moe_plan_small_kernel / moe_topk_kernel + moe_plan_kernel", "csrc/moe.cu", "trl_moe_plan", note="choice of experts, order by expert, tiles"),
+    "moe_rows": Kernel("moe_rows_kernel", "csrc/moe.cu", "trl_moe_rows", note="few rows: weight-streaming expert projections; fp32: moe_plain_kernel"),
+    "moe_gather": Kernel("moe_gather_kernel", "csrc/moe.cu", "trl_moe_gather"),
+    "moe_tc": Kernel("moe_tc_kernel", "csrc/moe_tc.cu", "trl_moe_tc", note="many rows: tcgen05 kind::f16, N follows the rows of an expert, gated epilogue from TMEM"),
+    "join_experts": Kernel("join_kernel", "csrc/join.cu", "trl_join_experts", note="weighted sum of a token's experts as the branch"),
+    "soft_cap": Kernel("cap_kernel", "csrc/join.cu", "trl_soft_cap", note="few rows: epilogue of linear_rows_kernel"),
     "batch_fill": Kernel("trl_batch_fill", "csrc/runtime.cpp", "trl_batch_fill", note="host runtime"),
     "pager": Kernel("trl_pager_*", "csrc/runtime.cpp", "trl_pager_alloc", note="host runtime"),
 })
