@@ -55,7 +55,7 @@ def _batch(lens, starts, slots=None):
 
 
 # ---- softmax attention ----------------------------------------------------------------------------------------
-SHAPES = [(1, 1, 16, 16), (6, 2, 48, 48), (4, 1, 64, 128), (3, 3, 20, 12), (20, 1, 128, 128), (4, 2, 256, 192), (8, 2, 128, 64), (5, 5, 72, 88)]
+SHAPES = [(1, 1, 16, 16), (6, 3, 40, 40), (7, 1, 64, 112), (3, 3, 20, 12), (20, 1, 128, 128), (4, 2, 256, 192), (8, 2, 128, 64), (5, 5, 72, 88)]
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-6), (torch.bfloat16, 6e-3)])
@@ -119,7 +119,7 @@ def test_one_key_far_back(ops, n, start, window):
         assert _rel(mid[-1], want) < 1e-2, at
 
 
-PREPS = [_spec(3, 1, 20, 20, tied=True, sink=True, cap=9.0), _spec(6, 2, 48, 32, conv=4), _spec(5, 5, 24, 40, norm="head", half=False, dims=8, window=9),
+PREPS = [_spec(3, 1, 20, 20, tied=True, sink=True, cap=9.0), _spec(6, 3, 56, 32, conv=4), _spec(5, 5, 24, 40, norm="head", half=False, dims=8, window=9),
          _spec(2, 1, 64, 16, conv=1, dims=32), _spec(16, 4, 128, 128, conv=3), _spec(4, 2, 40, 40, norm="head", half=True)]
 
 
