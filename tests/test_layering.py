@@ -8,7 +8,7 @@ ROOT = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))),
 
 # level of every top-level module / subpackage; imports may only point to the same or a lower level
 LEVEL = {
-    "config": 0, "mixers": 0, "zinutar_layout": 0, "fetotar_layout": 0, "deluvik_layout": 0, "formats": 0, "tokenizer": 0, "ledger": 0, "recipes": 0, "benchrec": 0, "build": 0,
+    "config": 0, "mixers": 0, "zinutar_layout": 0, "fetotar_layout": 0, "deluvik_layout": 0, "tobadra_layout": 0, "formats": 0, "tokenizer": 0, "ledger": 0, "recipes": 0, "benchrec": 0, "build": 0,
     "ops": 1, "tape": 1, "parallel": 1, "models": 1, "optim": 1,
     "batch": 2, "kv": 2, "kv_tiers": 2, "sparse": 2, "spec": 2, "graph": 2, "memory": 2, "kernel_cost": 2,
     "calibration": 2, "checkpoint": 2, "merge": 2, "mega": 2,

@@ -37,14 +37,15 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import ATTN, DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig
+from .config import ATTN, DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, TobadraConfig, ZinutarConfig
 from .formats import (FP8BlockTensor, NVFP4Tensor, dequantize_fp8_block, dequantize_nvfp4,
                       quantize_nvfp4)
 from .models.hybrid import HybridModel, linear_names, quantize_weight
 from .models.deluvik import DeluvikModel
 from .models.fetotar import FetotarModel
+from .models.tobadra import TobadraModel
 from .models.zinutar import ZinutarModel
-from . import deluvik_layout, fetotar_layout, zinutar_layout
+from . import deluvik_layout, fetotar_layout, tobadra_layout, zinutar_layout
 
 
 class CheckpointError(ValueError):
@@ -260,7 +261,7 @@ def assemble_master(cfg: ModelConfig, reader: _Reader) -> Dict[str, torch.Tensor
 
 
 STREAM_DESIGNS = {ZinutarConfig: (ZinutarModel, zinutar_layout), FetotarConfig: (FetotarModel, fetotar_layout),
-                  DeluvikConfig: (DeluvikModel, deluvik_layout)}
+                  DeluvikConfig: (DeluvikModel, deluvik_layout), TobadraConfig: (TobadraModel, tobadra_layout)}
 
 
 def load_stream_design(cfg: StreamDesign, path: str, device="cpu", dtype: Optional[torch.dtype] = None):

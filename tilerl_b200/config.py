@@ -1,9 +1,10 @@
 """Model configurations: the hybrid (gated-GQA attention + Gated-DeltaNet) decoder, and the stream designs
 (:class:`StreamDesign`: an fp32 residual stream, served in bf16 or fp32 on one GPU per process; no counterpart in the
 reference): Zinutar (:class:`ZinutarConfig`, a looped decoder of parallel blocks), Fetotar (:class:`FetotarConfig`,
-sandwich-normed layers of latent attention, Mamba-2 and mLSTM with a per-layer token input) and Deluvik
+sandwich-normed layers of latent attention, Mamba-2 and mLSTM with a per-layer token input), Deluvik
 (:class:`DeluvikConfig`, softmax attention with sinks, shared keys and short convolutions, a gated linear recurrence beside
-windowed attention, mixtures of experts, norms on every branch's output).
+windowed attention, mixtures of experts, norms on every branch's output) and Tobadra (:class:`TobadraConfig`, windowed attention
+over turned values, lightning attention and a per-channel delta rule, grouped experts, gated branches).
 
 One frozen dataclass describes every shape the kernels, the KV pools, the
 tensor-parallel shard tables and the cost model derive from.  Layer kinds are
@@ -22,8 +23,8 @@ from dataclasses import dataclass, replace
 from importlib import import_module
 from typing import Dict, Optional, Tuple
 
-from .mixers import (MIXERS, BandScalingSpec, ClampedGluSpec, GluSpec, LatentAttnSpec, LayerSpec, LruSpec, Mamba2Spec, MlstmSpec, MoeSpec,
-                     ParallelSpec, RotarySpec, SoftmaxAttnSpec, YarnSpec, take)
+from .mixers import (MIXERS, BandScalingSpec, ChannelDeltaSpec, ClampedGluSpec, DenseSpec, GluSpec, LatentAttnSpec, LayerSpec, LightningSpec,
+                     LruSpec, Mamba2Spec, MlstmSpec, MoeSpec, ParallelSpec, RotarySpec, RouterSpec, SoftmaxAttnSpec, YarnSpec, take)
 
 ATTN = "attn"
 GDN = "gdn"
@@ -230,6 +231,10 @@ class StreamDesign:
     n_gdn_layers = 0
     gdn_k_heads = gdn_v_heads = gdn_head_dim = gdn_conv_dim = 0
 
+    @classmethod
+    def from_dir(cls, j: Dict, path: str, name: str):
+        """The configuration of a checkpoint directory whose ``config.json`` is ``j``."""
+        return cls.from_json(j, name=name)
 
     @property
     def layout(self):
@@ -685,9 +690,175 @@ def deluvik_small() -> DeluvikConfig:
                            repeats=1, window=1024)
 
 
-ARCHITECTURES = {c.architecture: c for c in (ZinutarConfig, FetotarConfig, DeluvikConfig)}
+# ---- Tobadra: turned values, lightning attention, per-channel delta rule, grouped experts, gated branches ------------
+def tensor_shapes_in(path: str) -> Dict[str, Tuple[int, ...]]:
+    """Shapes of the tensors in a directory's safetensors files, from their headers."""
+    out: Dict[str, Tuple[int, ...]] = {}
+    for f in sorted(os.listdir(path)):
+        if f.endswith(".safetensors"):
+            with open(os.path.join(path, f), "rb") as fh:
+                head = json.loads(fh.read(int.from_bytes(fh.read(8), "little")))
+            out.update({k: tuple(v["shape"]) for k, v in head.items() if k != "__metadata__"})
+    return out
+
+
+@dataclass(frozen=True)
+class TobadraConfig(StreamDesign):
+    """Sizes and constants of a Tobadra model.  Every layer has its own mixer and feed-forward; attention layers number the KV
+    caches.  A layer with ``weights_of`` uses another layer's parameters and keeps a cache or state of its own."""
+    name: str
+    hidden: int
+    vocab: int
+    layers: Tuple[LayerSpec, ...]
+    canon: int                       # taps of the convolution on every mixer's input
+    logit_scale: float = 1.0
+    norm_eps: float = 1e-6
+    max_ctx: int = 1 << 20
+
+    architecture = "Tobadra"
+    tie_embeddings = True
+    MIXERS = (SoftmaxAttnSpec, LightningSpec, ChannelDeltaSpec)
+
+    def __post_init__(self) -> None:
+        object.__setattr__(self, "layers", tuple(self.layers))
+        if self.hidden <= 0 or self.vocab <= 0 or not self.layers or self.canon < 1:
+            raise ValueError("a model needs positive sizes, a tap and at least one layer")
+        for i, l in enumerate(self.layers):
+            if not isinstance(l.mixer, self.MIXERS):
+                raise ValueError(f"layer {i}: not a mixer of this design: {l.mixer}")
+            if l.weights_of is not None:
+                src = self.layers[l.weights_of] if 0 <= l.weights_of < len(self.layers) else None
+                if src is None or src.weights_of is not None or (src.mixer, src.mlp) != (l.mixer, l.mlp):
+                    raise ValueError(f"layer {i} cannot use the parameters of layer {l.weights_of}")
+
+    def source(self, layer: int) -> int:
+        """The layer whose parameters this one uses."""
+        src = self.layers[layer].weights_of
+        return layer if src is None else src
+
+    @property
+    def owners(self) -> Tuple[int, ...]:
+        """Layers with parameters of their own."""
+        return tuple(i for i, l in enumerate(self.layers) if l.weights_of is None)
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    def attn(self, layer: int) -> SoftmaxAttnSpec:
+        return self.layers[layer].mixer
+
+    @property
+    def cache_owners(self) -> Tuple[int, ...]:
+        """Layers with a KV cache, in the order of the caches."""
+        return tuple(i for i, l in enumerate(self.layers) if not l.mixer.recurrent)
+
+    def cache_index(self, layer: int) -> int:
+        return self.cache_owners.index(layer)
+
+    @property
+    def n_attn_layers(self) -> int:
+        return len(self.cache_owners)
+
+    @property
+    def n_q_heads(self) -> int:
+        return max([self.attn(i).heads for i in self.cache_owners] + [1])
+
+    @property
+    def n_kv_heads(self) -> int:
+        return max([self.attn(i).kv_heads for i in self.cache_owners] + [1])
+
+    def n_params(self) -> int:
+        from .tobadra_layout import tensor_shapes
+        return sum(math.prod(s) for s in tensor_shapes(self).values())
+
+    # ---- config.json -----------------------------------------------------------------------
+    @classmethod
+    def from_json(cls, j: Dict, name: str = "tobadra", max_ctx: Optional[int] = None, shapes: Optional[Dict] = None) -> "TobadraConfig":
+        """``shapes``: the checkpoint's tensor shapes, which hold the ranks of low-rank maps."""
+        take(j, ("architecture", "width", "vocab", "norm", "canon", "logit_scale", "layers"), "configuration")
+        take(j["norm"], ("eps",), "norm"), take(j["canon"], ("taps",), "canon")
+        layers = []
+        for i, l in enumerate(j["layers"]):
+            l = take({"mlp": None, "weights_of": None, **l}, ("type", "mixer", "mlp", "weights_of"), f"layer {i}")
+            m, f, src, where = l["mixer"], l["mlp"], l["weights_of"], f"layer {i} mixer"
+            if l["type"] == "attention":
+                m = SoftmaxAttnSpec.from_json(m, where, norm="none", half=True, windowed=True, bias=True, turned=True)
+                if m.rot.scaling is not None:
+                    raise ValueError(f"{where}: this design's rotations are not scaled")
+            elif l["type"] == "lightning":
+                m = LightningSpec.from_json(m, where)
+            elif l["type"] == "channel_delta":
+                ranks = [(shapes or {}).get(f"l{i if src is None else src}.mix.{n}") for n in ("a1", "g1")]
+                if None in ranks:
+                    raise ValueError(f"{where}: the checkpoint does not have the maps whose shapes tell its ranks")
+                m = ChannelDeltaSpec.from_json(m, where, *(r[0] for r in ranks))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+            if f is not None:
+                if f.get("kind") not in ("dense", "moe"):
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {f.get('kind')!r}")
+                f = DenseSpec.from_json(f, f"layer {i} mlp", "gelu") if f["kind"] == "dense" else MoeSpec.from_json_grouped(f, f"layer {i} mlp", "gelu_erf")
+            layers.append(LayerSpec(m, f, None if src is None else int(src)))
+        return cls(name=name, hidden=int(j["width"]), vocab=int(j["vocab"]), layers=tuple(layers), canon=int(j["canon"]["taps"]),
+                   logit_scale=float(j["logit_scale"]), norm_eps=float(j["norm"]["eps"]), **({} if max_ctx is None else {"max_ctx": max_ctx}))
+
+    @classmethod
+    def from_dir(cls, j: Dict, path: str, name: str) -> "TobadraConfig":
+        return cls.from_json(j, name=name, shapes=tensor_shapes_in(path))
+
+    def to_json(self) -> Dict:
+        layers = []
+        for l in self.layers:
+            layers.append({"type": l.mixer.type, "mixer": l.mixer.to_json(), "mlp": None if l.mlp is None else l.mlp.to_json()})
+            if l.weights_of is not None:
+                layers[-1]["weights_of"] = l.weights_of
+        return {"architecture": self.architecture, "width": self.hidden, "vocab": self.vocab, "norm": {"eps": self.norm_eps},
+                "canon": {"taps": self.canon}, "logit_scale": self.logit_scale, "layers": layers}
+
+
+def tobadra_attention(heads, kv_heads, dim, vdim, scale, window, dims, base=10000.0) -> SoftmaxAttnSpec:
+    """Windowed attention with biases whose values turn with their positions."""
+    return SoftmaxAttnSpec(heads, kv_heads, dim, vdim, scale, RotarySpec(dims, base, None, True), "none", window, bias=True, turned=True)
+
+
+def tobadra_moe(ff, experts, top, shared=0, scale=1.0, identity=0, groups=1, keep=1) -> MoeSpec:
+    return MoeSpec(ff, experts, top, shared, "gelu_erf", False, shared > 0, RouterSpec(scale, identity, groups, keep))
+
+
+def tobadra_tiny() -> TobadraConfig:
+    """Smoke model: every mixer, shared parameters, both feed-forwards and none, byte vocabulary of 320."""
+    moe, delta = tobadra_moe(40, 7, 2, 56, 1.3, 2, 3, 2), ChannelDeltaSpec(4, 2, 24, 16, 4, 12, 20)
+    return TobadraConfig(
+        name="tobadra-tiny", hidden=72, vocab=320, canon=3, logit_scale=0.5, norm_eps=1e-5, max_ctx=4096,
+        layers=(LayerSpec(tobadra_attention(4, 2, 24, 20, 0.2, 24, 16), DenseSpec(100, "gelu")),
+                LayerSpec(delta, moe), LayerSpec(LightningSpec(3, 16, 24, (0.7, 0.95, 0.995)), None),
+                LayerSpec(delta, moe, weights_of=1)))
+
+
+def tobadra_uniform(name: str, *, hidden: int, vocab: int, ff: int, expert_ff: int, experts: int, top: int, heads: int, kv_heads: int,
+                    repeats: int, window: int, dim: int = 128, rank: int = 128, identity: int = 0, groups: int = 1, keep: int = 1, **kw) -> TobadraConfig:
+    """A model of ``repeats`` x (channel delta, lightning, attention, channel delta) layers of one width; the first of the four has a
+    dense feed-forward, the others experts and a shared one."""
+    moe, layers = tobadra_moe(expert_ff, experts, top, expert_ff, 1.0, identity, groups, keep), []
+    delta = ChannelDeltaSpec(heads, heads, dim, dim, 4, rank, rank)
+    decay = tuple(1.0 - 2.0 ** (-4.0 - 6.0 * i / max(1, heads - 1)) for i in range(heads))
+    for _ in range(repeats):
+        layers += [LayerSpec(delta, DenseSpec(ff, "gelu")), LayerSpec(LightningSpec(heads, dim, dim, decay), moe),
+                   LayerSpec(tobadra_attention(heads, kv_heads, dim, dim, dim ** -0.5, window, dim), moe), LayerSpec(delta, moe)]
+    return TobadraConfig(name=name, hidden=hidden, vocab=vocab, layers=tuple(layers), canon=4, **kw)
+
+
+def tobadra_small() -> TobadraConfig:
+    """Four layers of a 1B-class width; profiler captures and GPU engine tests."""
+    return tobadra_uniform("tobadra-small", hidden=2048, vocab=32768, ff=8192, expert_ff=1024, experts=32, top=4, heads=16, kv_heads=4,
+                           repeats=1, window=1024, identity=8, groups=4, keep=2)
+
+
+ARCHITECTURES = {c.architecture: c for c in (ZinutarConfig, FetotarConfig, DeluvikConfig, TobadraConfig)}
 
 _REGISTRY = {
+    "tobadra-tiny": tobadra_tiny, "tobadra-small": tobadra_small,
     "deluvik-tiny": deluvik_tiny, "deluvik-small": deluvik_small,
     "fetotar-tiny": fetotar_tiny, "fetotar-small": fetotar_small,
     "zinutar-tiny": zinutar_tiny, "zinutar-small": zinutar_small, "zinutar-8b": zinutar_8b,
@@ -704,7 +875,7 @@ def config_from_dir(path: str):
         j = json.load(f)
     arch = j.get("architecture")
     if arch in ARCHITECTURES:
-        return ARCHITECTURES[arch].from_json(j, name=os.path.basename(os.path.normpath(path)))
+        return ARCHITECTURES[arch].from_dir(j, path, os.path.basename(os.path.normpath(path)))
     if j.get("name") in _REGISTRY:
         return _REGISTRY[j["name"]]()
     raise ValueError(f"{path}/config.json names neither a known architecture ({sorted(ARCHITECTURES)}) nor a known model")

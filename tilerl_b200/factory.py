@@ -20,19 +20,20 @@ from typing import Dict, Optional
 
 import torch
 
-from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig, get_config
+from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, TobadraConfig, ZinutarConfig, get_config
 from .engine import Engine, StepLimits
 from .formats import NVFP4Tensor
 from .kv import NoPrefixStore, PrefixStore, kv_pages, make_kv_pool, make_state_pool
 from .models.deluvik import DeluvikModel
 from .models.fetotar import FetotarModel
+from .models.tobadra import TobadraModel
 from .models.hybrid import HybridModel, linear_names, param_shapes, quantize_weight
 from .models.zinutar import ZinutarModel
 from .ops.backend import RefOps
 from .ops.ref import KV_BLOCK
 
 
-STREAM_MODELS = {ZinutarConfig: ZinutarModel, FetotarConfig: FetotarModel, DeluvikConfig: DeluvikModel}
+STREAM_MODELS = {ZinutarConfig: ZinutarModel, FetotarConfig: FetotarModel, DeluvikConfig: DeluvikModel, TobadraConfig: TobadraModel}
 
 
 def _seed_for(name: str, seed: int) -> int:

@@ -31,8 +31,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
-from . import deluvik_layout, fetotar_layout
-from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign
+from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, TobadraConfig
 from .fetotar_layout import LatentLayout, layout_of
 from .ops.ref import KV_BLOCK
 
@@ -273,7 +272,7 @@ def kv_pages(cfg, itemsize: int) -> Tuple[object, ...]:
     """Page layout of every KV cache of a design whose layers differ in size (one per execution of an attention layer)."""
     if isinstance(cfg, FetotarConfig):
         return tuple(LatentPage.of(layout_of(m), itemsize) for m in cfg.attn_mixers)
-    if isinstance(cfg, DeluvikConfig):
+    if isinstance(cfg, (DeluvikConfig, TobadraConfig)):
         return tuple(KvPage(a.kv_heads, a.dim, a.vdim, itemsize, False) for a in map(cfg.attn, cfg.cache_owners))
     return tuple(KvPage(a.kv_heads, a.dim, a.vdim, itemsize)
                  for a in (cfg.layers[run.layer].mixer for run in cfg.runs))
@@ -391,14 +390,15 @@ class GdnStatePool:
 
 def state_layouts(cfg) -> Tuple[object, ...]:
     """What a design's layers keep per sequence beside keys and values, in the order of the states."""
-    return (deluvik_layout if isinstance(cfg, DeluvikConfig) else fetotar_layout).state_layouts(cfg)
+    return cfg.layout.state_layouts(cfg)
 
 
 class RecurrentPool:
     """State slots of layers that differ in form and size: ``states [slots, planes, floats]`` fp32, every layer's record
     at a fixed offset (``fetotar_layout``: ``S [heads, dk, dv]``, then an mLSTM's key sum and running maximum;
-    ``deluvik_layout``: a vector, or nothing where only a convolution's inputs are kept), and a ring ``[slots, rows, channels]`` of convolution inputs indexed by ``position % rows``.  ``planes`` and
-    ``cur`` work as in :class:`GdnStatePool`."""
+    ``deluvik_layout``: a vector, or nothing where only a convolution's inputs are kept; ``tobadra_layout``: ``S``, or nothing),
+    and a ring ``[slots, rows, channels]`` of convolution inputs indexed by ``position % rows``.  ``planes`` and ``cur`` work as in
+    :class:`GdnStatePool`."""
 
     def __init__(self, cfg: FetotarConfig, num_slots: int, device="cpu", planes: int = 1, ring_dtype=torch.bfloat16):
         self.cfg, self.num_slots, self.planes = cfg, int(num_slots), int(planes)
@@ -469,7 +469,7 @@ class RecurrentPool:
 def make_state_pool(cfg, num_slots: int, device="cpu", *, planes: int = 1, ring_dtype=torch.bfloat16,
                     n_v_heads: Optional[int] = None, n_k_heads: Optional[int] = None):
     """The pool a configuration's recurrent layers keep their state in (it also hands out the slots of designs without any)."""
-    if isinstance(cfg, (FetotarConfig, DeluvikConfig)):
+    if isinstance(cfg, (FetotarConfig, DeluvikConfig, TobadraConfig)):
         return RecurrentPool(cfg, num_slots, device, planes=planes, ring_dtype=ring_dtype)
     return GdnStatePool(cfg, num_slots, device, planes=planes, ring_dtype=ring_dtype, n_v_heads=n_v_heads, n_k_heads=n_k_heads)
 

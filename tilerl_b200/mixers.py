@@ -222,10 +222,11 @@ MIXERS = {c.type: c for c in (LatentAttnSpec, Mamba2Spec, MlstmSpec)}
 @dataclass(frozen=True)
 class SoftmaxAttnSpec:
     """Causal softmax attention of ``heads`` query heads over ``kv_heads`` key / value heads (contiguous groups).  Queries and
-    keys are RMS-normalised with a weight, over the whole projection (``norm`` "all") or per head ("head"), then rotated.
-    Optional: a ``window`` (a query sees itself and the ``window - 1`` tokens before it), a soft cap on scores (``cap``), a
-    learned ``sink`` per head in the denominator, a short convolution of ``conv`` taps on every projection, values that are
-    the projected keys (``tied``), keys and values of an earlier layer (``kv_from``)."""
+    keys are RMS-normalised with a weight, over the whole projection (``norm`` "all") or per head ("head"), or not ("none"),
+    then rotated.  Optional: a ``window`` (a query sees itself and the ``window - 1`` tokens before it), a soft cap on scores
+    (``cap``), a learned ``sink`` per head in the denominator, a short convolution of ``conv`` taps on every projection, values
+    that are the projected keys (``tied``), keys and values of an earlier layer (``kv_from``), a ``bias`` on every projection,
+    values that are ``turned`` by their position over the whole head and whose weighted sum is turned back by the query's."""
     heads: int
     kv_heads: int
     dim: int
@@ -239,6 +240,11 @@ class SoftmaxAttnSpec:
     conv: int = 0
     tied: bool = False
     kv_from: Optional[int] = None
+    bias: bool = False
+    turned: bool = False
+
+    type = "attention"
+    recurrent = False
 
     def __post_init__(self) -> None:
         _positive("attention", self.heads, self.kv_heads, self.dim, self.vdim)
@@ -246,11 +252,17 @@ class SoftmaxAttnSpec:
             raise ValueError(f"attention needs heads a multiple of kv_heads: {self}")
         if self.rot.dims > self.dim:
             raise ValueError("more rotated dimensions than a head has")
-        if self.norm not in ("all", "head") or self.conv < 0 or (self.window is not None and self.window < 1) or \
+        if self.norm not in ("all", "head", "none") or self.conv < 0 or (self.window is not None and self.window < 1) or \
                 (self.cap is not None and self.cap <= 0):
             raise ValueError(f"attention: {self}")
         if self.tied and (self.dim != self.vdim or self.kv_from is not None):
             raise ValueError("values that are the keys have their size and their layer")
+        if self.turned and (self.tied or not self.rot.half or self.vdim % 2):
+            raise ValueError("turned values have an even size, are not the keys and turn in halves")
+
+    def value_frequencies(self) -> Tuple[float, ...]:
+        """Radians per position of every pair of a turned value (never scaled)."""
+        return RotarySpec(self.vdim, self.rot.base).frequencies()
 
     @property
     def channels(self) -> int:
@@ -264,7 +276,7 @@ class SoftmaxAttnSpec:
 
     @classmethod
     def from_json(cls, m: Dict, where: str, *, norm: str, half: bool, capped: bool = False, windowed: bool = False, conv: bool = False,
-                  sink: bool = False, tied: bool = False) -> "SoftmaxAttnSpec":
+                  sink: bool = False, tied: bool = False, bias: bool = False, turned: bool = False) -> "SoftmaxAttnSpec":
         """The keyword arguments say which of the optional parts the design's mixer has."""
         m = dict(m)
         source = m.pop("kv_from", None) if conv else None
@@ -273,7 +285,8 @@ class SoftmaxAttnSpec:
             take(m["mask"], ("size",), where + " mask")
         return cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
                    RotarySpec.from_json(m["rot"], where + " rot", BandScalingSpec, half), norm, int(m["mask"]["size"]) if windowed else None,
-                   float(m["softcap"]) if capped else None, sink, int(m["conv"]) if conv else 0, tied, None if source is None else int(source))
+                   float(m["softcap"]) if capped else None, sink, int(m["conv"]) if conv else 0, tied, None if source is None else int(source),
+                   bias, turned)
 
     def to_json(self) -> Dict:
         out: Dict = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale,
@@ -309,6 +322,66 @@ class LruSpec:
 
     def to_json(self) -> Dict:
         return asdict(self)
+
+
+@dataclass(frozen=True)
+class LightningSpec:
+    """Linear attention whose per-head sum of ``k v^T`` (``dim`` x ``vdim``) fades by a fixed factor a token (``decay``, one per
+    head); queries, keys and values pass silu, the heads' outputs one RMS norm together and a sigmoid gate."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]
+
+    type = "lightning"
+    recurrent = True
+
+    def __post_init__(self) -> None:
+        object.__setattr__(self, "decay", tuple(float(d) for d in self.decay))
+        _positive("lightning", self.heads, self.dim, self.vdim)
+        if len(self.decay) != self.heads or not all(0.0 < d <= 1.0 for d in self.decay):
+            raise ValueError(f"lightning: one decay in (0, 1] per head: {self}")
+
+    @classmethod
+    def from_json(cls, m: Dict, where: str) -> "LightningSpec":
+        take(m, ("heads", "dim", "vdim", "decay"), where)
+        return cls(int(m["heads"]), int(m["dim"]), int(m["vdim"]), tuple(m["decay"]))
+
+    def to_json(self) -> Dict:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "decay": list(self.decay)}
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """Delta rule with one decay per key channel: per head a sum of ``k u^T`` (``dim`` x ``vdim``) whose rows fade on their own,
+    ``u`` being the part of the value that the faded sum does not hold yet, scaled by a gate.  Queries and keys (``kv_heads``
+    heads, shared by contiguous groups) and values pass a short convolution of ``conv`` taps; the decays and the output gate
+    are maps of low rank (``decay_rank``, ``gate_rank``)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    decay_rank: int
+    gate_rank: int
+
+    type = "channel_delta"
+    recurrent = True
+
+    def __post_init__(self) -> None:
+        _positive("channel delta", self.heads, self.kv_heads, self.dim, self.vdim, self.conv, self.decay_rank, self.gate_rank)
+        if self.heads % self.kv_heads:
+            raise ValueError(f"channel delta needs heads a multiple of kv_heads: {self}")
+
+    @classmethod
+    def from_json(cls, m: Dict, where: str, decay_rank: int, gate_rank: int) -> "ChannelDeltaSpec":
+        """The ranks are no part of the dictionary: a checkpoint's tensors have them."""
+        names = ("heads", "kv_heads", "dim", "vdim", "conv")
+        take(m, names, where)
+        return cls(*(int(m[n]) for n in names), int(decay_rank), int(gate_rank))
+
+    def to_json(self) -> Dict:
+        return {n: getattr(self, n) for n in ("heads", "kv_heads", "dim", "vdim", "conv")}
 
 
 @dataclass(frozen=True)
@@ -365,20 +438,70 @@ class GluSpec:
 
 
 @dataclass(frozen=True)
+class DenseSpec:
+    """``W_down act(W_up h)``."""
+    ff: int
+    act: str                  # "gelu" (its tanh form), "gelu_erf" or "silu"
+    kind = "dense"
+
+    def __post_init__(self) -> None:
+        _positive("feed-forward", self.ff)
+        if self.act not in ("gelu", "gelu_erf", "silu"):
+            raise ValueError(f"unknown activation {self.act!r}")
+
+    @classmethod
+    def from_json(cls, f: Dict, where: str, act: str) -> "DenseSpec":
+        take(f, ("ff", "kind"), where)
+        return cls(int(f["ff"]), act)
+
+    def to_json(self) -> Dict:
+        return {"kind": self.kind, "ff": self.ff}
+
+
+@dataclass(frozen=True)
+class RouterSpec:
+    """Choice by scores that are the softmax over all outputs, plus a learned correction that the weights (scores times ``scale``)
+    do not see.  Outputs form ``groups`` equal groups of neighbours, of which the ``keep`` with the largest choice score can be
+    chosen from; the last ``identity`` outputs stand for the input itself."""
+    scale: float = 1.0
+    identity: int = 0
+    groups: int = 1
+    keep: int = 1
+
+    MAX_GROUPS = 64
+
+    def check(self, experts: int, top: int) -> None:
+        n = experts + self.identity
+        if self.identity < 0 or not 1 <= self.keep <= self.groups <= self.MAX_GROUPS or n % self.groups or n // self.groups * self.keep < top:
+            raise ValueError(f"router: {experts} experts, {top} chosen: {self}")
+
+
+@dataclass(frozen=True)
 class MoeSpec:
-    """``experts`` gated feed-forwards of width ``ff``, of which a token uses the ``top`` with the largest router logits, weighted
-    by the softmax over those; ``shared`` (0: none) is the width of one that every token uses."""
+    """``experts`` feed-forwards of width ``ff`` (``gated`` or plain), of which a token uses ``top``; ``shared`` (0: none) is the width
+    of one that every token uses, with weight one or (``shared_gate``) a sigmoid of the token's own.  Without ``router``, the
+    experts with the largest router logits are chosen, weighted by the softmax over those."""
     ff: int
     experts: int
     top: int
     shared: int = 0
     act: str = "silu"
+    gated: bool = True
+    shared_gate: bool = False
+    router: Optional[RouterSpec] = None
     kind = "moe"
 
     def __post_init__(self) -> None:
         _positive("experts", self.ff, self.experts, self.top)
-        if self.top > self.experts or self.shared < 0 or self.act not in ("gelu", "silu"):
+        if self.top > self.outputs or self.shared < 0 or self.act not in (("gelu", "silu") if self.gated else ("gelu", "gelu_erf", "silu")):
             raise ValueError(f"experts: {self}")
+        if self.router is not None:
+            self.router.check(self.experts, self.top)
+
+    @property
+    def outputs(self) -> int:
+        """Outputs of the router: experts, then the input itself."""
+        return self.experts + (self.router.identity if self.router else 0)
 
     @classmethod
     def from_json(cls, f: Dict, where: str) -> "MoeSpec":
@@ -389,8 +512,22 @@ class MoeSpec:
         return cls(int(f["expert"]["ff"]), int(f["router"]["experts"]), int(f["router"]["top"]),
                    0 if f["shared"] is None else int(f["shared"]["ff"]))
 
+    @classmethod
+    def from_json_grouped(cls, f: Dict, where: str, act: str) -> "MoeSpec":
+        """Plain experts behind a :class:`RouterSpec`, the shared one gated."""
+        f = take({"shared": None, **f}, ("kind", "expert", "router", "shared"), where)
+        r = take({"identity": 0, "groups": {"count": 1, "keep": 1}, **f["router"]}, ("experts", "top", "scale", "identity", "groups"), where + " router")
+        take(f["expert"], ("ff",), where + " expert"), take(r["groups"], ("count", "keep"), where + " groups")
+        if f["shared"] is not None:
+            take(f["shared"], ("ff",), where + " shared")
+        return cls(int(f["expert"]["ff"]), int(r["experts"]), int(r["top"]), 0 if f["shared"] is None else int(f["shared"]["ff"]), act, False,
+                   f["shared"] is not None, RouterSpec(float(r["scale"]), int(r["identity"]), int(r["groups"]["count"]), int(r["groups"]["keep"])))
+
     def to_json(self) -> Dict:
+        r = self.router
         out: Dict = {"kind": self.kind, "expert": {"ff": self.ff}, "router": {"experts": self.experts, "top": self.top}}
+        if r is not None:
+            out["router"].update(scale=r.scale, identity=r.identity, groups={"count": r.groups, "keep": r.keep})
         if self.shared:
             out["shared"] = {"ff": self.shared}
         return out
@@ -398,6 +535,8 @@ class MoeSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    """One layer: a mixer and, unless ``mlp`` is None, a feed-forward after it."""
+    """One layer: a mixer and, unless ``mlp`` is None, a feed-forward after it.  ``weights_of``: the earlier layer whose parameters
+    it uses (with a cache or state of its own)."""
     mixer: object
     mlp: Optional[object] = None
+    weights_of: Optional[int] = None

@@ -1,8 +1,8 @@
-"""fp32 torch form of the stream designs' mechanisms (latent and softmax attention, decayed scans, linear recurrence, experts,
-norms, gates) and, on top of them, the op surface :class:`RefMixers` that ``models/fetotar.py`` and ``models/deluvik.py`` call;
-mixed into :class:`~tilerl_b200.ops.backend.RefOps`.  The CUDA twins are :mod:`tilerl_b200.ops.cuda_mixers` and
-:mod:`tilerl_b200.ops.cuda_blocks`.  No counterpart in the
-reference.
+"""fp32 torch form of the stream designs' mechanisms (latent and softmax attention, decayed scans, delta rule, linear recurrence,
+experts, norms, gates) and, on top of them, the op surface :class:`RefMixers` that ``models/fetotar.py``, ``models/deluvik.py`` and
+``models/tobadra.py`` call; mixed into :class:`~tilerl_b200.ops.backend.RefOps`.  The CUDA twins are
+:mod:`tilerl_b200.ops.cuda_mixers`, :mod:`tilerl_b200.ops.cuda_blocks` and :mod:`tilerl_b200.ops.cuda_gated`.  No counterpart in
+the reference.
 """
 from __future__ import annotations
 
@@ -116,13 +116,27 @@ def lru_step(state, u, r, i, lam):
 
 
 def activate(z, act: str):
-    return gelu_tanh(z) if act == "gelu" else F.silu(z)
+    """"gelu" (its tanh form), "gelu_erf" or "silu"."""
+    return gelu_tanh(z) if act == "gelu" else F.gelu(z) if act == "gelu_erf" else F.silu(z)
 
 
 def choose(logits, top: int):
     """(experts ``[T, top]``, their weights): the largest logits (the first of equal ones), softmax over those."""
     best, idx = torch.sort(logits, dim=1, descending=True, stable=True)
     return idx[:, :top], torch.softmax(best[:, :top], dim=1)
+
+
+def choose_grouped(z, correction, top: int, r):
+    """(outputs ``[T, top]``, their weights): scores are the softmax over all outputs; the largest score plus correction among the
+    outputs of the ``r.keep`` groups whose largest is largest."""
+    s = torch.softmax(z, dim=1)
+    c = s + correction
+    t, n = c.shape
+    best = c.view(t, r.groups, -1).amax(2)
+    order = torch.sort(best, dim=1, descending=True, stable=True).indices[:, :r.keep]
+    kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, order, True).repeat_interleave(n // r.groups, dim=1)
+    idx = torch.sort(c.masked_fill(~kept, -math.inf), dim=1, descending=True, stable=True).indices[:, :top]
+    return idx, s.gather(1, idx) * r.scale
 
 
 # ---- decayed scans ---------------------------------------------------------------------------------------
@@ -154,6 +168,20 @@ def mlstm_step(state, n, m, q, k, v, i, f):
     return s, n, new, torch.einsum("hdv,hd->hv", s, q) / den[:, None]
 
 
+def unit_heads(x):
+    """Vectors of length one along the last dimension."""
+    return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
+
+
+def delta_step(state, q, k, v, log_keep, beta):
+    """``state [H, D, V]``; ``q, k, log_keep [H, D]``, ``v [H, V]``, ``beta [H]``: fade every row, write what of the value is not there
+    yet, read."""
+    s = torch.exp(log_keep)[:, :, None] * state
+    u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", s, k))
+    s = s + k[:, :, None] * u[:, None, :]
+    return s, torch.einsum("hdv,hd->hv", s, q)
+
+
 def grouped_rms(y, heads: int, vdim: int, dv: int, groups: int, eps: float):
     """RMS norm without a weight over ``groups`` equal parts of the true columns of ``y [T, heads * dv]``."""
     t = y.shape[0]
@@ -181,7 +209,7 @@ class RefMixers:
         """(fused projection rows, fp32 gate rows)."""
         return ref.linear(h, w[:n_in]).to(self.act_dtype), ref.linear(h, w[n_in:])
 
-    def project_f32(self, a, w):
+    def project_f32(self, a, w, name="branch"):
         return ref.linear(a, w)
 
     def project_logits(self, h, w, cap=0.0):
@@ -260,14 +288,18 @@ class RefMixers:
             ref.packed_kv_write(pool.layer(idx), pool.pages[idx], k.to(pool.dtype), v.to(pool.dtype), batch.slot_mapping, eps)
         return turn(q, batch.positions, freqs).to(self.act_dtype), torch.zeros(t, l.n_out, dtype=self.act_dtype, device=proj.device)
 
-    def softmax_attention(self, q, mid, a, sink, factor, batch, pool, idx):
-        """Attention output of every token, times ``factor``, into the first columns of ``mid``."""
+    def softmax_attention(self, q, mid, a, sink, factor, batch, pool, idx, turn=None):
+        """Attention output of every token, times ``factor``, into the first columns of ``mid``; with ``turn`` (cos and sin per token
+        and pair ``[T, dv / 2, 2]``) turned back first."""
         s = a.spec
         for i in range(q.shape[0]):
             p = int(batch.positions[i])
             k, v = ref.packed_kv_gather(pool.layer(idx), pool.pages[idx], pool.dtype, batch.block_table[int(batch.seq_ids[i])], p + 1)
             lo = 0 if s.window is None else max(0, p + 1 - s.window)
             o = softmax_attention(q[i].float(), k[lo:], v[lo:], s.scale, s.cap, sink)
+            if turn is not None:
+                (x, y), (c, sn) = o.chunk(2, dim=1), turn[i].unbind(1)
+                o = torch.cat([x * c + y * sn, y * c - x * sn], 1)
             mid[i, :a.n_out] = (o * factor).reshape(-1).to(self.act_dtype)
 
     # ---- gated linear recurrence -----------------------------------------------------------
@@ -313,6 +345,124 @@ class RefMixers:
 
     def join_experts(self, x, y, post, nxt, eps, n):
         return self.join(x, y, post, nxt, eps, n)
+
+    # ---- gated branches with a convolution on the next input ----------------------------------
+    def _input_conv(self, h, conv):
+        """``h`` plus its causal convolution, or None without one (``conv``: taps, batch, state pool, index of the inputs kept)."""
+        if conv is None:
+            return None
+        w, batch, spool, idx = conv
+        out = torch.empty_like(h)
+        for i in range(h.shape[0]):
+            ring = spool.ring_view(idx, int(batch.state_slots[int(batch.seq_ids[i])]))
+            out[i] = h[i] + (self._conv_inputs(h[i], ring, int(batch.positions[i]), w.shape[0]) * w).sum(0)
+        return out.to(self.act_dtype)
+
+    def embed_normed(self, table, vocab, ids, post, nxt, eps, n, conv):
+        """(stream, its normed row, that row convolved): the normed embedding."""
+        x = stream_norm(ref.embedding(table[:vocab], ids), post, eps, n)
+        h = stream_norm(x, nxt, eps, n).to(self.act_dtype)
+        return x, h, self._input_conv(h, conv)
+
+    def gated_join(self, x, y, bias, z, z_b, post, nxt, eps, n, conv):
+        """``x += norm_post((y + bias) sigmoid(z + z_b))``; returns (``norm_nxt(x)``, that row convolved)."""
+        y = (y if bias is None else y + bias) * torch.sigmoid(z + z_b)
+        h = self.join(x, y, post, nxt, eps, n)
+        return h, self._input_conv(h, conv)
+
+    def project_in(self, h, hc, w, n_in, n_gates, n_act=0, act="silu"):
+        """(rows of the mixer, the first ``n_act`` through ``act``; fp32 rows of its gates; fp32 rows of its branch's gate): the last
+        rows of ``w`` read ``h``, the others ``hc``."""
+        n = n_in + n_gates
+        proj = ref.linear(hc, w[:n_in])
+        proj[:, :n_act] = activate(proj[:, :n_act], act)
+        return proj.to(self.act_dtype), ref.linear(hc, w[n_in:n]), ref.linear(h, w[n:])
+
+    def up_act(self, h, w, n, act):
+        """(``act`` of the first ``n`` rows, the other rows in fp32)."""
+        return activate(ref.linear(h, w[:n]), act).to(self.act_dtype), ref.linear(h, w[n:])
+
+    def turned_prep(self, proj, l, bias, freqs, vfreqs, batch, pool, idx):
+        """Biased and turned queries ``[T, heads, dk]``; turned keys and values into the cache; the input of the output projection;
+        cos and sin of the values' turns."""
+        a, s, t = l.attn, l.attn.spec, proj.shape[0]
+        rows = proj.float() + bias
+        q, k, v = (rows[:, c:c + h * d].reshape(t, h, d) for c, h, d in ((0, s.heads, a.dk), (a.k0, s.kv_heads, a.dk), (a.v0, s.kv_heads, a.dv)))
+        q, k, v = (rotate_halves(x, batch.positions, f) for x, f in ((q, freqs), (k, freqs), (v, vfreqs)))
+        ref.packed_kv_write(pool.layer(idx), pool.pages[idx], k.to(pool.dtype), v.to(pool.dtype), batch.slot_mapping, 0.0)
+        ang = batch.positions.to(torch.float64)[:, None] * vfreqs.to(proj.device)[None, :]
+        turn = torch.stack([ang.cos(), ang.sin()], -1).float()
+        return q.to(self.act_dtype), torch.zeros(t, l.n_out, dtype=self.act_dtype, device=proj.device), turn
+
+    def _scan_tokens(self, l, batch, spool, sidx, step):
+        """``step(token, state, ring) -> (state, row)`` along every sequence; states move on in ``spool``."""
+        y = torch.zeros(batch.n_tokens, l.heads * l.dv, dtype=torch.float32, device=batch.positions.device)
+        for r in range(batch.n_seqs):
+            s0, n, slot = int(batch.q_start[r]), int(batch.q_len[r]), int(batch.state_slots[r])
+            if n == 0:
+                continue
+            keep = bool(batch.keep_steps) and batch.keep_rows[r]
+            live = spool.view(sidx, slot, int(spool.cur[slot]))[0]
+            state, ring = live.clone(), spool.ring_view(sidx, slot)
+            for j in range(n):
+                state, o = step(s0 + j, state, ring)
+                y[s0 + j] = o.reshape(-1)
+                if keep:
+                    spool.view(sidx, slot, j)[0].copy_(state)
+            if not keep:
+                live.copy_(state)
+        return y
+
+    def _gated_heads(self, y, z, norm, l, eps):
+        out = torch.zeros(y.shape[0], l.n_out, dtype=self.act_dtype, device=y.device)
+        out[:, :l.heads * l.dv] = (grouped_rms(y, l.heads, l.vdim, l.dv, l.norm_groups, eps) * norm * torch.sigmoid(z.float())).to(self.act_dtype)
+        return out
+
+    def lightning_mix(self, proj, log_decay, norm, l, batch, spool, sidx, eps):
+        keep = torch.exp(log_decay)[:, None, None]
+
+        def step(t, s, ring):
+            q, k, v = (proj[t, c:c + l.heads * d].float().view(l.heads, d) for c, d in ((0, l.dk), (l.k0, l.dk), (l.v0, l.dv)))
+            s = keep * s + k[:, :, None] * v[:, None, :]
+            return s, torch.einsum("hdv,hd->hv", s, q)
+        return self._gated_heads(self._scan_tokens(l, batch, spool, sidx, step), proj[:, l.g0:], norm, l, eps)
+
+    def delta_mix(self, proj, gates, w, norm, l, batch, spool, sidx, eps):
+        a = ref.linear(proj[:, l.a0:l.a0 + l.ra], w["a2"]) + w["dt_bias"]
+        log_keep = -torch.exp(w["a_log"])[None, :, None] * F.softplus(a).view(-1, l.heads, l.dk)
+        beta = torch.sigmoid(gates[:, :l.heads].float())
+        z = ref.linear(proj[:, l.g0:l.g0 + l.rg], w["g2"])
+        zero = torch.zeros(l.conv_c, device=proj.device)
+
+        def step(t, s, ring):
+            c = conv_rows(self._conv_inputs(proj[t, :l.conv_c], ring, int(batch.positions[t]), l.taps), w["conv"], zero).to(self.act_dtype).float()
+            q, k = (unit_heads(c[o:o + l.k0].view(l.kv_heads, l.dk)).repeat_interleave(l.per, 0) for o in (0, l.k0))
+            return delta_step(s, q * l.spec.dim ** -0.5, k, c[l.v0:].view(l.heads, l.dv), log_keep[t], beta[t])
+        return self._gated_heads(self._scan_tokens(l, batch, spool, sidx, step), z, norm, l, eps)
+
+    def routed_experts(self, h, z, correction, up, down, m):
+        """Weighted sum of the chosen experts' outputs, the shared one and the input's own share; ``z``: rows of the fused router."""
+        s = m.spec
+        idx, weight = choose_grouped(z[:, :s.outputs], correction[:s.outputs], s.top, s.router)
+        y = torch.zeros(h.shape[0], down.shape[1], dtype=torch.float32, device=h.device)
+        for e in range(s.outputs + m.pieces):
+            if e < s.outputs:
+                rows, place = torch.nonzero(idx == e, as_tuple=True)
+                scale = weight[rows, place][:, None]
+            else:
+                rows = torch.arange(h.shape[0], device=h.device)
+                scale = torch.sigmoid(z[:, s.outputs])[:, None] if s.shared_gate else 1.0
+            if not len(rows):
+                continue
+            if s.experts <= e < s.outputs:
+                y[rows] += scale * h[rows].float()
+                continue
+            j = e if e < s.experts else e - s.outputs + s.experts
+            y[rows] += scale * ref.linear(activate(ref.linear(h[rows], up[j]), s.act).to(self.act_dtype), down[j])
+        return y
+
+    def gated_join_experts(self, x, y, h, z, z_b, post, nxt, eps, n, conv):
+        return self.gated_join(x, y, None, z, z_b, post, nxt, eps, n, conv)
 
     # ---- recurrent mixers ------------------------------------------------------------------
     def recurrent_mix(self, proj, gates, w, l, batch, pool, idx, eps):
