@@ -3,7 +3,8 @@
 //
 //   qkv_prep_kernel             fused projection rows -> queries and cached keys / values of a token: an optional short convolution
 //                               (earlier rows from the slot's ring), RMS norm with a weight over the whole projection or per head,
-//                               rotation in halves or neighbouring pairs; two blocks per token.  Everything between the projection's
+//                               rotation in halves or neighbouring pairs; or no norm, a bias, and values that turn like keys; two blocks
+//                               per token.  Everything between the projection's
 //                               rounding and the final one is fp32.
 //   sm_attn_kernel<D, WM, WN>   tensor cores (mma.sync m16n8k16 bf16).  One block = (16 WM query rows, kv head, sequence, key split); a
 //                               row is a (token, head of the group) pair.  Keys come 64 at a time (four pages) into a ring of stages,
@@ -56,6 +57,9 @@ struct PrepArgs {
   int n_blocks;
   void* mid;                              // columns pad0 .. ldm - 1 are cleared
   int ldm, pad0;
+  const float* bias;                      // [n_in], added behind the convolution; or null
+  const double* vfreqs;                   // dv / 2 pairs (a value's halves) that turn with the position; or null
+  float2* turn;                           // [T, dv / 2] their cos and sin
 };
 
 // grid (token, part): part 0 = queries, part 1 = keys and values.  Weights of a tick take the read-only path (they are constants).
@@ -70,12 +74,19 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
   const int base = is_q ? 0 : a.k0, cols = is_q ? a.k0 : a.n_in - a.k0, heads = is_q ? a.heads : a.kv_heads;
   float* s_cs = s_row + cols;
   float* s_fac = s_cs + 2 * a.n_pairs;
+  float2* s_turn = reinterpret_cast<float2*>(s_fac + ((heads + 1) & ~1));
   pdl_wait();
   const int pos = a.positions[t], seq = a.seq_ids[t];
   const T* row = reinterpret_cast<const T*>(a.proj) + (size_t)t * a.ldp + base;
   T* ring = reinterpret_cast<T*>(a.ring) + (a.taps ? (size_t)a.slots[seq] * a.ring_slot + base : 0);
   const int t0 = a.q_start[seq];
   for (int i = tid; i < a.n_pairs; i += nt) pair_angle(pos, __ldg(a.freqs + i), 1.f, s_cs[2 * i], s_cs[2 * i + 1]);
+  if (!is_q && a.vfreqs)
+    for (int i = tid; i < a.dv / 2; i += nt) {
+      float2 cs;
+      pair_angle(pos, __ldg(a.vfreqs + i), 1.f, cs.x, cs.y);
+      s_turn[i] = cs, a.turn[(size_t)t * (a.dv / 2) + i] = cs;
+    }
   for (int c = tid * C; c < cols; c += nt * C) {
     const uint4 own = *reinterpret_cast<const uint4*>(row + c);
     float f[C];
@@ -101,6 +112,13 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
       for (int e = 0; e < C; ++e) f[e] = acc[e];
       if (a.write_ring) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.ring_rows) * a.ring_ld + c) = own;
     }
+    if (a.bias) {
+#pragma unroll
+      for (int e = 0; e < C; e += 4) {
+        const float4 b = __ldg(reinterpret_cast<const float4*>(a.bias + base + c + e));
+        f[e] += b.x, f[e + 1] += b.y, f[e + 2] += b.z, f[e + 3] += b.w;
+      }
+    }
 #pragma unroll
     for (int e = 0; e < C; e += 4) *reinterpret_cast<float4*>(s_row + c + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
   }
@@ -108,7 +126,9 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
     for (int c = a.pad0 + tid; c < a.ldm; c += nt) reinterpret_cast<T*>(a.mid)[(size_t)t * a.ldm + c] = from_f<T>(0.f);
   __syncthreads();
   // ---- norm factors (padding columns hold zeros)
-  if (a.norm_all) {
+  if (!a.q_norm) {
+    for (int h = tid; h < heads; h += nt) s_fac[h] = 1.f;
+  } else if (a.norm_all) {
     float ss = 0.f;
     for (int c = tid * 4; c < heads * a.dk; c += nt * 4) {
       const float4 v = *reinterpret_cast<const float4*>(s_row + c);
@@ -138,15 +158,16 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
   auto scaled = [&](const float* src, const float* w, float fac, int d, float (&o)[C]) {
 #pragma unroll
     for (int e = 0; e < C; e += 4) {
-      const float4 v = *reinterpret_cast<const float4*>(src + d + e), g = __ldg(reinterpret_cast<const float4*>(w + d + e));
+      const float4 v = *reinterpret_cast<const float4*>(src + d + e);
+      const float4 g = norm ? __ldg(reinterpret_cast<const float4*>(w + d + e)) : make_float4(1.f, 1.f, 1.f, 1.f);
       o[e] = v.x * fac * g.x, o[e + 1] = v.y * fac * g.y, o[e + 2] = v.z * fac * g.z, o[e + 3] = v.w * fac * g.w;
     }
   };
   for (int x = tid; x < heads * kch; x += nt) {
     const int h = x / kch, ci = x - h * kch, d0 = ci * C;
     const float* src = s_row + h * a.dk;
-    const float* w = norm + (a.norm_all ? h * a.dk : 0);
-    const float fac = s_fac[a.norm_all ? 0 : h];
+    const float* w = norm + (norm && a.norm_all ? h * a.dk : 0);
+    const float fac = s_fac[norm && a.norm_all ? 0 : h];
     float o[C];
     scaled(src, w, fac, d0, o);
     if (d0 < 2 * a.n_pairs) {
@@ -176,7 +197,7 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
           if (d < 2 * a.n_pairs) {
             const bool second = d >= a.n_pairs;
             const int p = second ? d - a.n_pairs : d, m = second ? p : d + a.n_pairs;
-            const float u = src[m] * fac * w[m], c = s_cs[2 * p], s = s_cs[2 * p + 1];
+            const float u = src[m] * fac * (norm ? w[m] : 1.f), c = s_cs[2 * p], s = s_cs[2 * p + 1];
             o[e] = second ? fmaf(o[e], c, u * s) : fmaf(o[e], c, -u * s);
           }
         }
@@ -200,6 +221,14 @@ __global__ void __launch_bounds__(512) qkv_prep_kernel(const PrepArgs a) {
       const float4 v = *reinterpret_cast<const float4*>(src + e);
       o[e] = v.x, o[e + 1] = v.y, o[e + 2] = v.z, o[e + 3] = v.w;
     }
+    if (a.vfreqs) {                                         // a chunk turns with the one half a head away
+      const int half = a.dv / 2, d0 = c * C;
+      const bool second = d0 >= half;
+      const float* other = second ? src - half : src + half;
+      const float2* cs = s_turn + (second ? d0 - half : d0);
+#pragma unroll
+      for (int e = 0; e < C; ++e) o[e] = second ? fmaf(o[e], cs[e].x, other[e] * cs[e].y) : fmaf(o[e], cs[e].x, -other[e] * cs[e].y);
+    }
     uint4* vd = reinterpret_cast<uint4*>(page0 + (size_t)h * page_bytes + KVB * kch * 16);
     vd[r * vch + page_chunk(c, r, vch)] = Chunk<T>::put(o);
   }
@@ -220,6 +249,7 @@ struct SmArgs {
   float2* ml;                          // [T, n_q, n_splits] (maximum in powers of two, sum)
   int n_q, n_kv, n_splits, n_stages, window, min_len, max_len;
   float scale, cap, factor;
+  const float2* turn;                  // [T, dv / 2]: finished rows are turned back by these (their halves pair up); or null
 };
 
 // Keys [lo, hi) that the rows [row0, row0 + rows) of a sequence see; lo is a page's first.
@@ -227,6 +257,10 @@ __device__ __forceinline__ int2 tile_keys(const SmArgs& a, int row0, int rows, i
   const int hi = a.positions[q0 + (min(row0 + rows, n_rows) - 1) / G] + 1;
   const int lo = a.window > 0 ? max(0, a.positions[q0 + row0 / G] - a.window + 1) & ~(KVB - 1) : 0;
   return make_int2(lo, hi);
+}
+// A pair of a finished row, turned back by its query's angle.
+__device__ __forceinline__ float2 turn_back(float u, float v, const float2& cs) {
+  return make_float2(fmaf(u, cs.x, v * cs.y), fmaf(v, cs.x, -u * cs.y));
 }
 // Pages per split (a multiple of a stage), and splits that hold keys.
 __device__ __forceinline__ int split_pages(int keys, int n_splits) {
@@ -521,6 +555,31 @@ sm_attn_kernel(const SmArgs a) {
   auto dst_out = [&](int row) { return reinterpret_cast<bf16*>(a.out) + (size_t)(q0 + row / G) * a.ldo + (size_t)(kvh * G + row % G) * dv; };
   if constexpr (WN == 1) {
     if (warp == NWC) return;
+    if (a.turn && used == 1) {                              // a pair's halves meet in the (idle) ring
+      const int lds = dv + 8, half = dv / 2;
+      float* so = reinterpret_cast<float*>(ring) + (size_t)wm * 16 * lds;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int r = (lane >> 2) + 8 * i, row = row0 + wm * 16 + r;
+        if (row >= n_rows) continue;
+        const float2 f = with_sink(mx[i], sum[i], a.sink, kvh * G + row % G);
+        const float g = f.x / f.y * a.factor;
+#pragma unroll
+        for (int nd = 0; nd < D / 8; ++nd)
+          if (FULL || nd < vch) *reinterpret_cast<float2*>(so + r * lds + nd * 8 + (lane & 3) * 2) = make_float2(o[nd][2 * i] * g, o[nd][2 * i + 1] * g);
+      }
+      __syncwarp();
+      for (int x = lane; x < 16 * (half / 2); x += 32) {
+        const int r = x / (half / 2), m = x % (half / 2) * 2, row = row0 + wm * 16 + r;
+        if (row >= n_rows) break;
+        const float4 cs = *reinterpret_cast<const float4*>(a.turn + (size_t)(q0 + row / G) * half + m);
+        const float2 u = *reinterpret_cast<const float2*>(so + r * lds + m), v = *reinterpret_cast<const float2*>(so + r * lds + half + m);
+        const float2 p0 = turn_back(u.x, v.x, make_float2(cs.x, cs.y)), p1 = turn_back(u.y, v.y, make_float2(cs.z, cs.w));
+        *reinterpret_cast<uint32_t*>(dst_out(row) + m) = f2_to_bf162_bits(p0.x, p1.x);
+        *reinterpret_cast<uint32_t*>(dst_out(row) + half + m) = f2_to_bf162_bits(p0.y, p1.y);
+      }
+      return;
+    }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int row = row0 + wm * 16 + (lane >> 2) + 8 * i;
@@ -553,10 +612,12 @@ sm_attn_kernel(const SmArgs a) {
       }
     }
     __syncthreads();
-    const int rows = min(ROWS, n_rows - row0);
-    for (int x = threadIdx.x; x < rows * dv; x += THREADS) {
-      const int r = x / dv, d = x % dv, row = row0 + r;
-      float top = -INFINITY, l = 0.f, v = 0.f;
+    const int rows = min(ROWS, n_rows - row0), half = dv / 2;
+    const bool turned = a.turn && used == 1;                // a thread takes both of a pair
+    const int cols = turned ? half : dv;
+    for (int x = threadIdx.x; x < rows * cols; x += THREADS) {
+      const int r = x / cols, d = x % cols, row = row0 + r;
+      float top = -INFINITY, l = 0.f, v = 0.f, v2 = 0.f;
 #pragma unroll
       for (int k = 0; k < WN; ++k) top = fmaxf(top, s_m[k][r]);
 #pragma unroll
@@ -564,8 +625,14 @@ sm_attn_kernel(const SmArgs a) {
         const float e = rel_weight(s_m[k][r], top);
         l = fmaf(s_l[k][r], e, l);
         v = fmaf(so[((size_t)k * ROWS + r) * dv + d], e, v);
+        if (turned) v2 = fmaf(so[((size_t)k * ROWS + r) * dv + half + d], e, v2);
       }
-      if (used == 1) {
+      if (turned) {
+        const float2 f = with_sink(top, l, a.sink, kvh * G + row % G);
+        const float g = f.x / f.y * a.factor;
+        const float2 p = turn_back(v * g, v2 * g, a.turn[(size_t)(q0 + row / G) * half + d]);
+        dst_out(row)[d] = __float2bfloat16(p.x), dst_out(row)[half + d] = __float2bfloat16(p.y);
+      } else if (used == 1) {
         const float2 f = with_sink(top, l, a.sink, kvh * G + row % G);
         dst_out(row)[d] = __float2bfloat16(v * (f.x / f.y * a.factor));
       } else {
@@ -614,8 +681,20 @@ __global__ void __launch_bounds__(CB_THREADS) sm_combine_kernel(const SmArgs a, 
   }
   s_v[threadIdx.x] = v;
   __syncthreads();
+  if (grp == 0)
+    for (int k = 1; k < n_g; ++k) v.x += s_v[k * pairs + threadIdx.x].x, v.y += s_v[k * pairs + threadIdx.x].y;
+  if (a.turn) {                                             // (uniform) a pair's halves meet in shared memory
+    __syncthreads();
+    s_v[threadIdx.x] = v;
+    __syncthreads();
+    if (grp == 0) {
+      const bool second = d >= dv / 2;
+      const float2 o = s_v[second ? threadIdx.x - pairs / 2 : threadIdx.x + pairs / 2];
+      const float4 cs = *reinterpret_cast<const float4*>(a.turn + (size_t)t * (dv / 2) + (second ? d - dv / 2 : d));
+      v = second ? make_float2(fmaf(v.x, cs.x, -o.x * cs.y), fmaf(v.y, cs.z, -o.y * cs.w)) : make_float2(fmaf(v.x, cs.x, o.x * cs.y), fmaf(v.y, cs.z, o.y * cs.w));
+    }
+  }
   if (grp) return;
-  for (int k = 1; k < n_g; ++k) v.x += s_v[k * pairs + threadIdx.x].x, v.y += s_v[k * pairs + threadIdx.x].y;
   *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(a.out) + (size_t)t * a.ldo + (size_t)h * dv + d) = f2_to_bf162_bits(v.x * g, v.y * g);
 }
 
@@ -685,13 +764,26 @@ __global__ void __launch_bounds__(256) sm_attn_plain_kernel(const SmArgs a) {
       }
     }
   }
-  if (!in) return;
   float g = 1.f;
   if (a.sink) {
     const float s = a.sink[h], top = fmaxf(m, s);
     g = expf(m - top), l = fmaf(l, g, expf(s - top));
   }
-  g = g / l * a.factor;
+  g = in ? g / l * a.factor : 0.f;
+  if (a.turn) {                                    // (uniform) a pair's halves meet where the values were
+    __syncthreads();
+    for (int i = 0; i < F_MAXD / 16; ++i)
+      if (c + 16 * i < dv) sv[r * dv + c + 16 * i] = acc[i] * g;
+    __syncwarp();                                  // a row's threads share a warp
+    if (!in) return;
+    for (int d = c; d < dv / 2; d += 16) {
+      const float2 p = turn_back(sv[r * dv + d], sv[r * dv + dv / 2 + d], a.turn[(size_t)t * (dv / 2) + d]);
+      T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.ldo + (size_t)h * dv + d;
+      out[0] = from_f<T>(p.x), out[dv / 2] = from_f<T>(p.y);
+    }
+    return;
+  }
+  if (!in) return;
   for (int i = 0; i < F_MAXD / 16; ++i)
     if (c + 16 * i < dv) reinterpret_cast<T*>(a.out)[(size_t)t * a.ldo + (size_t)h * dv + c + 16 * i] = from_f<T>(acc[i] * g);
 }
@@ -704,7 +796,8 @@ cudaError_t sm_launch_as(SmArgs a, int tiles, int B, const int* seq_ids, int n_t
   int stages = 4;
   while (stages > 2 && q_bytes + stages * stage > room) --stages;
   if (WM == 1 && stages < 3 && q_bytes + 3 * stage <= (size_t)SM_SMEM) stages = 3;
-  const size_t merge = WN > 1 ? (size_t)WN * ROWS * a.vch * 32 : 0;               // the merge of WN warps goes through the ring
+  // the merge of WN warps, or rows to be turned, go through the ring
+  const size_t merge = WN > 1 ? (size_t)WN * ROWS * a.vch * 32 : a.turn ? (size_t)ROWS * (a.vch * 32 + 32) : 0;
   const size_t smem = q_bytes + (stages * stage > merge ? stages * stage : merge);
   if (smem > (size_t)SM_SMEM) return cudaErrorInvalidValue;
   a.n_stages = stages;
@@ -736,12 +829,12 @@ TRL_API int trl_qkv_prep(const PrepArgs* args, int T, int f32, void* stream) {
   const PrepArgs& a = *args;
   const int per = f32 ? 4 : 8;
   const int widest = max(a.k0, a.n_in - a.k0);
-  const size_t smem = (size_t)(widest + 2 * a.n_pairs + max(a.heads, a.kv_heads) + 2) * sizeof(float);
+  const size_t smem = (size_t)(widest + 2 * a.n_pairs + max(a.heads, a.kv_heads) + 2 + (a.vfreqs ? a.dv : 0)) * sizeof(float);
   if (T <= 0 || a.ldp % per || a.n_in % 16 || a.n_in > a.ldp || a.dk % 16 || a.dv % 16 || a.heads <= 0 || a.kv_heads <= 0 || a.dim > a.dk ||
       2 * a.n_pairs > a.dim || a.k0 != a.heads * a.dk || a.n_in != (a.own ? a.v0 + a.kv_heads * a.dv : a.k0) || smem > 200 * 1024 ||
-      ((uintptr_t)a.proj & 15) || !a.q || !a.q_norm || (a.own && (!a.pages || !a.k_norm || ((uintptr_t)a.pages & 15))) ||
+      ((uintptr_t)a.proj & 15) || !a.q || (a.own && (!a.pages || !a.k_norm != !a.q_norm || ((uintptr_t)a.pages & 15))) ||
       (a.taps && (!a.conv || !a.ring || a.taps > a.ring_rows || a.ring_ld % per || a.ring_slot % per || ((uintptr_t)a.ring & 15))) ||
-      (a.mid && (a.pad0 < 0 || a.pad0 > a.ldm)))
+      (a.mid && (a.pad0 < 0 || a.pad0 > a.ldm)) || (a.vfreqs && (!a.turn || !a.own || a.v0 == a.k0)))
     return (int)cudaErrorInvalidValue;
   static bool configured = false;
   if (!configured) {
@@ -764,14 +857,14 @@ TRL_API int trl_softmax_attn_ok(int dk, int dv) { return dk <= 256 && dv <= 256;
 // q: [T, n_q * dk]; out: [T, ldo], first n_q * dv columns, times factor.  window 0: all earlier keys; cap 0: none; sink: fp32 [n_q] or
 // null.  Serves the sequences with min_len <= q_len <= max_len: wide = 0 in row tiles of 16 (key work split over four warps), wide = 1
 // in row tiles of trl_softmax_attn_rows(dk, dv), wide = 2 on CUDA cores (any length, no splits).  tiles: row tiles of the longest such
-// sequence.  part, ml: fp32 [T, n_q, n_splits, dv] and [T, n_q, n_splits, 2].
+// sequence.  turn: fp32 [T, dv / 2, 2] cos and sin by which finished rows are turned back, column d with d + dv / 2, or null.  part, ml: fp32 [T, n_q, n_splits, dv] and [T, n_q, n_splits, 2].
 TRL_API int trl_softmax_attn(const void* q, const void* pages, int n_blocks, const void* table, int max_blocks, const void* q_start,
                              const void* q_len, const void* positions, const void* seq_ids, const void* sink, void* out, int ldo, void* part,
                              void* ml, int T, int B, int tiles, int min_len, int max_len, int n_q, int n_kv, int dk, int dv, int n_splits,
-                             int wide, int window, float scale, float cap, float factor, int f32, void* stream) {
+                             int wide, int window, float scale, float cap, float factor, const void* turn, int f32, void* stream) {
   const int per = f32 ? 4 : 8;
   if (T <= 0 || B <= 0 || tiles <= 0 || n_kv <= 0 || n_q % n_kv || dk % 16 || dv % 16 || dk > F_MAXD || dv > F_MAXD || dk <= 0 || dv <= 0 ||
-      n_splits < 1 || n_splits > 64 || (n_splits > 1 && (!part || !ml)) || ldo % per || n_blocks <= 0 || window < 0 || cap < 0.f || ((uintptr_t)pages & 15) ||
+      n_splits < 1 || n_splits > 64 || (n_splits > 1 && (!part || !ml)) || ldo % per || n_blocks <= 0 || window < 0 || cap < 0.f || ((uintptr_t)turn & 15) || ((uintptr_t)pages & 15) ||
       ((uintptr_t)q & 15) || ((uintptr_t)out & 15) || (wide != 2 && (f32 || dk > 256 || dv > 256)))
     return (int)cudaErrorInvalidValue;
   SmArgs a;
@@ -780,7 +873,7 @@ TRL_API int trl_softmax_attn(const void* q, const void* pages, int n_blocks, con
   a.q_start = (const int*)q_start, a.q_len = (const int*)q_len, a.positions = (const int*)positions;
   a.sink = (const float*)sink, a.out = out, a.ldo = ldo, a.part = (float*)part, a.ml = (float2*)ml;
   a.n_q = n_q, a.n_kv = n_kv, a.n_splits = n_splits, a.n_stages = 2, a.window = window, a.min_len = min_len, a.max_len = max_len;
-  a.scale = scale, a.cap = cap, a.factor = factor;
+  a.scale = scale, a.cap = cap, a.factor = factor, a.turn = (const float2*)turn;
   cudaStream_t st = (cudaStream_t)stream;
   const int d = dk > dv ? dk : dv;
   const int* si = (const int*)seq_ids;

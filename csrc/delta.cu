@@ -1,0 +1,200 @@
+// Delta rule with one decay per key channel (models/tobadra.py).  Per head, with g_t the factors the rows of S keep:
+//
+//   S <- g_t S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
+//
+//   delta_prep_kernel    a tick's rows, a block per token: causal convolution and silu (earlier rows from the slot's ring), unit length of
+//                        every q / k head, log g = -exp(A) softplus(low + bias) per channel, beta = sigmoid(gate).
+//   delta_serial_kernel  token after token, 32 value columns of a head per block, the state in registers: decoding, windows of kept
+//                        states, short portions, and fp32 models.  o = (g S)^T q + (k . q) u, so a token needs one block barrier.
+//   (prompts: delta_mma.cu; the norm and gate behind it: scan_norm_kernel of scan.cu)
+//
+// q, k, decays, beta, state and sums are fp32; v is in the compute type, as its convolution leaves it.
+// Reference parity: the reference's delta rule has one decay per head (kernels_gdn.py of tilerl-kernels; no counterpart).
+#include "delta.cuh"
+
+namespace {
+
+template <typename T>
+__global__ void __launch_bounds__(512) delta_prep_kernel(const DeltaArgs a) {
+  constexpr int C = Chunk<T>::N;
+  extern __shared__ __align__(16) float s_row[];               // [2 k0] convolved q and k
+  pdl_launch_dependents(70);
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nt = blockDim.x, nw = nt >> 5;
+  const int pos = a.positions[t], seq = a.seq_ids[t], t0 = a.q_start[seq];
+  const T* row = reinterpret_cast<const T*>(a.rows) + (size_t)t * a.ldp;
+  T* ring = reinterpret_cast<T*>(a.ring) + (size_t)a.slots[seq] * a.ring_slot;
+  for (int c = tid * C; c < a.channels; c += nt * C) {
+    const uint4 own = *reinterpret_cast<const uint4*>(row + c);
+    float f[C], acc[C];
+    Chunk<T>::get(own, f);
+#pragma unroll
+    for (int e = 0; e < C; ++e) acc[e] = 0.f;
+    for (int back = 0; back < a.taps && back <= pos; ++back) {
+      if (back) {
+        const T* src = t - back >= t0 ? row - (size_t)back * a.ldp + c : ring + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + c;
+        Chunk<T>::get(*reinterpret_cast<const uint4*>(src), f);
+      }
+#pragma unroll
+      for (int e = 0; e < C; e += 4) {
+        const float4 w = __ldg(reinterpret_cast<const float4*>(a.conv_w + (size_t)(a.taps - 1 - back) * a.channels + c + e));
+        acc[e] = fmaf(f[e], w.x, acc[e]), acc[e + 1] = fmaf(f[e + 1], w.y, acc[e + 1]);
+        acc[e + 2] = fmaf(f[e + 2], w.z, acc[e + 2]), acc[e + 3] = fmaf(f[e + 3], w.w, acc[e + 3]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
+    if (a.write_ring) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.ring_rows) * a.ring_ld + c) = own;
+    const uint4 out = Chunk<T>::put(acc);
+    if (c >= a.v0) {
+      *reinterpret_cast<uint4*>(reinterpret_cast<T*>(a.v) + (size_t)t * a.heads * a.dv + c - a.v0) = out;
+    } else {
+      Chunk<T>::get(out, f);                                   // (as the compute type holds it)
+#pragma unroll
+      for (int e = 0; e < C; e += 4) *reinterpret_cast<float4*>(s_row + c + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+    }
+  }
+  const int n = a.heads * a.dk;
+  for (int c = tid * 4; c < n; c += nt * 4) {
+    const float4 x = load4(a.low + (size_t)t * n + c), b = __ldg(reinterpret_cast<const float4*>(a.dt_bias + c));
+    const float r = -expf(a.a_log[c / a.dk]);
+    *reinterpret_cast<float4*>(a.keep + (size_t)t * n + c) =
+        make_float4(r * softplus_x(x.x + b.x), r * softplus_x(x.y + b.y), r * softplus_x(x.z + b.z), r * softplus_x(x.w + b.w));
+  }
+  for (int h = tid; h < a.heads; h += nt) a.beta[(size_t)t * a.heads + h] = sigmoid_x(a.gates[(size_t)t * a.ldg + h]);
+  __syncthreads();
+  for (int h = warp; h < 2 * a.kv_heads; h += nw) {
+    const float* src = s_row + h * a.dk;
+    float ss = 0.f;
+    for (int d = lane; d < a.dk; d += 32) ss = fmaf(src[d], src[d], ss);
+    const bool is_q = h < a.kv_heads;
+    const float f = (is_q ? a.q_scale : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+    float* dst = (is_q ? a.q : a.k) + ((size_t)t * a.kv_heads + (is_q ? h : h - a.kv_heads)) * a.dk;
+    for (int d = lane; d < a.dk; d += 32) dst[d] = src[d] * f;
+  }
+}
+
+// grid (heads * column slices, sequences), 256 threads: lane = column, warp = dk / 8 state rows
+template <typename T, int RMAX>
+__global__ void __launch_bounds__(256, RMAX <= 16 ? 4 : 2) delta_serial_kernel(const DeltaArgs a) {
+  constexpr int DK = RMAX * 8, TB = RMAX <= 16 ? 16 : 8;
+  __shared__ float s_q[TB][DK], s_k[TB][DK], s_g[TB][DK], s_v[TB][32], s_beta[TB], s_kq[TB];
+  __shared__ float s_p[2][8][32], s_o[2][8][32];
+  pdl_launch_dependents(71);
+  const int n_sl = (a.dv + 31) / 32, h = blockIdx.x / n_sl, col0 = (blockIdx.x % n_sl) * 32, seq = blockIdx.y, kh = h / (a.heads / a.kv_heads);
+  const int T_ = a.q_len[seq], t0 = a.q_start[seq];
+  if (T_ < a.min_len || T_ > a.max_len) {
+    pdl_wait();                              // (a launch ends no sooner than those before it)
+    return;
+  }
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, R = a.dk / 8, col = col0 + lane;
+  const int slot = a.slots[seq], plane = a.cur[slot];
+  const bool keep_all = a.keep_flags && a.keep_flags[seq];
+  float* rec = a.states + (size_t)slot * a.slot_stride;
+  const size_t s_off = ((size_t)h * a.dk + warp * R) * a.dv + col;
+  float S[RMAX];
+  {
+    // (before the dependency wait: the state's last writer is the previous tick, and every tick has launches in between that let their
+    // dependents in only after their own wait)
+    const float* src = rec + (size_t)plane * a.plane_stride;
+#pragma unroll
+    for (int r = 0; r < RMAX; ++r) S[r] = r < R && col < a.dv ? src[s_off + (size_t)r * a.dv] : 0.f;
+  }
+  pdl_wait();
+  auto save = [&](int pl) {
+    float* dst = rec + (size_t)pl * a.plane_stride;
+#pragma unroll
+    for (int r = 0; r < RMAX; ++r)
+      if (r < R && col < a.dv) dst[s_off + (size_t)r * a.dv] = S[r];
+  };
+  const T* vb = reinterpret_cast<const T*>(a.v);
+  for (int i0 = 0; i0 < T_; i0 += TB) {
+    const int nb = min(TB, T_ - i0);
+    __syncthreads();
+    for (int x = tid; x < nb * a.dk; x += 256) {
+      const int j = x / a.dk, d = x % a.dk;
+      const size_t t = t0 + i0 + j;
+      s_q[j][d] = a.q[(t * a.kv_heads + kh) * a.dk + d];
+      s_k[j][d] = a.k[(t * a.kv_heads + kh) * a.dk + d];
+      s_g[j][d] = expf(a.keep[(t * a.heads + h) * a.dk + d]);
+    }
+    for (int x = tid; x < nb * 32; x += 256)
+      s_v[x >> 5][x & 31] = col0 + (x & 31) < a.dv ? to_f(vb[((size_t)(t0 + i0 + (x >> 5)) * a.heads + h) * a.dv + col0 + (x & 31)]) : 0.f;
+    if (tid < nb) s_beta[tid] = a.beta[(size_t)(t0 + i0 + tid) * a.heads + h];
+    __syncthreads();
+    for (int j = warp; j < nb; j += 8) {
+      float d = 0.f;
+      for (int c = lane; c < a.dk; c += 32) d = fmaf(s_q[j][c], s_k[j][c], d);
+      d = warp_sum(d);
+      if (lane == 0) s_kq[j] = d;
+    }
+    __syncthreads();
+    for (int j = 0; j < nb; ++j) {
+      const float *kr = &s_k[j][warp * R], *qr = &s_q[j][warp * R], *gr = &s_g[j][warp * R];
+      float p = 0.f, o = 0.f;
+#pragma unroll
+      for (int r = 0; r < RMAX; ++r) {
+        if (r < R) {
+          S[r] *= gr[r];
+          p = fmaf(kr[r], S[r], p);
+          o = fmaf(qr[r], S[r], o);
+        }
+      }
+      s_p[j & 1][warp][lane] = p, s_o[j & 1][warp][lane] = o;
+      __syncthreads();
+      p = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) p += s_p[j & 1][w][lane];
+      const float u = s_beta[j] * (s_v[j][lane] - p);
+#pragma unroll
+      for (int r = 0; r < RMAX; ++r)
+        if (r < R) S[r] = fmaf(kr[r], u, S[r]);
+      if (keep_all) save(i0 + j);
+      if (warp == 0 && col < a.dv) {
+        o = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) o += s_o[j & 1][w][lane];
+        a.o[((size_t)(t0 + i0 + j) * a.heads + h) * a.dv + col] = fmaf(s_kq[j], u, o);
+      }
+    }
+  }
+  if (!keep_all) save(plane);
+}
+
+template <typename T> cudaError_t serial_launch(const DeltaArgs& a, int B, cudaStream_t st) {
+  const dim3 grid(a.heads * ((a.dv + 31) / 32), B);
+  if (a.dk <= 32) return trl_launch(delta_serial_kernel<T, 4>, grid, dim3(256), 0, st, a);
+  if (a.dk <= 64) return trl_launch(delta_serial_kernel<T, 8>, grid, dim3(256), 0, st, a);
+  if (a.dk <= 128) return trl_launch(delta_serial_kernel<T, 16>, grid, dim3(256), 0, st, a);
+  return trl_launch(delta_serial_kernel<T, 32>, grid, dim3(256), 0, st, a);
+}
+
+}  // namespace
+
+// args: filled by the caller.  write_ring: the rows go into the ring (one token per sequence; else trl_ring_store does it afterwards).
+TRL_API int trl_delta_prep(const DeltaArgs* args, int T, int f32, void* stream) {
+  const DeltaArgs& a = *args;
+  const int per = f32 ? 4 : 8;
+  const size_t smem = (size_t)2 * a.k0 * sizeof(float);
+  if (T <= 0 || delta_args_bad(a) || smem > 200 * 1024 || a.taps < 1 || a.taps > a.ring_rows || a.ldp % per || a.channels > a.ldp || a.ldg < a.heads ||
+      a.ring_ld % per || a.ring_slot % per || !a.rows || !a.conv_w || !a.ring || !a.low || !a.dt_bias || !a.a_log || !a.gates || !a.positions ||
+      !a.seq_ids || !a.q_start || !a.slots || ((uintptr_t)a.rows & 15) || ((uintptr_t)a.ring & 15) || ((uintptr_t)a.low & 15) || ((uintptr_t)a.keep & 15))
+    return (int)cudaErrorInvalidValue;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const int threads = a.channels >= 4096 ? 512 : 256;
+  if (f32) return (int)trl_launch(delta_prep_kernel<float>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, a);
+  return (int)trl_launch(delta_prep_kernel<bf16>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, a);
+}
+
+// Serves sequences of min_len..max_len tokens, whose rows trl_delta_prep has prepared.
+TRL_API int trl_delta_serial(const DeltaArgs* args, int B, int f32, void* stream) {
+  const DeltaArgs& a = *args;
+  if (B <= 0 || delta_args_bad(a) || !a.states || !a.o || !a.cur || !a.q_start || !a.q_len || !a.slots) return (int)cudaErrorInvalidValue;
+  return (int)(f32 ? serial_launch<float>(a, B, (cudaStream_t)stream) : serial_launch<bf16>(a, B, (cudaStream_t)stream));
+}

@@ -1,9 +1,11 @@
-// Element-wise middle of sandwich-normed layers over an fp32 stream (models/fetotar.py):
+// Element-wise middle of sandwich-normed layers over an fp32 stream (models/fetotar.py, models/deluvik.py, models/tobadra.py):
 //
 //   join_kernel       x += norm_post(y) and h = norm_next(x) in the next projection's input type, a row per block; each
 //                     norm is a layer norm (weight and bias), an RMS norm (weight) or, for h, nothing but the rounding.
 //                     With a table it starts the stream instead: x = table[id] * scale.
-//                     The branch may also come as the rows of a token's experts, summed with their weights.
+//                     The branch may also come as the rows of a token's experts (or its own input), summed with their weights, may be
+//                     gated by its input (sigmoid) and, in ticks of one token per sequence, h may pass a short causal convolution.
+//   act_kernel        act(z), in place.
 //   glu_kernel        act(g) u over interleaved (gate, up) columns: silu, gelu (tanh form), or g sigmoid(1.702 g) (u + 1) with
 //                     the gate bounded above, up on both sides.
 //   cap_kernel        cap tanh(x / cap), in place.
@@ -50,20 +52,42 @@ __device__ __forceinline__ float4 apply_norm(const float4& v, const float2& st, 
   return o;
 }
 
+}  // namespace
+
+// Mirrored by tilerl_b200/ops/cuda_gated.py::JoinArgs, field by field (null pointers leave a step out).
+struct JoinArgs {
+  float* x;
+  const void* y;
+  const float *post, *next;
+  void* h;
+  const void* table;                   // starts the stream: rows of ld values of h's type
+  const int* ids;
+  const int* place;                    // rows y[place[t, j]], weighted; negative: the token's row of `own`
+  const float* weight;
+  const void* own;                     // of h's type; may be h itself
+  const float *bias, *z, *z_b;         // branch = (y + bias) sigmoid(z + z_b)
+  void* hc;                            // h plus its causal convolution (one token per sequence)
+  const float* conv_w;                 // [taps, ld]
+  void* ring;                          // earlier inputs: the layer's first column of slot 0
+  const int *positions, *seq_ids, *state_slots;
+  long ring_slot;
+  int post_kind, next_kind, V, ld, n, slots, y_bf16, ldz, taps, ring_rows, ring_ld;
+  float scale, eps;
+};
+
+namespace {
+
 template <typename T, int R>
-__global__ void __launch_bounds__(512)
-join_kernel(float* x, const float* y, const float* __restrict__ post, int post_kind, const float* __restrict__ next, int next_kind,
-            T* h, const T* __restrict__ table, const int* ids, float scale, int V, int ld, int n, float eps, const int* place,
-            const float* weight, int slots, int y_bf16) {
+__global__ void __launch_bounds__(512) join_kernel(const JoinArgs a) {
   __shared__ float red[32];
   pdl_launch_dependents(30);
   pdl_wait();
-  const int t = blockIdx.x;
-  float* xr = x + (size_t)t * ld;
+  const int t = blockIdx.x, ld = a.ld, n = a.n;
+  float* xr = a.x + (size_t)t * ld;
   float4 v[R];
-  if (table) {
-    int id = ids[t];
-    if (id < 0 || id >= V) {               // never read outside the table: zero row + error word {BOUNDS, 8, token, id}
+  if (a.table) {
+    int id = a.ids[t];
+    if (id < 0 || id >= a.V) {             // never read outside the table: zero row + error word {BOUNDS, 8, token, id}
       if (threadIdx.x == 0) trl_set_error(TRL_ERR_BOUNDS, 8, t, id);
       id = -1;
     }
@@ -72,14 +96,26 @@ join_kernel(float* x, const float* y, const float* __restrict__ post, int post_k
       const int k = (threadIdx.x + i * blockDim.x) * 4;
       v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (k < ld) {
-        if (id >= 0) v[i] = load4(table + (size_t)id * ld + k);
-        v[i].x *= scale, v[i].y *= scale, v[i].z *= scale, v[i].w *= scale;
-        *reinterpret_cast<float4*>(xr + k) = v[i];
+        if (id >= 0) v[i] = load4(reinterpret_cast<const T*>(a.table) + (size_t)id * ld + k);
+        v[i].x *= a.scale, v[i].y *= a.scale, v[i].z *= a.scale, v[i].w *= a.scale;
       }
+    }
+    if (a.post) {
+      const float2 st = row_stats<R>(v, a.post_kind, n, a.eps, red);
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int k = (threadIdx.x + i * blockDim.x) * 4;
+        if (k < ld) v[i] = apply_norm(v[i], st, a.post_kind, a.post, ld, k);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int k = (threadIdx.x + i * blockDim.x) * 4;
+      if (k < ld) *reinterpret_cast<float4*>(xr + k) = v[i];
     }
   } else {
     float4 xv[R];
-    const int parts = slots ? slots : 1;
+    const int parts = a.slots ? a.slots : 1;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       const int k = (threadIdx.x + i * blockDim.x) * 4;
@@ -87,38 +123,79 @@ join_kernel(float* x, const float* y, const float* __restrict__ post, int post_k
       if (k < ld) xv[i] = load4(xr + k);
     }
     for (int j = 0; j < parts; ++j) {        // rows y[place[t, j]], weighted; without slots the token's own row
-      const float wj = slots ? weight[(size_t)t * slots + j] : 1.f;
-      const size_t yr = (size_t)(slots ? place[(size_t)t * slots + j] : t) * ld;
+      const float wj = a.slots ? a.weight[(size_t)t * a.slots + j] : 1.f;
+      const int row = a.slots ? a.place[(size_t)t * a.slots + j] : t;
+      const size_t yr = (size_t)row * ld;
 #pragma unroll
       for (int i = 0; i < R; ++i) {
         const int k = (threadIdx.x + i * blockDim.x) * 4;
         if (k < ld) {
-          const float4 a = y_bf16 ? load4(reinterpret_cast<const bf16*>(y) + yr + k) : load4(y + yr + k);
-          v[i].x = fmaf(wj, a.x, v[i].x), v[i].y = fmaf(wj, a.y, v[i].y), v[i].z = fmaf(wj, a.z, v[i].z), v[i].w = fmaf(wj, a.w, v[i].w);
+          const float4 b = row < 0 ? load4(reinterpret_cast<const T*>(a.own) + (size_t)t * ld + k)
+                           : a.y_bf16 ? load4(reinterpret_cast<const bf16*>(a.y) + yr + k) : load4(reinterpret_cast<const float*>(a.y) + yr + k);
+          v[i].x = fmaf(wj, b.x, v[i].x), v[i].y = fmaf(wj, b.y, v[i].y), v[i].z = fmaf(wj, b.z, v[i].z), v[i].w = fmaf(wj, b.w, v[i].w);
         }
       }
     }
-    const float2 st = row_stats<R>(v, post_kind, n, eps, red);
+    if (a.z) {
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int k = (threadIdx.x + i * blockDim.x) * 4;
+        if (k < ld) {
+          if (a.bias) {
+            const float4 b = load4(a.bias + k);
+            v[i].x += b.x, v[i].y += b.y, v[i].z += b.z, v[i].w += b.w;
+          }
+          const float4 z = load4(a.z + (size_t)t * a.ldz + k), b = load4(a.z_b + k);
+          v[i].x *= sigmoid_x(z.x + b.x), v[i].y *= sigmoid_x(z.y + b.y), v[i].z *= sigmoid_x(z.z + b.z), v[i].w *= sigmoid_x(z.w + b.w);
+        }
+      }
+    }
+    const float2 st = row_stats<R>(v, a.post_kind, n, a.eps, red);
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       const int k = (threadIdx.x + i * blockDim.x) * 4;
       if (k < ld) {
-        const float4 o = apply_norm(v[i], st, post_kind, post, ld, k);
+        const float4 o = apply_norm(v[i], st, a.post_kind, a.post, ld, k);
         v[i] = make_float4(xv[i].x + o.x, xv[i].y + o.y, xv[i].z + o.z, xv[i].w + o.w);
         *reinterpret_cast<float4*>(xr + k) = v[i];
       }
     }
   }
-  T* hr = h + (size_t)t * ld;
+  T* hr = reinterpret_cast<T*>(a.h) + (size_t)t * ld;
   float2 st = make_float2(0.f, 1.f);
-  if (next_kind != NORM_NONE) st = row_stats<R>(v, next_kind, n, eps, red);
+  if (a.next_kind != NORM_NONE) st = row_stats<R>(v, a.next_kind, n, a.eps, red);
+  const int pos = a.taps ? a.positions[t] : 0;
+  T* rg = reinterpret_cast<T*>(a.ring) + (a.taps ? (size_t)a.state_slots[a.seq_ids[t]] * a.ring_slot : 0);
 #pragma unroll
   for (int i = 0; i < R; ++i) {
     const int k = (threadIdx.x + i * blockDim.x) * 4;
     if (k < ld) {
-      const float4 o = next_kind == NORM_NONE ? v[i] : apply_norm(v[i], st, next_kind, next, ld, k);
+      const float4 o = a.next_kind == NORM_NONE ? v[i] : apply_norm(v[i], st, a.next_kind, a.next, ld, k);
       store4<T>(hr + k, o.x, o.y, o.z, o.w);
+      if (a.taps) {                          // the convolution reads rounded rows, as it will find them in the ring
+        const float4 own = make_float4(to_f(from_f<T>(o.x)), to_f(from_f<T>(o.y)), to_f(from_f<T>(o.z)), to_f(from_f<T>(o.w)));
+        float4 c = own;
+        for (int back = 0; back < a.taps && back <= pos; ++back) {
+          const float4 f = back ? load4(rg + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + k) : own;
+          const float4 w = load4(a.conv_w + (size_t)(a.taps - 1 - back) * ld + k);
+          c.x = fmaf(f.x, w.x, c.x), c.y = fmaf(f.y, w.y, c.y), c.z = fmaf(f.z, w.z, c.z), c.w = fmaf(f.w, w.w, c.w);
+        }
+        store4<T>(reinterpret_cast<T*>(a.hc) + (size_t)t * ld + k, c.x, c.y, c.z, c.w);
+        store4<T>(rg + (size_t)(pos % a.ring_rows) * a.ring_ld + k, o.x, o.y, o.z, o.w);
+      }
     }
+  }
+}
+
+// act(z) of the first `cols` columns of every row, in place
+template <typename T>
+__global__ void __launch_bounds__(256) act_kernel(T* z, long ld, int c4, int act) {
+  pdl_launch_dependents(34);
+  pdl_wait();
+  T* row = z + (size_t)blockIdx.x * ld;
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < c4; i += 256 * gridDim.y) {
+    const float4 v = load4(row + 4 * i);
+    store4<T>(row + 4 * i, act_x(v.x, act), act_x(v.y, act), act_x(v.z, act), act_x(v.w, act));
   }
 }
 
@@ -161,14 +238,9 @@ side_kernel(const T* z, const T* __restrict__ side, const int* ids, T* out, int 
 }
 
 template <typename T>
-cudaError_t join_launch(void* x, const void* y, const void* post, int pk, const void* next, int nk, void* h, const void* table,
-                        const void* ids, float scale, int V, int T_, int ld, int n, float eps, const void* place, const void* weight,
-                        int slots, int y_bf16, cudaStream_t st) {
-  const int thr = ld >= 2048 ? 512 : (ld >= 1024 ? 256 : 128), need = (ld / 4 + thr - 1) / thr;
-#define JOIN(R)                                                                                                            \
-  return trl_launch(join_kernel<T, R>, dim3(T_), dim3(thr), 0, st, (float*)x, (const float*)y, (const float*)post, pk,     \
-                    (const float*)next, nk, (T*)h, (const T*)table, (const int*)ids, scale, V, ld, n, eps,                 \
-                    (const int*)place, (const float*)weight, slots, y_bf16)
+cudaError_t join_launch(const JoinArgs& a, int T_, cudaStream_t st) {
+  const int ld = a.ld, thr = ld >= 2048 ? 512 : (ld >= 1024 ? 256 : 128), need = (ld / 4 + thr - 1) / thr;
+#define JOIN(R) return trl_launch(join_kernel<T, R>, dim3(T_), dim3(thr), 0, st, a)
   if (need <= 1) JOIN(1);
   if (need <= 2) JOIN(2);
   if (need <= 4) JOIN(4);
@@ -179,27 +251,44 @@ cudaError_t join_launch(void* x, const void* y, const void* post, int pk, const 
 
 }  // namespace
 
-// post / next: fp32 [2, ld] weight and bias (kind 2), [1, ld] weight (kind 1); next kind 0: h is x rounded.  table: rows of
-// ld values in h's type (then y and post are unused).  ld up to 16384.
+// args: filled by the caller.  post / next: fp32 [2, ld] weight and bias (kind 2), [1, ld] weight (kind 1); next kind 0: h is x
+// rounded.  With a table, y is unused and post (or null) norms the row that starts the stream.  ld up to 16384.
+TRL_API int trl_join_args(const JoinArgs* args, int T, int f32, void* stream) {
+  const JoinArgs& a = *args;
+  const int per = f32 ? 4 : 8;
+  if (T <= 0 || a.ld % 64 || a.ld > 16384 || a.n <= 0 || a.n > a.ld || !a.x || !a.h || (!a.table && (!a.y || !a.post)) ||
+      (a.post && (a.post_kind < 1 || a.post_kind > 2)) || a.next_kind < 0 || a.next_kind > 2 || (a.next_kind && !a.next) || (a.table && !a.ids) ||
+      a.slots < 0 || (a.slots && (!a.place || !a.weight)) || (a.z && (!a.z_b || a.ldz % 4 || a.ldz < a.ld)) || (a.bias && !a.z) || a.taps < 0 ||
+      (a.taps && (!a.hc || !a.conv_w || !a.ring || !a.positions || !a.seq_ids || !a.state_slots || a.taps > a.ring_rows || a.ring_ld % per ||
+                  a.ring_slot % per || ((uintptr_t)a.ring & 15))))
+    return (int)cudaErrorInvalidValue;
+  return (int)(f32 ? join_launch<float>(a, T, (cudaStream_t)stream) : join_launch<bf16>(a, T, (cudaStream_t)stream));
+}
+
 TRL_API int trl_join(void* x, const void* y, const void* post, int post_kind, const void* next, int next_kind, void* h,
                      const void* table, const void* ids, float scale, int V, int T, int ld, int n, float eps, int f32, void* stream) {
-  if (T <= 0 || ld % 64 || ld > 16384 || n <= 0 || n > ld || (!table && (!y || !post || post_kind < 1 || post_kind > 2)) ||
-      next_kind < 0 || next_kind > 2 || (next_kind && !next) || (table && !ids))
-    return (int)cudaErrorInvalidValue;
-  cudaStream_t st = (cudaStream_t)stream;
-  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, 0, st)
-                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, table, ids, scale, V, T, ld, n, eps, nullptr, nullptr, 0, 0, st));
+  JoinArgs a = {};
+  a.x = (float*)x, a.y = y, a.post = table ? nullptr : (const float*)post, a.post_kind = post_kind, a.next = (const float*)next;
+  a.next_kind = next_kind, a.h = h, a.table = table, a.ids = (const int*)ids, a.scale = scale, a.V = V, a.ld = ld, a.n = n, a.eps = eps;
+  return trl_join_args(&a, T, f32, stream);
 }
 
 // The same with the branch of token t given as sum_j weight[t, j] y[place[t, j]] over `slots` rows, fp32 or bf16.
 TRL_API int trl_join_experts(void* x, const void* y, int y_bf16, const void* place, const void* weight, int slots, const void* post, int post_kind,
                              const void* next, int next_kind, void* h, int T, int ld, int n, float eps, int f32, void* stream) {
-  if (T <= 0 || ld % 64 || ld > 16384 || n <= 0 || n > ld || !y || !post || !place || !weight || slots <= 0 || post_kind < 1 || post_kind > 2 ||
-      next_kind < 0 || next_kind > 2 || (next_kind && !next))
-    return (int)cudaErrorInvalidValue;
-  cudaStream_t st = (cudaStream_t)stream;
-  return (int)(f32 ? join_launch<float>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, y_bf16, st)
-                   : join_launch<bf16>(x, y, post, post_kind, next, next_kind, h, nullptr, nullptr, 1.f, 0, T, ld, n, eps, place, weight, slots, y_bf16, st));
+  JoinArgs a = {};
+  a.x = (float*)x, a.y = y, a.y_bf16 = y_bf16, a.place = (const int*)place, a.weight = (const float*)weight, a.slots = slots;
+  a.post = (const float*)post, a.post_kind = post_kind, a.next = (const float*)next, a.next_kind = next_kind, a.h = h, a.ld = ld, a.n = n;
+  a.eps = eps, a.own = h;
+  return slots > 0 ? trl_join_args(&a, T, f32, stream) : (int)cudaErrorInvalidValue;
+}
+
+// act(z) of the first n columns (a multiple of 4) of T rows, in place.  act: ACT_* of packed.cuh.
+TRL_API int trl_act(void* z, int ld, int T, int n, int act, int f32, void* stream) {
+  if (T <= 0 || n <= 0 || n % 4 || n > ld || ld % 4 || ((uintptr_t)z & 15) || act < ACT_SILU || act > ACT_GELU_ERF) return (int)cudaErrorInvalidValue;
+  const dim3 grid(T, min((n / 4 + 255) / 256, 8));
+  if (f32) return (int)trl_launch(act_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, (float*)z, (long)ld, n / 4, act);
+  return (int)trl_launch(act_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, (bf16*)z, (long)ld, n / 4, act);
 }
 
 // x: n fp32 values, n a multiple of 4.

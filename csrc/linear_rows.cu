@@ -2,7 +2,8 @@
 //
 //   y[m, n] (store bf16 | store fp32 | += fp32) = sum_k x'[m, k] * W[n, k]
 //
-// or, in the epilogue, rows n >= n_split stored in fp32 beside the bf16 ones (gates of a recurrence), pairs of rows (gate, up)
+// or, in the epilogue, rows n >= n_split stored in fp32 beside the bf16 ones (gates of a recurrence or of a branch, whose rows may read
+// another input), the first rows through an activation, pairs of rows (gate, up)
 // joined by a gated activation, the soft cap of logits, or gelu(y) times a token's side-embedding row.
 // x' is the row itself (bf16) or rms(x) * norm_w of an fp32 stream row, rounded to bf16.  The weights are streamed
 // once: a warp owns 16 weight rows and a share of K, and every lane copies the 16-byte pieces it will itself feed to
@@ -25,7 +26,10 @@ enum { LR_STORE = 0, LR_STORE_F32 = 1, LR_ADD_F32 = 2, LR_GLU = 3, LR_SIDE = 4 }
 struct LrExtra {
   float* y2;                                                   // LR_STORE: fp32 rows n >= n_split
   int ldy2, n_split;
-  int act;                                                     // LR_GLU
+  int n_act;                                                   // LR_STORE: act (ACT_*) of rows n < n_act
+  const bf16* x2;                                              // rows n >= n_x2 (a multiple of 16) read this input
+  int n_x2;
+  int act;                                                     // LR_GLU: GLU_*
   float limit;
   float cap;                                                   // LR_STORE_F32: cap tanh(y / cap) (0: y)
   const int* ids;                                              // LR_SIDE: side[id * ld_side + off + n] for n < dim, 0 past it
@@ -116,9 +120,14 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
         *reinterpret_cast<uint4*>(dst + 8 * c) = *reinterpret_cast<const uint4*>(xr + 8 * c);
     }
   }
+  if (EPI == LR_STORE && ex.x2)
+    for (int m = 0; m < M; ++m)
+      for (int c = threadIdx.x; c < K / 8; c += LR_THREADS)
+        *reinterpret_cast<uint4*>(xs + (size_t)(M + m) * ldxs + 8 * c) = *reinterpret_cast<const uint4*>(ex.x2 + (size_t)m * ldx + 8 * c);
   __syncthreads();
   int slot = 0;
   for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
+    const bf16* xt = EPI == LR_STORE && ex.x2 && (tile * RW + wr) * 16 >= ex.n_x2 ? xs + (size_t)M * ldxs : xs;
     if (tile + (int)gridDim.x >= n_tiles) pdl_trigger();       // last tile: dependents may take the room this block leaves
     float acc[NT][4];
 #pragma unroll
@@ -139,7 +148,7 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
 #pragma unroll
           for (int i = 0; i < NT; ++i) {
             uint4 xv = make_uint4(0u, 0u, 0u, 0u);             // rows past M count as zeros
-            if (i * 8 + g < M) xv = *reinterpret_cast<const uint4*>(xs + (size_t)(i * 8 + g) * ldxs + ((j0 + u) << 5) + (t << 3));
+            if (i * 8 + g < M) xv = *reinterpret_cast<const uint4*>(xt + (size_t)(i * 8 + g) * ldxs + ((j0 + u) << 5) + (t << 3));
             lr_mma(acc[i], va[u].x, vb[u].x, va[u].y, vb[u].y, xv.x, xv.y);
             lr_mma(acc[i], va[u].z, vb[u].z, va[u].w, vb[u].w, xv.z, xv.w);
           }
@@ -172,7 +181,7 @@ linear_rows_kernel(const void* xin, int ldx, const bf16* __restrict__ w, const f
         reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(o);
       } else if (EPI == LR_STORE && n >= ex.n_split) {
         ex.y2[(size_t)m * ex.ldy2 + n - ex.n_split] = v;
-      } else if (EPI == LR_STORE) reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(v);
+      } else if (EPI == LR_STORE) reinterpret_cast<bf16*>(y)[(size_t)m * ldy + n] = __float2bfloat16(n < ex.n_act ? act_x(v, ex.act) : v);
       else if (EPI == LR_STORE_F32) reinterpret_cast<float*>(y)[(size_t)m * ldy + n] = ex.cap > 0.f ? ex.cap * tanhf(v / ex.cap) : v;
       else reinterpret_cast<float*>(y)[(size_t)m * ldy + n] += v;
     }
@@ -210,7 +219,8 @@ static int lr_launch(const void* x, int ldx, const void* w, const void* norm_w, 
   int KW = 1;
   while (KW < LR_WARPS && (K / 32 / (2 * KW) >= 16 || (long)groups * KW < 2L * lr_sms() * LR_WARPS)) KW *= 2;
   const int RW = LR_WARPS / KW, n_tiles = (groups + RW - 1) / RW, grid = min(n_tiles, lr_sms());
-  const size_t xb = (size_t)M * (K + LR_PAD) * sizeof(bf16);
+  const size_t xb = (size_t)M * (ex.x2 ? 2 : 1) * (K + LR_PAD) * sizeof(bf16);
+  if (xb + (size_t)LR_WARPS * 2 * LR_SLOT > (size_t)LR_SMEM) return (int)cudaErrorInvalidValue;
   const int nt = M <= 8 ? 1 : 2, depth = xb + LR_WARPS * 4 * LR_SLOT <= LR_SMEM ? 4 : 2;
   const size_t smem = xb + (size_t)LR_WARPS * depth * LR_SLOT;
   cudaError_t e = cudaErrorInvalidValue;
@@ -251,6 +261,18 @@ TRL_API int trl_linear_rows_split(const void* x, int ldx, const void* w, void* y
   if (!y2 || n_split < 0) return (int)cudaErrorInvalidValue;
   LrExtra ex = {};
   ex.y2 = (float*)y2, ex.ldy2 = ldy2, ex.n_split = n_split;
+  return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_STORE, ex, stream);
+}
+
+// The same with act (ACT_* of packed.cuh) on rows n < n_act, and rows n >= n_x2 (a multiple of 16) reading x2 (ldx, too; null: all read
+// x).  With x2, 2 M rows must fit trl_linear_rows_max(K).
+TRL_API int trl_linear_rows_mix(const void* x, int ldx, const void* x2, int n_x2, const void* w, void* y, int ldy, int n_split, void* y2, int ldy2,
+                                int M, int N, int K, int n_act, int act, void* stream) {
+  if (n_split < 0 || (n_split < N && !y2) || (n_split > 0 && !y) || n_act < 0 || n_act > n_split || act < ACT_NONE || act > ACT_GELU_ERF ||
+      (x2 && (n_x2 % 16 || n_x2 < 0 || ((uintptr_t)x2 & 15))))
+    return (int)cudaErrorInvalidValue;
+  LrExtra ex = {};
+  ex.y2 = (float*)y2, ex.ldy2 = ldy2, ex.n_split = n_split, ex.n_act = n_act, ex.act = act, ex.x2 = (const bf16*)x2, ex.n_x2 = n_x2;
   return lr_launch(x, ldx, w, nullptr, 0.f, 0, y, ldy, M, N, K, LR_STORE, ex, stream);
 }
 

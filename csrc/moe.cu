@@ -1,5 +1,7 @@
-// Mixture-of-experts feed-forwards (models/deluvik.py): every token uses the `top` experts with the largest router logits, weighted by
-// the softmax over those, and `pieces` experts that all tokens share (weight one).
+// Mixture-of-experts feed-forwards (models/deluvik.py, models/tobadra.py): every token uses the `top` experts with the largest router
+// logits, weighted by the softmax over those, and `pieces` experts that all tokens share (weight one).  Or (MoePlanArgs::outputs) scores
+// are the softmax over all outputs; a correction joins them for the choice only, which keeps to the groups of neighbours with the
+// largest best score; outputs past the experts stand for the token's own row; the shared experts have a gate per token.
 //
 //   moe_topk_kernel    router logits -> expert numbers and weights of every token, one warp per token.
 //   moe_plan_kernel    (moe_plan_small_kernel for a few pairs) one block: orders the (token, expert) pairs by expert and cuts every expert's rows into tiles.  Ticks of few
@@ -24,6 +26,9 @@ struct MoePlanArgs {
   MoeItem* items;
   int* n_items;
   int T, ldz, experts, top, pieces, tile, max_items;
+  // grouped choice (outputs 0: none): bias is the correction; gate_col: column of z with the shared experts' gate (-1: none)
+  int outputs, groups, keep, gate_col;
+  float scale;
 };
 
 namespace {
@@ -66,11 +71,82 @@ __device__ __forceinline__ void choose_experts(const MoePlanArgs& a, int t) {
   }
 }
 
+// The grouped choice.  Identity outputs count as expert number experts + pieces.
+__device__ __forceinline__ void choose_grouped(const MoePlanArgs& a, int t) {
+  const int lane = threadIdx.x & 31, slots = a.top + a.pieces, per = a.outputs / a.groups;
+  const float* z = a.z + (size_t)t * a.ldz;
+  float top = -INFINITY, sum = 0.f;
+  for (int e = lane; e < a.outputs; e += 32) top = fmaxf(top, z[e]);
+  top = warp_max(top);
+  for (int e = lane; e < a.outputs; e += 32) sum += expf(z[e] - top);
+  sum = warp_sum(sum);
+  auto score = [&](int e) { return expf(z[e] - top) / sum; };
+  auto choice = [&](int e) {
+    const float v = score(e) + a.bias[e];
+    return v == v ? v : -INFINITY;
+  };
+  unsigned kept[2] = {0xffffffffu, 0xffffffffu};
+  if (a.keep < a.groups) {
+    float best[2] = {-INFINITY, -INFINITY};                      // of groups lane and lane + 32
+    for (int g = 0; g < a.groups; ++g) {
+      float m = -INFINITY;
+      for (int e = g * per + lane; e < (g + 1) * per; e += 32) m = fmaxf(m, choice(e));
+      m = warp_max(m);
+      if (lane == (g & 31)) {
+        if (g < 32) best[0] = m;
+        else best[1] = m;
+      }
+    }
+    int ahead[2] = {0, 0};                                       // groups before this lane's
+    for (int g = 0; g < a.groups; ++g) {
+      const float m0 = __shfl_sync(0xffffffffu, best[0], g & 31), m1 = __shfl_sync(0xffffffffu, best[1], g & 31), m = g < 32 ? m0 : m1;
+      ahead[0] += m > best[0] || (m == best[0] && g < lane);
+      ahead[1] += m > best[1] || (m == best[1] && g < lane + 32);
+    }
+    kept[0] = __ballot_sync(0xffffffffu, lane < a.groups && ahead[0] < a.keep);
+    kept[1] = __ballot_sync(0xffffffffu, lane + 32 < a.groups && ahead[1] < a.keep);
+  }
+  float last = INFINITY;
+  int last_id = -1;
+  for (int j = 0; j < a.top; ++j) {
+    // the next in (choice score descending, number ascending) order after (last, last_id)
+    float best = -INFINITY;
+    int id = MP_MAXE;
+    for (int e = lane; e < a.outputs; e += 32) {
+      const int g = e / per;
+      if (!((g < 32 ? kept[0] >> g : kept[1] >> (g - 32)) & 1u)) continue;
+      const float v = choice(e);
+      const bool after = j == 0 || v < last || (v == last && e > last_id);
+      if (after && (v > best || (v == best && e < id))) best = v, id = e;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, id, o);
+      if (ov > best || (ov == best && oi < id)) best = ov, id = oi;
+    }
+    if (lane == 0) {
+      const int e = min(id, a.outputs - 1);
+      a.ids[(size_t)t * slots + j] = e < a.experts ? e : a.experts + a.pieces, a.weight[(size_t)t * slots + j] = score(e) * a.scale;
+    }
+    last = best, last_id = id;
+  }
+  for (int j = a.top + lane; j < slots; j += 32) {
+    const size_t p = (size_t)t * slots + j;
+    a.ids[p] = a.experts + j - a.top, a.weight[p] = a.gate_col >= 0 ? sigmoid_x(z[a.gate_col]) : 1.f;
+  }
+  __syncwarp();
+}
+__device__ __forceinline__ void choose_any(const MoePlanArgs& a, int t) {
+  if (a.outputs) choose_grouped(a, t);
+  else choose_experts(a, t);
+}
+
 __global__ void __launch_bounds__(256) moe_topk_kernel(const MoePlanArgs a) {
   pdl_launch_dependents(60);
   pdl_wait();
   const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (t < a.T) choose_experts(a, t);
+  if (t < a.T) choose_any(a, t);
 }
 
 __global__ void __launch_bounds__(MP_THREADS) moe_plan_kernel(const MoePlanArgs a, int choose) {
@@ -79,14 +155,15 @@ __global__ void __launch_bounds__(MP_THREADS) moe_plan_kernel(const MoePlanArgs 
   pdl_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, slots = a.top + a.pieces, n = a.experts + a.pieces, P = a.T * slots;
   if (choose)
-    for (int t = warp; t < a.T; t += MP_THREADS / 32) choose_experts(a, t);
+    for (int t = warp; t < a.T; t += MP_THREADS / 32) choose_any(a, t);
   for (int e = tid; e < MP_MAXE; e += MP_THREADS) s_cnt[e] = e >= a.experts && e < n ? a.T : 0;
   __syncthreads();
   for (int p = tid; p < P; p += MP_THREADS)
     if (p % slots < a.top) atomicAdd(&s_cnt[a.ids[p]], 1);
   __syncthreads();
   // exclusive sums of rows and of tiles over the experts, two a thread
-  const int c0 = s_cnt[2 * tid], c1 = s_cnt[2 * tid + 1], i0 = (c0 + a.tile - 1) / a.tile, i1 = (c1 + a.tile - 1) / a.tile;
+  const int c0 = s_cnt[2 * tid], c1 = s_cnt[2 * tid + 1];
+  const int i0 = 2 * tid < n ? (c0 + a.tile - 1) / a.tile : 0, i1 = 2 * tid + 1 < n ? (c1 + a.tile - 1) / a.tile : 0;      // (own rows have none)
   int rows = c0 + c1, items = i0 + i1;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -110,7 +187,7 @@ __global__ void __launch_bounds__(MP_THREADS) moe_plan_kernel(const MoePlanArgs 
   for (int p = tid; p < P; p += MP_THREADS) {
     const int t = p / slots, j = p % slots, e = a.ids[p];
     const int row = j < a.top ? atomicAdd(&s_off[e], 1) : s_off[e] + t;
-    a.place[p] = row, a.token[row] = t;
+    a.place[p] = e < n ? row : -1, a.token[row] = t;             // own rows stand at the list's end, without tiles
   }
 }
 
@@ -121,7 +198,7 @@ __global__ void __launch_bounds__(MQ_MAX) moe_plan_small_kernel(const MoePlanArg
   pdl_launch_dependents(61);
   pdl_wait();
   const int tid = threadIdx.x, slots = a.top + a.pieces, P = a.T * slots;
-  for (int t = tid >> 5; t < a.T; t += blockDim.x >> 5) choose_experts(a, t);
+  for (int t = tid >> 5; t < a.T; t += blockDim.x >> 5) choose_any(a, t);
   __syncthreads();
   const int e = tid < P ? a.ids[tid] : 0;
   s_e[tid] = e;
@@ -131,13 +208,14 @@ __global__ void __launch_bounds__(MQ_MAX) moe_plan_small_kernel(const MoePlanArg
     const int o = s_e[q];
     row += o < e || (o == e && q < tid), rank += o == e && q < tid, cnt += o == e;
   }
-  s_tiles[tid] = rank ? 0 : (cnt + a.tile - 1) / a.tile;        // an expert's tiles count, and are written, at its first pair
+  s_tiles[tid] = rank || e == a.experts + a.pieces ? 0 : (cnt + a.tile - 1) / a.tile;        // an expert's tiles count, and are written, at its first pair
   __syncthreads();
   if (tid >= P) return;
-  a.place[tid] = row, a.token[row] = tid / slots;
-  if (rank) return;
+  const bool own = e == a.experts + a.pieces;                   // the token's own row: at the list's end, without tiles
+  a.place[tid] = own ? -1 : row, a.token[row] = tid / slots;
+  if (rank || (own && row)) return;
   for (int q = 0; q < P; ++q) total += s_tiles[q], item += s_e[q] < e ? s_tiles[q] : 0;
-  for (int i = 0; i * a.tile < cnt; ++i)
+  for (int i = 0; !own && i * a.tile < cnt; ++i)
     if (item + i < a.max_items) a.items[item + i] = MoeItem{e, row + i * a.tile, min(a.tile, cnt - i * a.tile), 0};
   if (row == 0) *a.n_items = min(total, a.max_items);
 }
@@ -146,7 +224,6 @@ __global__ void __launch_bounds__(MQ_MAX) moe_plan_small_kernel(const MoePlanArg
 constexpr int MR_THREADS = 256, MR_WARPS = MR_THREADS / 32, MR_U = 4, MR_PAD = 32, MR_ROWS = 8;
 constexpr int MR_SLOT = MR_U * 2 * 512;                        // bytes of a ring stage of one warp
 constexpr int MR_SMEM = 216 * 1024;
-enum { MOE_UP = 0, MOE_DOWN = 1 };
 
 __device__ __forceinline__ void mr_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -159,8 +236,8 @@ __device__ __forceinline__ uint4 mr_lds(uint32_t a) {
   return v;
 }
 
-// x: UP [T, ldx] input rows by token, DOWN [rows, ldx] gated rows by place.  w: [experts, N, K].
-// y: UP bf16 [rows, ldy] act(gate) up, DOWN fp32 [rows, ldy].  A block walks consecutive row tiles of consecutive items.
+// x: UP, ACT [T, ldx] input rows by token, DOWN [rows, ldx] gated rows by place.  w: [experts, N, K].
+// y: UP bf16 [rows, ldy] act(gate) up, ACT the same with act(row) of every weight row, DOWN fp32 [rows, ldy].  A block walks consecutive row tiles of consecutive items.
 template <int KIND, int DEPTH>
 __global__ void __launch_bounds__(MR_THREADS)
 moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int ldy, const MoeItem* items, const int* n_items, const int* token,
@@ -172,7 +249,7 @@ moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int
   const int RW = MR_WARPS / KW, wr = warp / KW, wk = warp % KW, ldxs = K + MR_PAD;
   const uint32_t ring = (uint32_t)__cvta_generic_to_shared(mr_smem) + warp * DEPTH * MR_SLOT + lane * 16;
   const int steps = K >> 5, per = (steps + KW - 1) / KW, jb = min(steps, wk * per), je = min(steps, jb + per);
-  pdl_enter(62 + KIND);
+  pdl_enter(KIND == MOE_DOWN ? 63 : 62);
   pdl_wait();
   const long total = (long)*n_items * per_item;
   const int first = (int)(total * blockIdx.x / gridDim.x), end = (int)(total * (blockIdx.x + 1) / gridDim.x);
@@ -219,7 +296,7 @@ moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int
       it = items[item];
       __syncthreads();
       for (int m = 0; m < it.n; ++m) {
-        const bf16* src = x + (size_t)(KIND == MOE_UP ? token[it.row0 + m] : it.row0 + m) * ldx;
+        const bf16* src = x + (size_t)(KIND != MOE_DOWN ? token[it.row0 + m] : it.row0 + m) * ldx;
         for (int c = threadIdx.x; c < K / 8; c += MR_THREADS)
           *reinterpret_cast<uint4*>(xs + (size_t)m * ldxs + 8 * c) = *reinterpret_cast<const uint4*>(src + 8 * c);
       }
@@ -262,6 +339,7 @@ moe_rows_kernel(const bf16* x, int ldx, const bf16* __restrict__ w, void* y, int
       if (n >= N) continue;
       const float v = total_of(m, c);
       if (KIND == MOE_UP) reinterpret_cast<bf16*>(y)[(size_t)(it.row0 + m) * ldy + n / 2] = __float2bfloat16(glu_x(v, total_of(m, c + 1), act, 0.f));
+      else if (KIND == MOE_ACT) reinterpret_cast<bf16*>(y)[(size_t)(it.row0 + m) * ldy + n] = __float2bfloat16(act_x(v, act));
       else reinterpret_cast<float*>(y)[(size_t)(it.row0 + m) * ldy + n] = v;
     }
   }
@@ -294,7 +372,7 @@ moe_plain_kernel(const T* x, int ldx, const T* __restrict__ w, void* y, int ldy,
       for (int m = 0; m < MR_ROWS; ++m) {
         if (m < it.n) {
           float v[C];
-          Chunk<T>::get(*reinterpret_cast<const uint4*>(x + (size_t)(KIND == MOE_UP ? token[it.row0 + m] : it.row0 + m) * ldx + k), v);
+          Chunk<T>::get(*reinterpret_cast<const uint4*>(x + (size_t)(KIND != MOE_DOWN ? token[it.row0 + m] : it.row0 + m) * ldx + k), v);
 #pragma unroll
           for (int i = 0; i < W; ++i)
 #pragma unroll
@@ -308,6 +386,7 @@ moe_plain_kernel(const T* x, int ldx, const T* __restrict__ w, void* y, int ldy,
         const float a0 = warp_sum(acc[m][0]), a1 = warp_sum(acc[m][W - 1]);
         if (lane == 0) {
           if (KIND == MOE_UP) reinterpret_cast<T*>(y)[(size_t)(it.row0 + m) * ldy + n] = from_f<T>(glu_x(a0, a1, act, 0.f));
+          else if (KIND == MOE_ACT) reinterpret_cast<T*>(y)[(size_t)(it.row0 + m) * ldy + n] = from_f<T>(act_x(a0, act));
           else reinterpret_cast<float*>(y)[(size_t)(it.row0 + m) * ldy + n] = a0;
         }
       }
@@ -360,7 +439,10 @@ cudaError_t rows_launch(const void* x, int ldx, const void* w, void* y, int ldy,
 // T * slots / tile tiles.
 TRL_API int trl_moe_plan(const MoePlanArgs* args, void* stream) {
   const MoePlanArgs& a = *args;
-  if (a.T <= 0 || a.experts <= 0 || a.top <= 0 || a.top > a.experts || a.pieces < 0 || a.experts + a.pieces > MP_MAXE || a.ldz < a.experts ||
+  const int outputs = a.outputs ? a.outputs : a.experts;
+  if (a.T <= 0 || a.experts <= 0 || a.top <= 0 || a.top > outputs || a.pieces < 0 || a.experts + a.pieces >= MP_MAXE || outputs > MP_MAXE || a.ldz < outputs ||
+      (a.outputs && (a.outputs < a.experts || a.groups < 1 || a.groups > 64 || a.keep < 1 || a.keep > a.groups || a.outputs % a.groups ||
+                     a.outputs / a.groups * a.keep < a.top || a.gate_col >= a.ldz)) ||
       a.tile <= 0 || a.max_items <= 0 || !a.z || !a.bias || !a.ids || !a.weight || !a.place || !a.token || !a.items || !a.n_items)
     return (int)cudaErrorInvalidValue;
   const int choose = a.T <= 64;
@@ -373,10 +455,10 @@ TRL_API int trl_moe_plan(const MoePlanArgs* args, void* stream) {
   return (int)e;
 }
 
-// Up (kind 0) or down (kind 1) projections of all tiles (of at most 8 rows each).  likely: a guess of their number.  plain: CUDA cores.
+// Up (kind 0), down (kind 1) or plain up (kind 2) projections of all tiles (of at most 8 rows each).  likely: a guess of their number.  plain: CUDA cores.
 TRL_API int trl_moe_rows(const void* x, int ldx, const void* w, void* y, int ldy, const void* items, const void* n_items, const void* token,
                          int N, int K, int kind, int act, int likely, int f32, void* stream) {
-  if (N <= 0 || N % 2 || K < 64 || K % 64 || ldx % 8 || kind < 0 || kind > 1 || act < GLU_CLAMPED || act > GLU_GELU || likely <= 0 || !items ||
+  if (N <= 0 || N % 2 || K < 64 || K % 64 || ldx % 8 || kind < MOE_UP || kind > MOE_ACT || act < GLU_CLAMPED || act > (kind == MOE_ACT ? (int)ACT_GELU_ERF : (int)GLU_GELU) || likely <= 0 || !items ||
       !n_items || !token || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
@@ -388,17 +470,21 @@ TRL_API int trl_moe_rows(const void* x, int ldx, const void* w, void* y, int ldy
   return (int)trl_launch(moe_plain_kernel<TT, KK>, dim3(mr_sms() * 4), dim3(256), 0, st, (const TT*)x, ldx, (const TT*)w, y, ldy,   \
                          (const MoeItem*)items, (const int*)n_items, (const int*)token, N, K, act)
     if (f32 && kind == MOE_UP) MOE_PLAIN(float, MOE_UP);
+    if (f32 && kind == MOE_ACT) MOE_PLAIN(float, MOE_ACT);
     if (f32) MOE_PLAIN(float, MOE_DOWN);
     if (kind == MOE_UP) MOE_PLAIN(bf16, MOE_UP);
+    if (kind == MOE_ACT) MOE_PLAIN(bf16, MOE_ACT);
     MOE_PLAIN(bf16, MOE_DOWN);
 #undef MOE_PLAIN
   }
 #define MOE_ROWS(KK, DD, SZ) return (int)rows_launch<KK, DD>(x, ldx, w, y, ldy, items, n_items, token, groups, likely, N, K, act, SZ, st)
   if (deep <= (size_t)MR_SMEM) {
     if (kind == MOE_UP) MOE_ROWS(MOE_UP, 4, deep);
+    if (kind == MOE_ACT) MOE_ROWS(MOE_ACT, 4, deep);
     MOE_ROWS(MOE_DOWN, 4, deep);
   }
   if (kind == MOE_UP) MOE_ROWS(MOE_UP, 2, flat);
+  if (kind == MOE_ACT) MOE_ROWS(MOE_ACT, 2, flat);
   MOE_ROWS(MOE_DOWN, 2, flat);
 #undef MOE_ROWS
 }

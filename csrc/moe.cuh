@@ -6,3 +6,6 @@
 struct MoeItem {
   int expert, row0, n, pad;
 };
+
+// projections of the tiles: gated up (pairs of weight rows), down, plain up (an activation of every weight row)
+enum { MOE_UP = 0, MOE_DOWN = 1, MOE_ACT = 2 };

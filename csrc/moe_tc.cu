@@ -2,6 +2,7 @@
 //
 //   UP    out[r, j] = act(W[e, 2j] x[r]) * (W[e, 2j + 1] x[r])      bf16, rows ordered by expert (moe_plan_kernel)
 //   DOWN  out[r, n] = W[e, n] x[r]                                  bf16
+//   ACT   out[r, n] = act(W[e, n] x[r])                             bf16
 //
 // A tile is 128 weight rows (the MMA's A operand: TMEM lanes) by up to 256 rows of one expert (its B operand: TMEM columns).  The
 // instruction's N follows the rows an expert really has, in steps of 16, so a short expert costs what its rows cost.  K goes by in
@@ -41,7 +42,7 @@ __device__ __forceinline__ void tc_mma_bf16_lh(uint32_t d_tmem, uint32_t alo, ui
       : "memory");
 }
 
-template <bool UP>
+template <int KIND>
 __global__ void __launch_bounds__(MT_THREADS, 1)
 moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const TcArgs p) {
   extern __shared__ unsigned char mt_smem[];
@@ -136,7 +137,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
       tc_fence_after();
       // lane pairs (2j, 2j + 1) trade values so that the even lane ends with both of column c, the odd one with both of column c + 1
       const bool odd = lane & 1;
-      const int col = UP ? f >> 1 : f & ~1;
+      const int col = KIND == MOE_UP ? f >> 1 : f & ~1;
       bf16* out = p.out + (size_t)it.row0 * p.ldo + col;
       for (int c0 = half * (MT_N / 2); c0 < min(it.n, (half + 1) * (MT_N / 2)); c0 += 32) {
         uint32_t r[32];
@@ -149,7 +150,8 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
           const float lo = odd ? other : mine, up = odd ? mine : other;          // weight rows f & ~1 and f | 1
           const int row = c0 + c + odd;
           if (row < it.n && f < p.N) {
-            if (UP) out[(size_t)row * p.ldo] = __float2bfloat16(glu_x(lo, up, p.act, 0.f));
+            if (KIND == MOE_UP) out[(size_t)row * p.ldo] = __float2bfloat16(glu_x(lo, up, p.act, 0.f));
+            else if (KIND == MOE_ACT) *reinterpret_cast<uint32_t*>(out + (size_t)row * p.ldo) = f2_to_bf162_bits(act_x(lo, p.act), act_x(up, p.act));
             else *reinterpret_cast<uint32_t*>(out + (size_t)row * p.ldo) = f2_to_bf162_bits(lo, up);
           }
         }
@@ -197,11 +199,11 @@ int make_map(CUtensorMap* m, const void* base, uint64_t rows, uint64_t row_bytes
 // Most rows of an item.
 TRL_API int trl_moe_tc_tile() { return MT_N; }
 
-// x: bf16 [rows, K] ordered by expert; w: bf16 [experts, N, K]; K a multiple of 64, N even.  kind 0: up (out [rows, N / 2]), 1: down
-// (out [rows, N]); ldo: a multiple of 2.  items: of at most trl_moe_tc_tile() rows each.
+// x: bf16 [rows, K] ordered by expert; w: bf16 [experts, N, K]; K a multiple of 64, N even.  kind 0: up (out [rows, N / 2]), 1: down,
+// 2: plain up (out [rows, N]); ldo: a multiple of 2.  items: of at most trl_moe_tc_tile() rows each.
 TRL_API int trl_moe_tc(const void* x, const void* w, void* out, int ldo, const void* items, const void* n_items, int rows, int experts, int N,
                        int K, int kind, int act, void* stream) {
-  if (rows <= 0 || experts <= 0 || N <= 0 || N % 2 || K < 64 || K % 64 || ldo % 2 || kind < 0 || kind > 1 || act < GLU_CLAMPED || act > GLU_GELU ||
+  if (rows <= 0 || experts <= 0 || N <= 0 || N % 2 || K < 64 || K % 64 || ldo % 2 || kind < MOE_UP || kind > MOE_ACT || act < GLU_CLAMPED || act > (kind == MOE_ACT ? (int)ACT_GELU_ERF : (int)GLU_GELU) ||
       !items || !n_items || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & 3))
     return (int)cudaErrorInvalidValue;
   CUtensorMap mw, mx;
@@ -213,14 +215,16 @@ TRL_API int trl_moe_tc(const void* x, const void* w, void* out, int ldo, const v
     int dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    cudaError_t e = cudaFuncSetAttribute(moe_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(moe_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(moe_tc_kernel<MOE_UP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(moe_tc_kernel<MOE_ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(moe_tc_kernel<MOE_DOWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) {
       sms = 0;
       return (int)e;
     }
   }
   const TcArgs p = {(const MoeItem*)items, (const int*)n_items, (bf16*)out, N, K / 64, ldo, act, (N + MT_M - 1) / MT_M};
-  if (kind == 0) return (int)trl_launch(moe_tc_kernel<true>, dim3(sms), dim3(MT_THREADS), smem, (cudaStream_t)stream, mw, mx, p);
-  return (int)trl_launch(moe_tc_kernel<false>, dim3(sms), dim3(MT_THREADS), smem, (cudaStream_t)stream, mw, mx, p);
+  if (kind == MOE_ACT) return (int)trl_launch(moe_tc_kernel<MOE_ACT>, dim3(sms), dim3(MT_THREADS), smem, (cudaStream_t)stream, mw, mx, p);
+  if (kind == MOE_UP) return (int)trl_launch(moe_tc_kernel<MOE_UP>, dim3(sms), dim3(MT_THREADS), smem, (cudaStream_t)stream, mw, mx, p);
+  return (int)trl_launch(moe_tc_kernel<MOE_DOWN>, dim3(sms), dim3(MT_THREADS), smem, (cudaStream_t)stream, mw, mx, p);
 }

@@ -63,6 +63,14 @@ __device__ __forceinline__ float gelu_tanh_x(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+__device__ __forceinline__ float gelu_erf_x(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
+
+// plain activations
+enum { ACT_NONE = 0, ACT_SILU = 1, ACT_GELU = 2, ACT_GELU_ERF = 3 };
+__device__ __forceinline__ float act_x(float z, int act) {
+  return act == ACT_SILU ? z * sigmoid_x(z) : act == ACT_GELU ? gelu_tanh_x(z) : act == ACT_GELU_ERF ? gelu_erf_x(z) : z;
+}
+
 // gated feed-forwards: act(g) combined with u
 enum { GLU_CLAMPED = 0, GLU_SILU = 1, GLU_GELU = 2 };
 __device__ __forceinline__ float glu_x(float g, float u, int act, float limit) {

@@ -1,4 +1,4 @@
-// Decayed scans: S_t = keep_t S_(t-1) + add_t k_t v_t^T, o_t = S_t^T q_t per head, in two forms (models/fetotar.py).
+// Decayed scans: S_t = keep_t S_(t-1) + add_t k_t v_t^T, o_t = S_t^T q_t per head, in three forms (models/fetotar.py, models/tobadra.py).
 //
 //   Mamba-2   keep = exp(-exp(A) dt), add = dt, dt = softplus(raw + bias); k = B, q = C of the head's group and v = x, all
 //             after a causal convolution and silu; o += D x; then o silu(z), RMS norm in groups, weight.
@@ -6,7 +6,9 @@
 //             m_t = max(f + m_(t-1), i), keep = exp(f + m_(t-1) - m_t), add = exp(i - m_t); beside S the sum n of the keys,
 //             and o is divided by max(|n . q|, exp(-m)) + 1e-6; then RMS norm per head, weight, sigmoid gate.
 //
-//   scan_conv_kernel    convolution of a tick's rows (with or without silu, inputs with or without a bias); rows before the tick's
+//   fixed     keep = a constant of the head, add = 1; RMS norm over all heads, weight, sigmoid gate.
+//
+//   scan_conv_kernel    convolution of a tick's rows (with or without silu, inputs with or without a bias, with or without the input itself added); rows before the tick's
 //                       first token come from the slot's ring.
 //   conv_run_kernel     the same for prompts (up to 4 taps).
 //   ring_store_kernel   a tick's last convolution inputs into the ring.
@@ -23,12 +25,14 @@
 
 namespace {
 
+enum { CONV_SILU = 1, CONV_ADD = 2 };                         // silu of the sum; the input itself joins the sum
+
 // thread = one chunk of channels of one token
 template <typename T>
 __global__ void __launch_bounds__(128)
 scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ pre,
                  const T* ring, long ring_slot, int ring_rows, int ring_ld, const int* positions, const int* seq_ids,
-                 const int* q_start, const int* slots, T* out, int channels, int taps, int silu) {
+                 const int* q_start, const int* slots, T* out, int channels, int taps, int mode) {
   constexpr int C = Chunk<T>::N;
   pdl_launch_dependents(40);
   pdl_wait();
@@ -38,9 +42,13 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
   const T* rg = ring + (size_t)slots[seq] * ring_slot;
   float acc[C];
 #pragma unroll
-  for (int e = 0; e < C; e += 4) {
-    const float4 b = *reinterpret_cast<const float4*>(bias + c + e);
-    acc[e] = b.x, acc[e + 1] = b.y, acc[e + 2] = b.z, acc[e + 3] = b.w;
+  for (int e = 0; e < C; ++e) acc[e] = 0.f;
+  if (bias) {
+#pragma unroll
+    for (int e = 0; e < C; e += 4) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + c + e);
+      acc[e] = b.x, acc[e + 1] = b.y, acc[e + 2] = b.z, acc[e + 3] = b.w;
+    }
   }
   for (int j = 0; j < taps; ++j) {            // the last tap multiplies the token's own row
     const int back = taps - 1 - j;
@@ -52,6 +60,10 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
 #pragma unroll
       for (int e = 0; e < C; ++e) f[e] += pre[c + e];
     }
+    if ((mode & CONV_ADD) && back == 0) {
+#pragma unroll
+      for (int e = 0; e < C; ++e) acc[e] += f[e];
+    }
 #pragma unroll
     for (int e = 0; e < C; e += 4) {
       const float4 b = *reinterpret_cast<const float4*>(w + (size_t)j * channels + c + e);
@@ -59,7 +71,7 @@ scan_conv_kernel(const T* proj, int ldp, const float* __restrict__ w, const floa
       acc[e + 2] = fmaf(f[e + 2], b.z, acc[e + 2]), acc[e + 3] = fmaf(f[e + 3], b.w, acc[e + 3]);
     }
   }
-  if (silu) {
+  if (mode & CONV_SILU) {
 #pragma unroll
     for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
   }
@@ -72,7 +84,7 @@ template <typename T, int K>
 __global__ void __launch_bounds__(128)
 conv_run_kernel(const T* proj, int ldp, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ pre,
                 const T* ring, long ring_slot, int ring_rows, int ring_ld, const int* positions, const int* seq_ids,
-                const int* q_start, const int* slots, T* out, int n_tok, int channels, int taps, int silu) {
+                const int* q_start, const int* slots, T* out, int n_tok, int channels, int taps, int mode) {
   constexpr int C = Chunk<T>::N;
   pdl_launch_dependents(44);
   const int c = (blockIdx.y * 128 + threadIdx.x) * C, first = blockIdx.x * CR_RUN, end = min(n_tok, first + CR_RUN);
@@ -82,7 +94,7 @@ conv_run_kernel(const T* proj, int ldp, const float* __restrict__ w, const float
   }
   float wt[K][C], b[C], p[C], h[K][C];       // weight and input of `k` tokens back (inputs with their bias)
 #pragma unroll
-  for (int e = 0; e < C; ++e) b[e] = bias[c + e], p[e] = pre ? pre[c + e] : 0.f;
+  for (int e = 0; e < C; ++e) b[e] = bias ? bias[c + e] : 0.f, p[e] = pre ? pre[c + e] : 0.f;
 #pragma unroll
   for (int k = 0; k < K; ++k)
 #pragma unroll
@@ -110,7 +122,7 @@ conv_run_kernel(const T* proj, int ldp, const float* __restrict__ w, const float
 #pragma unroll
     for (int e = 0; e < C; ++e) {
       h[0][e] += p[e];
-      acc[e] = b[e];
+      acc[e] = b[e] + (mode & CONV_ADD ? h[0][e] : 0.f);
     }
 #pragma unroll
     for (int k = K - 1; k >= 0; --k)
@@ -120,7 +132,7 @@ conv_run_kernel(const T* proj, int ldp, const float* __restrict__ w, const float
     for (int k = K - 1; k > 0; --k)
 #pragma unroll
       for (int e = 0; e < C; ++e) h[k][e] = h[k - 1][e];
-    if (silu) {
+    if (mode & CONV_SILU) {
 #pragma unroll
       for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
     }
@@ -267,7 +279,7 @@ __global__ void __launch_bounds__(256, RMAX <= 16 ? 4 : 2) scan_serial_kernel(co
 #pragma unroll
           for (int w = 0; w < 8; ++w) d += s_den[j & 1][w];
           v /= fmaxf(fabsf(d), s_floor[j]) + 1e-6f;
-        } else {
+        } else if (KIND == SCAN_MAMBA2) {
           v = fmaf(a.skip[h], s_v[j][lane], v);
         }
         a.o[((size_t)(t0 + i0 + j) * a.heads + h) * a.dv + col] = v;
@@ -413,10 +425,10 @@ TRL_API int trl_ring_store(const void* rows, int ld, void* ring, long ring_slot,
 }
 
 // proj: rows whose first `channels` columns are convolved; w: [taps, channels]; pre (or null): bias of the inputs, which zeros before
-// a sequence's start do not get; ring: the layer's first column of slot 0.
+// a sequence's start do not get; bias may be null; mode: CONV_* bits; ring: the layer's first column of slot 0.
 TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* bias, const void* pre, const void* ring, long ring_slot,
                           int ring_rows, int ring_ld, const void* positions, const void* seq_ids, const void* q_start, const void* slots,
-                          void* out, int T, int channels, int taps, int silu, int f32, void* stream) {
+                          void* out, int T, int channels, int taps, int mode, int f32, void* stream) {
   const int per = f32 ? 4 : 8;
   if (T <= 0 || channels <= 0 || channels % 16 || taps < 1 || taps > ring_rows || ldp % per || ring_ld % per || ring_slot % per ||
       ((uintptr_t)ring & 15) || ((uintptr_t)proj & 15))
@@ -427,7 +439,7 @@ TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* 
 #define CONV_RUN(TT)                                                                                                               \
   return (int)trl_launch(conv_run_kernel<TT, 4>, runs, dim3(128), 0, (cudaStream_t)stream, (const TT*)proj, ldp, (const float*)w,  \
                          (const float*)bias, (const float*)pre, (const TT*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions, \
-                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (TT*)out, T, channels, taps, silu)
+                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (TT*)out, T, channels, taps, mode)
     if (f32) CONV_RUN(float);
     CONV_RUN(bf16);
 #undef CONV_RUN
@@ -435,13 +447,13 @@ TRL_API int trl_scan_conv(const void* proj, int ldp, const void* w, const void* 
   if (f32)
     return (int)trl_launch(scan_conv_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, (const float*)proj, ldp, (const float*)w,
                            (const float*)bias, (const float*)pre, (const float*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,
-                           (const int*)seq_ids, (const int*)q_start, (const int*)slots, (float*)out, channels, taps, silu);
+                           (const int*)seq_ids, (const int*)q_start, (const int*)slots, (float*)out, channels, taps, mode);
   return (int)trl_launch(scan_conv_kernel<bf16>, grid, dim3(128), 0, (cudaStream_t)stream, (const bf16*)proj, ldp, (const float*)w,
                          (const float*)bias, (const float*)pre, (const bf16*)ring, ring_slot, ring_rows, ring_ld, (const int*)positions,
-                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (bf16*)out, channels, taps, silu);
+                         (const int*)seq_ids, (const int*)q_start, (const int*)slots, (bf16*)out, channels, taps, mode);
 }
 
-// kind 0: Mamba-2, 1: mLSTM.  args: a ScanArgs (scan.cuh) filled by the caller.  Serves sequences of min_len..max_len tokens.
+// kind: SCAN_*.  args: a ScanArgs (scan.cuh) filled by the caller.  Serves sequences of min_len..max_len tokens.
 TRL_API int trl_scan_serial(const ScanArgs* a, int B, int kind, int f32, void* stream) {
   if (B <= 0 || scan_args_bad(*a, kind) || (a->taps && (kind != SCAN_MAMBA2 || a->taps > a->ring_rows || !a->conv_w || !a->conv_b || !a->ring ||
                                                         !a->positions || a->keep_flags)))
@@ -451,6 +463,7 @@ TRL_API int trl_scan_serial(const ScanArgs* a, int B, int kind, int f32, void* s
     return (int)(f32 ? serial_launch<float, SCAN_MAMBA2, true>(*a, B, st) : serial_launch<bf16, SCAN_MAMBA2, true>(*a, B, st));
   if (kind == SCAN_MAMBA2)
     return (int)(f32 ? serial_launch<float, SCAN_MAMBA2, false>(*a, B, st) : serial_launch<bf16, SCAN_MAMBA2, false>(*a, B, st));
+  if (kind == SCAN_FIXED) return (int)(f32 ? serial_launch<float, SCAN_FIXED, false>(*a, B, st) : serial_launch<bf16, SCAN_FIXED, false>(*a, B, st));
   return (int)(f32 ? serial_launch<float, SCAN_MLSTM, false>(*a, B, st) : serial_launch<bf16, SCAN_MLSTM, false>(*a, B, st));
 }
 

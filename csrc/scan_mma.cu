@@ -1,7 +1,7 @@
 // Decayed scans of prompts on tensor cores (mma.sync bf16): 64 tokens at a time, chunk after chunk (forms: scan.cu).
 //
 // Within a chunk every weight is one exponential of a difference: with L the running sum of the log decays, r_s the log
-// of what token s adds minus L_s, and M_t the running maximum of r and of the old state's m (mLSTM; -L_t for Mamba-2, whose
+// of what token s adds minus L_s, and M_t the running maximum of r and of the old state's m (mLSTM; -L_t for the others, whose
 // maximum is not tracked),
 //
 //   o_t = exp(m_0 - M_t) S_0^T q_t + sum_{s <= t} exp(r_s - M_t) b_s (q_t . k_s) v_s
@@ -116,15 +116,15 @@ __global__ void __launch_bounds__(SM_THREADS) scan_chunk_kernel(const ScanArgs a
     for (int e = 0; e < 2; ++e) {
       const int j = i0 + 2 * lane + e;
       g0[e] = g1[e] = 0.f;
-      if (j < T_) {
+      if (KIND != SCAN_FIXED && j < T_) {
         const float* row = a.gates + (size_t)(t0 + j) * a.ldg;
         g0[e] = row[h];
         if (KIND == SCAN_MLSTM) g1[e] = row[a.heads + h];
       }
     }
   };
-  const float bias0 = a.gate_b[h], bias1 = KIND == SCAN_MLSTM ? a.gate_b[a.heads + h] : 0.f;
-  const float rate = KIND == SCAN_MAMBA2 ? expf(a.a_log[h]) : 0.f, skip = KIND == SCAN_MAMBA2 ? a.skip[h] : 0.f;
+  const float bias0 = KIND != SCAN_FIXED ? a.gate_b[h] : 0.f, bias1 = KIND == SCAN_MLSTM ? a.gate_b[a.heads + h] : 0.f;
+  const float rate = KIND == SCAN_MAMBA2 ? expf(a.a_log[h]) : KIND == SCAN_FIXED ? a.a_log[h] : 0.f, skip = KIND == SCAN_MAMBA2 ? a.skip[h] : 0.f;
   fetch_gates(0);
   stage(0, 0);
   const int lrow = (lane & 7) + ((lane >> 3) & 1) * 8, lch = lane >> 4;      // rows / chunk of A and transposed B tiles
@@ -144,6 +144,8 @@ __global__ void __launch_bounds__(SM_THREADS) scan_chunk_kernel(const ScanArgs a
         if (KIND == SCAN_MAMBA2) {
           bb[e] = in ? softplus_x(g0[e] + bias0) : 0.f;
           la[e] = -rate * bb[e], add[e] = 0.f;
+        } else if (KIND == SCAN_FIXED) {
+          bb[e] = in ? 1.f : 0.f, la[e] = in ? rate : 0.f, add[e] = 0.f;
         } else {
           add[e] = in ? a.cap * tanhf((g0[e] + bias0) / a.cap) : -INFINITY;
           la[e] = in ? -softplus_x(-a.cap * tanhf((g1[e] + bias1) / a.cap)) : 0.f;
@@ -382,5 +384,6 @@ TRL_API int trl_scan_chunk(const ScanArgs* a, int B, int kind, int narrow, void*
       a->slot_stride % 2 || a->plane_stride % 2 || ((uintptr_t)a->rows & 15) || ((uintptr_t)a->states & 7))
     return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
+  if (kind == SCAN_FIXED) return (int)chunk_any<SCAN_FIXED>(*a, B, narrow, st);
   return (int)(kind == SCAN_MAMBA2 ? chunk_any<SCAN_MAMBA2>(*a, B, narrow, st) : chunk_any<SCAN_MLSTM>(*a, B, narrow, st));
 }

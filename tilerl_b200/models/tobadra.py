@@ -15,7 +15,7 @@ feed-forward's up rows, or behind the router's; one op gates and norms a branch,
 decode ticks, convolves it (:meth:`gated_join`).
 
 Parameter names: ``embed``, ``embed_norm``, ``final_norm`` and per layer with parameters of its own
-``L{i}.norm1|norm1b|canon|in|rg1_b|o``, the mixer's (``qkv_b|o_b``, ``norm``, ``conv|a2|g2|dt_bias|a_log``),
+``L{i}.norm1|norm1b|canon|in|rg1_b|o``, the mixer's (``qkv_b|o_b``, ``norm``, ``conv|low|dt_bias|a_log``),
 ``norm2|norm2b|rg2_b|up|down`` and ``router|correction``.
 """
 from __future__ import annotations
@@ -64,8 +64,8 @@ def _mixer_places(l, p: str, t: str, params, h: int):
     yield t + "a1", w_in[l.a0:l.a0 + s.decay_rank], None
     yield t + "g1", w_in[l.g0:l.g0 + s.gate_rank], None
     yield t + "b", w_in[l.n_in:l.n_in + l.heads], None
-    yield t + "a2", _rows(params[p + "a2"][:, :s.decay_rank], 0, l.heads, s.dim, l.dk), None
-    yield t + "g2", _rows(params[p + "g2"][:, :s.gate_rank], 0, l.heads, s.vdim, l.dv), None
+    yield t + "a2", _rows(params[p + "low"][:, :s.decay_rank], l.n_low, l.heads, s.dim, l.dk), None
+    yield t + "g2", _rows(params[p + "low"][:, :s.gate_rank], 0, l.heads, s.vdim, l.dv), None
     yield t + "dt_bias", params[p + "dt_bias"].view(l.heads, l.dk)[:, :s.dim], None
     yield t + "A_log", params[p + "a_log"], None
     yield t + "norm", params[p + "norm"][:l.vdim], None
@@ -227,7 +227,7 @@ class TobadraModel:
             proj, _, z = ops.project_in(h, hc, P[p + "in"], l.n_in, 0, l.g0, "silu")
             return ops.lightning_mix(proj, self.log_decay[i], self.head_norm[i], l, batch, state_pool, self.states[i], eps), z
         proj, gates, z = ops.project_in(h, hc, P[p + "in"], l.n_in, gate_rows(l))
-        w = {k: P[p + k] for k in ("conv", "a2", "g2", "dt_bias", "a_log")}
+        w = {k: P[p + k] for k in ("conv", "low", "dt_bias", "a_log")}
         return ops.delta_mix(proj, gates, w, self.head_norm[i], l, batch, state_pool, self.states[i], eps), z
 
     def forward(self, batch, ops, kv_pool, state_pool, *, last_only: bool = True, aux_layers: Sequence[int] = (),

@@ -27,6 +27,7 @@ import torch
 from ..formats import FP8BlockTensor, NVFP4Tensor
 from . import native as N
 from .cuda_blocks import BlockOps
+from .cuda_gated import GatedOps
 from .cuda_mixers import MixerOps
 from .cuda_stream import StreamOps
 
@@ -70,7 +71,7 @@ class Workspace:
         return t[:n].view(*shape)
 
 
-class CudaOps(StreamOps, MixerOps, BlockOps):
+class CudaOps(StreamOps, MixerOps, BlockOps, GatedOps):
     name = "cuda"
 
     def __init__(self, device="cuda", tp=None, comm=None, attn_splits: int = 0, use_tc_gemm: bool = True,

@@ -1,4 +1,4 @@
-"""CUDA ops of ``models/deluvik.py``: softmax attention with its preparation, gated linear recurrence, mixtures of experts.
+"""CUDA ops of ``models/deluvik.py`` (and, as far as it has them, ``models/tobadra.py``): softmax attention with its preparation, gated linear recurrence, mixtures of experts.
 
 Mixed into :class:`tilerl_b200.ops.cuda.CudaOps` beside :class:`~tilerl_b200.ops.cuda_mixers.MixerOps`, whose projections and joins
 they use.  The activation type is that of the weights: bf16 (the serving type) or fp32 (true fp32 everywhere).  No counterpart in
@@ -11,10 +11,11 @@ import ctypes
 import torch
 
 from . import native as N
-from .cuda_mixers import GLU_ACTS, _f32
-from .cuda_stream import EPI_STORE_F32, SHORT_ROWS
+from .cuda_mixers import ACTS, GLU_ACTS, _f32
+from .cuda_stream import SHORT_ROWS
 
 P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_long, ctypes.c_float
+MOE_UP, MOE_DOWN, MOE_ACT = 0, 1, 2
 MOE_TC_MIN = 16         # tokens from which on experts run as tensor-core tiles
 MOE_TILE = 8            # rows of a tile of the weight-streaming expert projections
 
@@ -29,7 +30,7 @@ class PrepArgs(ctypes.Structure):
     """``PrepArgs`` of ``csrc/attn_softmax.cu``."""
     _fields_ = _fields("proj ldp:i heads:i kv_heads:i dim:i dk:i dv:i k0:i v0:i n_in:i own:i taps:i conv ring ring_slot:l ring_rows:i ring_ld:i "
                        "write_ring:i q_norm k_norm norm_all:i freqs n_pairs:i half:i eps:f positions seq_ids q_start slots slot_mapping q pages "
-                       "n_blocks:i mid ldm:i pad0:i")
+                       "n_blocks:i mid ldm:i pad0:i bias vfreqs turn")
 
 
 class LruArgs(ctypes.Structure):
@@ -40,7 +41,8 @@ class LruArgs(ctypes.Structure):
 
 class MoePlan(ctypes.Structure):
     """``MoePlanArgs`` of ``csrc/moe.cu``."""
-    _fields_ = _fields("z bias ids weight place token items n_items T:i ldz:i experts:i top:i pieces:i tile:i max_items:i")
+    _fields_ = _fields("z bias ids weight place token items n_items T:i ldz:i experts:i top:i pieces:i tile:i max_items:i "
+                       "outputs:i groups:i keep:i gate_col:i scale:f")
 
 
 class BlockOps:
@@ -78,8 +80,9 @@ class BlockOps:
             self._ring_store(proj, al.n_in, ring, spool, batch)
         return q, mid
 
-    def softmax_attention(self, q, mid, al, sink, factor, batch, pool, idx):
-        """Attention output of every token, times ``factor``, into the first columns of ``mid``."""
+    def softmax_attention(self, q, mid, al, sink, factor, batch, pool, idx, turn=None):
+        """Attention output of every token, times ``factor``, into the first columns of ``mid``; with ``turn`` (cos and sin per token
+        and pair ``[T, dv / 2, 2]``) turned back first."""
         s, cache, table, lib = al.spec, pool.layer(idx), batch.block_table, self.lib
         t, g = q.shape[0], s.heads // s.kv_heads
         lens, kvs = batch.host_q_len, batch.host_kv_len
@@ -107,7 +110,7 @@ class BlockOps:
                 q.data_ptr(), cache.data_ptr(), cache.shape[0], table.data_ptr(), table.stride(0), batch.q_start.data_ptr(),
                 batch.q_len.data_ptr(), batch.positions.data_ptr(), batch.seq_ids.data_ptr(), N.ptr(sink), mid.data_ptr(), mid.stride(0),
                 N.ptr(part), N.ptr(ml), t, batch.n_seqs, tiles, lo, hi, s.heads, s.kv_heads, al.dk, al.dv, splits, wide, s.window or 0,
-                s.scale, s.cap or 0.0, factor, _f32(q), N.stream()), "softmax_attn")
+                s.scale, s.cap or 0.0, factor, N.ptr(turn), _f32(q), N.stream()), "softmax_attn")
             N.count(2 if splits > 1 else 1)
 
     def _softmax_splits(self, blocks: int, longest: int, wide: int, page_bytes: int) -> int:
@@ -156,21 +159,22 @@ class BlockOps:
     # ---- experts -----------------------------------------------------------------------------
     def _moe_plan(self, h, router, router_b, m, tile: int):
         """Router, choice and order by expert of a tick's (token, expert) pairs, in tiles of at most ``tile`` rows."""
-        t, s = h.shape[0], m.spec
-        z = self.ws.get("moe_router", (t, router.shape[0]), torch.float32)
-        if self._streams_mix(t, router):
-            self._linear_rows(h, router, z, EPI_STORE_F32)
-        else:
-            self._mm(h, router, z)
+        return self._moe_order(self.project_f32(h, router, "moe_router"), router_b, m, tile)
+
+    def _moe_order(self, z, bias, m, tile: int):
+        """The same from router logits; with the spec's ``router``, ``bias`` is the correction of its choice."""
+        t, s = z.shape[0], m.spec
         pairs = t * m.slots
         a = MoePlan()
         a.max_items = min(pairs, m.n) + pairs // tile
         ints = self.ws.get("moe_ints", (3 * pairs + 4,), torch.int32)
         weight, items = self.ws.get("moe_weight", (t, m.slots), torch.float32), self.ws.get("moe_items", (a.max_items, 4), torch.int32)
         n_items, ids, place, token = ints[:1], ints[4:4 + pairs], ints[4 + pairs:4 + 2 * pairs], ints[4 + 2 * pairs:]
-        a.z, a.bias, a.ids, a.weight, a.place = z.data_ptr(), router_b.data_ptr(), ids.data_ptr(), weight.data_ptr(), place.data_ptr()
+        a.z, a.bias, a.ids, a.weight, a.place = z.data_ptr(), bias.data_ptr(), ids.data_ptr(), weight.data_ptr(), place.data_ptr()
         a.token, a.items, a.n_items = token.data_ptr(), items.data_ptr(), n_items.data_ptr()
         a.T, a.ldz, a.experts, a.top, a.pieces, a.tile = t, z.stride(0), s.experts, s.top, m.pieces, tile
+        if s.router is not None:
+            a.outputs, a.groups, a.keep, a.scale, a.gate_col = s.outputs, s.router.groups, s.router.keep, s.router.scale, s.outputs if s.shared_gate else -1
         N.check(self.lib.trl_moe_plan(ctypes.byref(a), N.stream()), "moe_plan")
         N.count(1 if t <= 64 else 2)
         return a, place, weight
@@ -184,25 +188,29 @@ class BlockOps:
     def experts(self, h, router, router_b, gate_up, down, m):
         """Outputs of a tick's experts, ordered by expert, with the place and weight of every token's
         (:meth:`join_experts` sums them)."""
-        pairs, dt, act = h.shape[0] * m.slots, h.dtype, GLU_ACTS[m.spec.act]
+        return self._expert_rows(h, self.project_f32(h, router, "moe_router"), router_b, gate_up, down, m)
+
+    def _expert_rows(self, h, z, bias, up, down, m):
+        pairs, dt, act = h.shape[0] * m.slots, h.dtype, m.spec.act
+        kind, act = (MOE_UP, GLU_ACTS[act]) if m.spec.gated else (MOE_ACT, ACTS[act])
         if dt == torch.bfloat16 and h.shape[0] >= MOE_TC_MIN:
-            return self._experts_tc(h, router, router_b, gate_up, down, m, act)
-        plan, place, weight = self._moe_plan(h, router, router_b, m, MOE_TILE)
+            return self._experts_tc(h, z, bias, up, down, m, kind, act)
+        plan, place, weight = self._moe_order(z, bias, m, MOE_TILE)
         mid = self.ws.get(f"moe_mid_{dt}", (pairs, m.ff), dt)
         y = self.ws.get("moe_out", (pairs, down.shape[1]), torch.float32)
-        self._moe_rows(h, gate_up, mid, plan, 0, act, m)
-        self._moe_rows(mid, down, y, plan, 1, act, m)
+        self._moe_rows(h, up, mid, plan, kind, act, m)
+        self._moe_rows(mid, down, y, plan, MOE_DOWN, 0, m)
         return y, place, weight
 
-    def _experts_tc(self, h, router, router_b, gate_up, down, m, act: int):
+    def _experts_tc(self, h, z, bias, up, down, m, kind: int, act: int):
         """Many rows: tensor-core tiles of each expert's rows, gathered in order first; output rows in bf16."""
         pairs, w, bf, lib, st = h.shape[0] * m.slots, h.shape[1], torch.bfloat16, self.lib, N.stream()
-        plan, place, weight = self._moe_plan(h, router, router_b, m, lib.trl_moe_tc_tile())
+        plan, place, weight = self._moe_order(z, bias, m, lib.trl_moe_tc_tile())
         rows, mid, y = (self.ws.get(n, (pairs, k), bf) for n, k in (("moe_rows", w), ("moe_mid_tc", m.ff), ("moe_out_tc", down.shape[1])))
         N.check(lib.trl_moe_gather(h.data_ptr(), h.stride(0), plan.token, rows.data_ptr(), pairs, w, st), "moe_gather")
-        for x, wt, out, kind in ((rows, gate_up, mid, 0), (mid, down, y, 1)):
+        for x, wt, out, k, f in ((rows, up, mid, kind, act), (mid, down, y, MOE_DOWN, 0)):
             N.check(lib.trl_moe_tc(x.data_ptr(), wt.data_ptr(), out.data_ptr(), out.stride(0), plan.items, plan.n_items, pairs, wt.shape[0],
-                                   wt.shape[1], wt.shape[2], kind, act, st), "moe_tc")
+                                   wt.shape[1], wt.shape[2], k, f, st), "moe_tc")
         N.count(3)
         return y, place, weight
 

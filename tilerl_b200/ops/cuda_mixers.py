@@ -13,7 +13,9 @@ import torch
 from . import native as N
 from .cuda_stream import EPI_STORE, EPI_STORE_F32
 
-MAMBA2, MLSTM = 0, 1
+MAMBA2, MLSTM, FIXED = 0, 1, 2
+CONV_SILU, CONV_ADD = 1, 2
+ACTS = {"silu": 1, "gelu": 2, "gelu_erf": 3}
 GLU_CLAMPED = 0
 GLU_ACTS = {"silu": 1, "gelu": 2}
 MIX_ROWS_MAX = 8        # rows the weight-streaming projection serves
@@ -98,8 +100,8 @@ class MixerOps:
             return y
         return self._mm(h, w, y)
 
-    def project_f32(self, a, w):
-        y = self.ws.get("branch", (a.shape[0], w.shape[0]), torch.float32)
+    def project_f32(self, a, w, name="branch"):
+        y = self.ws.get(name, (a.shape[0], w.shape[0]), torch.float32)
         if self._streams_mix(a.shape[0], w):
             self._linear_rows(a, w, y, EPI_STORE_F32)
             return y
@@ -282,7 +284,7 @@ class MixerOps:
             N.check(self.lib.trl_scan_conv(
                 proj.data_ptr(), proj.stride(0), w["conv"].data_ptr(), w["conv_b"].data_ptr(), None, ring.data_ptr(), pool.ring.stride(0),
                 pool.ring_rows, pool.ring.stride(1), batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(),
-                batch.state_slots.data_ptr(), rows.data_ptr(), t, l.conv_c, l.taps, 1, _f32(proj), st), "scan_conv")
+                batch.state_slots.data_ptr(), rows.data_ptr(), t, l.conv_c, l.taps, CONV_SILU, _f32(proj), st), "scan_conv")
             N.count()
         if kind == MAMBA2:
             a.q0, a.k0, a.v0, a.per, a.q_scale, a.cap = l.q0, l.k0, 0, l.heads // l.groups, 1.0, 1.0
@@ -291,16 +293,25 @@ class MixerOps:
             a.q0, a.k0, a.v0, a.per, a.q_scale, a.cap = 0, l.k0, l.v0, 1, l.dim ** -0.5, l.cap
         a.rows, a.ld, a.gates, a.ldg = rows.data_ptr(), rows.stride(0), gates.data_ptr(), gates.stride(0)
         a.gate_b, a.a_log, a.skip = w["gate_b"].data_ptr(), N.ptr(w["a_log"]), N.ptr(w["skip"])
+        self._scan_state(a, o, l, batch, pool, idx)
+        self._scan(a, batch, kind, dt, st)
+        return self._scan_norm(o, proj[:, l.g0:], w["norm"], l, batch, pool, eps, kind, proj, ring)
+
+    @staticmethod
+    def _scan_state(a: ScanArgs, o, l, batch, pool, idx) -> None:
         a.states, a.slot_stride, a.plane_stride = pool.states.data_ptr() + 4 * pool.offsets[idx], pool.states.stride(0), pool.states.stride(1)
         a.cur, a.keep_flags = pool.cur.data_ptr(), N.ptr(batch.keep_flags) if batch.keep_steps else None
         a.q_start, a.q_len, a.slots = batch.q_start.data_ptr(), batch.q_len.data_ptr(), batch.state_slots.data_ptr()
         a.o, a.heads, a.dk, a.dv, a.min_len, a.max_len = o.data_ptr(), l.heads, l.dk, l.dv, 1, 1 << 30
-        self._scan(a, batch, kind, dt, st)
+
+    def _scan_norm(self, o, gate, norm, l, batch, pool, eps, kind: int, proj=None, ring=None):
+        """Normed and gated output of a scan (``kind`` MAMBA2: a tick's convolution inputs ``proj`` go into the ring, too)."""
+        t, dt = gate.shape[0], gate.dtype
         out = self.ws.get(f"mix_out_{dt}", (t, l.n_out), dt)
         N.check(self.lib.trl_scan_norm(
-            o.data_ptr(), proj[:, l.g0:].data_ptr(), proj.stride(0), w["norm"].data_ptr(), out.data_ptr(), l.n_out, t, l.heads, l.vdim, l.dv,
-            l.norm_groups, eps, proj.data_ptr(), N.ptr(ring), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1), l.conv_c,
+            o.data_ptr(), gate.data_ptr(), gate.stride(0), norm.data_ptr(), out.data_ptr(), l.n_out, t, l.heads, l.vdim, l.dv,
+            l.norm_groups, eps, N.ptr(proj), N.ptr(ring), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1), l.conv_c,
             batch.positions.data_ptr(), batch.seq_ids.data_ptr(), batch.q_start.data_ptr(), batch.q_len.data_ptr(),
-            batch.state_slots.data_ptr(), kind, _f32(proj), st), "scan_norm")
+            batch.state_slots.data_ptr(), kind, _f32(gate), N.stream()), "scan_norm")
         N.count()
         return out

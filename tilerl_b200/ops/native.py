@@ -88,6 +88,7 @@ _SIGS = {
     "trl_join": [P, P, P, I, P, I, P, P, P, F, I, I, I, I, F, I, P],
     "trl_glu": [P, P, L, I, F, I, P],
     "trl_join_experts": [P, P, I, P, P, I, P, I, P, I, P, I, I, I, F, I, P],
+    "trl_join_args": [P, I, I, P], "trl_act": [P, I, I, I, I, I, P],
     "trl_soft_cap": [P, L, F, P],
     "trl_linear_rows_cap": [P, I, P, P, I, I, I, I, F, P],
     "trl_ring_store": [P, I, P, L, I, I, I, P, P, P, P, P, I, I, P],
@@ -109,9 +110,11 @@ _SIGS = {
     "trl_scan_norm": [P, P, I, P, P, I, I, I, I, I, I, F, P, P, L, I, I, I, P, P, P, P, P, I, I, P],
     # softmax attention on packed pages, linear recurrence, experts (csrc/attn_softmax.cu, lru.cu, moe.cu)
     "trl_qkv_prep": [P, I, I, P],
-    "trl_softmax_attn": [P, P, I, P, I, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, F, I, P],
+    "trl_softmax_attn": [P, P, I, P, I, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, F, P, I, P],
     "trl_softmax_attn_rows": [I, I], "trl_softmax_attn_ok": [I, I],
     "trl_lru_scan": [P, I, I, P], "trl_lru_step": [P, I, I, P],
+    "trl_linear_rows_mix": [P, I, P, I, P, P, I, I, P, I, I, I, I, I, I, P],
+    "trl_delta_prep": [P, I, I, P], "trl_delta_serial": [P, I, I, P],
     "trl_moe_plan": [P, P],
     "trl_moe_rows": [P, I, P, P, I, P, P, P, I, I, I, I, I, I, P],
     "trl_moe_tc": [P, P, P, I, P, P, I, I, I, I, I, I, P], "trl_moe_tc_tile": [],

@@ -428,10 +428,10 @@ class RefMixers:
         return self._gated_heads(self._scan_tokens(l, batch, spool, sidx, step), proj[:, l.g0:], norm, l, eps)
 
     def delta_mix(self, proj, gates, w, norm, l, batch, spool, sidx, eps):
-        a = ref.linear(proj[:, l.a0:l.a0 + l.ra], w["a2"]) + w["dt_bias"]
+        a = ref.linear(proj[:, l.a0:l.g0], w["low"][l.n_low:]) + w["dt_bias"]
         log_keep = -torch.exp(w["a_log"])[None, :, None] * F.softplus(a).view(-1, l.heads, l.dk)
         beta = torch.sigmoid(gates[:, :l.heads].float())
-        z = ref.linear(proj[:, l.g0:l.g0 + l.rg], w["g2"])
+        z = ref.linear(proj[:, l.g0:l.n_in], w["low"][:l.n_low])
         zero = torch.zeros(l.conv_c, device=proj.device)
 
         def step(t, s, ring):

@@ -70,7 +70,8 @@ class LightningLayout:
 @dataclass(frozen=True)
 class DeltaLayout:
     """``in`` rows: ``[q kv_heads x dk | k kv_heads x dk | v heads x dv | decay map | gate map]``, then one fp32 write gate per head.
-    The first ``conv_c`` columns pass the convolution."""
+    The first ``conv_c`` columns pass the convolution.  Both maps go on from ``r`` columns to ``low`` rows: ``[gate heads x dv]``,
+    then the fp32 decays ``[heads x dk]``."""
     spec: ChannelDeltaSpec
 
     kind = "delta"
@@ -117,12 +118,8 @@ class DeltaLayout:
         return self.v0 + self.heads * self.dv
 
     @property
-    def ra(self) -> int:
-        return pad(self.spec.decay_rank, 64)
-
-    @property
-    def rg(self) -> int:
-        return pad(self.spec.gate_rank, 64)
+    def r(self) -> int:
+        return pad(max(self.spec.decay_rank, self.spec.gate_rank), 64)
 
     @property
     def a0(self) -> int:
@@ -130,11 +127,16 @@ class DeltaLayout:
 
     @property
     def g0(self) -> int:
-        return self.a0 + self.ra
+        return self.a0 + self.r
 
     @property
     def n_in(self) -> int:
-        return self.g0 + self.rg
+        return self.g0 + self.r
+
+    @property
+    def n_low(self) -> int:
+        """Rows of the output gate, before those of the decays."""
+        return self.heads * self.dv
 
     @property
     def n_gates(self) -> int:
@@ -258,7 +260,7 @@ def param_shapes(cfg) -> Dict[str, Tuple[Tuple[int, ...], str]]:
             out[p + "norm"] = ((l.heads * l.dv,), "f32")
         else:
             out[p + "norm"], out[p + "conv"] = ((l.dv,), "f32"), ((l.taps, l.conv_c), "f32")
-            out[p + "a2"], out[p + "g2"] = ((l.heads * l.dk, l.ra), "w"), ((l.heads * l.dv, l.rg), "w")
+            out[p + "low"] = ((l.n_low + l.heads * l.dk, l.r), "w")
             out[p + "dt_bias"], out[p + "a_log"] = ((l.heads * l.dk,), "f32"), ((l.heads,), "f32")
         if b.mlp is None:
             continue
