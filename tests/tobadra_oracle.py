@@ -149,7 +149,9 @@ def route(z, correction, r):
 def experts(h, w, p, f):
     r = f["router"]
     idx, weight = route(h @ w[p + "router"].T, w[p + "correction"], r)
-    out = sigmoid(h @ w[p + "shared.sg"].T) * plain_ff(h, w, p + "shared.", gelu_erf)
+    out = torch.zeros_like(h)
+    if f.get("shared") is not None:
+        out = sigmoid(h @ w[p + "shared.sg"].T) * plain_ff(h, w, p + "shared.", gelu_erf)
     for e in range(r["experts"] + r["identity"]):
         rows, place = torch.nonzero(idx == e, as_tuple=True)
         if len(rows):

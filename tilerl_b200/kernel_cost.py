@@ -15,7 +15,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Dict, List, Optional
 
-from .config import ATTN, DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, ZinutarConfig
+from .config import ATTN, DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, TobadraConfig, ZinutarConfig
 from .formats import FORMATS, nbytes
 from .parallel.mesh import tp_dims
 
@@ -134,12 +134,52 @@ def _deluvik_rows(cfg: DeluvikConfig, m: int, ctx: int, n_seqs: int, head_rows_m
     return rows
 
 
+def _tobadra_rows(cfg: TobadraConfig, m: int, ctx: int, n_seqs: int, head_rows_m: int) -> List[Row]:
+    """One forward of ``m`` tokens in ``n_seqs`` sequences that end at ``ctx`` tokens each."""
+    from .deluvik_layout import LayerLayout, MoeLayout
+    from .mixers import MoeSpec
+    from .tobadra_layout import gate_rows, head_rows, layouts, pad, router_rows, stream_width
+    w, q = stream_width(cfg), m // n_seqs
+    lin = lambda name, n, k, out=2: Row(name, 1, n * k * 2 + m * (k * 2 + n * out), 2.0 * m * n * k)
+    rows = [Row("embedding, norm, convolution", 1, m * w * (2 + 4 + 4), 0)]
+    for i, (b, l) in enumerate(zip(cfg.layers, layouts(cfg))):
+        rows.append(lin(f"L{i} in, branch gate", l.n_in + gate_rows(l) + w, w))
+        if isinstance(l, LayerLayout):
+            a, s = l.attn, l.attn.spec
+            seen = sum(min(p + 1, s.window) for p in range(ctx - q, ctx))            # (query, key) pairs of one sequence
+            keys = min(ctx, q + s.window - 1)
+            rows += [Row(f"L{i} attn.prep (bias, rotation, cache)", 1, m * a.n_in * 4.0, 0),
+                     Row(f"L{i} attn.softmax", 1, n_seqs * keys * s.kv_heads * (a.dk + a.dv) * 2 + m * s.heads * (a.dk + a.dv) * 2.0,
+                         2.0 * n_seqs * seen * s.heads * (a.dk + a.dv))]
+        else:
+            if l.kind == "delta":
+                rows += [lin(f"L{i} delta.decays and gate", l.n_low + l.heads * l.dk, l.r, 3), Row(f"L{i} delta.prep", 1, m * (l.conv_c * 4.0 + l.heads * l.dk * 8), 0)]
+            rows.append(Row(f"L{i} {l.kind}.scan", 1, n_seqs * l.state_floats * 8.0 + m * (l.n_in * 2 + l.heads * l.dv * 6.0),
+                            (4.0 if l.kind == "lightning" else 6.0) * m * l.heads * l.dk * l.dv))
+        rows += [lin(f"L{i} o", w, l.n_out, 4), Row(f"L{i} joins", 1 + (b.mlp is not None), m * w * (4 + 4 + 8 + 4.0), 0)]
+        if isinstance(b.mlp, MoeSpec):
+            e = MoeLayout(b.mlp)
+            used = e.pieces + e.spec.experts * (1.0 - (1.0 - e.spec.top / e.spec.outputs) ** m)     # experts some token chooses
+            slots = e.pieces + e.spec.top * e.spec.experts / e.spec.outputs                          # of a token, on average
+            rows.append(lin(f"L{i} router, branch gate", router_rows(b.mlp) + w, w, 4))
+            for name, n, k, out in (("up", e.ff, w, 2), ("down", w, e.ff, 4)):
+                rows.append(Row(f"L{i} experts {name}", 1, used * n * k * 2 + m * slots * (k * 2 + n * out), 2.0 * m * slots * n * k))
+        elif b.mlp is not None:
+            ff = pad(b.mlp.ff, 64)
+            rows += [lin(f"L{i} up, branch gate", ff + w, w), lin(f"L{i} down", w, ff, 4)]
+    rows.append(Row("logits", 1, head_rows(cfg) * w * 2 + head_rows_m * (w * 2 + head_rows(cfg) * 4), 2.0 * head_rows_m * head_rows(cfg) * w))
+    return rows
+
+
+_STREAM_ROWS = {FetotarConfig: _fetotar_rows, DeluvikConfig: _deluvik_rows, TobadraConfig: _tobadra_rows}
+
+
 def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
     """One decode (or verify) tick on one TP rank."""
     if isinstance(cfg, StreamDesign):
         b, c = s.batch, s.ctx
-        if isinstance(cfg, (FetotarConfig, DeluvikConfig)):
-            return (_fetotar_rows if isinstance(cfg, FetotarConfig) else _deluvik_rows)(cfg, b * s.width, c, b, b * s.width)
+        if type(cfg) in _STREAM_ROWS:
+            return _STREAM_ROWS[type(cfg)](cfg, b * s.width, c, b, b * s.width)
         return _zinutar_rows(cfg, b * s.width, b * s.width * c, b * c, b * s.width)
     d = tp_dims(cfg, s.tp)
     m = s.batch * s.width
@@ -175,10 +215,8 @@ def tick_rows(cfg: ModelConfig, s: TickShape) -> List[Row]:
 def prefill_rows(cfg: ModelConfig, tokens: int, tp: int = 1, terms: int = 2) -> List[Row]:
     """One prefill of ``tokens`` tokens (one sequence) on one TP rank; ``terms`` NVFP4
     activation terms per token multiply the tensor-core work."""
-    if isinstance(cfg, FetotarConfig):
-        return _fetotar_rows(cfg, tokens, tokens, 1, 1)
-    if isinstance(cfg, DeluvikConfig):
-        return _deluvik_rows(cfg, tokens, tokens, 1, 1)
+    if type(cfg) in _STREAM_ROWS:
+        return _STREAM_ROWS[type(cfg)](cfg, tokens, tokens, 1, 1)
     if isinstance(cfg, StreamDesign):
         return _zinutar_rows(cfg, tokens, tokens * (tokens + 1) / 2, tokens, 1)
     d = tp_dims(cfg, tp)
