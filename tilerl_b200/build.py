@@ -35,7 +35,7 @@ NVCC_FLAGS = [
 GROUPS = {"Zinutar": ("core.cu", "stream.cu", "linear_rows.cu", "attn_sigmoid.cu", "misc.cu", "runtime.cpp"),
           "Fetotar": ("core.cu", "join.cu", "linear_rows.cu", "latent.cu", "latent_mma.cu", "scan.cu", "scan_mma.cu", "misc.cu", "runtime.cpp"),
           "Deluvik": ("core.cu", "join.cu", "linear_rows.cu", "attn_softmax.cu", "lru.cu", "moe.cu", "moe_tc.cu", "scan.cu", "misc.cu", "runtime.cpp"),
-          "Tobadra": ("core.cu", "join.cu", "linear_rows.cu", "attn_softmax.cu", "moe.cu", "moe_tc.cu", "scan.cu", "scan_mma.cu", "delta.cu", "misc.cu",
+          "Tobadra": ("core.cu", "join.cu", "linear_rows.cu", "attn_softmax.cu", "moe.cu", "moe_tc.cu", "scan.cu", "scan_mma.cu", "delta.cu", "delta_mma.cu", "misc.cu",
                       "runtime.cpp")}
 
 

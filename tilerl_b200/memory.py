@@ -121,19 +121,21 @@ def workspace_bytes(cfg: ModelConfig, tokens: int, tp: int = 1) -> int:
     if isinstance(cfg, TobadraConfig):
         from .deluvik_layout import LayerLayout, MoeLayout
         from .mixers import MoeSpec
-        from .tobadra_layout import delta_chunk_floats, head_rows, layouts, pad, router_rows, stream_width
+        from .tobadra_layout import head_rows, layouts, pad, router_rows, stream_width
         ls, w = layouts(cfg), stream_width(cfg)
         moe = [MoeLayout(b.mlp) for b in cfg.layers if isinstance(b.mlp, MoeSpec)]
         up = max([pad(b.mlp.ff, 64) for b in cfg.layers if b.mlp is not None and not isinstance(b.mlp, MoeSpec)] + [0])
         # fp32 stream, branch output and branch gate, bf16 normed and convolved rows, fused projection rows, mixer output, feed-forward;
-        # queries and turns; a scan's fp32 rows; a delta rule's decays, gate, fp32 q and k, v and chunk factors; of every used expert the
+        # queries and turns; a scan's fp32 rows; a delta rule's decays, gate, fp32 q and k, v; of every used expert the
         # input row, the row between and the output row
         per = w * (4 + 4 + 4 + 2 + 2) + 2 * max(l.n_in for l in ls) + 2 * max(l.n_out for l in ls) + 2 * up
         per += max([2 * l.attn.k0 + 4 * l.attn.dv for l in ls if isinstance(l, LayerLayout)] + [0])
         per += max([4 * l.heads * l.dv for l in ls if not isinstance(l, LayerLayout)] + [0])
-        per += max([4 * l.heads * l.dk + 4 * l.n_low + 8 * l.k0 + 4 * delta_chunk_floats(l) for l in ls if getattr(l, "kind", "") == "delta"] + [0])
+        per += max([4 * l.heads * l.dk + 4 * l.n_low + 8 * l.k0 for l in ls if getattr(l, "kind", "") == "delta"] + [0])
         per += max([m.slots * (w * 6 + m.ff * 2) + 4 * (router_rows(m.spec) + w) for m in moe] + [0])
-        return tokens * per + head_rows(cfg) * 4 * 64
+        # (a delta rule's chunks go through a scratch of at most a quarter of a GiB)
+        chunks = (1 << 28) if any(getattr(l, "kind", "") == "delta" for l in ls) else 0
+        return tokens * per + head_rows(cfg) * 4 * 64 + chunks
     if isinstance(cfg, StreamDesign):
         from .zinutar_layout import BlockLayout, head_rows, stream_width
         ls = [BlockLayout.of(b) for b in cfg.layers]

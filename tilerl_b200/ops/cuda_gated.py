@@ -29,6 +29,16 @@ class DeltaArgs(ctypes.Structure):
                        "kv_heads:i dk:i dv:i min_len:i max_len:i q_scale:f")
 
 
+class DeltaSel(ctypes.Structure):
+    """``DeltaSel`` of ``csrc/delta_mma.cu``."""
+    _fields_ = _fields("n:i c0:i nc:i pad:i") + [("seq", ctypes.c_int * 64)]
+
+
+DELTA_SHORT = 16            # tokens of a sequence up to which the delta rule goes token by token
+DELTA_DK = 128              # state rows its chunked form takes
+DELTA_BYTES = 1 << 28       # most scratch of a launch's chunks
+
+
 class GatedOps:
     # ---- joins ---------------------------------------------------------------------------
     def _join_conv(self, a: JoinArgs, x, h, post, nxt, eps, n, conv):
@@ -178,9 +188,29 @@ class GatedOps:
         N.count()
         if not single:
             self._ring_store(proj, l.conv_c, ring, pool, batch)
-        N.check(self.lib.trl_delta_serial(ctypes.byref(a), batch.n_seqs, _f32(proj), st), "delta_serial")
-        N.count()
+        self._delta_scan(a, batch, dt, st)
         return self._scan_norm(o, z, norm, l, batch, pool, eps, MLSTM)
+
+    def _delta_scan(self, a: DeltaArgs, batch, dt, st) -> None:
+        """Prompts chunk by chunk on tensor cores, everything else token by token."""
+        lens, lib = batch.host_q_len, self.lib
+        long = [i for i, n in enumerate(lens) if n > DELTA_SHORT] if dt == torch.bfloat16 and a.dk <= DELTA_DK and not a.keep_flags else []
+        step = lib.trl_delta_chunk_tokens()
+        for g in range(0, len(long), 64):
+            seqs = long[g:g + 64]
+            chunks = max((lens[i] + step - 1) // step for i in seqs)
+            per = len(seqs) * a.heads * lib.trl_delta_record(a.dk, a.dv)
+            nc = max(1, min(chunks, DELTA_BYTES // per))
+            a.chunk = self.ws.get("delta_chunks", (nc * per // 4,), torch.float32).data_ptr()
+            narrow = int(len(seqs) * a.heads * ((a.dv + 63) // 64) < self.sms)
+            for c0 in range(0, chunks, nc):
+                sel = DeltaSel(len(seqs), c0, min(nc, chunks - c0), 0, (ctypes.c_int * 64)(*seqs))
+                N.check(lib.trl_delta_chunk(ctypes.byref(a), ctypes.byref(sel), narrow, st), "delta_chunk")
+                N.count(2)
+        if len(long) < len(lens):
+            a.min_len, a.max_len = 1, DELTA_SHORT if long else 1 << 30
+            N.check(lib.trl_delta_serial(ctypes.byref(a), batch.n_seqs, int(dt == torch.float32), st), "delta_serial")
+            N.count()
 
     # ---- experts -----------------------------------------------------------------------------
     def routed_experts(self, h, z, correction, up, down, m):

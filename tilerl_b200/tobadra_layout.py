@@ -155,11 +155,6 @@ class DeltaLayout:
         return self.heads * self.dk * self.dv
 
 
-def delta_chunk_floats(l: DeltaLayout) -> int:
-    """fp32 values a token of a prompt has between the two kernels of the chunked delta rule."""
-    return 0
-
-
 def layout_of(m):
     if isinstance(m, SoftmaxAttnSpec):
         return LayerLayout(AttnLayout(m), None)
