@@ -190,7 +190,7 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN)
     ap.add_argument("--gen", type=int, default=GEN_LEN)
     ap.add_argument("--no-control", action="store_true", help="skip the unfused same-box control at N > 1")
-    ap.add_argument("--design", default=None, choices=["zinutar", "fetotar", "deluvik"],
+    ap.add_argument("--design", default=None, choices=["zinutar", "fetotar", "deluvik", "tobadra"],
                     help="measure another design beside the closest hybrid form at equal size instead (tilerl_b200/suites/<design>.py; "
                          "its own flags follow)")
     args, rest = ap.parse_known_args()

@@ -6,6 +6,7 @@
 //                        every q / k head, log g = -exp(A) softplus(low + bias) per channel, beta = sigmoid(gate).
 //   delta_serial_kernel  token after token, 32 value columns of a head per block, the state in registers: decoding, windows of kept
 //                        states, short portions, and fp32 models.  o = (g S)^T q + (k . q) u, so a token needs one block barrier.
+//   delta_step_kernel    one token per sequence from projection rows to normed and gated ones (heads up to 128 x 128).
 //   (prompts: delta_mma.cu; the norm and gate behind it: scan_norm_kernel of scan.cu)
 //
 // q, k, decays, beta, state and sums are fp32; v is in the compute type, as its convolution leaves it.
@@ -14,8 +15,13 @@
 
 namespace {
 
+// silu of a short convolution
+template <typename T> __device__ __forceinline__ float conv_silu(float x) {
+  return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : x * sigmoid_x(x);
+}
+
 template <typename T>
-__global__ void __launch_bounds__(512) delta_prep_kernel(const DeltaArgs a) {
+__global__ void __launch_bounds__(512, 2) delta_prep_kernel(const DeltaArgs a) {
   constexpr int C = Chunk<T>::N;
   extern __shared__ __align__(16) float s_row[];               // [2 k0] convolved q and k
   pdl_launch_dependents(70);
@@ -27,14 +33,13 @@ __global__ void __launch_bounds__(512) delta_prep_kernel(const DeltaArgs a) {
   for (int c = tid * C; c < a.channels; c += nt * C) {
     const uint4 own = *reinterpret_cast<const uint4*>(row + c);
     float f[C], acc[C];
-    Chunk<T>::get(own, f);
 #pragma unroll
     for (int e = 0; e < C; ++e) acc[e] = 0.f;
-    for (int back = 0; back < a.taps && back <= pos; ++back) {
-      if (back) {
-        const T* src = t - back >= t0 ? row - (size_t)back * a.ldp + c : ring + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + c;
-        Chunk<T>::get(*reinterpret_cast<const uint4*>(src), f);
-      }
+#pragma unroll 4
+    for (int back = 0; back < a.taps; ++back) {
+      if (back > pos) break;
+      const T* src = t - back >= t0 ? row - (size_t)back * a.ldp + c : ring + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + c;
+      Chunk<T>::get(*reinterpret_cast<const uint4*>(src), f);
 #pragma unroll
       for (int e = 0; e < C; e += 4) {
         const float4 w = __ldg(reinterpret_cast<const float4*>(a.conv_w + (size_t)(a.taps - 1 - back) * a.channels + c + e));
@@ -43,7 +48,7 @@ __global__ void __launch_bounds__(512) delta_prep_kernel(const DeltaArgs a) {
       }
     }
 #pragma unroll
-    for (int e = 0; e < C; ++e) acc[e] *= sigmoid_x(acc[e]);
+    for (int e = 0; e < C; ++e) acc[e] = conv_silu<T>(acc[e]);
     if (a.write_ring) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.ring_rows) * a.ring_ld + c) = own;
     const uint4 out = Chunk<T>::put(acc);
     if (c >= a.v0) {
@@ -161,6 +166,86 @@ __global__ void __launch_bounds__(256, RMAX <= 16 ? 4 : 2) delta_serial_kernel(c
   if (!keep_all) save(plane);
 }
 
+// One token per sequence, preparation and norm included: grid (heads, sequences); a warp owns 32 columns and a quarter of the rows.
+constexpr int DT_COLS = 128;
+template <typename T, int RMAX>
+__global__ void __launch_bounds__(512, 2) delta_step_kernel(const DeltaArgs a, const T* gate, int ldg, const float* __restrict__ norm, T* out, int ldo,
+                                                         int vdim, float eps) {
+  __shared__ float s_q[4 * RMAX], s_k[4 * RMAX], s_g[4 * RMAX], s_v[DT_COLS], s_p[4][DT_COLS], s_o[4][DT_COLS], s_sum[3], s_ss[4];
+  pdl_launch_dependents(74);
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nt = blockDim.x;
+  if (a.q_len[seq] == 0) {
+    pdl_wait();
+    return;
+  }
+  const int grp = warp & 3, col = (warp >> 2) * 32 + lane, R = a.dk / 4, t = a.q_start[seq], slot = a.slots[seq];
+  const bool in = col < a.dv;
+  float* st = a.states + (size_t)slot * a.slot_stride + (size_t)a.cur[slot] * a.plane_stride + ((size_t)h * a.dk + grp * R) * a.dv + col;
+  float S[RMAX];
+#pragma unroll
+  for (int r = 0; r < RMAX; ++r) S[r] = r < R && in ? st[(size_t)r * a.dv] : 0.f;      // (before the wait: see delta_serial_kernel)
+  pdl_wait();
+  const int per = a.heads / a.kv_heads, kh = h / per, pos = a.positions[t];
+  const T* row = reinterpret_cast<const T*>(a.rows) + (size_t)t * a.ldp;
+  T* ring = reinterpret_cast<T*>(a.ring) + (size_t)slot * a.ring_slot;
+  for (int x = tid; x < 2 * a.dk + a.dv; x += nt) {
+    const bool is_v = x >= 2 * a.dk, is_k = !is_v && x >= a.dk;
+    const int c = is_v ? a.v0 + h * a.dv + x - 2 * a.dk : is_k ? a.k0 + kh * a.dk + x - a.dk : kh * a.dk + x;
+    const T own = row[c];
+    float v = 0.f;
+#pragma unroll 4
+    for (int j = 0; j < a.taps; ++j) {
+      const int back = a.taps - 1 - j;
+      if (back <= pos) v = fmaf(to_f(back ? ring[(size_t)((pos - back) % a.ring_rows) * a.ring_ld + c] : own), a.conv_w[(size_t)j * a.channels + c], v);
+    }
+    v = to_f(from_f<T>(conv_silu<T>(v)));
+    if (is_v) s_v[x - 2 * a.dk] = v;
+    else if (is_k) s_k[x - a.dk] = v;
+    else s_q[x] = v;
+    if (is_v || h % per == 0) ring[(size_t)(pos % a.ring_rows) * a.ring_ld + c] = own;      // (no block reads this row of the ring)
+  }
+  const float rate = -expf(a.a_log[h]);
+  for (int d = tid; d < a.dk; d += nt) s_g[d] = expf(rate * softplus_x(a.low[((size_t)t * a.heads + h) * a.dk + d] + a.dt_bias[h * a.dk + d]));
+  __syncthreads();
+  if (warp < 3) {                              // q . q, k . k, q . k
+    const float *x = warp == 1 ? s_k : s_q, *y = warp == 0 ? s_q : s_k;
+    float d = 0.f;
+    for (int c = lane; c < a.dk; c += 32) d = fmaf(x[c], y[c], d);
+    d = warp_sum(d);
+    if (lane == 0) s_sum[warp] = d;
+  }
+  float p = 0.f, o = 0.f;
+#pragma unroll
+  for (int r = 0; r < RMAX; ++r)
+    if (r < R) {
+      S[r] *= s_g[grp * R + r];
+      p = fmaf(s_k[grp * R + r], S[r], p), o = fmaf(s_q[grp * R + r], S[r], o);
+    }
+  s_p[grp][col] = p, s_o[grp][col] = o;
+  __syncthreads();
+  const float fq = a.q_scale / sqrtf(s_sum[0] + 1e-6f), fk = 1.f / sqrtf(s_sum[1] + 1e-6f);
+  p = (s_p[0][col] + s_p[1][col] + s_p[2][col] + s_p[3][col]) * fk;
+  const float beta = sigmoid_x(a.gates[(size_t)t * a.ldg + h]), u = in ? beta * (s_v[col] - p) : 0.f;
+#pragma unroll
+  for (int r = 0; r < RMAX; ++r)
+    if (r < R && in) st[(size_t)r * a.dv] = fmaf(s_k[grp * R + r] * fk, u, S[r]);
+  float y = 0.f;
+  if (grp == 0) {
+    if (in) y = fmaf(s_sum[2] * fq * fk, u, (s_o[0][col] + s_o[1][col] + s_o[2][col] + s_o[3][col]) * fq);
+    const float ss = warp_sum(y * y);          // (padding columns hold zeros)
+    if (lane == 0) s_ss[warp >> 2] = ss;
+  }
+  __syncthreads();
+  if (grp == 0) {
+    float ss = 0.f;
+    for (int w = 0; w * 32 < a.dv; ++w) ss += s_ss[w];
+    const int c = h * a.dv + col;
+    if (in) out[(size_t)t * ldo + c] = from_f<T>(y * inv_rms(ss, vdim, eps) * norm[c] * sigmoid_x(to_f(gate[(size_t)t * ldg + c])));
+  }
+  if (h == 0)
+    for (int c = a.heads * a.dv + tid; c < ldo; c += nt) out[(size_t)t * ldo + c] = from_f<T>(0.f);
+}
+
 template <typename T> cudaError_t serial_launch(const DeltaArgs& a, int B, cudaStream_t st) {
   const dim3 grid(a.heads * ((a.dv + 31) / 32), B);
   if (a.dk <= 32) return trl_launch(delta_serial_kernel<T, 4>, grid, dim3(256), 0, st, a);
@@ -187,7 +272,7 @@ TRL_API int trl_delta_prep(const DeltaArgs* args, int T, int f32, void* stream) 
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const int threads = a.channels >= 4096 ? 512 : 256;
+  const int threads = T <= 148 && a.channels >= 4096 ? 512 : 256;
   if (f32) return (int)trl_launch(delta_prep_kernel<float>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, a);
   return (int)trl_launch(delta_prep_kernel<bf16>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, a);
 }
@@ -197,4 +282,30 @@ TRL_API int trl_delta_serial(const DeltaArgs* args, int B, int f32, void* stream
   const DeltaArgs& a = *args;
   if (B <= 0 || delta_args_bad(a) || !a.states || !a.o || !a.cur || !a.q_start || !a.q_len || !a.slots) return (int)cudaErrorInvalidValue;
   return (int)(f32 ? serial_launch<float>(a, B, (cudaStream_t)stream) : serial_launch<bf16>(a, B, (cudaStream_t)stream));
+}
+
+// Heads that trl_delta_step takes.
+TRL_API int trl_delta_step_ok(int dk, int dv) { return dk <= 128 && dv <= DT_COLS; }
+
+// One token per sequence, no kept states: rows -> out [T, ldo], normed per head (over vdim values), times norm [heads * dv], times
+// sigmoid(gate [T, ldg]); the state moves on and the rows go into the ring.  a.q, a.k, a.v, a.keep, a.beta and a.o are not used.
+TRL_API int trl_delta_step(const DeltaArgs* args, int B, const void* gate, int ldg, const void* norm, void* out, int ldo, int vdim, float eps,
+                           int f32, void* stream) {
+  const DeltaArgs& a = *args;
+  if (B <= 0 || a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dk <= 0 || a.dk % 16 || a.dv <= 0 || a.dv % 16 || !trl_delta_step_ok(a.dk, a.dv) ||
+      a.keep_flags || !a.states || !a.cur || !a.q_start || !a.q_len || !a.slots || !a.positions || !a.rows || !a.conv_w || !a.ring || !a.low || !a.dt_bias ||
+      !a.a_log || !a.gates || a.taps < 1 || a.taps > a.ring_rows || a.ldg < a.heads || !gate || !norm || !out || ldo < a.heads * a.dv ||
+      ldg < a.heads * a.dv || vdim < 1 || vdim > a.dv || a.k0 != a.kv_heads * a.dk || a.v0 != 2 * a.k0 || a.channels != a.v0 + a.heads * a.dv)
+    return (int)cudaErrorInvalidValue;
+  const dim3 grid(a.heads, B), block((a.dv + 31) / 32 * 128);
+  cudaStream_t st = (cudaStream_t)stream;
+#define DELTA_STEP(TT, RR)                                                                                                             \
+  return (int)trl_launch(delta_step_kernel<TT, RR>, grid, block, 0, st, a, (const TT*)gate, ldg, (const float*)norm, (TT*)out, ldo, vdim, eps)
+  if (f32) {
+    if (a.dk <= 64) DELTA_STEP(float, 16);
+    DELTA_STEP(float, 32);
+  }
+  if (a.dk <= 64) DELTA_STEP(bf16, 16);
+  DELTA_STEP(bf16, 32);
+#undef DELTA_STEP
 }

@@ -11,7 +11,7 @@
 //                       fp32; goes out as one record whose tiles have the order in which the scan's shared memory wants them.
 //   delta_scan_kernel   a block per (head, 32 or 64 value columns, sequence), four warps on mma.sync: chunk after chunk, the state in fp32
 //                       registers.  Every operand enters its products as a bf16 pair (value and rest; three products), so it keeps 16
-//                       bits of mantissa; sums are fp32.  The next record is copied (cp.async) while this one is used.
+//                       bits of mantissa; sums are fp32.  Each half of a record is copied (cp.async) while the other half is used.
 // Reference parity: the reference's chunked delta rule has one decay per head (no counterpart).
 #include "delta.cuh"
 
@@ -221,13 +221,13 @@ __global__ void __launch_bounds__(DF_THREADS) delta_form_kernel(const DeltaArgs 
 }
 
 template <int DK, int DV> struct ScanSm {
-  static constexpr int HEAD = Rec<DK>::U, STAGE = HEAD + DV / 32 * Rec<DK>::USLICE, VROW = DV * 2;
-  __align__(128) unsigned char st[2][STAGE];
+  static constexpr int HEAD = Rec<DK>::U, VROW = DV * 2;
+  __align__(128) unsigned char st[HEAD], u[DV / 32 * Rec<DK>::USLICE];
   __align__(128) unsigned char s_hi[DK * VROW], s_lo[DK * VROW], d_hi[DC * VROW], d_lo[DC * VROW];
 };
 
 template <int DK, int DV>
-__global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs a, const DeltaSel sel) {
+__global__ void __launch_bounds__(DS_THREADS, 2) delta_scan_kernel(const DeltaArgs a, const DeltaSel sel) {
   using R = Rec<DK>;
   using SM = ScanSm<DK, DV>;
   constexpr int MT = DK / 64, NT = DV / 8, NH = NT / 2, VROW = SM::VROW;
@@ -243,18 +243,25 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs 
   const int slot = a.slots[seq];
   float* s_rec = a.states + (size_t)slot * a.slot_stride + (size_t)a.cur[slot] * a.plane_stride + (size_t)h * a.dk * a.dv + col0;
   auto u32 = [](const void* p) { return (uint32_t)__cvta_generic_to_shared(p); };
-  const uint32_t st_a[2] = {u32(sm.st[0]), u32(sm.st[1])}, sh_a = u32(sm.s_hi), sl_a = u32(sm.s_lo), dh_a = u32(sm.d_hi), dl_a = u32(sm.d_lo);
+  const uint32_t base = u32(sm.st), u_a = u32(sm.u), sh_a = u32(sm.s_hi), sl_a = u32(sm.s_lo), dh_a = u32(sm.d_hi), dl_a = u32(sm.d_lo);
   const size_t rec_bytes = R::bytes(a.dv);
   const unsigned char* recs = reinterpret_cast<const unsigned char*>(a.chunk) + ((size_t)blockIdx.y * sel.nc * a.heads + h) * rec_bytes;
   const int u_bytes = min(DV / 32, (a.dv + 31) / 32 - slice * (DV / 32)) * R::USLICE;
-  auto stage = [&](int c, int b) {
+  // a record comes in two parts: what the products with the state need (W, q, U), then what those with u need (k, N, factors)
+  auto stage1 = [&](int c) {
     const unsigned char* src = recs + (size_t)(c - sel.c0) * a.heads * rec_bytes;
-#pragma unroll 4
-    for (int x = tid * 16; x < SM::HEAD; x += DS_THREADS * 16) cp16(st_a[b] + x, src + x);
-    for (int x = tid * 16; x < u_bytes; x += DS_THREADS * 16) cp16(st_a[b] + SM::HEAD + x, src + R::U + slice * (DV / 32) * R::USLICE + x);
+#pragma unroll 8
+    for (int x = tid * 16; x < 4 * R::TILE; x += DS_THREADS * 16) cp16(base + x, src + x);
+    for (int x = tid * 16; x < u_bytes; x += DS_THREADS * 16) cp16(u_a + x, src + R::U + slice * (DV / 32) * R::USLICE + x);
     cp_commit();
   };
-  stage(first, 0);
+  auto stage2 = [&](int c) {
+    const unsigned char* src = recs + (size_t)(c - sel.c0) * a.heads * rec_bytes;
+#pragma unroll 8
+    for (int x = 4 * R::TILE + tid * 16; x < SM::HEAD; x += DS_THREADS * 16) cp16(base + x, src + x);
+    cp_commit();
+  };
+  stage1(first);
 
   // rows of the state this warp owns: 16 (MT warp + mt) .. + 15
   float S[MT][NT][4];
@@ -286,12 +293,10 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs 
   const int lrow = (lane & 7) + ((lane >> 3) & 1) * 8, lch = lane >> 4;      // rows / chunk of A and transposed B tiles
   const int brow = (lane & 7) + (lane >> 4) * 8, bch = (lane >> 3) & 1;      // of transposed A tiles
   const int mrow = 16 * (warp & 1), n0 = (warp >> 1) * NH;                   // this warp's tokens and columns (in eights)
-  int b = 0;
-  for (int c = first; c < last; ++c, b ^= 1) {
+  for (int c = first; c < last; ++c) {
     cp_wait<0>();
-    __syncthreads();                        // this chunk's record and the state's copy are in; the other stage is free
-    if (c + 1 < last) stage(c + 1, b ^ 1);
-    const uint32_t base = st_a[b];
+    __syncthreads();                        // the first part and the state's copy are in; the second part's place is free
+    stage2(c);
     // ---- P = W S, O = q S of this warp's 16 tokens and columns; main products and rests in sums of their own
     float P[NH][4], O[NH][4], X[NH][4], Y[NH][4];
 #pragma unroll
@@ -326,13 +331,15 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs 
       for (int i = 0; i < 2; ++i) {
         const int r = mrow + g8 + 8 * i, cc = (n0 + nt) * 8 + 2 * t4;
         float2 u = make_float2(0.f, 0.f);
-        if (col0 + cc < a.dv) u = *reinterpret_cast<const float2*>(sm.st[b] + SM::HEAD + (cc >> 5) * R::USLICE + (r * 32 + (cc & 31)) * 4);
+        if (col0 + cc < a.dv) u = *reinterpret_cast<const float2*>(sm.u + (cc >> 5) * R::USLICE + (r * 32 + (cc & 31)) * 4);
         uint32_t hi, lo;
         split2(u.x - (P[nt][2 * i] + X[nt][2 * i]), u.y - (P[nt][2 * i + 1] + X[nt][2 * i + 1]), hi, lo);
         const uint32_t o = tile_off<VROW>(r, n0 + nt) + t4 * 4;
         *reinterpret_cast<uint32_t*>(sm.d_hi + o) = hi, *reinterpret_cast<uint32_t*>(sm.d_lo + o) = lo;
       }
-    __syncthreads();
+    cp_wait<0>();
+    __syncthreads();                        // u and the second part are in; the first part's place is free
+    if (c + 1 < last) stage1(c + 1);
     // ---- O += N u
 #pragma unroll
     for (int kt = 0; kt < DC / 16; ++kt) {
@@ -367,7 +374,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaArgs 
       }
     }
     // ---- S = e^(G_C) S + (decayed keys)^T u
-    const float* eg = reinterpret_cast<const float*>(sm.st[b] + R::G);
+    const float* eg = reinterpret_cast<const float*>(sm.st + R::G);
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       const float f0 = eg[(MT * warp + mt) * 16 + g8], f1 = eg[(MT * warp + mt) * 16 + g8 + 8];
@@ -417,6 +424,7 @@ template <int DK, int DV> cudaError_t scan_launch(const DeltaArgs& a, const Delt
   if (!configured) {
     const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(ScanSm<DK, DV>));
     if (e != cudaSuccess) return e;
+    cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     configured = true;
   }
   return trl_launch(k, dim3(a.heads * ((a.dv + DV - 1) / DV), s.n), dim3(DS_THREADS), sizeof(ScanSm<DK, DV>), st, a, s);
@@ -427,6 +435,7 @@ template <int DK> cudaError_t chunk_launch(const DeltaArgs& a, const DeltaSel& s
   if (!configured) {
     const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(FormSmem<DK>));
     if (e != cudaSuccess) return e;
+    cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
     configured = true;
   }
   const cudaError_t e = trl_launch(k, dim3(s.nc, a.heads, s.n), dim3(DF_THREADS), sizeof(FormSmem<DK>), st, a, s);

@@ -77,8 +77,11 @@ struct JoinArgs {
 
 namespace {
 
-template <typename T, int R>
-__global__ void __launch_bounds__(512) join_kernel(const JoinArgs a) {
+template <typename T> __device__ __forceinline__ float gate_x(float z) { return sizeof(T) == 2 ? sigmoid_f(z) : sigmoid_x(z); }
+
+// GATED: branches with a gate, rows of the token itself, a convolution on the result.
+template <typename T, int R, bool GATED>
+__global__ void __launch_bounds__(512, R <= 2 ? 2 : 1) join_kernel(const JoinArgs a) {
   __shared__ float red[32];
   pdl_launch_dependents(30);
   pdl_wait();
@@ -114,13 +117,14 @@ __global__ void __launch_bounds__(512) join_kernel(const JoinArgs a) {
       if (k < ld) *reinterpret_cast<float4*>(xr + k) = v[i];
     }
   } else {
-    float4 xv[R];
+    float4 xv[R], zv[R];
     const int parts = a.slots ? a.slots : 1;
 #pragma unroll
     for (int i = 0; i < R; ++i) {
       const int k = (threadIdx.x + i * blockDim.x) * 4;
-      v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      v[i] = xv[i] = zv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (k < ld) xv[i] = load4(xr + k);
+      if (GATED && k < ld) zv[i] = load4(a.z + (size_t)t * a.ldz + k);
     }
     for (int j = 0; j < parts; ++j) {        // rows y[place[t, j]], weighted; without slots the token's own row
       const float wj = a.slots ? a.weight[(size_t)t * a.slots + j] : 1.f;
@@ -130,13 +134,13 @@ __global__ void __launch_bounds__(512) join_kernel(const JoinArgs a) {
       for (int i = 0; i < R; ++i) {
         const int k = (threadIdx.x + i * blockDim.x) * 4;
         if (k < ld) {
-          const float4 b = row < 0 ? load4(reinterpret_cast<const T*>(a.own) + (size_t)t * ld + k)
+          const float4 b = GATED && row < 0 ? load4(reinterpret_cast<const T*>(a.own) + (size_t)t * ld + k)
                            : a.y_bf16 ? load4(reinterpret_cast<const bf16*>(a.y) + yr + k) : load4(reinterpret_cast<const float*>(a.y) + yr + k);
           v[i].x = fmaf(wj, b.x, v[i].x), v[i].y = fmaf(wj, b.y, v[i].y), v[i].z = fmaf(wj, b.z, v[i].z), v[i].w = fmaf(wj, b.w, v[i].w);
         }
       }
     }
-    if (a.z) {
+    if constexpr (GATED) {
 #pragma unroll
       for (int i = 0; i < R; ++i) {
         const int k = (threadIdx.x + i * blockDim.x) * 4;
@@ -145,8 +149,8 @@ __global__ void __launch_bounds__(512) join_kernel(const JoinArgs a) {
             const float4 b = load4(a.bias + k);
             v[i].x += b.x, v[i].y += b.y, v[i].z += b.z, v[i].w += b.w;
           }
-          const float4 z = load4(a.z + (size_t)t * a.ldz + k), b = load4(a.z_b + k);
-          v[i].x *= sigmoid_x(z.x + b.x), v[i].y *= sigmoid_x(z.y + b.y), v[i].z *= sigmoid_x(z.z + b.z), v[i].w *= sigmoid_x(z.w + b.w);
+          const float4 b = load4(a.z_b + k);
+          v[i].x *= gate_x<T>(zv[i].x + b.x), v[i].y *= gate_x<T>(zv[i].y + b.y), v[i].z *= gate_x<T>(zv[i].z + b.z), v[i].w *= gate_x<T>(zv[i].w + b.w);
         }
       }
     }
@@ -164,20 +168,20 @@ __global__ void __launch_bounds__(512) join_kernel(const JoinArgs a) {
   T* hr = reinterpret_cast<T*>(a.h) + (size_t)t * ld;
   float2 st = make_float2(0.f, 1.f);
   if (a.next_kind != NORM_NONE) st = row_stats<R>(v, a.next_kind, n, a.eps, red);
-  const int pos = a.taps ? a.positions[t] : 0;
-  T* rg = reinterpret_cast<T*>(a.ring) + (a.taps ? (size_t)a.state_slots[a.seq_ids[t]] * a.ring_slot : 0);
+  const int taps = GATED ? a.taps : 0, pos = taps ? a.positions[t] : 0;
+  T* rg = reinterpret_cast<T*>(a.ring) + (taps ? (size_t)a.state_slots[a.seq_ids[t]] * a.ring_slot : 0);
 #pragma unroll
   for (int i = 0; i < R; ++i) {
     const int k = (threadIdx.x + i * blockDim.x) * 4;
     if (k < ld) {
       const float4 o = a.next_kind == NORM_NONE ? v[i] : apply_norm(v[i], st, a.next_kind, a.next, ld, k);
       store4<T>(hr + k, o.x, o.y, o.z, o.w);
-      if (a.taps) {                          // the convolution reads rounded rows, as it will find them in the ring
+      if (GATED && taps) {                   // the convolution reads rounded rows, as it will find them in the ring
         const float4 own = make_float4(to_f(from_f<T>(o.x)), to_f(from_f<T>(o.y)), to_f(from_f<T>(o.z)), to_f(from_f<T>(o.w)));
         float4 c = own;
-        for (int back = 0; back < a.taps && back <= pos; ++back) {
+        for (int back = 0; back < taps && back <= pos; ++back) {
           const float4 f = back ? load4(rg + (size_t)((pos - back) % a.ring_rows) * a.ring_ld + k) : own;
-          const float4 w = load4(a.conv_w + (size_t)(a.taps - 1 - back) * ld + k);
+          const float4 w = load4(a.conv_w + (size_t)(taps - 1 - back) * ld + k);
           c.x = fmaf(f.x, w.x, c.x), c.y = fmaf(f.y, w.y, c.y), c.z = fmaf(f.z, w.z, c.z), c.w = fmaf(f.w, w.w, c.w);
         }
         store4<T>(reinterpret_cast<T*>(a.hc) + (size_t)t * ld + k, c.x, c.y, c.z, c.w);
@@ -239,8 +243,15 @@ side_kernel(const T* z, const T* __restrict__ side, const int* ids, T* out, int 
 
 template <typename T>
 cudaError_t join_launch(const JoinArgs& a, int T_, cudaStream_t st) {
-  const int ld = a.ld, thr = ld >= 2048 ? 512 : (ld >= 1024 ? 256 : 128), need = (ld / 4 + thr - 1) / thr;
-#define JOIN(R) return trl_launch(join_kernel<T, R>, dim3(T_), dim3(thr), 0, st, a)
+  // (the stream's first row has no gate: with a convolution it takes the gated form, whose steps look at their pointers)
+  const bool gated = a.z || a.taps;
+  const int ld = a.ld, thr = ld >= (gated && T_ > 148 ? 4096 : 2048) ? 512 : (ld >= 1024 ? 256 : 128);
+  const int need = (ld / 4 + thr - 1) / thr;
+#define JOIN(R)                                                                            \
+  {                                                                                        \
+    if (gated) return trl_launch(join_kernel<T, R, true>, dim3(T_), dim3(thr), 0, st, a);  \
+    return trl_launch(join_kernel<T, R, false>, dim3(T_), dim3(thr), 0, st, a);            \
+  }
   if (need <= 1) JOIN(1);
   if (need <= 2) JOIN(2);
   if (need <= 4) JOIN(4);
@@ -258,7 +269,7 @@ TRL_API int trl_join_args(const JoinArgs* args, int T, int f32, void* stream) {
   const int per = f32 ? 4 : 8;
   if (T <= 0 || a.ld % 64 || a.ld > 16384 || a.n <= 0 || a.n > a.ld || !a.x || !a.h || (!a.table && (!a.y || !a.post)) ||
       (a.post && (a.post_kind < 1 || a.post_kind > 2)) || a.next_kind < 0 || a.next_kind > 2 || (a.next_kind && !a.next) || (a.table && !a.ids) ||
-      a.slots < 0 || (a.slots && (!a.place || !a.weight)) || (a.z && (!a.z_b || a.ldz % 4 || a.ldz < a.ld)) || (a.bias && !a.z) || a.taps < 0 ||
+      a.slots < 0 || (a.slots && (!a.place || !a.weight)) || (a.z && (!a.z_b || a.ldz % 4 || a.ldz < a.ld || a.table)) || (a.taps && !a.z && !a.table) || (a.bias && !a.z) || a.taps < 0 ||
       (a.taps && (!a.hc || !a.conv_w || !a.ring || !a.positions || !a.seq_ids || !a.state_slots || a.taps > a.ring_rows || a.ring_ld % per ||
                   a.ring_slot % per || ((uintptr_t)a.ring & 15))))
     return (int)cudaErrorInvalidValue;

@@ -173,17 +173,24 @@ class GatedOps:
         else:
             self._mm(proj[:, l.g0:l.n_in], low[:l.n_low], z)
             self._mm(proj[:, l.a0:l.g0], low[l.n_low:], keep)
-        o, q, k, beta = f32("scan_o", l.heads * l.dv), f32("delta_q", l.k0), f32("delta_k", l.k0), f32("delta_beta", l.heads)
-        v, ring, single = self.ws.get(f"delta_v_{dt}", (t, l.heads * l.dv), dt), pool.ring_view(idx, 0), batch.max_q_len == 1
+        ring, single = pool.ring_view(idx, 0), batch.max_q_len == 1
         a = DeltaArgs()
         a.rows, a.ldp, a.conv_w, a.taps, a.channels, a.k0, a.v0 = proj.data_ptr(), proj.stride(0), w["conv"].data_ptr(), l.taps, l.conv_c, l.k0, l.v0
         a.ring, a.ring_slot, a.ring_rows, a.ring_ld, a.write_ring = ring.data_ptr(), pool.ring.stride(0), pool.ring_rows, pool.ring.stride(1), int(single)
-        a.low, a.keep, a.dt_bias, a.a_log, a.gates, a.ldg = keep.data_ptr(), keep.data_ptr(), w["dt_bias"].data_ptr(), w["a_log"].data_ptr(), gates.data_ptr(), gates.stride(0)
-        a.q, a.k, a.v, a.beta, a.o, a.q_scale = q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), o.data_ptr(), l.spec.dim ** -0.5
+        a.low, a.dt_bias, a.a_log, a.gates, a.ldg = keep.data_ptr(), w["dt_bias"].data_ptr(), w["a_log"].data_ptr(), gates.data_ptr(), gates.stride(0)
         a.states, a.slot_stride, a.plane_stride = pool.states.data_ptr() + 4 * pool.offsets[idx], pool.states.stride(0), pool.states.stride(1)
         a.cur, a.keep_flags = pool.cur.data_ptr(), N.ptr(batch.keep_flags) if batch.keep_steps else None
         a.q_start, a.q_len, a.slots, a.positions, a.seq_ids = (x.data_ptr() for x in (batch.q_start, batch.q_len, batch.state_slots, batch.positions, batch.seq_ids))
-        a.heads, a.kv_heads, a.dk, a.dv, a.min_len, a.max_len = l.heads, l.kv_heads, l.dk, l.dv, 1, 1 << 30
+        a.heads, a.kv_heads, a.dk, a.dv, a.min_len, a.max_len, a.q_scale = l.heads, l.kv_heads, l.dk, l.dv, 1, 1 << 30, l.spec.dim ** -0.5
+        if single and not batch.keep_steps and self.lib.trl_delta_step_ok(l.dk, l.dv):
+            out = self.ws.get(f"mix_out_{dt}", (t, l.n_out), dt)
+            N.check(self.lib.trl_delta_step(ctypes.byref(a), batch.n_seqs, z.data_ptr(), z.stride(0), norm.data_ptr(), out.data_ptr(), l.n_out, l.vdim, eps,
+                                            _f32(proj), st), "delta_step")
+            N.count()
+            return out
+        o, q, k, beta = f32("scan_o", l.heads * l.dv), f32("delta_q", l.k0), f32("delta_k", l.k0), f32("delta_beta", l.heads)
+        v = self.ws.get(f"delta_v_{dt}", (t, l.heads * l.dv), dt)
+        a.keep, a.q, a.k, a.v, a.beta, a.o = keep.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), o.data_ptr()
         N.check(self.lib.trl_delta_prep(ctypes.byref(a), t, _f32(proj), st), "delta_prep")
         N.count()
         if not single:
@@ -202,7 +209,7 @@ class GatedOps:
             per = len(seqs) * a.heads * lib.trl_delta_record(a.dk, a.dv)
             nc = max(1, min(chunks, DELTA_BYTES // per))
             a.chunk = self.ws.get("delta_chunks", (nc * per // 4,), torch.float32).data_ptr()
-            narrow = int(len(seqs) * a.heads * ((a.dv + 63) // 64) < self.sms)
+            narrow = int(len(seqs) * a.heads * ((a.dv + 31) // 32) <= 2 * self.sms)          # (two blocks share an SM)
             for c0 in range(0, chunks, nc):
                 sel = DeltaSel(len(seqs), c0, min(nc, chunks - c0), 0, (ctypes.c_int * 64)(*seqs))
                 N.check(lib.trl_delta_chunk(ctypes.byref(a), ctypes.byref(sel), narrow, st), "delta_chunk")

@@ -115,6 +115,7 @@ _SIGS = {
     "trl_lru_scan": [P, I, I, P], "trl_lru_step": [P, I, I, P],
     "trl_linear_rows_mix": [P, I, P, I, P, P, I, I, P, I, I, I, I, I, I, P],
     "trl_delta_prep": [P, I, I, P], "trl_delta_serial": [P, I, I, P],
+    "trl_delta_step": [P, I, P, I, P, P, I, I, F, I, P], "trl_delta_step_ok": [I, I],
     "trl_delta_chunk": [P, P, I, P], "trl_delta_record": [I, I], "trl_delta_chunk_tokens": [],
     "trl_moe_plan": [P, P],
     "trl_moe_rows": [P, I, P, P, I, P, P, P, I, I, I, I, I, I, P],

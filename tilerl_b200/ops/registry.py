@@ -193,6 +193,14 @@ register("any", "sm100", {
     "moe_tc": Kernel("moe_tc_kernel", "csrc/moe_tc.cu", "trl_moe_tc", note="many rows: tcgen05 kind::f16, N follows the rows of an expert, gated epilogue from TMEM"),
     "join_experts": Kernel("join_kernel", "csrc/join.cu", "trl_join_experts", note="weighted sum of a token's experts as the branch"),
     "soft_cap": Kernel("cap_kernel", "csrc/join.cu", "trl_soft_cap", note="few rows: epilogue of linear_rows_kernel"),
+    "act": Kernel("act_kernel", "csrc/join.cu", "trl_act", note="few rows: epilogue of linear_rows_kernel"),
+    "gated_join": Kernel("join_kernel", "csrc/join.cu", "trl_join_args", note="branch gate, bias, own share of a token's experts; decode ticks: convolution of the next input"),
+    "project_in": Kernel("linear_rows_kernel", "csrc/linear_rows.cu", "trl_linear_rows_mix", note="rows of two inputs, activation of the first rows; prompts: library products"),
+    "delta_prep": Kernel("delta_prep_kernel", "csrc/delta.cu", "trl_delta_prep", note="convolution, unit heads, decays per channel, write gates; bf16 or fp32"),
+    "delta_decode": Kernel("delta_step_kernel", "csrc/delta.cu", "trl_delta_step", note="from projection rows to normed and gated ones, one token per sequence"),
+    "delta_serial": Kernel("delta_serial_kernel", "csrc/delta.cu", "trl_delta_serial", note="fp32 state in registers; kept states, short portions, fp32 models"),
+    "delta_prefill": Kernel("delta_form_kernel + delta_scan_kernel", "csrc/delta_mma.cu", "trl_delta_chunk",
+                            note="32-token chunks: triangular form for all chunks at once, then state to state on tensor cores"),
     "batch_fill": Kernel("trl_batch_fill", "csrc/runtime.cpp", "trl_batch_fill", note="host runtime"),
     "pager": Kernel("trl_pager_*", "csrc/runtime.cpp", "trl_pager_alloc", note="host runtime"),
 })

@@ -12,6 +12,7 @@ JSON line:
   whole models and single kernels;
 * ``fetotar`` (:mod:`.fetotar`): the Fetotar design beside the hybrid with Gated-DeltaNet layers, likewise;
 * ``deluvik`` (:mod:`.deluvik`): the Deluvik design beside the hybrid with mostly attention layers, likewise;
+* ``tobadra`` (:mod:`.tobadra`): the Tobadra design beside the hybrid with mostly Gated-DeltaNet layers, likewise;
 * ``grpo`` (:mod:`.grpo`): one-GPU GRPO step with LoRA adapters, split rollout / train;
 * ``grpo-zero3`` (:mod:`.grpo_zero3`, started under ``torchrun``): GRPO step with ZeRO-3 training
   and a tensor-parallel NVFP4 rollout engine on the same GPUs.
@@ -32,6 +33,7 @@ SUITES = {
     "zinutar": ("zinutar", []),
     "fetotar": ("fetotar", []),
     "deluvik": ("deluvik", []),
+    "tobadra": ("tobadra", []),
     "grpo": ("grpo", []),
     "grpo-zero3": ("grpo_zero3", []),
 }
