@@ -118,7 +118,7 @@ def kernels(size: str, reps: int, hbm_gbs: float, tflops: float):
     alp = {"q_norm": torch.ones(256, device=dev), "k_norm": torch.ones(256, device=dev)}
     nq, nkv = ch.n_q_heads, ch.n_kv_heads
     dw = {k: P["L0." + k] for k in ("conv", "low", "dt_bias", "a_log")}
-    for b, n, ctx in ((1, 1, 4096), (16, 1, 4096), (64, 1, 4096), (1, 512, 512), (1, 2048, 2048), (1, 8192, 8192), (4, 2048, 4096)):
+    for b, n, ctx in ((1, 1, 1024), (16, 1, 1024), (64, 1, 1024), (64, 1, 4096), (1, 512, 512), (1, 2048, 2048), (1, 8192, 8192), (4, 2048, 4096)):
         pages = ctx // 16 + 2
         seqs = [dict(tokens=[1] * n, start=ctx - n, blocks=list(range(1 + i * pages, 1 + (i + 1) * pages)), slot=i + 1) for i in range(b)]
         batch, t = Batch.build(seqs, dev), b * n
