@@ -31,6 +31,7 @@ from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
+from . import fetotar_layout
 from .config import DeluvikConfig, FetotarConfig, ModelConfig, StreamDesign, TobadraConfig
 from .fetotar_layout import LatentLayout, layout_of
 from .ops.ref import KV_BLOCK
@@ -390,7 +391,7 @@ class GdnStatePool:
 
 def state_layouts(cfg) -> Tuple[object, ...]:
     """What a design's layers keep per sequence beside keys and values, in the order of the states."""
-    return cfg.layout.state_layouts(cfg)
+    return getattr(cfg, "layout", fetotar_layout).state_layouts(cfg)
 
 
 class RecurrentPool:
