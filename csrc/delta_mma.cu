@@ -151,18 +151,20 @@ __global__ void __launch_bounds__(DF_THREADS) delta_form_kernel(const DeltaArgs 
   }
   __syncthreads();
   if (warp == 0) {
-    // ---- T: lane j solves its column by forward substitution
-    float t[DC];
+    // ---- the two diagonal blocks of T: a lane solves a column of its block by forward substitution
+    const int o = lane & 16, j = lane & 15;
+    float t[16];
 #pragma unroll
-    for (int i = 0; i < DC; ++i) {
-      float v0 = i == lane ? 1.f : 0.f, v1 = 0.f;
+    for (int i = 0; i < 16; ++i) {
+      float v0 = i == j ? 1.f : 0.f, v1 = 0.f;
 #pragma unroll
       for (int m = 0; m < i; ++m) {
-        if (m & 1) v1 = fmaf(-sm.A[i][m], t[m], v1);
-        else v0 = fmaf(-sm.A[i][m], t[m], v0);
+        if (m & 1) v1 = fmaf(-sm.A[o + i][o + m], t[m], v1);
+        else v0 = fmaf(-sm.A[o + i][o + m], t[m], v0);
       }
       t[i] = v0 + v1;
-      sm.T[i][lane] = t[i];
+      sm.T[o + i][lane] = t[i];
+      if (o) sm.T[i][lane] = 0.f;
     }
   } else {
     // ---- decayed queries and keys
@@ -171,17 +173,38 @@ __global__ void __launch_bounds__(DF_THREADS) delta_form_kernel(const DeltaArgs 
       const int y = is_k ? x - DC * (DK / 8) : x, r = y / (DK / 8), ch = y % (DK / 8);
       uint32_t hi[4], lo[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
+      for (int e = 0; e < 4; e += 2) {
         const int d = ch * 8 + 2 * e;
-        float f[2];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) f[i] = is_k ? sm.k[r][d + i] * ex2_f(sm.G[DC - 1][d + i] - sm.G[r][d + i]) : sm.q[r][d + i] * ex2_f(sm.G[r][d + i]);
-        split2(f[0], f[1], hi[e], lo[e]);
+        const float4 f = *reinterpret_cast<const float4*>(is_k ? &sm.k[r][d] : &sm.q[r][d]);
+        float4 g = *reinterpret_cast<const float4*>(&sm.G[r][d]);
+        if (is_k) {
+          const float4 end = *reinterpret_cast<const float4*>(&sm.G[DC - 1][d]);
+          g = make_float4(end.x - g.x, end.y - g.y, end.z - g.z, end.w - g.w);
+        }
+        split2(f.x * ex2_f(g.x), f.y * ex2_f(g.y), hi[e], lo[e]);
+        split2(f.z * ex2_f(g.z), f.w * ex2_f(g.w), hi[e + 1], lo[e + 1]);
       }
       unsigned char* dst = rec + (is_k ? 4 : 2) * R::TILE + tile_off<R::ROW>(r, ch);
       *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
       *reinterpret_cast<uint4*>(dst + R::TILE) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
+  }
+  __syncthreads();
+  // ---- the block below: -T22 (A21 T11), the inner product where A is not needed any more
+  if (tid < 256) {
+    const int i = tid >> 4, j = tid & 15;
+    float v = 0.f;
+#pragma unroll
+    for (int m = 0; m < 16; ++m) v = fmaf(sm.A[16 + i][m], sm.T[m][j], v);
+    sm.A[i][j] = v;
+  }
+  __syncthreads();
+  if (tid < 256) {
+    const int i = tid >> 4, j = tid & 15;
+    float v = 0.f;
+#pragma unroll
+    for (int m = 0; m < 16; ++m) v = fmaf(-sm.T[16 + i][16 + m], sm.A[m][j], v);
+    sm.T[16 + i][j] = v;
   }
   __syncthreads();
   // ---- W and U: a thread per column (pairs of lanes store W together)

@@ -158,6 +158,18 @@ def test_served_parameters_hold_every_tensor_and_only_zeros_besides(name):
     assert set(dict(again.tensors())) == set(w)
 
 
+def test_parameters_used_by_way_of_another_layer():
+    cfg = CONFIGS["mixed"]
+    j = cfg.to_json()
+    j["layers"].append({**json.loads(json.dumps(j["layers"][0])), "weights_of": 0})            # layer 0 uses those of layer 3
+    from tilerl_b200.tobadra_layout import tensor_shapes
+    more = TobadraConfig.from_json(j, shapes=tensor_shapes(cfg))
+    assert more.source(6) == 3 and more.owners == cfg.owners and tensor_shapes(more) == tensor_shapes(cfg)
+    j["layers"][3]["weights_of"] = 6
+    with pytest.raises(ValueError):
+        TobadraConfig.from_json(j, shapes=tensor_shapes(cfg))
+
+
 def test_configuration_refuses_what_it_does_not_know():
     from tilerl_b200.tobadra_layout import tensor_shapes
     cfg = CONFIGS["mixed"]

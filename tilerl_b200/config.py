@@ -702,6 +702,18 @@ def tensor_shapes_in(path: str) -> Dict[str, Tuple[int, ...]]:
     return out
 
 
+def _parameter_layer(weights_of, layer: int) -> int:
+    """The layer whose parameters ``layer`` uses, by way of others that use them, too."""
+    at = layer
+    for _ in weights_of:
+        if weights_of[at] is None:
+            return at
+        at = int(weights_of[at])
+        if not 0 <= at < len(weights_of):
+            break
+    raise ValueError(f"layer {layer} uses the parameters of no layer")
+
+
 @dataclass(frozen=True)
 class TobadraConfig(StreamDesign):
     """Sizes and constants of a Tobadra model.  Every layer has its own mixer and feed-forward; attention layers number the KV
@@ -726,15 +738,13 @@ class TobadraConfig(StreamDesign):
         for i, l in enumerate(self.layers):
             if not isinstance(l.mixer, self.MIXERS):
                 raise ValueError(f"layer {i}: not a mixer of this design: {l.mixer}")
-            if l.weights_of is not None:
-                src = self.layers[l.weights_of] if 0 <= l.weights_of < len(self.layers) else None
-                if src is None or src.weights_of is not None or (src.mixer, src.mlp) != (l.mixer, l.mlp):
-                    raise ValueError(f"layer {i} cannot use the parameters of layer {l.weights_of}")
+            src = self.layers[_parameter_layer([x.weights_of for x in self.layers], i)]
+            if (src.mixer, src.mlp) != (l.mixer, l.mlp):
+                raise ValueError(f"layer {i} cannot use the parameters of layer {l.weights_of}")
 
     def source(self, layer: int) -> int:
         """The layer whose parameters this one uses."""
-        src = self.layers[layer].weights_of
-        return layer if src is None else src
+        return _parameter_layer([x.weights_of for x in self.layers], layer)
 
     @property
     def owners(self) -> Tuple[int, ...]:
@@ -789,7 +799,8 @@ class TobadraConfig(StreamDesign):
             elif l["type"] == "lightning":
                 m = LightningSpec.from_json(m, where)
             elif l["type"] == "channel_delta":
-                ranks = [(shapes or {}).get(f"l{i if src is None else src}.mix.{n}") for n in ("a1", "g1")]
+                own = _parameter_layer([x.get("weights_of") for x in j["layers"]], i)
+                ranks = [(shapes or {}).get(f"l{own}.mix.{n}") for n in ("a1", "g1")]
                 if None in ranks:
                     raise ValueError(f"{where}: the checkpoint does not have the maps whose shapes tell its ranks")
                 m = ChannelDeltaSpec.from_json(m, where, *(r[0] for r in ranks))
