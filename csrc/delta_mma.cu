@@ -90,62 +90,67 @@ __global__ void __launch_bounds__(DF_THREADS) delta_form_kernel(const DeltaArgs 
     reinterpret_cast<float*>(rec + R::G)[tid] = ex2_f(s);
   }
   __syncthreads();
-  // ---- A and N in tiles of two by two, two threads (halves of the channels) a tile
+  // ---- A and N in tiles of four by four, eight threads (shares of the channels) a tile
   {
-    const int tile = tid >> 1, half = tid & 1;
-    const bool on = tile < 136;
-    int ti = (int)((sqrtf(8.f * (float)tile + 1.f) - 1.f) * 0.5f);
-    while (ti * (ti + 1) / 2 > tile) --ti;
+    const int tile = tid >> 3, sl = tid & 7;
+    int ti = 0;
     while ((ti + 1) * (ti + 2) / 2 <= tile) ++ti;
-    if (!on) ti = 0;
-    const int tj = on ? tile - ti * (ti + 1) / 2 : 0, r = 2 * ti, c = 2 * tj;
+    const int tj = tile - ti * (ti + 1) / 2, r = 4 * ti, c = 4 * tj;
     const bool diag = ti == tj;
-    float kk[2][2] = {}, qk[2][2] = {};
-#pragma unroll 2
-    for (int s = 0; s < Q4 / 2; ++s) {
-      const int d = (2 * s + half) * 4;
-      float kr[2][4], qr[2][4], kc[2][4], gr[4], gc[4], Gr[4], Gc[4];
-      auto get = [&](float (&o)[4], const float* p) {
-        const float4 v = *reinterpret_cast<const float4*>(p);
-        o[0] = v.x, o[1] = v.y, o[2] = v.z, o[3] = v.w;
-      };
-      get(kr[0], &sm.k[r][d]), get(kr[1], &sm.k[r + 1][d]), get(qr[0], &sm.q[r][d]), get(qr[1], &sm.q[r + 1][d]);
-      get(kc[0], &sm.k[c][d]), get(kc[1], &sm.k[c + 1][d]), get(gr, &sm.g[r + 1][d]), get(gc, &sm.g[c + 1][d]);
-      get(Gr, &sm.G[r][d]), get(Gc, &sm.G[c + 1][d]);
+    float acc[32];                                               // k . k, then q . k, row by row
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        // e^(G_i - G_j): the closest pair of rows, the others by factors (on the diagonal: one, one, and one factor)
-        const float e01 = diag ? 0.f : ex2_f(Gr[e] - Gc[e]), e00 = diag ? 1.f : e01 * gc[e];
-        const float e11 = diag ? 1.f : e01 * gr[e], e10 = e00 * gr[e];
-        const float x00 = kc[0][e] * e00, x10 = kc[0][e] * e10, x01 = kc[1][e] * e01, x11 = kc[1][e] * e11;
-        kk[0][0] = fmaf(kr[0][e], x00, kk[0][0]), kk[0][1] = fmaf(kr[0][e], x01, kk[0][1]);
-        kk[1][0] = fmaf(kr[1][e], x10, kk[1][0]), kk[1][1] = fmaf(kr[1][e], x11, kk[1][1]);
-        qk[0][0] = fmaf(qr[0][e], x00, qk[0][0]), qk[0][1] = fmaf(qr[0][e], x01, qk[0][1]);
-        qk[1][0] = fmaf(qr[1][e], x10, qk[1][0]), qk[1][1] = fmaf(qr[1][e], x11, qk[1][1]);
+    for (int i = 0; i < 32; ++i) acc[i] = 0.f;
+#pragma unroll 1
+    for (int s = 0; s < DK / 16; ++s) {
+      const int d = (8 * s + sl) * 2;
+      auto get = [&](const float* p) { return *reinterpret_cast<const float2*>(p); };
+      float2 kr[4], qr[4], kc[4], gr[4], gc[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) kr[i] = get(&sm.k[r + i][d]), qr[i] = get(&sm.q[r + i][d]), kc[i] = get(&sm.k[c + i][d]);
+#pragma unroll
+      for (int i = 1; i < 4; ++i) gr[i] = get(&sm.g[r + i][d]), gc[i] = get(&sm.g[c + i][d]);
+      const float2 Gr = get(&sm.G[r][d]), Gc = get(&sm.G[c + 3][d]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        auto at = [&](const float2& v) { return e ? v.y : v.x; };
+        // e^(G_i - G_j): the closest pair of rows, the others by factors (on the diagonal: one, and factors below it)
+        float E[4];
+        E[3] = diag ? 0.f : ex2_f(at(Gr) - at(Gc));
+        E[2] = E[3] * at(gc[3]), E[1] = E[2] * at(gc[2]), E[0] = diag ? 1.f : E[1] * at(gc[1]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if (i) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) E[j] = diag && j == i ? 1.f : E[j] * at(gr[i]);
+          }
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float x = at(kc[j]) * E[j];
+            acc[i * 4 + j] = fmaf(at(kr[i]), x, acc[i * 4 + j]), acc[16 + i * 4 + j] = fmaf(at(qr[i]), x, acc[16 + i * 4 + j]);
+          }
+        }
       }
     }
+    // the eight shares: every step halves what a thread holds, until it has one row of one product
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+    for (int m = 4, n = 16; m > 0; m >>= 1, n >>= 1)
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        kk[i][j] += __shfl_xor_sync(0xffffffffu, kk[i][j], 1), qk[i][j] += __shfl_xor_sync(0xffffffffu, qk[i][j], 1);
+      for (int i = 0; i < n; ++i) {
+        const float mine = sl & m ? acc[n + i] : acc[i], other = sl & m ? acc[i] : acc[n + i];
+        acc[i] = mine + __shfl_xor_sync(0xffffffffu, other, m);
       }
-    if (on && half == 0) {
+    const int row = r + (sl & 3);
+    if (sl < 4) {
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j) sm.A[r + i][c + j] = c + j < r + i ? sm.beta[r + i] * kk[i][j] : 0.f;
-    } else if (on) {
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        uint32_t hi, lo;
-        split2(qk[i][0], diag && i == 0 ? 0.f : qk[i][1], hi, lo);
-        const uint32_t o = tile_off<R::NROW>(r + i, c >> 3) + (c & 7) * 2;
-        *reinterpret_cast<uint32_t*>(rec + R::N + o) = hi, *reinterpret_cast<uint32_t*>(rec + R::N + R::NTILE + o) = lo;
-        if (!diag) {                                             // the mirrored tile lies above the diagonal
-          const uint32_t m = tile_off<R::NROW>(c + i, r >> 3) + (r & 7) * 2;
-          *reinterpret_cast<uint32_t*>(rec + R::N + m) = 0u, *reinterpret_cast<uint32_t*>(rec + R::N + R::NTILE + m) = 0u;
-        }
+      for (int j = 0; j < 4; ++j) sm.A[row][c + j] = c + j < row ? sm.beta[row] * acc[j] : 0.f;
+    } else {
+      uint2 hi, lo;                                              // (zeros above the diagonal)
+      split2(acc[0], acc[1], hi.x, lo.x), split2(acc[2], acc[3], hi.y, lo.y);
+      const uint32_t o = tile_off<R::NROW>(row, c >> 3) + (c & 7) * 2;
+      *reinterpret_cast<uint2*>(rec + R::N + o) = hi, *reinterpret_cast<uint2*>(rec + R::N + R::NTILE + o) = lo;
+      if (!diag) {                                               // the mirrored tile lies above the diagonal
+        const uint32_t m = tile_off<R::NROW>(c + (sl & 3), r >> 3) + (r & 7) * 2;
+        *reinterpret_cast<uint2*>(rec + R::N + m) = make_uint2(0u, 0u), *reinterpret_cast<uint2*>(rec + R::N + R::NTILE + m) = make_uint2(0u, 0u);
       }
     }
   }

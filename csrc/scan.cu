@@ -308,9 +308,11 @@ struct NormArgs {
   const int *positions, *seq_ids, *q_start, *q_len, *slots;
 };
 
-// one block per token
-constexpr int NORM_R = 8;
-template <typename T, int KIND>
+// gates behind a recurrence's norm
+template <typename T> __device__ __forceinline__ float gate_x(float z) { return sizeof(T) == 2 ? sigmoid_f(z) : sigmoid_x(z); }
+
+// one block per token; NORM_R: float4 a thread keeps of a row
+template <typename T, int KIND, int NORM_R>
 __global__ void __launch_bounds__(256) scan_norm_kernel(const NormArgs a) {
   extern __shared__ float s_y[];               // [heads * vdim], true columns only
   __shared__ float red[32];
@@ -340,7 +342,7 @@ __global__ void __launch_bounds__(256) scan_norm_kernel(const NormArgs a) {
 #pragma unroll
     for (int i = 0; i < NORM_R; ++i)
       if (i < nr) {
-        const float4 s = make_float4(sigmoid_x(z[i].x), sigmoid_x(z[i].y), sigmoid_x(z[i].z), sigmoid_x(z[i].w));
+        const float4 s = make_float4(gate_x<T>(z[i].x), gate_x<T>(z[i].y), gate_x<T>(z[i].z), gate_x<T>(z[i].w));
         if (KIND == SCAN_MAMBA2) v[i].x *= z[i].x * s.x, v[i].y *= z[i].y * s.y, v[i].z *= z[i].z * s.z, v[i].w *= z[i].w * s.w;
         z[i] = s;
         const float ss = warp_sum(v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w);
@@ -484,8 +486,11 @@ TRL_API int trl_scan_norm(const void* o, const void* gate, int ldp, const void* 
   a.q_start = (const int*)q_start, a.q_len = (const int*)q_len, a.slots = (const int*)slots;
   cudaStream_t st = (cudaStream_t)stream;
 #define NORM_AS(TT, KK)                                                                                                    \
+  if (heads * vdim <= 4096) NORM_R_AS(TT, KK, 4)                                                                           \
+  else NORM_R_AS(TT, KK, 8)
+#define NORM_R_AS(TT, KK, RR)                                                                                              \
   {                                                                                                                        \
-    auto k = scan_norm_kernel<TT, KK>;                                                                                     \
+    auto k = scan_norm_kernel<TT, KK, RR>;                                                                                     \
     static bool configured = false;                                                                                        \
     if (!configured) {                                                                                                     \
       const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);              \
@@ -501,4 +506,5 @@ TRL_API int trl_scan_norm(const void* o, const void* gate, int ldp, const void* 
   if (f32) NORM_AS(float, SCAN_MLSTM)
   NORM_AS(bf16, SCAN_MLSTM)
 #undef NORM_AS
+#undef NORM_R_AS
 }
